@@ -156,6 +156,18 @@ class Req:
         self._grow[have] = next_token.view(())
         self.input_ids = self._grow[: have + 1]
 
+    def extend_host(self, tokens: torch.Tensor) -> None:
+        """Appends tokens that are given, not sampled, to the host copy; the next forwards run them."""
+        have, n = len(self.input_ids), len(tokens)
+        if have + n > self.max_device_len:
+            raise RuntimeError("the request's length limit is used up")
+        if self._grow is None:
+            self._grow = torch.empty(self.max_device_len, dtype=self.input_ids.dtype)
+            self._grow[:have] = self.input_ids
+        self._grow[have:have + n] = tokens
+        self.input_ids = self._grow[: have + n]
+        self.device_len = have + n
+
     def observe_generated_token(self, token_id: int, *, think_end_token_id: int) -> None:
         self.reasoning_state = advance_reasoning_state(self.reasoning_state, token_id,
                                                        think_end_token_id=think_end_token_id)
@@ -179,6 +191,7 @@ class Batch:
     num_token_non_padded: int = 0
     reasoning_states: Any = None
     max_context: int = 0         # largest device_len in the batch (bounds index-surface widths)
+    seg_off: Any = None          # prefill: [B+1] int32 device, row ranges of the requests
 
     @property
     def is_prefill(self) -> bool:

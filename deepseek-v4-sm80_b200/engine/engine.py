@@ -17,10 +17,10 @@ from typing import Any, Dict, List, Optional
 import torch
 
 from ..core import Batch, Req
-from ..dsv4_release import DSV4_RELEASE, RECIPES
-from ..kvcache.pool import DSV4KVPool, PoolSizes, bytes_per_page, bytes_per_req_slot, bytes_per_swa_slot
-from ..models.config import ModelConfig
-from ..models.deepseek_v4 import DSV4Model, ForwardBatch, GreedyTail
+from ..dsv4_release import RECIPES
+from ..kvcache.paged import PoolSizes
+from ..models.base import ForwardBatch, GreedyTail
+from ..models.registry import family_of, parse_config, swa_slot_plan  # noqa: F401
 from ..parallel import comm as comm_mod
 from ..parallel.info import set_tp_info
 from ..utils.logger import init_logger, set_log_rank
@@ -42,19 +42,6 @@ class ForwardOutput:
     status: Any = None           # ops.native.StatusProbe whose snapshot was queued behind this forward (CUDA only)
 
 
-def swa_slot_plan(max_running_req: int, prefill_budget: int, page_size: int, window: int) -> int:
-    """Sliding-window slots to reserve: the pages of one full prefill forward, one spare, and per running request its
-    hard share (:func:`minisgl.scheduler.cache.slots_per_request`: window pages, the page being written, the step
-    overlap scheduling keeps in flight) plus ``ceil(window / ps)`` for the tail of the cached path it locks in the
-    prefix tree.  Admission divides the pool by the hard share (``CacheManager.request_capacity``); the tree's part is
-    an allowance that keeps prefix-hit resume points alive and is given up first under pressure.
-    (The reference reserves at least 8 per request, python/minisgl/engine/engine.py:569-584.)"""
-    from ..scheduler.cache import slots_per_request
-
-    per_req = slots_per_request(window, page_size) + div_ceil(window, page_size)
-    return div_ceil(prefill_budget, page_size) + 1 + max_running_req * per_req
-
-
 class Engine:
     def __init__(self, config: EngineConfig):
         self.config = config = self._adjust_config(config)
@@ -74,8 +61,14 @@ class Engine:
             self.stream = torch.cuda.Stream(self.device)
         else:
             self.stream = None
-        self.model_config: ModelConfig = config.model_config or self._load_model_config(config.model_path)
+        self.model_config = config.model_config or self._load_model_config(config.model_path)
         cfg = self.model_config
+        self.family = family_of(cfg)
+        if config.dtype not in self.family.dtypes:
+            raise ValueError(f"{self.family.name} models are served in {[str(d) for d in self.family.dtypes]}, not "
+                             f"{config.dtype}")
+        if tp.size > self.family.max_tp:
+            raise ValueError(f"{self.family.name} models run on at most {self.family.max_tp} GPU(s), not {tp.size}")
         self.page_size = config.page_size
         self.cpu_group, self.comm = comm_mod.init_distributed(
             tp, self.device, config.distributed_addr, config.distributed_timeout, fused=config.use_pynccl,
@@ -94,8 +87,8 @@ class Engine:
             buckets=self.graph_policy.buckets, num_context_classes=len(self.context_classes),
             hidden_size=cfg.hidden_size)
         self.kv_plan = self._plan_kv()
-        self.pool = DSV4KVPool(cfg, PoolSizes(self.kv_plan["num_pages"], self.kv_plan["swa_slots"],
-                                              config.max_running_req, self.page_size), self.device)
+        self.pool = self.family.pool(cfg, PoolSizes(self.kv_plan["num_pages"], self.kv_plan["swa_slots"],
+                                                    config.max_running_req, self.page_size), self.device, config.dtype)
         self.num_pages = self.kv_plan["num_pages"]
         self.max_seq_len = self.kv_plan["max_seq_len"]
         self.page_table = torch.zeros(config.max_running_req + 1, align_ceil(self.max_seq_len, self.page_size),
@@ -105,7 +98,7 @@ class Engine:
         row = self.pool.dummy_page * ps + torch.arange(self.page_table.shape[1], dtype=torch.int32) % ps
         self.page_table[self.dummy_slot] = row.to(self.device)
         self.last_token = torch.zeros(config.max_running_req + 1, dtype=torch.int32, device=self.device)
-        self.model = DSV4Model(cfg, self.weights, self.pool, self.comm, config.moe_mode)
+        self.model = self.family.build(cfg, self.weights, self.pool, self.comm, config.moe_mode, config.dtype)
         self.model_prepare_report = self.model.prepare_report()
         logger.info_rank0("model prepared: %s", {k: v for k, v in self.model_prepare_report.items()
                                                  if k != "derived_bytes"})
@@ -165,31 +158,26 @@ class Engine:
         return rank % max(torch.cuda.device_count(), 1)
 
     @staticmethod
-    def _load_model_config(path: str) -> ModelConfig:
+    def _load_model_config(path: str):
         from ..utils.hf import cached_load_hf_config
 
-        return ModelConfig.from_hf(cached_load_hf_config(path))
+        return parse_config(cached_load_hf_config(path))
 
     def _load_weights(self) -> Dict[str, torch.Tensor]:
         cfg, tp = self.model_config, self.config.tp_info
         if self.config.use_dummy_weight or not self.config.model_path:
-            from ..models import synth
-
             from ..env import ENV
 
-            return synth.random_weights(cfg, self.device, tp.rank, tp.size, self.config.moe_mode, self.config.seed,
-                                        fast_experts=self.is_cuda,
-                                        draw_on_host=self.is_cuda and bool(ENV.DUMMY_WEIGHT_ON_HOST))
-        from ..models.weight import load_checkpoint
+            return self.family.draw(cfg, self.device, tp.rank, tp.size, self.config.moe_mode, self.config.seed,
+                                    bool(ENV.DUMMY_WEIGHT_ON_HOST))
         from ..utils.hf import download_hf_weight
 
-        return load_checkpoint(download_hf_weight(self.config.model_path), cfg, self.device, tp.rank, tp.size,
-                               self.config.moe_mode)
+        return self.family.load(download_hf_weight(self.config.model_path), cfg, self.device, tp.rank, tp.size,
+                                self.config.moe_mode)
 
     def _context_classes(self) -> List[int]:
         limit = self.config.max_seq_len_override or self.model_config.max_position
-        classes = [c for c in (4 * self.model_config.index_topk, DSV4_RELEASE.graph_short_context) if c < limit]
-        return classes + [limit]
+        return self.family.context_classes(self.model_config, limit) + [limit]
 
     # ------------------------------------------------------------------ memory
     def _sync_free_memory(self) -> int:
@@ -212,9 +200,8 @@ class Engine:
         cfg, c = self.model_config, self.config
         ps = self.page_size
         limit = c.max_seq_len_override or cfg.max_position
-        swa_slots = swa_slot_plan(c.max_running_req, c.max_prefill_length, ps, cfg.window_size)
-        per_page = bytes_per_page(cfg, ps)
-        fixed = swa_slots * bytes_per_swa_slot(cfg, ps) + (c.max_running_req + 1) * bytes_per_req_slot(cfg)
+        kv = self.family.budget(cfg, c, c.dtype)
+        swa_slots, per_page, fixed = kv.window_slots, kv.bytes_per_page, kv.fixed_bytes
         want_pages = min(c.max_running_req * div_ceil(limit, ps) + div_ceil(c.max_prefill_length, ps), 1 << 18)
         if self.is_cuda:
             free = self._sync_free_memory()
@@ -224,7 +211,7 @@ class Engine:
             budget -= table_bytes
             num_pages = graph_memory.select_num_pages(budget_bytes=budget, bytes_per_page=per_page,
                                                       override=c.num_page_override,
-                                                      min_pages=div_ceil(c.max_prefill_length, ps) + 1)
+                                                      min_pages=kv.min_pages)
             if c.num_page_override is None:
                 num_pages = min(num_pages, want_pages)
         else:
@@ -248,7 +235,39 @@ class Engine:
     def make_forward_batch(self, batch: Batch) -> ForwardBatch:
         return ForwardBatch(batch.input_ids, batch.positions, batch.slots, batch.out_loc, batch.last_idx,
                             self.page_table, batch.is_prefill, batch.max_context, None,
-                            token_feedback=self.last_token if batch.is_decode else None)
+                            token_feedback=self.last_token if batch.is_decode else None, seg_off=batch.seg_off,
+                            seg_lens=batch.chunk_lens if batch.is_prefill else None)
+
+    def _run(self, batch: Batch, greedy: bool):
+        """Launches one forward: (logits, greedy tokens or None).  Decode batches replay a captured graph when there is
+        one of their size."""
+        if batch.is_decode and batch.input_ids is None:
+            # decode rows take their token from last_token[slot] inside the embedding kernel, which fills this buffer
+            batch.input_ids = torch.empty(batch.positions.shape[0], dtype=torch.int32, device=self.device)
+        if self.graph_runner is not None and batch.is_decode and self.graph_runner.can_replay(batch):
+            logits, toks = self.graph_runner.replay(batch)
+            return (logits, toks) if greedy else (self.comm.all_gather_last(logits), None)
+        if greedy:
+            return self.model.forward(self.make_forward_batch(batch), GreedyTail(self.last_token))
+        return self.model.forward(self.make_forward_batch(batch)), None
+
+    def force_tokens(self, slots: torch.Tensor, tokens: torch.Tensor) -> None:
+        """Makes ``tokens`` (instead of the last samples) the next input of the request slots' decode rows."""
+        self.last_token[slots.long().to(self.device)] = tokens.to(self.device, torch.int32)
+
+    def forward_logits(self, batch: Batch, rows: List[int]) -> torch.Tensor:
+        """Runs one prepared batch without sampling: fp32 logits [len(rows), vocab] of the given rows of the batch."""
+        if batch.is_prefill:
+            batch.last_idx = torch.tensor(rows, dtype=torch.int64, device=self.device)
+        keep = None
+        if batch.is_decode and self.graph_runner is not None:
+            keep = self.last_token.clone()      # a captured decode step ends with sampling: undo its token feedback
+        logits, _ = self._run(batch, False)
+        if keep is not None:
+            self.last_token.copy_(keep)
+        if batch.is_prefill:
+            return logits
+        return logits[torch.tensor(rows, dtype=torch.int64, device=self.device)]
 
     def forward_batch(self, batch: Batch, args: BatchSamplingArgs) -> ForwardOutput:
         t_ev = None
@@ -258,18 +277,7 @@ class Engine:
         # Greedy batches are sampled by the forward's last kernel (argmax over the vocabulary-parallel logits with
         # the shards' candidates exchanged in-kernel), which also stores the token as the request's next input.
         greedy = args.all_greedy and args.mask_ids is None
-        toks = None
-        if batch.is_decode and batch.input_ids is None:
-            # decode rows take their token from last_token[slot] inside the embedding kernel, which fills this buffer
-            batch.input_ids = torch.empty(batch.positions.shape[0], dtype=torch.int32, device=self.device)
-        if self.graph_runner is not None and batch.is_decode and self.graph_runner.can_replay(batch):
-            logits, toks = self.graph_runner.replay(batch)
-            if not greedy:
-                logits = self.comm.all_gather_last(logits)
-        elif greedy:
-            logits, toks = self.model.forward(self.make_forward_batch(batch), GreedyTail(self.last_token))
-        else:
-            logits = self.model.forward(self.make_forward_batch(batch))
+        logits, toks = self._run(batch, greedy)
         for req in batch.reqs:
             req.complete_one()
         if greedy:

@@ -16,7 +16,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..core import Batch
-from ..models.deepseek_v4 import ForwardBatch, GreedyTail
+from ..models.base import ForwardBatch, GreedyTail
 from ..ops import native
 from ..utils.logger import init_logger
 from .graph_policy import pick_bucket
@@ -60,7 +60,7 @@ class GraphRunner:
         self.buffer = GraphCaptureBuffer(self.max_bs, engine.device)
         # every graph writes its logits shard into the same static buffer: a per-graph output would pin
         # bucket x vocab floats for each of the dozens of (bucket, context class) graphs of a serving recipe
-        self.buffer.logits = torch.empty(self.max_bs, engine.weights["head.weight"].shape[0], dtype=torch.float32,
+        self.buffer.logits = torch.empty(self.max_bs, engine.model.logits_width, dtype=torch.float32,
                                          device=engine.device)
         self.graphs: Dict[Tuple[int, int], torch.cuda.CUDAGraph] = {}
         self.logits: Dict[Tuple[int, int], torch.Tensor] = {}

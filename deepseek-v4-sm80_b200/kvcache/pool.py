@@ -23,21 +23,12 @@ The last page id and the last table slot are reserved for the dummy request that
 from __future__ import annotations
 
 from collections import OrderedDict
-
-from dataclasses import dataclass
-from typing import List, Optional
+from typing import List
 
 import torch
 
 from ..models.config import ModelConfig
-
-
-@dataclass
-class PoolSizes:
-    num_pages: int
-    num_swa_slots: int
-    num_req_slots: int
-    page_size: int
+from .paged import PagedPool, PoolSizes
 
 
 def bytes_per_page(cfg: ModelConfig, page_size: int) -> int:
@@ -62,18 +53,21 @@ def bytes_per_req_slot(cfg: ModelConfig) -> int:
     return (len(cfg.c4_layers) * 8 * (4 * d + 4 * di) + len(cfg.c128_layers) * 128 * 2 * d) * 4
 
 
-class DSV4KVPool:
+class DSV4KVPool(PagedPool):
+    has_window = True
+    prefix_align = 128        # the ratio-128 compressor's ring holds no partial group at such boundaries
+
     def __init__(self, cfg: ModelConfig, sizes: PoolSizes, device, dtype=torch.bfloat16):
-        self.cfg, self.sizes, self.device = cfg, sizes, torch.device(device)
+        super().__init__(sizes, device)
+        self.cfg = cfg
         ps = sizes.page_size
         assert ps % 4 == 0, "page size must be a multiple of the C4 ratio"
-        self.page_size = ps
         self.c4_rpp = ps // 4
         self.c128_rpp = max(ps // 128, 1)
         d, di = cfg.head_dim, cfg.index_head_dim
         n4, n128 = len(cfg.c4_layers), len(cfg.c128_layers)
         P, S, R = sizes.num_pages + 1, sizes.num_swa_slots + 1, sizes.num_req_slots + 1
-        self.dummy_page, self.dummy_swa, self.dummy_slot = P - 1, S - 1, R - 1
+        self.dummy_swa = S - 1
         self.layer_c4 = {l: i for i, l in enumerate(cfg.c4_layers)}
         self.layer_c128 = {l: i for i, l in enumerate(cfg.c128_layers)}
         z = dict(device=self.device)
@@ -92,62 +86,27 @@ class DSV4KVPool:
         # host-side ownership
         self._swa_map_host = [-1] * P
         self._swa_map_host[self.dummy_page] = self.dummy_swa
-        self.free_pages: List[int] = list(range(sizes.num_pages - 1, -1, -1))
         self.free_swa: List[int] = list(range(sizes.num_swa_slots - 1, -1, -1))
-        self.page_ref = [0] * P
         self.swa_pins = [0] * P          # users of a page's window storage (running requests + the radix tree)
         self._tree_pinned: "OrderedDict[int, None]" = OrderedDict()   # pages the prefix tree pins, oldest pin first
         self.swa_version = 0
         # pages nobody pins any more but that still own a window slot, oldest first: their rows stay readable (a later
         # prefix hit can resume on them) until another page needs the slot
         self._reclaimable: "OrderedDict[int, None]" = OrderedDict()
-        self.counters = {"swa_taken": 0, "swa_released": 0, "swa_reclaimed": 0, "pages_taken": 0, "pages_released": 0}
+        self.counters.update({"swa_taken": 0, "swa_released": 0, "swa_reclaimed": 0})
 
-    # ------------------------------------------------------------------ pages
-    @property
-    def num_free_pages(self) -> int:
-        return len(self.free_pages)
+    def _on_freed(self, pages: List[int]) -> None:
+        for p in pages:
+            self.swa_pins[p] = 0
+            self._tree_pinned.pop(p, None)
+        self.release_swa(pages)
 
+    # ------------------------------------------------------------------ SWA slots
     @property
     def num_free_swa(self) -> int:
         """Window slots a new page can get: unused ones plus those of unpinned pages (reclaimed on demand)."""
         return len(self.free_swa) + len(self._reclaimable)
 
-    def alloc_pages(self, n: int, with_swa: bool = True) -> List[int]:
-        if n > len(self.free_pages) or (with_swa and n > self.num_free_swa):
-            raise RuntimeError(f"KV pool exhausted: want {n} pages, free {len(self.free_pages)} pages / "
-                               f"{self.num_free_swa} SWA slots")
-        pages = [self.free_pages.pop() for _ in range(n)]
-        for p in pages:
-            assert self.page_ref[p] == 0, f"page {p} handed out while referenced"
-            self.page_ref[p] = 1
-        self.counters["pages_taken"] += n
-        if with_swa:
-            self.attach_swa(pages)
-        return pages
-
-    def ref_pages(self, pages) -> None:
-        for p in pages:
-            assert self.page_ref[p] > 0, f"page {p} referenced while free"
-            self.page_ref[p] += 1
-
-    def unref_pages(self, pages) -> None:
-        """Drops one reference; a page whose count reaches zero returns to the free list with its SWA slot."""
-        freed = []
-        for p in pages:
-            assert self.page_ref[p] > 0, f"double free of page {p}"
-            self.page_ref[p] -= 1
-            if self.page_ref[p] == 0:
-                freed.append(p)
-        if freed:
-            for p in freed:
-                self.swa_pins[p] = 0
-                self._tree_pinned.pop(p, None)
-            self.release_swa(freed)
-            self.free_pages.extend(freed)
-            self.counters["pages_released"] += len(freed)
-
-    # ------------------------------------------------------------------ SWA slots
     def reclaim_swa(self, n: int) -> int:
         """Takes the window slots of up to n unpinned pages back, least recently unpinned first."""
         victims = []
@@ -284,7 +243,6 @@ class DSV4KVPool:
         return v
 
     def assert_no_leak(self) -> None:
-        assert len(self.free_pages) == self.sizes.num_pages, (len(self.free_pages), self.sizes.num_pages)
+        super().assert_no_leak()
         assert len(self.free_swa) == self.sizes.num_swa_slots, (len(self.free_swa), self.sizes.num_swa_slots)
-        assert all(r == 0 for r in self.page_ref[:-1])
         assert all(s == -1 for s in self._swa_map_host[:-1])

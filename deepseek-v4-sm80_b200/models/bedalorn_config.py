@@ -1,0 +1,149 @@
+"""Configuration of the Bedalorn design: a list of layers, each with its own mixer (latent attention or recurrent time
+mixing) and feed-forward (dense, mixture of experts, or none), and an optional range of layers that runs several times
+with the same weights."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Any, Dict, List, Optional, Tuple
+
+ARCHITECTURE = "Bedalorn"
+
+
+@dataclass(frozen=True)
+class LatentAttentionSpec:
+    heads: int
+    dim: int          # query / key dimensions per head
+    vdim: int         # value dimensions per head
+    kv_rank: int
+    scale: float
+
+
+@dataclass(frozen=True)
+class WKVSpec:
+    heads: int
+    dim: int
+
+
+@dataclass(frozen=True)
+class DenseSpec:
+    ff: int
+
+
+@dataclass(frozen=True)
+class ExpertsSpec:
+    ff: int
+    experts: int
+    top: int
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: Any
+    ff: Any           # DenseSpec, ExpertsSpec or None
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class LayerRun:
+    """One pass of one layer.  ``enters``: the number of the loop pass that begins right before it, or None."""
+
+    layer: int
+    enters: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class BedalornConfig:
+    layers: Tuple[LayerSpec, ...]
+    hidden_size: int
+    vocab_size: int
+    norm_eps: float
+    logit_scale: float
+    loop: Optional[LoopSpec] = None
+    max_position: int = 1 << 20      # positions enter no computation: a limit of the page table, not of the design
+    eos_token_id: int = -1           # none unless the configuration names one
+    bos_token_id: int = -1
+    architectures: tuple = (ARCHITECTURE,)
+    model_type: str = "bedalorn"
+    window_size: int = 0
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def runs(self) -> List[LayerRun]:
+        """The layer runs of one forward, in order."""
+        n, lp = len(self.layers), self.loop
+        if lp is None:
+            return [LayerRun(i) for i in range(n)]
+        out = [LayerRun(i) for i in range(lp.start)]
+        for t in range(lp.times):
+            out += [LayerRun(i, t if i == lp.start else None) for i in range(lp.start, lp.stop)]
+        return out + [LayerRun(i) for i in range(lp.stop, n)]
+
+    def run_stores(self) -> list:
+        """What every run keeps between forwards (kvcache/latent_pool.py)."""
+        out = []
+        for r in self.runs:
+            m = self.layers[r.layer].mixer
+            out.append(("latent", m.kv_rank) if isinstance(m, LatentAttentionSpec) else ("state", m.heads, m.dim))
+        return out
+
+    # ------------------------------------------------------------------ config.json
+    @staticmethod
+    def from_dict(raw: Dict[str, Any]) -> "BedalornConfig":
+        if raw.get("architecture") != ARCHITECTURE:
+            raise ValueError(f"architecture {raw.get('architecture')!r} is not {ARCHITECTURE}")
+        layers = tuple(_layer(i, e) for i, e in enumerate(raw["layers"]))
+        loop = raw.get("loop")
+        if loop:
+            loop = LoopSpec(int(loop["start"]), int(loop["stop"]), int(loop["times"]))
+            if not (0 <= loop.start < loop.stop <= len(layers) and loop.times >= 1):
+                raise ValueError(f"loop {loop} does not fit {len(layers)} layers")
+        return BedalornConfig(
+            layers=layers, hidden_size=int(raw["width"]), vocab_size=int(raw["vocab"]),
+            norm_eps=float(raw["norm"]["eps"]), logit_scale=float(raw["logit_scale"]), loop=loop or None,
+            max_position=int(raw.get("max_position_embeddings") or 1 << 20),
+            eos_token_id=int(raw["eos_token_id"]) if raw.get("eos_token_id") is not None else -1,
+            bos_token_id=int(raw["bos_token_id"]) if raw.get("bos_token_id") is not None else -1)
+
+    def to_dict(self) -> Dict[str, Any]:
+        """The inverse of from_dict."""
+        def mlp(f):
+            if f is None:
+                return None
+            if isinstance(f, DenseSpec):
+                return {"kind": "dense", "ff": f.ff}
+            return {"kind": "moe", "expert": {"ff": f.ff}, "router": {"experts": f.experts, "top": f.top}}
+
+        def layer(s):
+            latent = isinstance(s.mixer, LatentAttentionSpec)
+            return {"type": "latent_attention" if latent else "wkv", "mixer": dict(vars(s.mixer)), "mlp": mlp(s.ff)}
+
+        return {"architecture": ARCHITECTURE, "layers": [layer(s) for s in self.layers], "width": self.hidden_size,
+                "vocab": self.vocab_size, "norm": {"eps": self.norm_eps}, "logit_scale": self.logit_scale,
+                "loop": dict(vars(self.loop)) if self.loop else None, "max_position_embeddings": self.max_position}
+
+
+def _layer(i: int, e: Dict[str, Any]) -> LayerSpec:
+    m, kind, f = e["mixer"], e["type"], e.get("mlp")
+    if kind == "latent_attention":
+        mixer = LatentAttentionSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["kv_rank"]), float(m["scale"]))
+    elif kind == "wkv":
+        mixer = WKVSpec(int(m["heads"]), int(m["dim"]))
+    else:
+        raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+    if f is None:
+        return LayerSpec(mixer, None)
+    if f["kind"] == "dense":
+        return LayerSpec(mixer, DenseSpec(int(f["ff"])))
+    if f["kind"] == "moe":
+        r = f["router"]
+        return LayerSpec(mixer, ExpertsSpec(int(f["expert"]["ff"]), int(r["experts"]), int(r["top"])))
+    raise ValueError(f"layer {i}: unknown feed-forward {f['kind']!r}")

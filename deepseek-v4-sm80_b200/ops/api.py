@@ -14,6 +14,8 @@ from . import ref
 gemm_bf16 = _gemm.gemm_bf16
 gemm_fp8 = _gemm.gemm_fp8
 gemm_bf16_grouped = _gemm.gemm_bf16_grouped
+linear = _gemm.linear
+grouped_linear = _gemm.grouped_linear
 
 
 def _cu():
@@ -255,6 +257,65 @@ def moe_experts(y, idx, w, w13, s13, w2, s2, limit, expert_base: int = 0):
     local = idx - expert_base
     local = torch.where((local >= 0) & (local < e_local) & (idx >= 0), local, torch.full_like(local, -1))
     return ref.moe_experts(y, local, w, w13, s13, w2, s2, limit)
+
+
+# --------------------------------------------------------------------------- fp32 residual stream, experts in bf16
+def _layers(t):
+    """The bodies of the operators below: kernels for CUDA tensors, plain PyTorch for CPU tensors."""
+    from . import cuda_layers, ref_layers
+
+    return cuda_layers if t.is_cuda else ref_layers
+
+
+def embed_residual(ids, weight, dtype, feedback=None, slots=None, want_act: bool = False):
+    """(x fp32 [T, D], the same rows as activations of ``dtype`` or None); feedback / slots as in :func:`embed`."""
+    return _layers(ids).embed_residual(ids, weight, dtype, feedback, slots, want_act)
+
+
+def residual_norm(x, gain, eps: float, dtype, mul: float = 1.0, rows=None, add=None, add2=None, vec=None, experts=None,
+                  cast: bool = False):
+    """Adds whatever is given to the fp32 stream x (in place): ``add`` / ``add2`` [T, D] fp32, ``vec`` [D] fp32,
+    ``experts`` = (expert rows [T*k, D], weights [T, k], ids [T, k]).  Then returns x / rms(x) * gain * mul as
+    activations; with gain None nothing is normed and the sum itself is returned if ``cast`` is set.  ``rows``: the rows
+    wanted (nothing is added then)."""
+    return _layers(x).residual_norm(x, gain, eps, dtype, mul, rows, add, add2, vec, experts, cast)
+
+
+def route_topk(h, weight, bias, top: int, num_valid=None):
+    """Router of a softmax-over-the-selected mixture: logits z = h W^T + b in fp32, the ``top`` largest (lower id on
+    ties) and the softmax over them.  Rows >= num_valid get id -1."""
+    return _layers(h).route_topk(h, weight, bias, top, num_valid)
+
+
+def gated_experts(h, idx, wts, w13, w2):
+    """silu(gate) * up experts: w13 [E, 2, F, D] (gate, up), w2 [E, D, F], bf16.  Returns the chosen experts' outputs
+    [T*k, D], not weighted yet (``residual_norm`` adds them up)."""
+    return _layers(h).gated_experts(h, idx, wts, w13, w2)
+
+
+# --------------------------------------------------------------------------- latent attention, recurrent mixing
+def latent_store(x, gain, eps: float, cache, fb):
+    """cache[out_loc[t]] = x[t] / rms(x[t]) * gain (x may be a column slice)."""
+    return _layers(x).latent_store(x, gain, eps, cache, fb)
+
+
+def latent_attention(q, cache, fb, scale: float):
+    """Causal attention of every (token, head) row over its request's cached latents, which are keys and values alike:
+    q [T, H, R] (key up-projection absorbed) -> [T, H, R]."""
+    return _layers(q).latent_attention(q, cache, fb, scale)
+
+
+def shift_mix(x, gain, eps: float, mu, prev, tail, fb, dtype):
+    """Norm and token shift: h = x / rms(x) * gain, h' = the previous token's h; returns [T, n*D], mix m being
+    h + (h' - h) mu[m].  prev [slots+1, D]: every slot's last h, read by the first row of a portion.  tail: scratch of
+    the same shape (``wkv`` moves a portion's last row from there to prev)."""
+    return _layers(x).shift_mix(x, gain, eps, mu, prev, tail, fb, dtype)
+
+
+def wkv(p, a, w0, u, gain, state, prev, tail, fb, heads: int, eps: float):
+    """Recurrence with decay exp(-exp(a + w0)), bonus u, per-head norm, gain and silu gate (csrc/wkv.cu).  p [T, 4*H*d]:
+    r | k | v | g; a fp32 [T, H*d]; state fp32 [slots+1, H, d, d] is advanced.  Returns [T, H*d]."""
+    return _layers(p).wkv(p, a, w0, u, gain, state, prev, tail, fb, heads, eps)
 
 
 # --------------------------------------------------------------------------- sampling

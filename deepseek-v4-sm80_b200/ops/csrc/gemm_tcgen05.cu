@@ -28,6 +28,7 @@
 //   * fused all-reduce: the epilogue publishes the partial tile to the rank's symmetric buffer and reduces the peers'
 //     tiles over NVLink (comm.cuh).
 #include "comm.cuh"
+#include "vec.cuh"
 
 namespace {
 
@@ -71,6 +72,7 @@ struct GemmArgs {
   int sp_mode;
   int* sp_counters;          // [row blocks], zero between launches (sp_mode 2)
   SpCtx sp;
+  int act;                   // epilogue activation (GemmAct), applied to the complete sum before it is added or stored
 };
 
 __device__ __forceinline__ void store_row_chunk(__nv_bfloat16* dst, const float* v, int ncols_valid) {
@@ -427,6 +429,10 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       }
       write_out = false;
     }
+    if (write_out && g.act) {
+#pragma unroll
+      for (int j = 0; j < BN; ++j) acc[j] = gemm_act(acc[j], g.act);
+    }
     if (write_out && grow < M) {
 #pragma unroll
       for (int c = 0; c < BN / 32; ++c) {
@@ -500,6 +506,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
 #pragma unroll
           for (int j = 0; j < 4; ++j)
             if (col + j < N) {
+              if (g.act) v4[j] = gemm_act(v4[j], g.act);
               if (g.accumulate_out) v4[j] += (float)dst[j];
               dst[j] = (OutT)v4[j];
             }
@@ -527,6 +534,7 @@ struct LaunchOpts {
   int sp_mode = 0;
   const SpCtx* sp = nullptr;
   int* sp_counters = nullptr;
+  int act = 0;
 };
 
 int g_weight_prefetch = 0;  // set by dsv4_gemm_set_weight_prefetch
@@ -559,7 +567,7 @@ int launch_gemm(const void* x, const void* w, OutT* out, int M, int N, int K, in
   }
   GemmArgs g{M, N, K, ldo, sa, sb, o.sb_ld ? o.sb_ld : (K + 127) / 128, accumulate_out, o.a_col_pb, o.b_row_pb,
              o.out_col_pb, o.splits, o.ws, o.counters, o.deposit_only, g_weight_prefetch, o.cluster, o.partial_stride,
-             o.sp_mode, o.sp_counters, o.sp ? *o.sp : SpCtx{}};
+             o.sp_mode, o.sp_counters, o.sp ? *o.sp : SpCtx{}, o.act};
   if (o.sp_mode && (!o.sp || o.sp->rows_per_rank % kBM || o.batches != 1)) return 106;
   if (o.sp_mode >= 2 && (o.splits != 1 || !o.sp_counters)) return 107;
   if (o.cluster) {
@@ -616,15 +624,17 @@ DSV4_API long long dsv4_gemm_splitk_ws_elems(int M, int N, int bn, int batches, 
 // out dtype: 0 = bf16, 1 = fp32.  ld* are row strides in elements.  bn = 0 picks the tile width.
 // batches > 1: batch b uses A columns [b*K, (b+1)*K) of x (ldx covers all batches), W rows [b*N, (b+1)*N) and output
 // columns [b*N, (b+1)*N).  splits > 1 needs ws (dsv4_gemm_splitk_ws_elems floats) and counters (>= tiles ints, zero).
+// act: epilogue activation (GemmAct in vec.cuh).
 DSV4_API int dsv4_gemm_bf16(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int ldw, int ldo,
                             int out_fp32, int accumulate_out, int bn, int batches, int splits, float* ws, int* counters,
-                            cudaStream_t stream) {
+                            int act, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if ((K % 8) || (ldx % 8) || (ldw % 8)) return 110;
   LaunchOpts o;
   o.batches = batches < 1 ? 1 : batches;
   o.splits = splits < 1 ? 1 : splits;
   o.ws = ws, o.counters = counters;
+  o.act = act;
   if (o.batches > 1) o.a_col_pb = K, o.b_row_pb = N, o.out_col_pb = N, o.a_cols = K * o.batches, o.b_rows = N * o.batches;
   if (o.splits > 1 && bn == 0) return 116;
   if (o.splits > 1 && (!ws || !counters)) o.cluster = 1;  // no workspace given: reduce inside a thread-block cluster

@@ -1,0 +1,495 @@
+// Latent attention without positions over a paged cache of latents: all heads of a token read the same row c_j (K = V =
+// c_j, `rank` values), because the per-head up-projections of keys and values are absorbed into the query and into the
+// output:  score = (W_uk^T q) . c_j * scale,   o_lat = sum_j softmax_j c_j,   o = W_uv o_lat.
+//
+// q and o are [T][heads][rank].  The (token, head) rows of a request are consecutive, and all of them see a prefix of the
+// same keys, so a CTA takes M = 16 .. 64 consecutive rows of one request -- heads of one token in decode, several tokens
+// in prefill -- and streams the request's latents once for all of them.  Position i sees every j <= i.
+//   S phase : 8 warps share the M x 64 score tile (mma.sync m16n8k16, bf16 in, fp32 accumulate)
+//   softmax : online (max, sum) per row in fp32, probabilities to shared memory as bf16
+//   PV phase: warp w owns rank / 8 output columns of all M rows in registers
+// Latent rows are fetched with cp.async into 128B-swizzled shared memory, double buffered.  grid.y splits the keys of a
+// row tile when the row tiles alone leave SMs idle; latent_merge_kernel adds the partial results in split order.
+//
+// latent_attn_row_kernel computes the same with one warp per row on the CUDA cores, in fp32 throughout: models served in
+// 32-bit floats, and ranks the tensor-core kernel does not take.
+#include "vec.cuh"
+
+namespace {
+
+struct LatArgs {
+  const int* slots;
+  const int* pos;
+  const int* page_table;
+  int ld_pt;
+  const int* seg_off;    // [nseg + 1] row ranges of the requests, or null: every row is a request's only one
+  int nseg;
+  const int* num_valid;  // rows (tokens) >= *num_valid are padding, or null
+  int rows;              // tokens
+  int heads, rank;
+  float scale;
+  int nsplit;
+  float* part_acc;       // [T * heads][nsplit][rank]
+  float* part_ml;        // [T * heads][nsplit][2]
+};
+
+// ------------------------------------------------------------------ latent norm + store
+// cache[out_loc[t]] = x[t] / rms(x[t]) * gain.  One warp per token.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__ x, int ldx,
+                                                           const float* __restrict__ gain, float eps,
+                                                           T* __restrict__ cache, const int* __restrict__ out_loc,
+                                                           int rows, int rank) {
+  pdl_entry();
+  const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= rows) return;
+  const T* r = x + (size_t)t * ldx;
+  float ss = 0.f;
+  for (int i = lane; i < rank; i += 32) {
+    const float v = ld_f(r + i);
+    ss += v * v;
+  }
+  const float sc = 1.f / sqrtf(warp_sum(ss) / rank + eps);
+  const int loc = out_loc[t];
+  if (loc < 0) return;
+  for (int i = lane; i < rank; i += 32) st_f(cache + (size_t)loc * rank + i, ld_f(r + i) * sc * gain[i]);
+}
+
+// ------------------------------------------------------------------ row tiles
+// Which M consecutive (token, head) rows tile `b` covers: rows [row0, row1) of the request whose last token is t_last.
+template <int M>
+__device__ __forceinline__ bool find_tile(const LatArgs& a, int b, int& row0, int& row1) {
+  const int lane = threadIdx.x & 31;
+  if (!a.seg_off) {
+    const int tpt = (a.heads + M - 1) / M;
+    const int t = b / tpt;
+    if (t >= a.rows) return false;
+    row0 = t * a.heads + (b % tpt) * M;
+    row1 = min(row0 + M, (t + 1) * a.heads);
+    return true;
+  }
+  int base = 0;
+  for (int s0 = 0; s0 < a.nseg; s0 += 32) {  // every warp does the same prefix sum over the requests' tile counts
+    const int s = s0 + lane;
+    int lo = 0, hi = 0;
+    if (s < a.nseg) lo = a.seg_off[s] * a.heads, hi = a.seg_off[s + 1] * a.heads;
+    const int cnt = (hi - lo + M - 1) / M;
+    int inc = cnt;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, inc, o);
+      if (lane >= o) inc += v;
+    }
+    const unsigned in = __ballot_sync(0xffffffffu, b < base + inc);
+    if (in) {
+      const int w = __ffs(in) - 1;
+      const int first = __shfl_sync(0xffffffffu, base + inc - cnt, w);
+      const int rlo = __shfl_sync(0xffffffffu, lo, w), rhi = __shfl_sync(0xffffffffu, hi, w);
+      row0 = rlo + (b - first) * M;
+      row1 = min(row0 + M, rhi);
+      return true;
+    }
+    base += __shfl_sync(0xffffffffu, inc, 31);
+  }
+  return false;
+}
+
+// ------------------------------------------------------------------ tensor-core kernel
+__device__ __forceinline__ void cpa16_zfill(void* smem, const void* g, bool valid) {
+  const int sz = valid ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem)), "l"(g), "r"(sz) : "memory");
+}
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// 16-byte chunk c of row r sits at chunk (c ^ (r & 7)) within its group of eight
+__device__ __forceinline__ int swz(int r, int c) { return (c & ~7) | ((c ^ r) & 7); }
+
+constexpr int kKT = 64;   // keys per tile
+constexpr int kSP = kKT + 4;  // floats per score row
+
+template <int RP, int MT>
+struct LatCfg {
+  static constexpr int M = MT * 16;
+  static constexpr int RG = MT == 4 ? 2 : 1;       // warp row groups of the S phase
+  static constexpr int WM = MT / RG;               // m16 tiles per warp
+  static constexpr int KG = 8 / RG;                // key groups
+  static constexpr int WN = kKT / KG / 8;          // n8 tiles per warp
+  static constexpr int DW = RP / 8;                // output columns per warp
+  static constexpr int NT = DW / 8;
+  static constexpr int SMEM = M * RP * 2 + 2 * kKT * RP * 2 + M * kSP * 4 + M * kKT * 2 + 4 * M * 4;
+};
+
+template <int RP, int MT>
+__global__ void __launch_bounds__(256) latent_attn_kernel(const __nv_bfloat16* __restrict__ q,
+                                                          const __nv_bfloat16* __restrict__ cache,
+                                                          __nv_bfloat16* __restrict__ o, const LatArgs a) {
+  pdl_entry();
+  using C = LatCfg<RP, MT>;
+  constexpr int M = C::M, WM = C::WM, WN = C::WN, NT = C::NT;
+  extern __shared__ __align__(128) uint8_t lat_smem[];
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(lat_smem);  // [M][RP] swizzled
+  __nv_bfloat16* kv = qs + M * RP;                                 // [2][kKT][RP] swizzled
+  float* ss = reinterpret_cast<float*>(kv + 2 * kKT * RP);         // [M][kSP]
+  __nv_bfloat16* pb = reinterpret_cast<__nv_bfloat16*>(ss + M * kSP);  // [M][kKT] swizzled
+  float* ms = reinterpret_cast<float*>(pb + M * kKT);
+  float* ls = ms + M;
+  float* alpha = ls + M;
+  int* see = reinterpret_cast<int*>(alpha + M);                    // keys the row sees
+
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int split = blockIdx.y, R = a.rank, rch = R / 8;
+  int row0, row1;
+  if (!find_tile<M>(a, blockIdx.x, row0, row1)) return;
+  if (a.num_valid && row0 / a.heads >= *a.num_valid) return;
+  const int t_last = (row1 - 1) / a.heads;
+  const int keys = a.pos[t_last] + 1;   // of the tile's last token, the one that sees most
+  const int* pt = a.page_table + (size_t)a.slots[t_last] * a.ld_pt;
+
+  const int ktiles = (keys + kKT - 1) / kKT;
+  const int per = (ktiles + a.nsplit - 1) / a.nsplit;
+  const int kt0 = split * per, kt1 = min(kt0 + per, ktiles);
+  if (kt0 >= kt1) {  // nothing for this split: an empty partial
+    if (a.nsplit > 1)
+      for (int r = row0 + tid; r < row1; r += 256) {
+        float* ml = a.part_ml + ((size_t)r * a.nsplit + split) * 2;
+        ml[0] = -1e30f, ml[1] = 0.f;
+      }
+    return;
+  }
+
+  for (int i = tid; i < M * (RP / 8); i += 256) {
+    const int r = i / (RP / 8), c = i % (RP / 8);
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (row0 + r < row1 && c < rch) v = reinterpret_cast<const uint4*>(q + (size_t)(row0 + r) * R)[c];
+    reinterpret_cast<uint4*>(qs + r * RP)[swz(r, c)] = v;
+  }
+  if (tid < M) {
+    ms[tid] = -1e30f, ls[tid] = 0.f;
+    see[tid] = row0 + tid < row1 ? a.pos[(row0 + tid) / a.heads] + 1 : 0;
+  }
+
+  // four threads fetch one latent row
+  const int fk = tid >> 2, fp = tid & 3;
+  auto key_loc = [&](int kt) {
+    const int key = kt * kKT + fk;
+    return (kt < kt1 && key < keys) ? pt[key] : -1;
+  };
+  auto issue = [&](int loc, int buf) {
+    __nv_bfloat16* dst = kv + ((size_t)buf * kKT + fk) * RP;
+    const __nv_bfloat16* src = cache + (size_t)max(loc, 0) * R;
+#pragma unroll
+    for (int c = fp; c < RP / 8; c += 4) {
+      const bool in = loc >= 0 && c < rch;
+      cpa16_zfill(dst + swz(fk, c) * 8, in ? src + c * 8 : cache, in);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+
+  float acc[MT][NT][4];
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < NT; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
+
+  issue(key_loc(kt0), kt0 & 1);
+  int loc_next = key_loc(kt0 + 1);
+  const float sc2 = a.scale * 1.4426950408889634f;  // scores in powers of two
+  const int rg = warp / C::KG, kg = warp % C::KG;
+  for (int kt = kt0; kt < kt1; ++kt) {
+    const int buf = kt & 1;
+    if (kt + 1 < kt1) {
+      issue(loc_next, buf ^ 1);
+      loc_next = key_loc(kt + 2);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const __nv_bfloat16* kb = kv + (size_t)buf * kKT * RP;
+    // ---- scores: rows [rg * WM * 16, +WM * 16) x keys [kg * WN * 8, +WN * 8)
+    {
+      float s[2][WM][WN][4] = {};
+#pragma unroll 2
+      for (int ks = 0; ks < RP / 16; ks += 2) {
+        uint32_t bf[WN][4];
+#pragma unroll
+        for (int j = 0; j < WN; ++j) {
+          const int br = (kg * WN + j) * 8 + (lane & 7);
+          ldsm4(bf[j], kb + br * RP + swz(br, ks * 2 + (lane >> 3)) * 8);
+        }
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int i = 0; i < WM; ++i) {
+            const int ar = (rg * WM + i) * 16 + (lane & 15);
+            uint32_t af[4];
+            ldsm4(af, qs + ar * RP + swz(ar, (ks + h) * 2 + (lane >> 4)) * 8);
+#pragma unroll
+            for (int j = 0; j < WN; ++j) mma16816(s[h][i][j], af, bf[j][2 * h], bf[j][2 * h + 1]);
+          }
+      }
+#pragma unroll
+      for (int i = 0; i < WM; ++i)
+#pragma unroll
+        for (int j = 0; j < WN; ++j) {
+          const int r = (rg * WM + i) * 16 + (lane >> 2), c = (kg * WN + j) * 8 + (lane & 3) * 2;
+          *reinterpret_cast<float2*>(ss + r * kSP + c) =
+              make_float2((s[0][i][j][0] + s[1][i][j][0]) * sc2, (s[0][i][j][1] + s[1][i][j][1]) * sc2);
+          *reinterpret_cast<float2*>(ss + (r + 8) * kSP + c) =
+              make_float2((s[0][i][j][2] + s[1][i][j][2]) * sc2, (s[0][i][j][3] + s[1][i][j][3]) * sc2);
+        }
+    }
+    __syncthreads();
+    // ---- online softmax
+    {
+      constexpr int TPR = 256 / M, PER = kKT / TPR;  // threads per row, keys per thread (4, 8 or 16)
+      const int r = tid / TPR, seg = tid % TPR;
+      const int lim = see[r] - kt * kKT - seg * PER;
+      float v[PER];
+      float mx = -1e30f;
+#pragma unroll
+      for (int i = 0; i < PER; i += 4) {
+        const float4 f = *reinterpret_cast<const float4*>(ss + r * kSP + seg * PER + i);
+        v[i] = f.x, v[i + 1] = f.y, v[i + 2] = f.z, v[i + 3] = f.w;
+      }
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        v[i] = i < lim ? v[i] : -INFINITY;
+        mx = fmaxf(mx, v[i]);
+      }
+#pragma unroll
+      for (int off = TPR / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+      const float m_old = ms[r], m_new = fmaxf(m_old, mx);
+      float sum = 0.f;
+      __align__(16) __nv_bfloat16 e[PER];
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        e[i] = f2bf(exp2f(v[i] - m_new));
+        sum += bf2f(e[i]);   // the weights as they enter the product add up to what they are divided by
+      }
+#pragma unroll
+      for (int off = TPR / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+      if constexpr (PER >= 8) {
+#pragma unroll
+        for (int i = 0; i < PER; i += 8)
+          reinterpret_cast<uint4*>(pb + r * kKT)[swz(r, (seg * PER + i) / 8)] = *reinterpret_cast<uint4*>(e + i);
+      } else {
+        *reinterpret_cast<uint2*>(pb + r * kKT + swz(r, seg / 2) * 8 + (seg & 1) * 4) = *reinterpret_cast<uint2*>(e);
+      }
+      __syncwarp();
+      if (seg == 0) {
+        const float al = exp2f(m_old - m_new);
+        alpha[r] = al;
+        ms[r] = m_new;
+        ls[r] = ls[r] * al + sum;
+      }
+    }
+    __syncthreads();
+    // ---- o += P C: all rows, output columns [warp * DW, +DW)
+    {
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        const float a0 = alpha[i * 16 + (lane >> 2)], a1 = alpha[i * 16 + (lane >> 2) + 8];
+#pragma unroll
+        for (int j = 0; j < NT; ++j) acc[i][j][0] *= a0, acc[i][j][1] *= a0, acc[i][j][2] *= a1, acc[i][j][3] *= a1;
+      }
+#pragma unroll
+      for (int kk = 0; kk < kKT / 16; ++kk) {
+        uint32_t pf[MT][4];
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+          const int pr = i * 16 + (lane & 15);
+          ldsm4(pf[i], pb + pr * kKT + swz(pr, kk * 2 + (lane >> 4)) * 8);
+        }
+        const int vr = kk * 16 + (lane & 15);
+#pragma unroll
+        for (int j = 0; j < NT; j += 2) {
+          uint32_t vf[4];
+          ldsm4_t(vf, kb + vr * RP + swz(vr, warp * (C::DW / 8) + j + (lane >> 4)) * 8);
+#pragma unroll
+          for (int i = 0; i < MT; ++i) {
+            mma16816(acc[i][j], pf[i], vf[0], vf[1]);
+            mma16816(acc[i][j + 1], pf[i], vf[2], vf[3]);
+          }
+        }
+      }
+    }
+    __syncthreads();
+  }
+  // ---- result or partial
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int r = i * 16 + (lane >> 2) + half * 8, row = row0 + r;
+      if (row >= row1) continue;
+      const float inv = 1.f / ls[r];
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const int c = warp * C::DW + j * 8 + (lane & 3) * 2;
+        if (c >= R) continue;
+        const float x = acc[i][j][half * 2], y = acc[i][j][half * 2 + 1];
+        if (a.nsplit > 1)
+          *reinterpret_cast<float2*>(a.part_acc + ((size_t)row * a.nsplit + split) * R + c) = make_float2(x, y);
+        else
+          *reinterpret_cast<__nv_bfloat162*>(o + (size_t)row * R + c) = __floats2bfloat162_rn(x * inv, y * inv);
+      }
+    }
+  if (a.nsplit > 1 && tid < M && row0 + tid < row1) {
+    float* ml = a.part_ml + ((size_t)(row0 + tid) * a.nsplit + split) * 2;
+    ml[0] = ms[tid], ml[1] = ls[tid];
+  }
+}
+
+// o[row] = sum_s acc_s 2^(m_s - M) / sum_s l_s 2^(m_s - M)
+__global__ void __launch_bounds__(128) latent_merge_kernel(__nv_bfloat16* __restrict__ o, const LatArgs a) {
+  pdl_entry();
+  const int row = blockIdx.x, n = a.nsplit;
+  if (a.num_valid && row / a.heads >= *a.num_valid) return;
+  const float* ml = a.part_ml + (size_t)row * n * 2;
+  float mx = -1e30f, l = 0.f;
+  for (int s = 0; s < n; ++s) mx = fmaxf(mx, ml[s * 2]);
+  for (int s = 0; s < n; ++s) l += ml[s * 2 + 1] * exp2f(ml[s * 2] - mx);
+  const float inv = 1.f / l;
+  for (int c = threadIdx.x; c < a.rank; c += 128) {
+    float v = 0.f;
+    for (int s = 0; s < n; ++s)
+      if (ml[s * 2 + 1] > 0.f) v = fmaf(a.part_acc[((size_t)row * n + s) * a.rank + c], exp2f(ml[s * 2] - mx), v);
+    o[(size_t)row * a.rank + c] = f2bf(v * inv);
+  }
+}
+
+// ------------------------------------------------------------------ one warp per row, fp32 arithmetic
+template <typename T, int NI>
+__global__ void __launch_bounds__(128) latent_attn_row_kernel(const T* __restrict__ q, const T* __restrict__ cache,
+                                                              T* __restrict__ o, const LatArgs a) {
+  pdl_entry();
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, R = a.rank;
+  if (row >= a.rows * a.heads) return;
+  const int t = row / a.heads;
+  if (a.num_valid && t >= *a.num_valid) return;
+  const int keys = a.pos[t] + 1;
+  const int* pt = a.page_table + (size_t)a.slots[t] * a.ld_pt;
+  float qv[NI], acc[NI];
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int c = i * 32 + lane;
+    qv[i] = c < R ? ld_f(q + (size_t)row * R + c) * a.scale : 0.f;
+    acc[i] = 0.f;
+  }
+  float m = -1e30f, l = 0.f;
+  for (int k0 = 0; k0 < keys; k0 += 32) {
+    const int mine = k0 + lane < keys ? pt[k0 + lane] : 0;
+    const int n = min(32, keys - k0);
+    for (int k = 0; k < n; ++k) {
+      const T* c = cache + (size_t)__shfl_sync(0xffffffffu, mine, k) * R;
+      float cv[NI], s = 0.f;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        cv[i] = i * 32 + lane < R ? ld_f(c + i * 32 + lane) : 0.f;
+        s = fmaf(qv[i], cv[i], s);
+      }
+      s = warp_sum(s);
+      const float mn = fmaxf(m, s), al = expf(m - mn), p = expf(s - mn);
+      l = l * al + p;
+      m = mn;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) acc[i] = fmaf(p, cv[i], acc[i] * al);
+    }
+  }
+  const float inv = 1.f / l;
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int c = i * 32 + lane;
+    if (c < R) st_f(o + (size_t)row * R + c, acc[i] * inv);
+  }
+}
+
+template <int RP, int MT>
+int launch_lat(const void* q, const void* cache, void* o, const LatArgs& a, int tiles, cudaStream_t st) {
+  using C = LatCfg<RP, MT>;
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(latent_attn_kernel<RP, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM) !=
+        cudaSuccess)
+      return 631;
+    set = true;
+  }
+  dsv4_launch(latent_attn_kernel<RP, MT>, dim3(tiles, a.nsplit), 256, C::SMEM, st, (const __nv_bfloat16*)q,
+              (const __nv_bfloat16*)cache, (__nv_bfloat16*)o, a);
+  if (a.nsplit > 1)
+    dsv4_launch(latent_merge_kernel, a.rows * a.heads, 128, 0, st, (__nv_bfloat16*)o, a);
+  return (int)cudaGetLastError();
+}
+template <int RP>
+int dispatch_lat(int m, const void* q, const void* cache, void* o, const LatArgs& a, int tiles, cudaStream_t st) {
+  switch (m) {
+    case 16: return launch_lat<RP, 1>(q, cache, o, a, tiles, st);
+    case 32: return launch_lat<RP, 2>(q, cache, o, a, tiles, st);
+    case 64: return launch_lat<RP, 4>(q, cache, o, a, tiles, st);
+    default: return 632;
+  }
+}
+template <typename T>
+int launch_row(const void* q, const void* cache, void* o, const LatArgs& a, cudaStream_t st) {
+  const int grid = (a.rows * a.heads + 3) / 4;
+  const T *tq = (const T*)q, *tc = (const T*)cache;
+  if (a.rank <= 128)
+    dsv4_launch(latent_attn_row_kernel<T, 4>, grid, 128, 0, st, tq, tc, (T*)o, a);
+  else if (a.rank <= 256)
+    dsv4_launch(latent_attn_row_kernel<T, 8>, grid, 128, 0, st, tq, tc, (T*)o, a);
+  else if (a.rank <= 512)
+    dsv4_launch(latent_attn_row_kernel<T, 16>, grid, 128, 0, st, tq, tc, (T*)o, a);
+  else if (a.rank <= 1024)
+    dsv4_launch(latent_attn_row_kernel<T, 32>, grid, 128, 0, st, tq, tc, (T*)o, a);
+  else
+    return 633;
+  return (int)cudaGetLastError();
+}
+
+}  // namespace
+
+DSV4_API int dsv4_latent_store(const void* x, int ldx, const float* gain, float eps, void* cache, const int* out_loc,
+                               int rows, int rank, int fp32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const int grid = (rows + 3) / 4;
+  if (fp32)
+    dsv4_launch(latent_store_kernel<float>, grid, 128, 0, st, (const float*)x, ldx, gain, eps, (float*)cache, out_loc,
+                rows, rank);
+  else
+    dsv4_launch(latent_store_kernel<__nv_bfloat16>, grid, 128, 0, st, (const __nv_bfloat16*)x, ldx, gain, eps,
+                (__nv_bfloat16*)cache, out_loc, rows, rank);
+  return (int)cudaGetLastError();
+}
+
+// m: rows per CTA (16, 32 or 64; 0 = the one-warp-per-row kernel), tiles: row tiles of that height over all requests.
+// nsplit > 1 needs part_acc [T * heads, nsplit, rank] and part_ml [T * heads, nsplit, 2].
+DSV4_API int dsv4_latent_attention(const void* q, const void* cache, void* o, const int* slots, const int* pos,
+                                   const int* page_table, int ld_pt, const int* seg_off, int nseg,
+                                   const int* num_valid, int rows, int heads, int rank, float scale, int m, int tiles,
+                                   int nsplit, float* part_acc, float* part_ml, int fp32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (nsplit < 1 || nsplit > 65535 || (nsplit > 1 && (!part_acc || !part_ml))) return 634;
+  const LatArgs a{slots, pos, page_table, ld_pt, seg_off, nseg, num_valid, rows, heads, rank, scale, nsplit, part_acc, part_ml};
+  if (m == 0) return fp32 ? launch_row<float>(q, cache, o, a, st) : launch_row<__nv_bfloat16>(q, cache, o, a, st);
+  if (fp32 || rank % 8) return 635;
+  if (rank <= 128) return dispatch_lat<128>(m, q, cache, o, a, tiles, st);
+  if (rank <= 256) return dispatch_lat<256>(m, q, cache, o, a, tiles, st);
+  if (rank <= 384) return dispatch_lat<384>(m, q, cache, o, a, tiles, st);
+  if (rank <= 512) return dispatch_lat<512>(m, q, cache, o, a, tiles, st);
+  return 636;
+}

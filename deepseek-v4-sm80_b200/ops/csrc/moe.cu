@@ -33,6 +33,8 @@ struct PlanHeader {
 // ------------------------------------------------------------------ router post-processing
 // scores fp32 [n_part][T,E] (split-K partial products, summed here) -> p = sqrt(softplus) | sigmoid ; select top-k of p + bias (ties: lower id) or the hash
 // table row; w = p[idx] / (sum + 1e-8) * scaling.  Rows >= num_valid get (-1, 0).
+// scoring 3: the bias belongs to the logits, the k largest z = score + bias are selected and weighted with the softmax
+// over the selected logits only (p = e^(z - max z); the largest is always selected, so the sum is at least 1).
 __global__ void moe_topk_kernel(const float* __restrict__ scores, const float* __restrict__ bias,
                                 const int* __restrict__ tid2eid, const int* __restrict__ token_ids,
                                 const int* __restrict__ num_valid, int* __restrict__ idx, float* __restrict__ wts,
@@ -66,7 +68,14 @@ __global__ void moe_topk_kernel(const float* __restrict__ scores, const float* _
     }
   }
   float smax = -INFINITY;
-  if (scoring == 2) {
+  if (scoring == 3 && bias) {
+#pragma unroll
+    for (int i = 0; i < MAXPER; ++i) {
+      const int j = lane + i * 32;
+      if (i < per && j < e) sc[i] += bias[j];
+    }
+  }
+  if (scoring >= 2) {
 #pragma unroll
     for (int i = 0; i < MAXPER; ++i) {
       const int j = lane + i * 32;
@@ -93,6 +102,7 @@ __global__ void moe_topk_kernel(const float* __restrict__ scores, const float* _
         ssum += v;
       }
       p[i] = v;
+      if (scoring == 3) sel[i] = s;
     }
   }
   if (scoring == 2) {
@@ -103,7 +113,7 @@ __global__ void moe_topk_kernel(const float* __restrict__ scores, const float* _
 #pragma unroll
   for (int i = 0; i < MAXPER; ++i) {
     const int j = lane + i * 32;
-    if (i < per && j < e) sel[i] = p[i] + (bias ? bias[j] : 0.f);
+    if (scoring != 3 && i < per && j < e) sel[i] = p[i] + (bias ? bias[j] : 0.f);
   }
   float wsum = 0.f;
   float myw = 0.f;

@@ -1,0 +1,192 @@
+// The residual stream of models that keep it in 32-bit floats: embedding gather, and RMSNorm fused with whatever is
+// added to the stream right before it (a projection's output, a learned vector, the weighted outputs of the chosen
+// experts).  T is the activation type the next projection reads (bf16, or fp32 for models served in 32-bit).
+#include "vec.cuh"
+
+namespace {
+
+// x[t] = embed[id], also as activations (x0, may be null).  feedback as in embed_kernel: the token of row t is
+// feedback[slots[t]] and is written to ids[t].
+template <typename T>
+__global__ void __launch_bounds__(256) embed_residual_kernel(int* __restrict__ ids, const int* __restrict__ feedback,
+                                                             const int* __restrict__ slots,
+                                                             const __nv_bfloat16* __restrict__ w,
+                                                             float* __restrict__ x, T* __restrict__ x0, int d) {
+  pdl_entry();
+  const int t = blockIdx.x;
+  int id;
+  if (feedback) {
+    id = feedback[slots[t]];
+    if (threadIdx.x == 0) ids[t] = id;
+  } else {
+    id = ids[t];
+  }
+  const __nv_bfloat16* src = w + (size_t)id * d;
+  for (int i = threadIdx.x; i < d; i += blockDim.x) {
+    const float v = bf2f(src[i]);
+    x[(size_t)t * d + i] = v;
+    if (x0) st_f(x0 + (size_t)t * d + i, v);
+  }
+}
+
+struct NormArgs {
+  float* x;             // [rows, d] stream (row stride d), updated in place when something is added
+  const long long* rows_idx;  // not null: output row r is the norm of stream row rows_idx[r] (nothing is added then)
+  const float* add;     // [rows, d] or null
+  const float* add2;    // [rows, d] or null
+  const float* vec;     // [d] or null
+  const float* wts;     // [rows, topk]: weights of the expert rows below
+  const int* eidx;      // [rows, topk]: expert ids, negative = no expert ran for this place
+  int topk;             // 0: no expert rows
+  const float* gain;    // [d]; null: no norm, only the additions (out, if given, receives the sum as activations)
+  float eps, mul;       // out = x / rms(x) * gain * mul
+  int d;
+};
+
+// One CTA per row.  The row stays in registers between the two passes when it has at most 8 x 4 values per thread.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) residual_norm_kernel(const NormArgs a, const T* __restrict__ erows,
+                                                            T* __restrict__ out) {
+  pdl_entry();
+  __shared__ float sh[32];
+  const int r = blockIdx.x, d = a.d;
+  const size_t src = (size_t)(a.rows_idx ? a.rows_idx[r] : r) * d;
+  const bool adds = a.add || a.add2 || a.vec || a.topk > 0;
+  float ss = 0.f;
+  if constexpr (VEC) {
+    constexpr int NV = 8;
+    float4 keep[NV];
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int i = (n * 256 + threadIdx.x) * 4;
+      if (i >= d) continue;
+      float4 v = *reinterpret_cast<const float4*>(a.x + src + i);
+      if (adds) {
+        if (a.add) {
+          const float4 u = *reinterpret_cast<const float4*>(a.add + src + i);
+          v.x += u.x, v.y += u.y, v.z += u.z, v.w += u.w;
+        }
+        if (a.add2) {
+          const float4 u = *reinterpret_cast<const float4*>(a.add2 + src + i);
+          v.x += u.x, v.y += u.y, v.z += u.z, v.w += u.w;
+        }
+        if (a.vec) {
+          const float4 u = *reinterpret_cast<const float4*>(a.vec + i);
+          v.x += u.x, v.y += u.y, v.z += u.z, v.w += u.w;
+        }
+        if (a.topk > 0) {
+          float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+          for (int k = 0; k < a.topk; ++k) {
+            if (a.eidx[r * a.topk + k] < 0) continue;
+            const float w = a.wts[r * a.topk + k];
+            const float4 u = ld_f4(erows + ((size_t)r * a.topk + k) * d + i);
+            s.x += w * u.x, s.y += w * u.y, s.z += w * u.z, s.w += w * u.w;
+          }
+          v.x += s.x, v.y += s.y, v.z += s.z, v.w += s.w;
+        }
+        *reinterpret_cast<float4*>(a.x + src + i) = v;
+      }
+      keep[n] = v;
+      if (!a.gain && out) st_f4(out + (size_t)r * d + i, v);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    if (!a.gain) return;
+    ss = cta_sum(ss, sh);
+    const float sc = a.mul / sqrtf(ss / d + a.eps);
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int i = (n * 256 + threadIdx.x) * 4;
+      if (i >= d) continue;
+      const float4 g = *reinterpret_cast<const float4*>(a.gain + i);
+      st_f4(out + (size_t)r * d + i,
+            make_float4(keep[n].x * sc * g.x, keep[n].y * sc * g.y, keep[n].z * sc * g.z, keep[n].w * sc * g.w));
+    }
+  } else {
+    for (int i = threadIdx.x; i < d; i += 256) {
+      float v = a.x[src + i];
+      if (adds) {
+        if (a.add) v += a.add[src + i];
+        if (a.add2) v += a.add2[src + i];
+        if (a.vec) v += a.vec[i];
+        float s = 0.f;
+        for (int k = 0; k < a.topk; ++k)
+          if (a.eidx[r * a.topk + k] >= 0)
+            s += a.wts[r * a.topk + k] * ld_f(erows + ((size_t)r * a.topk + k) * d + i);
+        v += s;
+        a.x[src + i] = v;
+      }
+      if (!a.gain && out) st_f(out + (size_t)r * d + i, v);
+      ss += v * v;
+    }
+    if (!a.gain) return;
+    ss = cta_sum(ss, sh);
+    const float sc = a.mul / sqrtf(ss / d + a.eps);
+    for (int i = threadIdx.x; i < d; i += 256)  // each thread re-reads what it wrote itself
+      st_f(out + (size_t)r * d + i, a.x[src + i] * sc * a.gain[i]);
+  }
+}
+
+// silu(gate) * up: gu [rows, 2 f] (gate columns first) -> out [rows, f]
+template <typename T>
+__global__ void __launch_bounds__(256) silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, long long total,
+                                                       int f) {
+  pdl_entry();
+  const long long i = blockIdx.x * 256ll + threadIdx.x;
+  if (i >= total) return;
+  const long long r = i / f;
+  const int c = (int)(i % f);
+  const float g = ld_f(gu + r * 2 * f + c), u = ld_f(gu + r * 2 * f + f + c);
+  st_f(out + i, g / (1.f + expf(-g)) * u);
+}
+
+template <typename T>
+int launch_norm(const NormArgs& a, const void* erows, void* out, int rows, cudaStream_t st) {
+  const bool vec = a.d % 4 == 0 && a.d <= 8192;
+  if (vec)
+    dsv4_launch(residual_norm_kernel<T, true>, rows, 256, 0, st, a, (const T*)erows, (T*)out);
+  else
+    dsv4_launch(residual_norm_kernel<T, false>, rows, 256, 0, st, a, (const T*)erows, (T*)out);
+  return (int)cudaGetLastError();
+}
+
+}  // namespace
+
+// fp32: the activation type (0 = bf16, 1 = fp32).
+DSV4_API int dsv4_embed_residual(int* ids, const int* feedback, const int* slots, const void* w, float* x, void* x0,
+                                 int t, int d, int fp32, cudaStream_t st) {
+  if (t <= 0) return 0;
+  if (feedback && !slots) return 600;
+  if (fp32)
+    dsv4_launch(embed_residual_kernel<float>, t, 256, 0, st, ids, feedback, slots, (const __nv_bfloat16*)w, x,
+                (float*)x0, d);
+  else
+    dsv4_launch(embed_residual_kernel<__nv_bfloat16>, t, 256, 0, st, ids, feedback, slots, (const __nv_bfloat16*)w, x,
+                (__nv_bfloat16*)x0, d);
+  return (int)cudaGetLastError();
+}
+
+// x (+= add + add2 + vec + sum_k wts[k] * erows[k]);  out = x / rms(x) * gain * mul.  rows_idx (no additions then):
+// gathers the rows first.
+DSV4_API int dsv4_residual_norm(float* x, const long long* rows_idx, const float* add, const float* add2,
+                                const float* vec, const void* erows, const float* wts, const int* eidx, int topk,
+                                const float* gain, float eps, float mul, void* out, int rows, int d, int fp32,
+                                cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (rows_idx && (add || add2 || vec || topk)) return 601;
+  if (topk > 0 && (!erows || !wts || !eidx)) return 602;
+  if (gain && !out) return 603;
+  const NormArgs a{x, rows_idx, add, add2, vec, wts, eidx, topk, gain, eps, mul, d};
+  return fp32 ? launch_norm<float>(a, erows, out, rows, st) : launch_norm<__nv_bfloat16>(a, erows, out, rows, st);
+}
+
+DSV4_API int dsv4_silu_mul(const void* gu, void* out, int rows, int f, int fp32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  const long long total = (long long)rows * f;
+  const unsigned grid = (unsigned)((total + 255) / 256);
+  if (fp32)
+    dsv4_launch(silu_mul_kernel<float>, grid, 256, 0, st, (const float*)gu, (float*)out, total, f);
+  else
+    dsv4_launch(silu_mul_kernel<__nv_bfloat16>, grid, 256, 0, st, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, total,
+                f);
+  return (int)cudaGetLastError();
+}

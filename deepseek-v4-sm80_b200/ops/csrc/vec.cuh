@@ -1,0 +1,50 @@
+// Element access shared by the kernels that exist for bf16 and for fp32 activations.
+#pragma once
+#include "common.cuh"
+
+__device__ __forceinline__ float ld_f(const float* p) { return *p; }
+__device__ __forceinline__ float ld_f(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void st_f(float* p, float v) { *p = v; }
+__device__ __forceinline__ void st_f(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ float4 ld_f4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ld_f4(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void st_f4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void st_f4(__nv_bfloat16* p, const float4& v) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 u;
+  u.x = *reinterpret_cast<uint32_t*>(&a);
+  u.y = *reinterpret_cast<uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = u;
+}
+// sum over the CTA (blockDim.x a multiple of 32, at most 1024); sh: 32 floats
+__device__ __forceinline__ float cta_sum(float v, float* sh) {
+  v = warp_sum(v);
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = blockDim.x >> 5;
+  __syncthreads();
+  if (l == 0) sh[w] = v;
+  __syncthreads();
+  return warp_sum(l < nw ? sh[l] : 0.f);
+}
+
+// Epilogue activations of the projections (the numbers are part of the host interface).
+enum GemmAct : int { kActNone = 0, kActRelu2 = 1, kActTanh = 2 };
+__device__ __forceinline__ float gemm_act(float v, int act) {
+  if (act == kActRelu2) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+  }
+  return act == kActTanh ? tanhf(v) : v;
+}
+
+// First and last row of a request's rows in the batch: rows of a request stand together at consecutive positions.
+__device__ __forceinline__ bool seg_first(const int* slots, const int* pos, int t) {
+  return t == 0 || slots[t - 1] != slots[t] || pos[t - 1] + 1 != pos[t];
+}
+__device__ __forceinline__ bool seg_last(const int* slots, const int* pos, int t, int rows) {
+  return t + 1 >= rows || slots[t + 1] != slots[t] || pos[t + 1] != pos[t] + 1;
+}

@@ -109,13 +109,21 @@ def _ws(m, n, bn, batches, splits, device):
             _counters(device))
 
 
-def gemm_bf16(x, w, out=None, out_dtype=torch.bfloat16, accumulate=False, bn=0, splits=0):
-    """bf16 x bf16 -> bf16 / fp32 with fp32 accumulation."""
+# epilogue activations of the projections (csrc/vec.cuh: GemmAct), applied to the fp32 sum
+ACTS = {None: 0, "relu2": 1, "tanh": 2}
+
+
+def _act(y, act):
+    return y if act is None else y.clamp_min(0).square() if act == "relu2" else y.tanh()
+
+
+def gemm_bf16(x, w, out=None, out_dtype=torch.bfloat16, accumulate=False, bn=0, splits=0, act=None):
+    """bf16 x bf16 -> bf16 / fp32 with fp32 accumulation; act: activation of the sum, before it is added or stored."""
     x2 = _as2d(x)
     m, k = x2.shape
     n = w.shape[0]
     if not x.is_cuda:
-        y = (x2.float() @ w.float().t())
+        y = _act(x2.float() @ w.float().t(), act)
         if out is not None:
             y = y.reshape(out.shape)
             y = y + out.float() if accumulate else y
@@ -132,7 +140,46 @@ def gemm_bf16(x, w, out=None, out_dtype=torch.bfloat16, accumulate=False, bn=0, 
     ws, cnt = _ws(m, n, bn, 1, splits, x.device)
     nv.call("gemm_bf16", nv.ptr(x2), nv.ptr(w), nv.ptr(o2), I(m), I(n), I(k), I(x2.stride(0)), I(w.stride(0)),
             I(o2.stride(0)), I(1 if out.dtype == torch.float32 else 0), I(1 if accumulate else 0), I(bn), I(1),
-            I(splits), nv.ptr(ws), nv.ptr(cnt))
+            I(splits), nv.ptr(ws), nv.ptr(cnt), I(ACTS[act]))
+    return out
+
+
+def _tma_ok(x2, w, k: int) -> bool:
+    """bf16 operands whose rows all start on 16 bytes, as TMA wants them."""
+    return (x2.dtype == torch.bfloat16 and k % 8 == 0 and x2.stride(0) % 8 == 0 and w.stride(0) % 8 == 0
+            and x2.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
+
+
+def linear(x, w, out=None, out_dtype=None, accumulate=False, act=None):
+    """``x [T, K] @ w [N, K]^T`` for bf16 weights and bf16 or fp32 activations (rows may be strided).  bf16 runs on the
+    tensor cores; fp32 activations, and bf16 rows that TMA cannot fetch, on the fp32 kernel (csrc/gemm_simt.cu)."""
+    return grouped_linear(x, w, 1, out, out_dtype, accumulate, act)
+
+
+def grouped_linear(x, w, groups: int, out=None, out_dtype=None, accumulate=False, act=None):
+    """``groups`` projections side by side in one launch: x [T, G*K] (rows may be strided), w [G*N, K] -> [T, G*N],
+    group g reading its own K columns."""
+    t, k = x.shape[0], x.shape[1] // groups
+    n = w.shape[0] // groups
+    if out is None:
+        out = torch.empty(t, groups * n, dtype=out_dtype or x.dtype, device=x.device)
+    if not x.is_cuda:
+        y = torch.einsum("tgk,gnk->tgn", x.reshape(t, groups, k).float(), w.reshape(groups, n, k).float())
+        y = _act(y.reshape(t, groups * n), act)
+        out.copy_(y + out.float() if accumulate else y)
+        return out
+    assert w.dtype == torch.bfloat16 and w.stride(-1) == 1 and x.stride(-1) == 1 and out.stride(-1) == 1
+    f32 = I(1 if out.dtype == torch.float32 else 0)
+    if _tma_ok(x, w, k):
+        bn, splits = pick_tiling(t, n, (k + 63) // 64, groups, False, 0, 0)
+        ws, cnt = _ws(t, n, bn, groups, splits, x.device)
+        nv.call("gemm_bf16", nv.ptr(x), nv.ptr(w), nv.ptr(out), I(t), I(n), I(k), I(x.stride(0)), I(w.stride(0)),
+                I(out.stride(0)), f32, I(1 if accumulate else 0), I(bn), I(groups), I(splits), nv.ptr(ws), nv.ptr(cnt),
+                I(ACTS[act]))
+    else:
+        nv.call("gemm_simt", nv.ptr(x), nv.ptr(w), nv.ptr(out), I(t), I(n), I(k), I(x.stride(0)), I(w.stride(0)),
+                I(out.stride(0)), I(1 if x.dtype == torch.float32 else 0), f32, I(1 if accumulate else 0),
+                I(ACTS[act]), I(groups))
     return out
 
 
@@ -194,7 +241,7 @@ def gemm_bf16_grouped(x, w, groups: int, out=None):
     bn, splits = pick_tiling(t, n, (k + 63) // 64, groups, False, 0, 0)
     ws, cnt = _ws(t, n, bn, groups, splits, x.device)
     nv.call("gemm_bf16", nv.ptr(x), nv.ptr(w), nv.ptr(out), I(t), I(n), I(k), I(x.stride(0)), I(w.stride(0)),
-            I(out.stride(0)), I(0), I(0), I(bn), I(groups), I(splits), nv.ptr(ws), nv.ptr(cnt))
+            I(out.stride(0)), I(0), I(0), I(bn), I(groups), I(splits), nv.ptr(ws), nv.ptr(cnt), I(0))
     return out
 
 

@@ -1,0 +1,111 @@
+"""Plain-PyTorch statement of the operators of the layered models (fp32 residual stream, latent attention without
+positions, recurrent time mixing, bf16 experts): the bodies CPU tensors run on.  fp32 arithmetic, results in the
+activation type."""
+from __future__ import annotations
+
+import torch
+
+
+def _rms(x, eps):
+    return x * torch.rsqrt(x.square().mean(-1, keepdim=True) + eps)
+
+
+def segments(fb):
+    """Row ranges [a, b) of the requests of a forward."""
+    if fb.seg_off is None:
+        n = fb.positions.shape[0]
+        return [(i, i + 1) for i in range(n)]
+    off = fb.seg_off.tolist()
+    return list(zip(off[:-1], off[1:]))
+
+
+def embed_residual(ids, weight, dtype, feedback, slots, want_act):
+    if feedback is not None:
+        ids.copy_(feedback[slots.long()])
+    x = weight[ids.long()].float()
+    return x, (x.to(dtype) if want_act else None)
+
+
+def residual_norm(x, gain, eps, dtype, mul, rows, add, add2, vec, experts, cast):
+    for a in (add, add2, vec):
+        if a is not None:
+            x += a
+    if experts is not None:
+        erows, wts, idx = experts
+        w = torch.where(idx >= 0, wts, torch.zeros_like(wts))
+        x += (erows.float().view(*idx.shape, -1) * w[..., None]).sum(1)
+    if gain is None:
+        return x.to(dtype) if cast else None
+    y = x if rows is None else x[rows]
+    return (_rms(y, eps) * gain * mul).to(dtype)
+
+
+def route_topk(h, weight, bias, top, num_valid):
+    z = h.float() @ weight.float().t() + bias
+    idx = torch.sort(z, dim=-1, descending=True, stable=True).indices[:, :top]
+    w = torch.softmax(torch.gather(z, 1, idx), -1)
+    idx = idx.to(torch.int32)
+    if num_valid is not None:
+        idx[int(num_valid):] = -1
+        w[int(num_valid):] = 0
+    return idx, w
+
+
+def gated_experts(h, idx, wts, w13, w2):
+    t, k = idx.shape
+    out = torch.zeros(t, k, h.shape[1], dtype=h.dtype)
+    for e in range(w13.shape[0]):
+        at = (idx == e).nonzero()
+        if len(at) == 0:
+            continue
+        x = h[at[:, 0]].float()
+        g, u = x @ w13[e, 0].float().t(), x @ w13[e, 1].float().t()
+        act = (g * torch.sigmoid(g) * u).to(h.dtype).float()
+        out[at[:, 0], at[:, 1]] = (act @ w2[e].float().t()).to(h.dtype)
+    return out.view(t * k, -1)
+
+
+def latent_store(x, gain, eps, cache, fb):
+    ok = fb.out_loc >= 0
+    cache[fb.out_loc[ok].long()] = (_rms(x[ok].float(), eps) * gain).to(cache.dtype)
+
+
+def latent_attention(q, cache, fb, scale):
+    out = torch.empty_like(q)
+    for a, b in segments(fb):
+        n = int(fb.positions[b - 1]) + 1
+        c = cache[fb.page_table[int(fb.slots[a]), :n].long()].float()
+        s = torch.einsum("thr,jr->thj", q[a:b].float(), c) * scale
+        hidden = torch.arange(n)[None, :] > fb.positions[a:b].long()[:, None]
+        p = torch.softmax(s.masked_fill(hidden[:, None, :], float("-inf")), -1)
+        out[a:b] = torch.einsum("thj,jr->thr", p, c).to(q.dtype)
+    return out
+
+
+def shift_mix(x, gain, eps, mu, prev, tail, fb, dtype):
+    h = _rms(x, eps) * gain
+    hp = torch.cat([h[:1], h[:-1]], 0)
+    for a, b in segments(fb):
+        s = int(fb.slots[a])
+        hp[a] = 0 if int(fb.positions[a]) == 0 else prev[s]
+        (prev if b - a == 1 else tail)[s] = h[b - 1]
+    return torch.cat([h + (hp - h) * m for m in mu], -1).to(dtype)
+
+
+def wkv(p, a, w0, u, gain, state, prev, tail, fb, heads, eps):
+    t, hd = a.shape
+    d = hd // heads
+    r, k, v, g = (c.view(t, heads, d) for c in p.float().chunk(4, -1))
+    w = torch.exp(-torch.exp(a + w0)).view(t, heads, d)
+    o = torch.empty(t, heads, d)
+    for lo, hi in segments(fb):
+        slot = int(fb.slots[lo])
+        s = torch.zeros_like(state[slot]) if int(fb.positions[lo]) == 0 else state[slot].clone()
+        for i in range(lo, hi):
+            kv = k[i][:, :, None] * v[i][:, None, :]
+            o[i] = ((s + u.view(heads, d)[:, :, None] * kv) * r[i][:, :, None]).sum(1)
+            s = w[i][:, :, None] * s + kv
+        state[slot] = s
+        if hi - lo > 1:
+            prev[slot] = tail[slot]
+    return ((_rms(o, eps) * gain.view(heads, d) * (g * torch.sigmoid(g))).view(t, hd)).to(p.dtype)

@@ -20,7 +20,7 @@ from typing import Optional, Tuple
 import torch
 import torch.distributed as dist
 
-from ..models.deepseek_v4 import Comm
+from ..models.base import Comm
 from ..utils.logger import init_logger
 from .info import DistributedInfo
 

@@ -38,7 +38,8 @@ def slots_per_request(window: int, page_size: int) -> int:
 class CacheManager:
     def __init__(self, pool, page_table: torch.Tensor, page_size: int, window: int, enable_prefix_cache: bool = True):
         self.pool, self.page_table, self.ps, self.window = pool, page_table, page_size, window
-        self.radix: Optional[RadixPrefixCache] = RadixPrefixCache(pool, page_size, window) if enable_prefix_cache else None
+        self.radix: Optional[RadixPrefixCache] = (
+            RadixPrefixCache(pool, page_size, window, pool.prefix_align) if enable_prefix_cache else None)
         self.device = page_table.device
         self.counters = {"alloc_pages": 0, "evictions": 0, "swa_unpinned": 0, "alloc_failures": 0, "dedup_pages": 0,
                          "tree_pins_dropped": 0}
@@ -55,7 +56,10 @@ class CacheManager:
     def request_capacity(self, prefill_budget: int) -> int:
         """How many requests the window-slot pool can carry at once: what is left of the pool after one prefill
         forward's pages (at most half of it) and a spare, divided by each request's share; never less than one (a
-        lone request always fits: its chunk shrinks to what the pool can hold)."""
+        lone request always fits: its chunk shrinks to what the pool can hold).  Without windows the table slots are
+        the only limit."""
+        if not self.pool.has_window:
+            return self.pool.sizes.num_req_slots
         total = self.pool.sizes.num_swa_slots
         chunk = min(div_ceil(prefill_budget, self.ps) + 1, total // 2)
         return max((total - chunk) // slots_per_request(self.window, self.ps), 1)
@@ -142,6 +146,8 @@ class CacheManager:
         how many.  The next forward of the request starts at ``cached_len`` (the next prefill chunk, or the next decode
         token), whose window reaches back to ``cached_len - window + 1``.  ``device_len`` must not be used here:
         while a prompt is prefilled in chunks it already is the full prompt length."""
+        if not self.pool.has_window:
+            return 0
         target = max(req.cached_len - self.window, 0) // self.ps
         target = min(target, len(req.pages))
         frontier = getattr(req, "swa_pin_frontier", 0)
@@ -203,6 +209,8 @@ class CacheManager:
         """Invariant of every forward: each page that the sliding windows of positions [first_pos, last_pos] reach
         still owns window storage and is pinned by somebody.  Checked by the scheduler before each launch when
         ``check_window`` is set (tests, MINISGL_DEBUG_BOUNDS=1)."""
+        if not self.pool.has_window:
+            return
         lo = max(first_pos - self.window + 1, 0) // self.ps
         hi = last_pos // self.ps
         for i in range(lo, hi + 1):

@@ -61,7 +61,7 @@ class Scheduler:
         self.tp = config.tp_info
         self.table = TableManager(e.config.max_running_req)
         self.cache = CacheManager(e.pool, e.page_table, self.ps, e.model_config.window_size,
-                                  enable_prefix_cache=config.cache_type == "radix")
+                                  enable_prefix_cache=config.cache_type == "radix" and e.pool.prefix_reusable)
         self.decode = DecodeManager(self.ps)
         self.prefill = PrefillManager(self.cache, self.table, self.decode, self.ps, e.max_seq_len)
         self.policy = MixedPhaseFairPolicy(isolated_prefill_budget=config.max_extend_tokens)
@@ -210,6 +210,8 @@ class Scheduler:
             self.bytes_h2d += host.numel() * 4
             batch.input_ids, batch.positions, batch.slots, batch.out_loc = dev[0], dev[1], dev[2], dev[3]
             batch.last_idx = torch.tensor(last, dtype=torch.int64).to(self.device, non_blocking=True)
+            batch.seg_off = torch.tensor([0] + [i + 1 for i in last], dtype=torch.int32).to(self.device,
+                                                                                            non_blocking=True)
             batch.num_token_non_padded = total
             batch.padded_reqs = list(reqs)
             batch.max_context = max(r.cached_len + n for r, n in zip(reqs, batch.chunk_lens))
