@@ -44,6 +44,11 @@ def parse():
     ap.add_argument("--moe-mode", default="ep", choices=["ep", "tp"])
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--no-fused-comm", action="store_true")
+    ap.add_argument("--design", default="", choices=["", "bedalorn"],
+                    help="instead of the headline: prefill / decode throughput of this design beside DeepSeek-V4 at equal "
+                         "size (one JSON line per model and workload, one GPU)")
+    ap.add_argument("--sizes", default="small,large", help="with --design: model sizes to run")
+    ap.add_argument("--profile", action="store_true", help="with --design: add per-launcher device times")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)  # fewer than three untimed steps would leave clocks and caches cold
     return args
@@ -146,10 +151,15 @@ def main():
     if args.impl == "reference":
         run_reference(args)
         return
+    sys.path.insert(0, ROOT)
+    if args.design:
+        from minisgl.benchmark import designs
+
+        designs.main(args.sizes.split(","), args.profile)
+        return
     import torch
     import torch.distributed as dist
 
-    sys.path.insert(0, ROOT)
     rank = int(os.environ.get("RANK", 0))
     world = int(os.environ.get("WORLD_SIZE", 1))
     local = int(os.environ.get("LOCAL_RANK", 0))
