@@ -60,7 +60,10 @@ def _decode_once(llm, batch: int, context: int) -> None:
     reqs = []
     for i in range(batch):
         r = Req(torch.zeros(context, dtype=torch.int32), llm.table.allocate(), context - 1, 1, i, SamplingParams())
-        llm.cache.allocate(r, context)
+        for upto in range(256, context + 256, 256):    # window storage follows, as it does while a prompt is prefilled
+            r.cached_len = min(upto, context) - 1
+            llm.cache.allocate(r, min(upto, context))
+            llm.cache.release_swa_behind(r)
         reqs.append(r)
     b = Batch(reqs, "decode")
     llm._prepare_batch(b)

@@ -192,6 +192,7 @@ class Batch:
     reasoning_states: Any = None
     max_context: int = 0         # largest device_len in the batch (bounds index-surface widths)
     seg_off: Any = None          # prefill: [B+1] int32 device, row ranges of the requests
+    seg_ends: Any = None         # prefill: context length of every request after the forward (host list)
 
     @property
     def is_prefill(self) -> bool:

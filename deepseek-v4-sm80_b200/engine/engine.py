@@ -236,7 +236,8 @@ class Engine:
         return ForwardBatch(batch.input_ids, batch.positions, batch.slots, batch.out_loc, batch.last_idx,
                             self.page_table, batch.is_prefill, batch.max_context, None,
                             token_feedback=self.last_token if batch.is_decode else None, seg_off=batch.seg_off,
-                            seg_lens=batch.chunk_lens if batch.is_prefill else None)
+                            seg_lens=batch.chunk_lens if batch.is_prefill else None, seg_ends=batch.seg_ends,
+                            seg_slots=[r.table_idx for r in batch.reqs] if batch.is_prefill else None)
 
     def _run(self, batch: Batch, greedy: bool):
         """Launches one forward: (logits, greedy tokens or None).  Decode batches replay a captured graph when there is

@@ -31,6 +31,7 @@ class ForwardBatch:
     seg_off: Optional[torch.Tensor] = None    # [B+1] int32
     seg_lens: Optional[List[int]] = None      # the same lengths on the host
     seg_ends: Optional[List[int]] = None      # context length of every request after this forward (host)
+    seg_slots: Optional[List[int]] = None     # table slot of every request (host)
 
 
 @dataclass

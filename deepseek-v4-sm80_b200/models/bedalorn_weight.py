@@ -85,7 +85,7 @@ def build_weights(cfg: BedalornConfig, get: Callable[[str], torch.Tensor], devic
         if isinstance(m, LatentAttentionSpec):
             w[q + "qc"] = torch.cat([mat(q + "q"), mat(q + "dkv")], 0)
             w[q + "latent.gain"] = vec(q + "dkv.norm")
-            uk = mat(q + "uk")
+            uk = w[q + "uk"] = mat(q + "uk")
             w[q + "uk_t"] = uk.view(m.heads, m.dim, m.kv_rank).transpose(1, 2).reshape(-1, m.dim).contiguous()
             w[q + "uv"] = mat(q + "uv")
         else:

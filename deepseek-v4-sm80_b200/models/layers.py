@@ -12,21 +12,25 @@ from .base import ForwardBatch
 
 class LatentAttention:
     """Causal attention without positions over one cached latent row per token.  The per-head key up-projection is
-    absorbed into the query and the value up-projection into the output, so the latents are read once for all heads."""
+    absorbed into the query and the value up-projection into the output, so the latents are read once for all heads; long
+    prompt portions expand the latents to keys and values instead, which costs fewer operations per pair."""
 
     def __init__(self, w: Dict[str, torch.Tensor], prefix: str, heads: int, dim: int, vdim: int, rank: int, scale: float,
                  eps: float):
         self.heads, self.dim, self.vdim, self.rank, self.scale, self.eps = heads, dim, vdim, rank, scale, eps
         self.qc, self.gain = w[prefix + "qc"], w[prefix + "latent.gain"]
-        self.uk_t, self.uv, self.o = w[prefix + "uk_t"], w[prefix + "uv"], w[prefix + "o"]
+        self.uk, self.uk_t, self.uv, self.o = (w[prefix + n] for n in ("uk", "uk_t", "uv", "o"))
 
     def __call__(self, h: torch.Tensor, x: torch.Tensor, cache: torch.Tensor, fb: ForwardBatch) -> None:
         t, hq = h.shape[0], self.heads * self.dim
         qc = O.linear(h, self.qc)
         O.latent_store(qc[:, hq:], self.gain, self.eps, cache, fb)
-        q = O.grouped_linear(qc[:, :hq], self.uk_t, self.heads).view(t, self.heads, self.rank)
-        lat = O.latent_attention(q, cache, fb, self.scale)
-        v = O.grouped_linear(lat.view(t, self.heads * self.rank), self.uv, self.heads)
+        if fb.is_prefill and O.prefers_expanded(qc, fb, self.heads, self.dim, self.vdim, self.rank):
+            v = O.expanded_attention(qc[:, :hq], cache, fb, self.uk, self.uv, self.heads, self.scale)
+        else:
+            q = O.grouped_linear(qc[:, :hq], self.uk_t, self.heads).view(t, self.heads, self.rank)
+            lat = O.latent_attention(q, cache, fb, self.scale)
+            v = O.grouped_linear(lat.view(t, self.heads * self.rank), self.uv, self.heads)
         O.linear(v, self.o, out=x, accumulate=True)
 
 

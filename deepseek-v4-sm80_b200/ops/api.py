@@ -305,6 +305,17 @@ def latent_attention(q, cache, fb, scale: float):
     return _layers(q).latent_attention(q, cache, fb, scale)
 
 
+def prefers_expanded(q, fb, heads: int, dim: int, vdim: int, rank: int) -> bool:
+    """Whether :func:`expanded_attention` is the cheaper form for this forward (long prompt portions)."""
+    return _layers(q).prefers_expanded(q.dtype, fb, heads, dim, vdim, rank)
+
+
+def expanded_attention(q, cache, fb, uk, uv, heads: int, scale: float):
+    """The same attention with keys W_uk c and values W_uv c expanded from the requests' cached latents:
+    q [T, H*dim] (a column slice), uk [H*dim, R], uv [H*vdim, R] -> [T, H*vdim]."""
+    return _layers(q).expanded_attention(q, cache, fb, uk, uv, heads, scale)
+
+
 def shift_mix(x, gain, eps: float, mu, prev, tail, fb, dtype):
     """Norm and token shift: h = x / rms(x) * gain, h' = the previous token's h; returns [T, n*D], mix m being
     h + (h' - h) mu[m].  prev [slots+1, D]: every slot's last h, read by the first row of a portion.  tail: scratch of

@@ -47,12 +47,13 @@ int dsv4_make_tmap_2d(CUtensorMap* out, const void* base, int elem, uint64_t inn
 }
 
 int dsv4_make_tmap_3d(CUtensorMap* out, const void* base, uint64_t inner, uint64_t mid, uint64_t outer,
-                      uint64_t mid_stride_bytes, uint64_t outer_stride_bytes, uint32_t box_inner, uint32_t box_mid) {
+                      uint64_t mid_stride_bytes, uint64_t outer_stride_bytes, uint32_t box_inner, uint32_t box_mid,
+                      uint32_t box_outer) {
   EncodeTiledFn fn = get_encode_fn();
   if (!fn) return 1;
   cuuint64_t dims[3] = {inner, mid, outer};
   cuuint64_t strides[2] = {mid_stride_bytes, outer_stride_bytes};
-  cuuint32_t box[3] = {box_inner, box_mid, 1};
+  cuuint32_t box[3] = {box_inner, box_mid, box_outer};
   cuuint32_t estr[3] = {1, 1, 1};
   CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,

@@ -398,7 +398,8 @@ inline cudaError_t dsv4_launch_cluster(void (*kernel)(KArgs...), dim3 grid, dim3
 // swizzle: 0 = none, 3 = 128 B.
 int dsv4_make_tmap_2d(CUtensorMap* out, const void* base, int elem, uint64_t inner, uint64_t outer,
                       uint64_t row_stride_bytes, uint32_t box_inner, uint32_t box_outer, int swizzle);
-// 3-D bf16 tensor map (contiguous dimension first), 128-byte swizzle, box (box_inner, box_mid, 1).  Coordinates past an
+// 3-D bf16 tensor map (contiguous dimension first), 128-byte swizzle, box (box_inner, box_mid, box_outer).  Coordinates past an
 // extent read zeros, so neighbouring slices of the outer dimensions never leak into a tile.
 int dsv4_make_tmap_3d(CUtensorMap* out, const void* base, uint64_t inner, uint64_t mid, uint64_t outer,
-                      uint64_t mid_stride_bytes, uint64_t outer_stride_bytes, uint32_t box_inner, uint32_t box_mid);
+                      uint64_t mid_stride_bytes, uint64_t outer_stride_bytes, uint32_t box_inner, uint32_t box_mid,
+                      uint32_t box_outer = 1);

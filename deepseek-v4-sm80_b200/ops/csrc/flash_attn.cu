@@ -1,0 +1,320 @@
+// Causal multi-head attention of long prompt portions on tcgen05, keys and values expanded from the cached latents.
+//
+// The absorbed form (latent_attn.cu) multiplies every (query, key) pair over the whole latent rank, twice.  For a portion
+// of many tokens it is cheaper to expand the request's latents once,  K = C W_uk^T  and  V^T = W_uv C^T  (two plain
+// projections; the second one comes out with the keys contiguous, which is the K-major operand of the PV product), and to
+// run ordinary attention over `dim` and `vdim` per head.
+//
+// One CTA: one head, 256 consecutive queries of one request as two 128-row tiles that share every key / value tile (128
+// keys).  The tensor core works on one tile while the softmax warps work on the other:
+//   warp 0      TMA producer: Q once, then K and V^T tiles through two-stage rings
+//   warp 1      tcgen05.mma issuer:  S_t = Q_t K^T,  O_t += P_t V  (P_t is read from tensor memory)
+//   warps 2-5   softmax of tile 0, warps 6-9 of tile 1: one thread per row; P_t overwrites S_t in place as bf16
+// Tensor memory: S0 | S1 | O0 | O1, 128 columns each.  O stays there; it is rescaled only when a row's maximum has grown by
+// more than 2^8 since the last time (the sums stay far from overflow, the quotient does not depend on it).
+#include "vec.cuh"
+
+namespace {
+
+constexpr int kQT = 128;                     // queries per tile, keys per tile
+constexpr int kBlk = kQT * 128;              // bytes of a [128 rows][64 elements] operand block
+constexpr int kFThreads = 320;
+constexpr int kColO = 256;
+
+struct FlashArgs {
+  const int* items;     // [n_items][5]: first query row, queries, context position of the first, first key row, keys
+  int heads, dim, vdim, ldo;
+  float scale2;         // scale * log2(e)
+};
+
+struct FlashBars {
+  uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_ready[2], o_full[2];
+  uint32_t tmem;
+  int abort_flag;
+};
+
+template <int NB>     // 64-wide blocks of dim
+struct FlashCfg {
+  static constexpr int kQ = 2 * NB * kBlk, kK = NB * kBlk, kV = 2 * kBlk;
+  static constexpr int kSmem = kQ + 2 * (kK + kV) + 1024 + (int)sizeof(FlashBars);
+};
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <int NB>
+__global__ void __launch_bounds__(kFThreads, 1)
+flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                  const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out, const FlashArgs a) {
+  using C = FlashCfg<NB>;
+  extern __shared__ uint8_t fsm_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(fsm_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* qs = smem;                       // [2 tiles][NB] blocks
+  uint8_t* ks = qs + C::kQ;                 // [2 stages][NB] blocks
+  uint8_t* vs = ks + 2 * C::kK;             // [2 stages][2] blocks of [vdim rows][64 keys]
+  FlashBars* b = reinterpret_cast<FlashBars*>(vs + 2 * C::kV);
+  volatile int* abort_flag = &b->abort_flag;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int head = blockIdx.x;
+
+  if (threadIdx.x == 0) {
+    mbar_init(&b->q_full, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&b->k_full[i], 1), mbar_init(&b->k_empty[i], 1);
+      mbar_init(&b->v_full[i], 1), mbar_init(&b->v_empty[i], 1);
+      mbar_init(&b->s_full[i], 1), mbar_init(&b->o_full[i], 1);
+      mbar_init(&b->p_ready[i], 128);
+    }
+    b->abort_flag = 0;
+    mbar_fence_init();
+    tma_prefetch_desc(&tmQ);
+    tma_prefetch_desc(&tmK);
+    tma_prefetch_desc(&tmV);
+  }
+  if (warp == 1) {
+    tmem_alloc(&b->tmem, 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = b->tmem;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int* it = a.items + blockIdx.y * 5;
+  const int q0 = it[0], nq = it[1], pos0 = it[2], kv0 = it[3], nkeys = it[4];
+  const int n = (nkeys + kQT - 1) / kQT;    // key tiles: every key the last query sees
+  const int vp = (a.vdim + 15) & ~15;       // columns of the PV product
+  const uint32_t v_bytes = 2u * (uint32_t)vp * 128u;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      mbar_expect_tx(&b->q_full, C::kQ);
+      for (int t = 0; t < 2; ++t)
+        for (int j = 0; j < NB; ++j) tma_load_3d(qs + (t * NB + j) * kBlk, &tmQ, &b->q_full, j * 64, head, q0 + t * kQT);
+      for (int i = 0; i < n; ++i) {
+        const int s = i & 1;
+        const uint32_t ph = ((i >> 1) & 1) ^ 1;
+        if (i >= 2 && !mbar_wait<32>(&b->k_empty[s], ph, abort_flag, 81)) break;
+        mbar_expect_tx(&b->k_full[s], C::kK);
+        for (int j = 0; j < NB; ++j)
+          tma_load_3d(ks + s * C::kK + j * kBlk, &tmK, &b->k_full[s], j * 64, head, kv0 + i * kQT);
+        if (i >= 2 && !mbar_wait<32>(&b->v_empty[s], ph, abort_flag, 82)) break;
+        mbar_expect_tx(&b->v_full[s], v_bytes);
+        for (int j = 0; j < 2; ++j)
+          tma_load_3d(vs + s * C::kV + j * kBlk, &tmV, &b->v_full[s], kv0 + i * kQT + j * 64, 0, head);
+      }
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t kIdS = umma_idesc(128, kQT, 1, 1);
+      const uint32_t id_o = umma_idesc(128, vp, 1, 1);
+      auto scores = [&](int t, int i) {
+        const uint8_t* kt = ks + (i & 1) * C::kK;
+#pragma unroll
+        for (int k = 0; k < NB * 4; ++k)
+          umma_f16(tmem + t * 128, umma_desc_k128(qs + (t * NB + k / 4) * kBlk, (k & 3) * 32),
+                   umma_desc_k128(kt + k / 4 * kBlk, (k & 3) * 32), kIdS, k > 0);
+      };
+      auto values = [&](int t, int i) {
+        const uint8_t* vt = vs + (i & 1) * C::kV;
+#pragma unroll
+        for (int k = 0; k < 8; ++k)
+          umma_f16_ta(tmem + kColO + t * 128, tmem + t * 128 + k * 8,
+                      umma_desc_k128(vt + k / 4 * kBlk, (k & 3) * 32), id_o, i > 0 || k > 0);
+      };
+      bool ok = mbar_wait(&b->q_full, 0, abort_flag, 83) && mbar_wait(&b->k_full[0], 0, abort_flag, 84);
+      tc_fence_after();
+      if (ok) {
+        for (int t = 0; t < 2; ++t) {
+          scores(t, 0);
+          umma_commit(&b->s_full[t]);
+        }
+        umma_commit(&b->k_empty[0]);
+      }
+      for (int i = 0; i < n && ok; ++i) {
+        const bool more = i + 1 < n;
+        ok = mbar_wait(&b->v_full[i & 1], (i >> 1) & 1, abort_flag, 85);
+        for (int t = 0; t < 2 && ok; ++t) {
+          ok = mbar_wait(&b->p_ready[t], i & 1, abort_flag, 86);
+          if (!ok) break;
+          tc_fence_after();
+          values(t, i);
+          if (more) {
+            // S_t may only be written now: P_t, which sits on it, has been consumed by the product before (MMAs of one
+            // thread run in order)
+            if (t == 0) ok = mbar_wait(&b->k_full[(i + 1) & 1], ((i + 1) >> 1) & 1, abort_flag, 87);
+            if (!ok) break;
+            tc_fence_after();
+            scores(t, i + 1);
+            umma_commit(&b->s_full[t]);
+          } else {
+            umma_commit(&b->o_full[t]);
+          }
+        }
+        if (ok) {
+          umma_commit(&b->v_empty[i & 1]);
+          if (more) umma_commit(&b->k_empty[(i + 1) & 1]);
+        }
+      }
+    }
+  } else {
+    const int t = (warp - 2) >> 2, quarter = warp & 3;
+    const int row = t * kQT + quarter * 32 + lane;            // query within the item
+    const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
+    const uint32_t sp = tmem + t * 128 + lane_base, op = tmem + kColO + t * 128 + lane_base;
+    const int last = row < nq ? pos0 + row : -1;              // last key the row sees
+    const int first_masked = (pos0 + t * kQT + quarter * 32 + 1) / kQT;  // key tiles before it are seen whole by the warp
+    float m = -1e30f, l = 0.f;
+    bool ok = true;
+    for (int i = 0; i < n; ++i) {
+      ok = mbar_wait<16>(&b->s_full[t], i & 1, abort_flag, 88);
+      if (!ok) break;
+      tc_fence_after();
+      float s[kQT];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        uint32_t r[32];
+        tmem_ld_32x32(sp + c * 32, r);
+        tmem_ld_wait();
+#pragma unroll
+        for (int j = 0; j < 32; ++j) s[c * 32 + j] = __uint_as_float(r[j]);
+      }
+      if (i >= first_masked || row >= nq) {
+        const int lim = last - i * kQT;
+#pragma unroll
+        for (int j = 0; j < kQT; ++j)
+          if (j > lim) s[j] = -INFINITY;
+      }
+      float mx = s[0];
+#pragma unroll
+      for (int j = 1; j < kQT; ++j) mx = fmaxf(mx, s[j]);
+      mx *= a.scale2;
+      const bool grow = mx > m + 8.f;
+      if (__any_sync(0xffffffffu, grow)) {
+        const float mn = grow ? mx : m, f = ex2(m - mn);
+        m = mn;
+        l *= f;
+        if (i > 0) {
+#pragma unroll 1
+          for (int c = 0; c < vp; c += 16) {
+            uint32_t r[16];
+            tmem_ld_32x16(op + c, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * f);
+            tmem_st_32x16(op + c, r);
+          }
+        }
+      }
+      float sum0 = 0.f, sum1 = 0.f;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        uint32_t pk[16];
+#pragma unroll
+        for (int j = 0; j < 16; ++j) {
+          const float p0 = ex2(fmaf(s[c * 32 + 2 * j], a.scale2, -m)), p1 = ex2(fmaf(s[c * 32 + 2 * j + 1], a.scale2, -m));
+          sum0 += p0, sum1 += p1;
+          const __nv_bfloat162 p = __floats2bfloat162_rn(p0, p1);
+          pk[j] = *reinterpret_cast<const uint32_t*>(&p);
+        }
+        tmem_st_32x16(sp + c * 16, pk);
+      }
+      l += sum0 + sum1;
+      tmem_st_wait();
+      tc_fence_before();
+      mbar_arrive(&b->p_ready[t]);
+    }
+    if (ok && mbar_wait<16>(&b->o_full[t], 0, abort_flag, 89)) {
+      tc_fence_after();
+      const float inv = 1.f / l;
+      __nv_bfloat16* dst = out + (size_t)(q0 + row) * a.ldo + head * a.vdim;
+#pragma unroll 1
+      for (int c = 0; c < vp; c += 16) {
+        uint32_t r[16];
+        tmem_ld_32x16(op + c, r);
+        tmem_ld_wait();
+        if (row < nq) {
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            if (c + h * 8 >= a.vdim) break;      // vdim is a multiple of 8
+            uint4 u;
+            __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+              p[j] = __floats2bfloat162_rn(__uint_as_float(r[h * 8 + 2 * j]) * inv,
+                                           __uint_as_float(r[h * 8 + 2 * j + 1]) * inv);
+            *reinterpret_cast<uint4*>(dst + c + h * 8) = u;
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) tmem_dealloc(tmem, 512);
+}
+
+// ctx[dst + j] = cache[page_table[slot][j]] for the keys j of every listed request, zeros in the padding behind them.
+// list: [segs][3] = slot, keys, first row of the copy; rows [dst, dst of the next request) belong to a request.
+__global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* __restrict__ cache, uint4* __restrict__ ctx,
+                                                            const int* __restrict__ list, int segs, int total,
+                                                            const int* __restrict__ page_table, int ld_pt, int r8) {
+  pdl_entry();
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= total) return;
+  int lo = 0, hi = segs - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (list[mid * 3 + 2] <= row) lo = mid; else hi = mid - 1;
+  }
+  const int j = row - list[lo * 3 + 2];
+  const bool in = j < list[lo * 3 + 1];
+  const size_t src = in ? (size_t)page_table[(size_t)list[lo * 3] * ld_pt + j] * r8 : 0;
+  for (int i = lane; i < r8; i += 32) ctx[(size_t)row * r8 + i] = in ? cache[src + i] : make_uint4(0, 0, 0, 0);
+}
+
+template <int NB>
+int launch_flash(const CUtensorMap& q, const CUtensorMap& k, const CUtensorMap& v, void* out, const FlashArgs& a,
+                 int n_items, cudaStream_t st) {
+  using C = FlashCfg<NB>;
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(flash_attn_kernel<NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmem) != cudaSuccess)
+      return 655;
+    set = true;
+  }
+  dsv4_launch(flash_attn_kernel<NB>, dim3(a.heads, n_items), kFThreads, C::kSmem, st, q, k, v, (__nv_bfloat16*)out, a);
+  return (int)cudaGetLastError();
+}
+
+}  // namespace
+
+DSV4_API int dsv4_latent_gather(const void* cache, void* ctx, const int* list, int segs, int total,
+                                const int* page_table, int ld_pt, int rank, cudaStream_t st) {
+  if (total <= 0) return 0;
+  if (rank % 8 || segs < 1) return 650;
+  dsv4_launch(latent_gather_kernel, (total + 3) / 4, 128, 0, st, (const uint4*)cache, (uint4*)ctx, list, segs, total,
+              page_table, ld_pt, rank / 8);
+  return (int)cudaGetLastError();
+}
+
+// q: bf16 [rows, heads * dim] (row stride ldq), k: [kv_rows, heads * dim], vt: [heads * vdim, kv_rows] (row stride
+// kv_rows), out: [rows, heads * vdim].  items as in FlashArgs, at most 256 queries each; first key rows are multiples of 8.
+DSV4_API int dsv4_flash_attention(const void* q, int ldq, const void* k, const void* vt, void* out, const int* items,
+                                  int n_items, int rows, int kv_rows, int heads, int dim, int vdim, float scale,
+                                  cudaStream_t st) {
+  if (n_items <= 0) return 0;
+  if (dim % 8 || vdim % 8 || ldq % 8 || kv_rows % 8 || dim < 8 || dim > 128 || vdim < 8 || vdim > 128 || n_items > 65535)
+    return 651;
+  CUtensorMap tq, tk, tv;
+  if (dsv4_make_tmap_3d(&tq, q, dim, heads, rows, (uint64_t)dim * 2, (uint64_t)ldq * 2, 64, 1, kQT)) return 652;
+  if (dsv4_make_tmap_3d(&tk, k, dim, heads, kv_rows, (uint64_t)dim * 2, (uint64_t)heads * dim * 2, 64, 1, kQT)) return 653;
+  const int vp = (vdim + 15) & ~15;
+  if (dsv4_make_tmap_3d(&tv, vt, kv_rows, vdim, heads, (uint64_t)kv_rows * 2, (uint64_t)vdim * kv_rows * 2, 64, vp)) return 654;
+  const FlashArgs a{items, heads, dim, vdim, heads * vdim, scale * 1.4426950408889634f};
+  return dim <= 64 ? launch_flash<1>(tq, tk, tv, out, a, n_items, st) : launch_flash<2>(tq, tk, tv, out, a, n_items, st);
+}

@@ -2,6 +2,8 @@
 moe_bf16.cu, gemm_simt.cu), one function per facade op in :mod:`minisgl.ops.api`.  Activations are bf16 or fp32."""
 from __future__ import annotations
 
+import os
+
 import torch
 
 from . import native as nv
@@ -136,6 +138,72 @@ def latent_attention(q, cache, fb, scale):
             nv.ptr(fb.num_valid), I(t), I(h), I(r), F(scale), I(m), I(tiles), I(nsplit), nv.ptr(acc), nv.ptr(ml),
             _f32(q.dtype))
     return o
+
+
+# MINISGL_LATENT_PREFILL: auto (by cost), expanded (wherever the kernel can) or absorbed
+LATENT_PREFILL = os.environ.get("MINISGL_LATENT_PREFILL", "auto")
+EXPAND_BYTES = 4 << 30                        # bound of the expanded keys and values of one call
+ABSORBED_TFLOPS, EXPANDED_TFLOPS, GEMM_TFLOPS, EXPAND_US = 200.0, 500.0, 450.0, 25.0    # measured rates
+
+
+def prefers_expanded(q_dtype, fb, heads: int, dim: int, vdim: int, rank: int) -> bool:
+    """Whether a prefill forward should expand its requests' latents to keys and values (csrc/flash_attn.cu) instead of
+    attending over the latents: expanding costs every request's whole context once, and then a query pays dim + vdim per
+    key instead of twice the rank."""
+    if fb.seg_ends is None or q_dtype != torch.bfloat16 or LATENT_PREFILL == "absorbed":
+        return False
+    if dim % 8 or vdim % 8 or rank % 8 or dim > 128 or vdim > 128:
+        return False
+    ctx = sum(-(-s // KV_ALIGN) * KV_ALIGN for s in fb.seg_ends)
+    if 2 * ctx * (heads * (dim + vdim) + rank) > EXPAND_BYTES:
+        return False
+    if LATENT_PREFILL == "expanded":
+        return True
+    pairs = sum(n * (s - n / 2) for n, s in zip(fb.seg_lens, fb.seg_ends))
+    tiled = sum(-(-n // 256) * 256 * (s - n / 2 + 64) for n, s in zip(fb.seg_lens, fb.seg_ends))
+    absorbed = 4e-6 * heads * rank * pairs / ABSORBED_TFLOPS \
+        + 2e-6 * sum(fb.seg_lens) * heads * rank * (dim + vdim) / GEMM_TFLOPS
+    expanded = 2e-6 * heads * (dim + vdim) * (tiled / EXPANDED_TFLOPS + ctx * rank / GEMM_TFLOPS) + EXPAND_US
+    return expanded < absorbed
+
+
+KV_ALIGN = 64       # a request's expanded keys start at a multiple of this (16-byte TMA boundaries of V^T)
+
+
+def _expanded_plan(fb, device):
+    """(request list [n, 3], work items [m, 5], expanded rows), one per forward: the same for all layers.  Items are
+    ordered by the number of keys they see, longest first."""
+    plan = getattr(fb, "expanded_plan", None)
+    if plan is None:
+        reqs, items, at, row = [], [], 0, 0
+        for n, s, slot in zip(fb.seg_lens, fb.seg_ends, fb.seg_slots):
+            reqs.append((slot, s, at))
+            for q in range(0, n, 256):
+                m = min(256, n - q)
+                items.append((row + q, m, s - n + q, at, s - n + q + m))
+            at += -(-s // KV_ALIGN) * KV_ALIGN
+            row += n
+        items.sort(key=lambda i: -i[4])
+        host = torch.tensor([v for t in (*reqs, *items) for v in t], dtype=torch.int32).pin_memory()
+        dev = host.to(device, non_blocking=True)
+        k = 3 * len(reqs)
+        plan = fb.expanded_plan = (dev[:k], dev[k:], len(reqs), len(items), at)
+    return plan
+
+
+@tensors(q="bf16[_,_]s", cache="bf16[_,R]", uk="bf16[_,R]", uv="bf16[_,R]")
+def expanded_attention(q, cache, fb, uk, uv, heads, scale):
+    t, dim, vdim, rank = q.shape[0], uk.shape[0] // heads, uv.shape[0] // heads, cache.shape[1]
+    reqs, items, n_reqs, n_items, rows = _expanded_plan(fb, q.device)
+    ctx = torch.empty(rows, rank, dtype=q.dtype, device=q.device)
+    pt = fb.page_table
+    nv.call("latent_gather", nv.ptr(cache), nv.ptr(ctx), nv.ptr(reqs), I(n_reqs), I(rows), nv.ptr(pt), I(pt.stride(0)),
+            I(rank))
+    k, vt = linear(ctx, uk), linear(uv, ctx)
+    out = torch.empty(t, heads * vdim, dtype=q.dtype, device=q.device)
+    nv.call("flash_attention", nv.ptr(q), I(q.stride(0)), nv.ptr(k), nv.ptr(vt), nv.ptr(out), nv.ptr(items), I(n_items),
+            I(t), I(rows), I(heads), I(dim), I(vdim), F(scale))
+    return out
 
 
 # --------------------------------------------------------------------------- recurrent time mixing

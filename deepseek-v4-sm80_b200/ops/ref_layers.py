@@ -82,6 +82,24 @@ def latent_attention(q, cache, fb, scale):
     return out
 
 
+def prefers_expanded(q_dtype, fb, heads, dim, vdim, rank):
+    return False
+
+
+def expanded_attention(q, cache, fb, uk, uv, heads, scale):
+    t, vdim = q.shape[0], uv.shape[0] // heads
+    out = torch.empty(t, heads * vdim, dtype=q.dtype)
+    for a, b in segments(fb):
+        n = int(fb.positions[b - 1]) + 1
+        c = cache[fb.page_table[int(fb.slots[a]), :n].long()].float()
+        k, v = (c @ uk.float().t()).view(n, heads, -1), (c @ uv.float().t()).view(n, heads, vdim)
+        s = torch.einsum("thd,jhd->thj", q[a:b].float().reshape(b - a, heads, -1), k) * scale
+        hidden = torch.arange(n)[None, :] > fb.positions[a:b].long()[:, None]
+        p = torch.softmax(s.masked_fill(hidden[:, None, :], float("-inf")), -1)
+        out[a:b] = torch.einsum("thj,jhd->thd", p, v).reshape(b - a, -1).to(q.dtype)
+    return out
+
+
 def shift_mix(x, gain, eps, mu, prev, tail, fb, dtype):
     h = _rms(x, eps) * gain
     hp = torch.cat([h[:1], h[:-1]], 0)

@@ -214,7 +214,8 @@ class Scheduler:
                                                                                             non_blocking=True)
             batch.num_token_non_padded = total
             batch.padded_reqs = list(reqs)
-            batch.max_context = max(r.cached_len + n for r, n in zip(reqs, batch.chunk_lens))
+            batch.seg_ends = [r.cached_len + n for r, n in zip(reqs, batch.chunk_lens)]
+            batch.max_context = max(batch.seg_ends)
         if isinstance(e.sampler, ReasoningSampler):
             states = [int(r.reasoning_state) for r in reqs]
             return e.sampler.prepare(batch, states)
