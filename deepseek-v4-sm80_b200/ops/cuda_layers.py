@@ -217,12 +217,45 @@ def shift_mix(x, gain, eps, mu, prev, tail, fb, dtype):
     return out
 
 
+# Portions of at least WKV_CHUNK_MIN tokens run the recurrence in chunks (csrc/wkv_chunk.cu).  In 32-bit serving it stays
+# token by token: decays are then products of the decays themselves, not exponentials of sums.  WKV_CHUNKED overrides.
+WKV_CHUNKED = None
+WKV_CHUNK_MIN, WKV_CHUNK = 64, 32
+
+
+def _chunk_plan(fb, device):
+    """(chunks [n, 2], segments [m, 4]) of a forward for the chunked recurrence; the same for all layers."""
+    plan = getattr(fb, "chunk_plan", None)
+    if plan is None:
+        chunks, segs, row = [], [], 0
+        for n, slot in zip(fb.seg_lens, fb.seg_slots):
+            c0 = len(chunks)
+            chunks += [(row + i, min(WKV_CHUNK, n - i)) for i in range(0, n, WKV_CHUNK)]
+            segs.append((slot, c0, len(chunks) - c0, row))
+            row += n
+        host = torch.tensor([v for t in (*chunks, *segs) for v in t], dtype=torch.int32).pin_memory()
+        dev = host.to(device, non_blocking=True)
+        k = 2 * len(chunks)
+        plan = fb.chunk_plan = (dev[:k], dev[k:], len(chunks), len(segs))
+    return plan
+
+
 @tensors(p="bf16|f32[T,_]", a="f32[T,N]", w0="f32[N]", u="f32[N]", gain="f32[N]", state="f32[S,_,_,_]",
          prev="f32[S,W]", tail="f32[S,W]")
 def wkv(p, a, w0, u, gain, state, prev, tail, fb, heads, eps):
     t, hd = a.shape
     assert p.shape[1] == 4 * hd and state.shape[1] == heads
     out = torch.empty(t, hd, dtype=p.dtype, device=p.device)
+    chunked = WKV_CHUNKED if WKV_CHUNKED is not None else p.dtype == torch.bfloat16
+    if chunked and fb.seg_lens is not None and max(fb.seg_lens) >= WKV_CHUNK_MIN:
+        d = hd // heads
+        chunks, segs, n_chunks, n_segs = _chunk_plan(fb, p.device)
+        us = torch.empty(n_chunks, heads, d, d, dtype=torch.float32, device=p.device)
+        decay = torch.empty(n_chunks, heads, d, dtype=torch.float32, device=p.device)
+        nv.call("wkv_chunked", nv.ptr(p), nv.ptr(a), nv.ptr(w0), nv.ptr(u), nv.ptr(gain), nv.ptr(state), nv.ptr(prev),
+                nv.ptr(tail), I(prev.shape[1]), nv.ptr(fb.positions), nv.ptr(fb.seg_off), nv.ptr(chunks), I(n_chunks),
+                nv.ptr(segs), I(n_segs), nv.ptr(us), nv.ptr(decay), I(heads), I(d), F(eps), nv.ptr(out), _f32(p.dtype))
+        return out
     segs = t if fb.seg_off is None else fb.seg_off.shape[0] - 1
     nv.call("wkv_scan", nv.ptr(p), nv.ptr(a), nv.ptr(w0), nv.ptr(u), nv.ptr(gain), nv.ptr(state), nv.ptr(prev),
             nv.ptr(tail), I(prev.shape[1]), nv.ptr(fb.slots), nv.ptr(fb.positions), nv.ptr(fb.seg_off), I(segs),

@@ -198,3 +198,138 @@ def test_latent_store(dtype):
         if i != 3:
             want[int(fb.out_loc[i])] = P.rms(x[i, 12:].to(F), 1e-2) * gain.to(F)
     assert err(cache, want) < TOL[dtype]
+
+
+# --------------------------------------------------------------------------- recurrent time mixing
+def plain_shift_mix(x, gain, eps, mu, prev):
+    h = P.rms(x.to(F), eps) * gain.to(F)
+    hp = P.token_shift(h, prev.to(F))
+    return torch.cat([h + (hp - h) * m.to(F) for m in mu], -1), h[-1]
+
+
+@BOTH
+@pytest.mark.parametrize("d", [96, 50, 1024])
+def test_shift_mix(d, dtype):
+    """First rows of a request, of a later portion and single rows; what every portion leaves in its slot."""
+    segs = [(0, 0, 3), (1, 7, 4), (2, 0, 1), (3, 9, 1)]
+    fb, _ = make_fb(segs, DEV)
+    x, gain, mu = rand(9, d), rand(d, seed=1), rand(5, d, seed=2)
+    prev, tail = rand(7, d, seed=3), torch.full((7, d), 9.0)
+    pc, tc = prev.to(DEV), tail.to(DEV)
+    got = O.shift_mix(x.to(DEV), gain.to(DEV), 1e-3, mu.to(DEV), pc, tc, fb, dtype)
+    row = 0
+    for slot, start, n in segs:
+        want, last = plain_shift_mix(x[row:row + n], gain, 1e-3, mu, prev[slot] if start else torch.zeros(d))
+        assert err(got[row:row + n], want) < TOL[dtype]
+        assert err((pc if n == 1 else tc)[slot][None], last[None]) < 1e-5
+        row += n
+
+
+def wkv_case(segs, heads, d, dtype, seed=0, w0=None):
+    fb, _ = make_fb(segs, DEV)
+    t, hd = sum(n for _, _, n in segs), heads * d
+    p, a = rand(t, 4 * hd, seed=seed).to(dtype), rand(t, hd, seed=seed + 1)
+    w0 = rand(hd, seed=seed + 2) - 2.0 if w0 is None else torch.full((hd,), float(w0))
+    u, gain = rand(hd, seed=seed + 3), rand(hd, seed=seed + 4)
+    state, prev, tail = rand(7, heads, d, d, seed=seed + 5), rand(7, 64, seed=seed + 6), rand(7, 64, seed=seed + 7)
+    return fb, p, a, w0, u, gain, state, prev, tail
+
+
+def check_wkv(segs, heads, d, dtype, tol, w0=None):
+    fb, p, a, w0, u, gain, state, prev, tail = wkv_case(segs, heads, d, dtype, w0=w0)
+    hd = heads * d
+    sc, pc = state.to(DEV), prev.to(DEV)
+    got = O.wkv(p.to(DEV), a.to(DEV), w0.to(DEV), u.to(DEV), gain.to(DEV), sc, pc, tail.to(DEV), fb, heads, 1e-4)
+    row = 0
+    for slot, start, n in segs:
+        r, k, v, g = (c.reshape(n, heads, d) for c in p[row:row + n].to(F).split(hd, 1))
+        w = torch.exp(-torch.exp(a[row:row + n].to(F) + w0.to(F))).view(n, heads, d)
+        s0 = state[slot].to(F) if start else torch.zeros(heads, d, d, dtype=F)
+        o, s = P.wkv_recurrence(r, k, v, w, u.to(F).view(heads, d), s0)
+        want = (P.rms(o, 1e-4) * gain.to(F).view(heads, d) * P.silu(g)).reshape(n, hd)
+        assert err(got[row:row + n], want) < tol
+        assert err(sc[slot].flatten(0, 1), s.flatten(0, 1)) < 3e-5
+        assert torch.equal(pc[slot].cpu(), tail[slot] if n > 1 else prev[slot])
+        row += n
+
+
+WKV_SEGS = [[(0, 0, 1), (1, 5, 1)], [(2, 0, 40)], [(3, 8, 17), (0, 0, 2), (5, 1, 1), (4, 100, 33)]]
+
+
+@BOTH
+@pytest.mark.parametrize("heads,d", [(1, 8), (3, 16), (2, 20), (2, 32), (2, 41), (2, 64), (1, 128)])
+@pytest.mark.parametrize("segs", WKV_SEGS)
+def test_wkv_token_by_token(heads, d, segs, dtype):
+    check_wkv(segs, heads, d, dtype, TOL[dtype])
+
+
+@BOTH
+@pytest.mark.parametrize("heads,d", [(1, 8), (3, 16), (2, 20), (2, 32), (2, 41), (2, 64), (1, 128)])
+@pytest.mark.parametrize("segs", [[(1, 0, 64)], [(2, 3, 200)], [(3, 8, 65), (0, 0, 2), (5, 1, 1), (4, 100, 33), (1, 0, 96)]])
+def test_wkv_in_chunks(heads, d, segs, dtype, monkeypatch):
+    monkeypatch.setattr(C, "WKV_CHUNKED", True)
+    check_wkv(segs, heads, d, dtype, TOL[dtype])
+
+
+@pytest.mark.parametrize("w0", [-12, -1, 2, 6])
+def test_wkv_chunks_with_slow_and_fast_decays(w0, monkeypatch):
+    """A state that hardly decays over hundreds of tokens, and decays that leave nothing of the token before."""
+    monkeypatch.setattr(C, "WKV_CHUNKED", True)
+    check_wkv([(1, 0, 300), (2, 50, 70)], 2, 32, torch.float32, 1e-4, w0=w0)
+
+
+# --------------------------------------------------------------------------- mixture of experts
+@BOTH
+@pytest.mark.parametrize("experts,top", [(1, 1), (5, 2), (8, 8), (40, 1), (100, 6)])
+def test_router(experts, top, dtype):
+    t, d = 33, 72
+    h, w, b = rand(t, d).to(dtype), rand(experts, d, seed=1, dtype=torch.bfloat16), rand(experts, seed=2)
+    idx, wts = O.route_topk(h.to(DEV), w.to(DEV), b.to(DEV), top)
+    z = h.to(F) @ w.to(F).T + b.to(F)
+    want = torch.sort(z, -1, descending=True).indices[:, :top]
+    assert torch.equal(idx.cpu().long(), want)
+    assert err(wts, torch.softmax(torch.gather(z, 1, want), -1)) < 1e-5
+
+
+def test_router_bias_changes_the_choice_and_the_weights():
+    h = torch.zeros(1, 16, dtype=torch.bfloat16, device=DEV)
+    w = torch.zeros(4, 16, dtype=torch.bfloat16, device=DEV)
+    idx, wts = O.route_topk(h, w, torch.tensor([0.0, 3.0, -1.0, 2.0], device=DEV), 2)
+    assert idx.tolist() == [[1, 3]]
+    assert torch.allclose(wts.cpu(), torch.softmax(torch.tensor([[3.0, 2.0]]), -1), atol=1e-6)
+
+
+@BOTH
+@pytest.mark.parametrize("t,d,f,experts,top", [(1, 64, 40, 3, 2), (9, 96, 72, 5, 2), (60, 136, 200, 4, 3), (300, 64, 48, 4, 2),
+                                               (700, 256, 136, 6, 4), (20, 50, 36, 3, 1)])
+def test_experts(t, d, f, experts, top, dtype):
+    """Every route-tile width, sizes that fill no tile, experts without a token, rows whose ids are -1."""
+    h = rand(t, d).to(dtype)
+    w13 = rand(experts, 2, f, d, seed=1, std=d ** -0.5, dtype=torch.bfloat16)
+    w2 = rand(experts, d, f, seed=2, std=f ** -0.5, dtype=torch.bfloat16)
+    g = torch.Generator().manual_seed(5)
+    idx = torch.stack([torch.randperm(experts, generator=g)[:top] for _ in range(t)]).to(torch.int32)
+    idx[idx == 1] = 0 if top == 1 else idx[idx == 1]
+    if t > 4:
+        idx[3] = -1
+    wts = rand(t, top, seed=6)
+    got = O.gated_experts(h.to(DEV), idx.to(DEV), wts.to(DEV), w13.to(DEV), w2.to(DEV)).view(t, top, d)
+    for i in range(0, t, max(t // 25, 1)):
+        for j in range(top):
+            e = int(idx[i, j])
+            if e < 0:
+                continue
+            x = h[i].to(F)
+            want = w2[e].to(F) @ (P.silu(w13[e, 0].to(F) @ x) * (w13[e, 1].to(F) @ x))
+            assert err(got[i, j][None], want[None]) < 1.5 * TOL[dtype]
+
+
+@BOTH
+def test_embedding_feedback(dtype):
+    w = rand(50, 72, dtype=torch.bfloat16)
+    ids = torch.zeros(3, dtype=torch.int32, device=DEV)
+    feedback = torch.tensor([4, 9, 49, 0], dtype=torch.int32, device=DEV)
+    slots = torch.tensor([2, 0, 1], dtype=torch.int32, device=DEV)
+    x, act = O.embed_residual(ids, w.to(DEV), dtype, feedback, slots, True)
+    assert ids.tolist() == [49, 4, 9]
+    assert torch.equal(x.cpu(), w[[49, 4, 9]].float()) and torch.equal(act.cpu(), w[[49, 4, 9]].to(dtype))
