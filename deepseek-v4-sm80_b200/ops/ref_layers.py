@@ -23,7 +23,7 @@ def embed_residual(ids, weight, dtype, feedback, slots, want_act):
     if feedback is not None:
         ids.copy_(feedback[slots.long()])
     x = weight[ids.long()].float()
-    return x, (x.to(dtype) if want_act else None)
+    return x, (x.to(dtype, copy=True) if want_act else None)    # the stream changes in place
 
 
 def residual_norm(x, gain, eps, dtype, mul, rows, add, add2, vec, experts, cast):
@@ -35,7 +35,7 @@ def residual_norm(x, gain, eps, dtype, mul, rows, add, add2, vec, experts, cast)
         w = torch.where(idx >= 0, wts, torch.zeros_like(wts))
         x += (erows.float().view(*idx.shape, -1) * w[..., None]).sum(1)
     if gain is None:
-        return x.to(dtype) if cast else None
+        return x.to(dtype, copy=True) if cast else None
     y = x if rows is None else x[rows]
     return (_rms(y, eps) * gain * mul).to(dtype)
 
