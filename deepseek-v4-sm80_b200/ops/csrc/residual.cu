@@ -43,8 +43,8 @@ struct NormArgs {
   int d;
 };
 
-// One CTA per row.  The row stays in registers between the two passes when it has at most 8 x 4 values per thread.
-template <typename T, bool VEC>
+// One CTA per row.  NV > 0: the row stays in registers between the two passes, NV x 4 values per thread.
+template <typename T, int NV>
 __global__ void __launch_bounds__(256) residual_norm_kernel(const NormArgs a, const T* __restrict__ erows,
                                                             T* __restrict__ out) {
   pdl_entry();
@@ -53,8 +53,7 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const NormArgs a, co
   const size_t src = (size_t)(a.rows_idx ? a.rows_idx[r] : r) * d;
   const bool adds = a.add || a.add2 || a.vec || a.topk > 0;
   float ss = 0.f;
-  if constexpr (VEC) {
-    constexpr int NV = 8;
+  if constexpr (NV > 0) {
     float4 keep[NV];
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
@@ -76,6 +75,7 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const NormArgs a, co
         }
         if (a.topk > 0) {
           float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
           for (int k = 0; k < a.topk; ++k) {
             if (a.eidx[r * a.topk + k] < 0) continue;
             const float w = a.wts[r * a.topk + k];
@@ -141,11 +141,17 @@ __global__ void __launch_bounds__(256) silu_mul_kernel(const T* __restrict__ gu,
 
 template <typename T>
 int launch_norm(const NormArgs& a, const void* erows, void* out, int rows, cudaStream_t st) {
-  const bool vec = a.d % 4 == 0 && a.d <= 8192;
-  if (vec)
-    dsv4_launch(residual_norm_kernel<T, true>, rows, 256, 0, st, a, (const T*)erows, (T*)out);
+  auto go = [&](auto kern) { dsv4_launch(kern, rows, 256, 0, st, a, (const T*)erows, (T*)out); };
+  if (a.d % 4 || a.d > 8192)
+    go(residual_norm_kernel<T, 0>);
+  else if (a.d <= 1024)
+    go(residual_norm_kernel<T, 1>);
+  else if (a.d <= 2048)
+    go(residual_norm_kernel<T, 2>);
+  else if (a.d <= 4096)
+    go(residual_norm_kernel<T, 4>);
   else
-    dsv4_launch(residual_norm_kernel<T, false>, rows, 256, 0, st, a, (const T*)erows, (T*)out);
+    go(residual_norm_kernel<T, 8>);
   return (int)cudaGetLastError();
 }
 

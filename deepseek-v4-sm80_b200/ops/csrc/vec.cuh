@@ -21,6 +21,23 @@ __device__ __forceinline__ void st_f4(__nv_bfloat16* p, const float4& v) {
   u.y = *reinterpret_cast<uint32_t*>(&b);
   *reinterpret_cast<uint2*>(p) = u;
 }
+// W consecutive values, W = 1 or 4 (then aligned to four elements)
+template <int W>
+__device__ __forceinline__ void ld_w(const float* p, float (&v)[W]) {
+  if constexpr (W == 4) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    v[0] = f.x, v[1] = f.y, v[2] = f.z, v[3] = f.w;
+  } else {
+    v[0] = *p;
+  }
+}
+template <int W, typename T>
+__device__ __forceinline__ void st_w(T* p, const float (&v)[W]) {
+  if constexpr (W == 4)
+    st_f4(p, make_float4(v[0], v[1], v[2], v[3]));
+  else
+    st_f(p, v[0]);
+}
 // sum over the CTA (blockDim.x a multiple of 32, at most 1024); sh: 32 floats
 __device__ __forceinline__ float cta_sum(float v, float* sh) {
   v = warp_sum(v);

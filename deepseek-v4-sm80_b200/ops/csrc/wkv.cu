@@ -15,7 +15,7 @@ namespace {
 // zeros at position 0);  out[t][m] = h + (h' - h) * mu[m] for the n_mix mixes.  A request's last row goes to the slot:
 // directly if it is also the first one, else to `tail` (other CTAs may still have to read the slot), from where
 // wkv_scan_kernel moves it.
-template <typename T>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) shift_mix_kernel(const float* __restrict__ x, const float* __restrict__ gain,
                                                         float eps, const float* __restrict__ mu, int n_mix,
                                                         float* __restrict__ prev, float* __restrict__ tail,
@@ -23,17 +23,21 @@ __global__ void __launch_bounds__(256) shift_mix_kernel(const float* __restrict_
                                                         T* __restrict__ out, int rows, int d) {
   pdl_entry();
   __shared__ float sh[32];
+  constexpr int W = VEC ? 4 : 1;   // columns per access
   const int t = blockIdx.x, tid = threadIdx.x;
   const bool first = seg_first(slots, pos, t), last = seg_last(slots, pos, t, rows);
   const float* xc = x + (size_t)t * d;
   const float* xp = xc - d;  // only read when !first
   float sc = 0.f, sp = 0.f;
-  for (int i = tid; i < d; i += 256) {
-    const float v = xc[i];
-    sc += v * v;
-    if (!first) {
-      const float q = xp[i];
-      sp += q * q;
+#pragma unroll 2
+  for (int i = tid * W; i < d; i += 256 * W) {
+    float v[W], q[W];
+    ld_w<W>(xc + i, v);
+    if (!first) ld_w<W>(xp + i, q);
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+      sc += v[j] * v[j];
+      if (!first) sp += q[j] * q[j];
     }
   }
   const float rc = 1.f / sqrtf(cta_sum(sc, sh) / d + eps);
@@ -41,19 +45,28 @@ __global__ void __launch_bounds__(256) shift_mix_kernel(const float* __restrict_
   const bool fresh = pos[t] == 0;
   float* ps = prev + (size_t)slots[t] * d;
   float* ts = tail + (size_t)slots[t] * d;
-  for (int i = tid; i < d; i += 256) {
-    const float g = gain[i];
-    const float h = xc[i] * rc * g;
-    const float hp = first ? (fresh ? 0.f : ps[i]) : xp[i] * rp * g;
-    const float dh = hp - h;
-    T* o = out + (size_t)t * n_mix * d + i;
-    for (int m = 0; m < n_mix; ++m) st_f(o + (size_t)m * d, h + dh * mu[m * d + i]);
-    if (last) {
-      if (first)
-        ps[i] = h;
-      else
-        ts[i] = h;
+#pragma unroll 2
+  for (int i = tid * W; i < d; i += 256 * W) {
+    float g[W], h[W], hp[W], m[W], r[W];
+    ld_w<W>(gain + i, g);
+    ld_w<W>(xc + i, h);
+    if (!first)
+      ld_w<W>(xp + i, hp);
+    else if (!fresh)
+      ld_w<W>(ps + i, hp);
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+      h[j] *= rc * g[j];
+      hp[j] = (first ? (fresh ? 0.f : hp[j]) : hp[j] * rp * g[j]) - h[j];
     }
+    T* o = out + (size_t)t * n_mix * d + i;
+    for (int n = 0; n < n_mix; ++n) {
+      ld_w<W>(mu + (size_t)n * d + i, m);
+#pragma unroll
+      for (int j = 0; j < W; ++j) r[j] = h[j] + hp[j] * m[j];
+      st_w<W>(o + (size_t)n * d, r);
+    }
+    if (last) st_w<W>((first ? ps : ts) + i, h);
   }
 }
 
@@ -245,6 +258,17 @@ __global__ void __launch_bounds__(ScanCfg<DP>::THREADS) wkv_scan_kernel(const T*
   }
 }
 
+template <typename T>
+void launch_shift(const float* x, const float* gain, float eps, const float* mu, int n_mix, float* prev, float* tail,
+                  const int* slots, const int* pos, void* out, int rows, int d, cudaStream_t st) {
+  if (d % 4 == 0)
+    dsv4_launch(shift_mix_kernel<T, true>, rows, 256, 0, st, x, gain, eps, mu, n_mix, prev, tail, slots, pos, (T*)out,
+                rows, d);
+  else
+    dsv4_launch(shift_mix_kernel<T, false>, rows, 256, 0, st, x, gain, eps, mu, n_mix, prev, tail, slots, pos, (T*)out,
+                rows, d);
+}
+
 template <typename T, int DP>
 int launch_scan(const void* p, void* y, const ScanArgs& a, int segs, cudaStream_t st) {
   const size_t smem = ScanCfg<DP>::smem(sizeof(T));
@@ -275,11 +299,9 @@ DSV4_API int dsv4_shift_mix(const float* x, const float* gain, float eps, const 
   if (rows <= 0) return 0;
   if (n_mix < 1) return 622;
   if (fp32)
-    dsv4_launch(shift_mix_kernel<float>, rows, 256, 0, st, x, gain, eps, mu, n_mix, prev, tail, slots, pos, (float*)out,
-                rows, d);
+    launch_shift<float>(x, gain, eps, mu, n_mix, prev, tail, slots, pos, out, rows, d, st);
   else
-    dsv4_launch(shift_mix_kernel<__nv_bfloat16>, rows, 256, 0, st, x, gain, eps, mu, n_mix, prev, tail, slots, pos,
-                (__nv_bfloat16*)out, rows, d);
+    launch_shift<__nv_bfloat16>(x, gain, eps, mu, n_mix, prev, tail, slots, pos, out, rows, d, st);
   return (int)cudaGetLastError();
 }
 

@@ -37,7 +37,9 @@ struct ChunkCfg {
   static constexpr int CG = DP / 4, THREADS = 8 * CG;
   static constexpr int LD = DP + 4;                    // row stride of the [token][channel] arrays
   static constexpr int SMEM_STATE = (2 * kC * LD + kC * DP) * 4;
-  static constexpr int SMEM_OUT = (3 * kC * LD + 2 * kC * DP + DP * DP + kC * (kC + 4) + DP * (kC + 4)) * 4;
+  // the state moves into the space of log decays, r and k once A is complete, where it fits
+  static constexpr bool ALIAS = DP * DP <= 3 * kC * LD;
+  static constexpr int SMEM_OUT = (3 * kC * LD + kC * DP + (ALIAS ? 0 : DP * DP) + kC * (kC + 4) + DP * (kC + 4)) * 4;
 };
 
 // Inclusive running sums of log w over the chunk's tokens, one channel per thread (channels past d stay zero).
@@ -103,7 +105,7 @@ __global__ void __launch_bounds__(ChunkCfg<DP>::THREADS) wkv_chunk_state_kernel(
   __syncthreads();
   for (int i = tid; i < kC * DP; i += C::THREADS) {
     const int t = i / DP, e = i % DP;
-    ks[t * LD + e] *= expf(ls[(kC - 1) * LD + e] - ls[t * LD + e]);
+    ks[t * LD + e] *= __expf(ls[(kC - 1) * LD + e] - ls[t * LD + e]);
   }
   __syncthreads();
   const int rg = tid / C::CG, cg = tid % C::CG;
@@ -137,39 +139,43 @@ __global__ void __launch_bounds__(ChunkCfg<DP>::THREADS) wkv_chunk_state_kernel(
   if (tid < d) a.decay[((size_t)c * a.heads + head) * d + tid] = expf(ls[(kC - 1) * LD + tid]);
 }
 
-// One thread per state element.  segs: [n][4] = slot, first chunk, chunks, first row.
-__global__ void __launch_bounds__(256) wkv_chunk_carry_kernel(float* __restrict__ us, const float* __restrict__ decay,
+// One thread per W consecutive state elements of one key (W = 4 when d allows).  segs: [n][4] = slot, first chunk, chunks,
+// first row.
+template <int W>
+__global__ void __launch_bounds__(128) wkv_chunk_carry_kernel(float* __restrict__ us, const float* __restrict__ decay,
                                                               float* __restrict__ state, float* __restrict__ prev,
                                                               const float* __restrict__ tail, int width,
                                                               const int* __restrict__ segs, const int* __restrict__ pos,
                                                               const int* __restrict__ seg_rows, int heads, int d) {
   pdl_entry();
-  const int seg = blockIdx.x, head = blockIdx.y, e = blockIdx.z * 256 + threadIdx.x;
+  const int seg = blockIdx.x, head = blockIdx.y, e = (blockIdx.z * 128 + threadIdx.x) * W;
   const int slot = segs[seg * 4], c0 = segs[seg * 4 + 1], n = segs[seg * 4 + 2], row = segs[seg * 4 + 3];
   const size_t dd = (size_t)d * d, step = (size_t)heads * dd, pstep = (size_t)heads * d;
   if (e < d * d) {
     float* st = state + ((size_t)slot * heads + head) * dd + e;
-    float s = pos[row] == 0 ? 0.f : *st;
+    float s[W] = {};
+    if (pos[row] != 0) ld_w<W>(st, s);
     float* u = us + ((size_t)c0 * heads + head) * dd + e;
     const float* w = decay + ((size_t)c0 * heads + head) * d + e / d;
     constexpr int B = 8;
     for (int c = 0; c < n; c += B) {
-      float uv[B], wv[B];
+      float uv[B][W], wv[B];
 #pragma unroll
       for (int j = 0; j < B; ++j)
-        if (c + j < n) uv[j] = u[(c + j) * step], wv[j] = w[(c + j) * pstep];
+        if (c + j < n) ld_w<W>(u + (c + j) * step, uv[j]), wv[j] = w[(c + j) * pstep];
 #pragma unroll
       for (int j = 0; j < B; ++j)
         if (c + j < n) {
-          u[(c + j) * step] = s;
-          s = fmaf(wv[j], s, uv[j]);
+          st_w<W>(u + (c + j) * step, s);
+#pragma unroll
+          for (int q = 0; q < W; ++q) s[q] = fmaf(wv[j], s[q], uv[j][q]);
         }
     }
-    *st = s;
+    st_w<W>(st, s);
   }
   if (seg_rows[seg + 1] - seg_rows[seg] > 1 && blockIdx.z == 0) {  // the token shift's last row (wkv.cu: shift_mix_kernel)
     const int per = (width + heads - 1) / heads;
-    for (int i = head * per + threadIdx.x; i < min((head + 1) * per, width); i += 256)
+    for (int i = head * per + threadIdx.x; i < min((head + 1) * per, width); i += 128)
       prev[(size_t)slot * width + i] = tail[(size_t)slot * width + i];
   }
 }
@@ -185,25 +191,20 @@ __global__ void __launch_bounds__(ChunkCfg<DP>::THREADS) wkv_chunk_out_kernel(co
   float* rs = ls + kC * LD;          // [kC][LD] r
   float* ks = rs + kC * LD;          // [kC][LD] k
   float* vs = ks + kC * LD;          // [kC][DP]
-  float* gs = vs + kC * DP;          // [kC][DP] gate projections
-  float* ss = gs + kC * DP;          // [DP][DP] state before the chunk
-  float* at = ss + DP * DP;          // [kC (s)][TL (t)] A transposed
+  float* at = vs + kC * DP;          // [kC (s)][TL (t)] A transposed
   float* rt = at + kC * TL;          // [DP][TL] r e^{L_{t-1}} transposed
+  float* ss = C::ALIAS ? ls : rt + DP * TL;  // [DP][DP] state before the chunk
   const int c = blockIdx.x, head = blockIdx.y, d = a.d, tid = threadIdx.x, hd = a.heads * d;
   const int t0 = a.chunks[c * 2], m = a.chunks[c * 2 + 1];
   load_rows<T, DP>(p, a, t0, m, head, 0, rs, LD);
   load_rows<T, DP>(p, a, t0, m, head, 1, ks, LD);
   load_rows<T, DP>(p, a, t0, m, head, 2, vs, DP);
-  load_rows<T, DP>(p, a, t0, m, head, 3, gs, DP);
+  constexpr int NS = DP * DP / 4 / C::THREADS;
   const float* sg = a.us + ((size_t)c * a.heads + head) * d * d;
+  float4 sv[NS];                     // in flight while A is computed
   if (d == DP) {
-    for (int i = tid; i < DP * DP / 4; i += C::THREADS)
-      reinterpret_cast<float4*>(ss)[i] = reinterpret_cast<const float4*>(sg)[i];
-  } else {
-    for (int i = tid; i < DP * DP; i += C::THREADS) {
-      const int k = i / DP, e = i % DP;
-      ss[i] = (k < d && e < d) ? sg[(size_t)k * d + e] : 0.f;
-    }
+#pragma unroll
+    for (int n = 0; n < NS; ++n) sv[n] = reinterpret_cast<const float4*>(sg)[tid + n * C::THREADS];
   }
   log_decays<DP>(a, t0, m, head, ls);
   for (int i = tid; i < kC * TL; i += C::THREADS) at[i] = 0.f;
@@ -211,7 +212,7 @@ __global__ void __launch_bounds__(ChunkCfg<DP>::THREADS) wkv_chunk_out_kernel(co
   // r e^{L_{t-1}}, key-major
   for (int i = tid; i < kC * DP; i += C::THREADS) {
     const int t = i % kC, e = i / kC;
-    rt[e * TL + t] = rs[t * LD + e] * (t > 0 ? expf(ls[(t - 1) * LD + e]) : 1.f);
+    rt[e * TL + t] = rs[t * LD + e] * (t > 0 ? __expf(ls[(t - 1) * LD + e]) : 1.f);
   }
   // A inside the two diagonal blocks of 16 tokens, the pair's own exponent per channel; s == t is the bonus
   for (int i = tid; i < 2 * 136; i += C::THREADS) {
@@ -221,7 +222,17 @@ __global__ void __launch_bounds__(ChunkCfg<DP>::THREADS) wkv_chunk_out_kernel(co
     const float *rp = rs + (b + t) * LD, *kp = ks + (b + s) * LD;
     float acc = 0.f;
     if (s == t) {
-      for (int e = 0; e < d; ++e) acc = fmaf(rp[e] * a.u[head * d + e], kp[e], acc);
+      const float* up = a.u + head * d;
+      if (d % 4 == 0) {
+#pragma unroll 4
+        for (int e = 0; e < d; e += 4) {
+          const float4 r = *reinterpret_cast<const float4*>(rp + e), k = *reinterpret_cast<const float4*>(kp + e);
+          const float4 u = *reinterpret_cast<const float4*>(up + e);
+          acc = fmaf(r.x * u.x, k.x, fmaf(r.y * u.y, k.y, fmaf(r.z * u.z, k.z, fmaf(r.w * u.w, k.w, acc))));
+        }
+      } else {
+        for (int e = 0; e < d; ++e) acc = fmaf(rp[e] * up[e], kp[e], acc);
+      }
     } else {
       const float *lt = ls + (b + t - 1) * LD, *lp = ls + (b + s) * LD;
 #pragma unroll 4
@@ -242,8 +253,8 @@ __global__ void __launch_bounds__(ChunkCfg<DP>::THREADS) wkv_chunk_out_kernel(co
   for (int i = tid; i < 16 * DP; i += C::THREADS) {
     const int t = i / DP, e = i % DP;
     const float l15 = ls[15 * LD + e];
-    rs[(16 + t) * LD + e] *= expf(ls[(15 + t) * LD + e] - l15);
-    ks[t * LD + e] *= expf(l15 - ls[t * LD + e]);
+    rs[(16 + t) * LD + e] *= __expf(ls[(15 + t) * LD + e] - l15);
+    ks[t * LD + e] *= __expf(l15 - ls[t * LD + e]);
   }
   __syncthreads();
   for (int i = tid; i < 256; i += C::THREADS) {
@@ -256,6 +267,16 @@ __global__ void __launch_bounds__(ChunkCfg<DP>::THREADS) wkv_chunk_out_kernel(co
       acc = fmaf(r.x, k.x, fmaf(r.y, k.y, fmaf(r.z, k.z, fmaf(r.w, k.w, acc))));
     }
     at[s * TL + 16 + t] = acc;
+  }
+  __syncthreads();
+  if (d == DP) {
+#pragma unroll
+    for (int n = 0; n < NS; ++n) reinterpret_cast<float4*>(ss)[tid + n * C::THREADS] = sv[n];
+  } else {
+    for (int i = tid; i < DP * DP; i += C::THREADS) {
+      const int k = i / DP, e = i % DP;
+      ss[i] = (k < d && e < d) ? sg[(size_t)k * d + e] : 0.f;
+    }
   }
   __syncthreads();
   // o: four tokens x four value columns per thread
@@ -282,11 +303,12 @@ __global__ void __launch_bounds__(ChunkCfg<DP>::THREADS) wkv_chunk_out_kernel(co
     for (int off = C::CG / 2; off > 0; off >>= 1) q += __shfl_xor_sync(0xffffffffu, q, off);
     if (t >= m) continue;
     const float inv = 1.f / sqrtf(q / d + a.eps);
+    const T* gp = p + (size_t)(t0 + t) * a.ld + 3 * hd + head * d + cg * 4;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int e = cg * 4 + j;
       if (e >= d) break;
-      const float g = gs[t * DP + e];
+      const float g = ld_f(gp + j);
       o[i][j] *= inv * a.gain[head * d + e] * (g / (1.f + expf(-g)));
     }
     T* dst = y + (size_t)(t0 + t) * hd + head * d + cg * 4;
@@ -314,8 +336,12 @@ int launch_chunks(const void* p, void* y, const ChunkArgs& a, int n_chunks, floa
   }
   const dim3 grid(n_chunks, a.heads);
   dsv4_launch(wkv_chunk_state_kernel<T, DP>, grid, C::THREADS, C::SMEM_STATE, st, (const T*)p, a);
-  dsv4_launch(wkv_chunk_carry_kernel, dim3(n_segs, a.heads, (a.d * a.d + 255) / 256), 256, 0, st, a.us, a.decay, state,
-              prev, tail, width, segs, pos, seg_rows, a.heads, a.d);
+  if (a.d % 4 == 0)
+    dsv4_launch(wkv_chunk_carry_kernel<4>, dim3(n_segs, a.heads, (a.d * a.d / 4 + 127) / 128), 128, 0, st, a.us, a.decay,
+                state, prev, tail, width, segs, pos, seg_rows, a.heads, a.d);
+  else
+    dsv4_launch(wkv_chunk_carry_kernel<1>, dim3(n_segs, a.heads, (a.d * a.d + 127) / 128), 128, 0, st, a.us, a.decay,
+                state, prev, tail, width, segs, pos, seg_rows, a.heads, a.d);
   dsv4_launch(wkv_chunk_out_kernel<T, DP>, grid, C::THREADS, C::SMEM_OUT, st, (const T*)p, (T*)y, a);
   return (int)cudaGetLastError();
 }

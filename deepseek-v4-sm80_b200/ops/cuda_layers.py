@@ -82,12 +82,12 @@ def gated_experts(h, idx, wts, w13, w2):
     new = lambda n: torch.empty(routes, n, dtype=h.dtype, device=h.device)
     act, rows = new(f), new(d)
     if mma:
-        xs = new(d)
+        xs, sms = new(d), I(num_sms(h.device))
         nv.call("moe_gather_rows", nv.ptr(h), nv.ptr(xs), nv.ptr(plan), I(routes), I(max_tiles), I(top), I(d))
         nv.call("moe_bf16_gemm", I(1), I(nt), nv.ptr(w13), nv.ptr(xs), nv.ptr(plan), I(routes), I(max_tiles),
-                nv.ptr(act), I(e), I(f), I(d))
+                nv.ptr(act), I(e), I(f), I(d), sms)
         nv.call("moe_bf16_gemm", I(2), I(nt), nv.ptr(w2), nv.ptr(act), nv.ptr(plan), I(routes), I(max_tiles),
-                nv.ptr(rows), I(e), I(d), I(f))
+                nv.ptr(rows), I(e), I(d), I(f), sms)
         return rows
     gu = new(2 * f)
     nv.call("moe_gemm_simt", nv.ptr(h), nv.ptr(w13), nv.ptr(gu), nv.ptr(plan), I(routes), I(max_tiles), I(e), I(2 * f),
@@ -143,7 +143,7 @@ def latent_attention(q, cache, fb, scale):
 # MINISGL_LATENT_PREFILL: auto (by cost), expanded (wherever the kernel can) or absorbed
 LATENT_PREFILL = os.environ.get("MINISGL_LATENT_PREFILL", "auto")
 EXPAND_BYTES = 4 << 30                        # bound of the expanded keys and values of one call
-ABSORBED_TFLOPS, EXPANDED_TFLOPS, GEMM_TFLOPS, EXPAND_US = 200.0, 500.0, 450.0, 25.0    # measured rates
+ABSORBED_TFLOPS, EXPANDED_TFLOPS, GEMM_TFLOPS, EXPAND_US = 200.0, 900.0, 600.0, 25.0    # measured rates
 
 
 def prefers_expanded(q_dtype, fb, heads: int, dim: int, vdim: int, rank: int) -> bool:

@@ -150,6 +150,13 @@ def _tma_ok(x2, w, k: int) -> bool:
             and x2.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
+PREFILL_MIN_TILES = 100     # 128 x 256 output tiles from which the persistent kernel (csrc/gemm_prefill.cu) fills the GPU
+
+
+def prefill_tiles(m: int, n: int, groups: int) -> int:
+    return -(-m // 128) * -(-n // 256) * groups if m > 128 else 0
+
+
 def linear(x, w, out=None, out_dtype=None, accumulate=False, act=None):
     """``x [T, K] @ w [N, K]^T`` for bf16 weights and bf16 or fp32 activations (rows may be strided).  bf16 runs on the
     tensor cores; fp32 activations, and bf16 rows that TMA cannot fetch, on the fp32 kernel (csrc/gemm_simt.cu)."""
@@ -171,6 +178,10 @@ def grouped_linear(x, w, groups: int, out=None, out_dtype=None, accumulate=False
     assert w.dtype == torch.bfloat16 and w.stride(-1) == 1 and x.stride(-1) == 1 and out.stride(-1) == 1
     f32 = I(1 if out.dtype == torch.float32 else 0)
     if _tma_ok(x, w, k):
+        if prefill_tiles(t, n, groups) >= PREFILL_MIN_TILES:
+            nv.call("gemm_prefill", nv.ptr(x), nv.ptr(w), nv.ptr(out), I(t), I(n), I(k), I(x.stride(0)), I(w.stride(0)),
+                    I(out.stride(0)), f32, I(1 if accumulate else 0), I(ACTS[act]), I(groups), I(NUM_SMS_HINT))
+            return out
         bn, splits = pick_tiling(t, n, (k + 63) // 64, groups, False, 0, 0)
         ws, cnt = _ws(t, n, bn, groups, splits, x.device)
         nv.call("gemm_bf16", nv.ptr(x), nv.ptr(w), nv.ptr(out), I(t), I(n), I(k), I(x.stride(0)), I(w.stride(0)),

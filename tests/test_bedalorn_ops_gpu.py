@@ -67,6 +67,24 @@ def test_linear(m, k, n, act, dtype):
     assert err(acc, y + base.to(F)) < 2e-5
 
 
+@pytest.mark.parametrize("m,k,n,groups,act", [(4000, 72, 1030, 1, "relu2"), (1300, 200, 2600, 1, None), (2050, 40, 264, 7, "tanh"),
+                                              (129, 64, 13000, 1, None)])
+def test_projections_of_many_rows(m, k, n, groups, act):
+    """The persistent kernel: ragged tiles in every direction, batches, fp32 accumulation and bf16 results."""
+    from minisgl.ops.gemm import PREFILL_MIN_TILES, prefill_tiles
+
+    assert prefill_tiles(m, n, groups) >= PREFILL_MIN_TILES
+    x, w = rand(m, groups * k + 8, dtype=torch.bfloat16), rand(groups * n, k, seed=1, std=k ** -0.5, dtype=torch.bfloat16)
+    f = {"relu2": lambda v: v.clamp_min(0) ** 2, "tanh": torch.tanh, None: lambda v: v}[act]
+    want = f(torch.cat([x[:, i * k:(i + 1) * k].float() @ w[i * n:(i + 1) * n].float().T for i in range(groups)], 1))
+    xs = x.to(DEV)[:, : groups * k]
+    assert err(O.grouped_linear(xs, w.to(DEV), groups, act=act), want) < 1e-2
+    base = rand(m, groups * n, seed=2)
+    acc = base.to(DEV)
+    O.grouped_linear(xs, w.to(DEV), groups, out=acc, accumulate=True, act=act)
+    assert err(acc, want + base) < 1e-4
+
+
 @BOTH
 def test_grouped_linear_reads_column_slices(dtype):
     t, groups, k, n = 70, 3, 40, 24
