@@ -65,6 +65,7 @@ def _decode_once(llm, batch: int, context: int) -> None:
             llm.cache.allocate(r, min(upto, context))
             llm.cache.release_swa_behind(r)
         reqs.append(r)
+    llm.engine.last_token.copy_(torch.randint(0, llm.engine.model_config.vocab_size, llm.engine.last_token.shape))
     b = Batch(reqs, "decode")
     llm._prepare_batch(b)
     llm.engine.forward_batch(b, llm.engine.sampler.prepare(b))

@@ -69,6 +69,10 @@ class Engine:
                              f"{config.dtype}")
         if tp.size > self.family.max_tp:
             raise ValueError(f"{self.family.name} models run on at most {self.family.max_tp} GPU(s), not {tp.size}")
+        if self.is_cuda:
+            from ..ops import native
+
+            native.prefer_kernel_set(self.family.kernel_set)
         self.page_size = config.page_size
         self.cpu_group, self.comm = comm_mod.init_distributed(
             tp, self.device, config.distributed_addr, config.distributed_timeout, fused=config.use_pynccl,

@@ -3,7 +3,7 @@ and build its KV pool and build its model; the engine, the scheduler and the com
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Any, Callable, Dict, List, Tuple
+from typing import Any, Callable, Dict, List, Optional, Tuple
 
 import torch
 
@@ -37,6 +37,7 @@ class ModelFamily:
     pool: Callable[..., Any]                        # (cfg, PoolSizes, device, dtype)
     build: Callable[..., Any]                       # (cfg, weights, pool, comm, moe_mode, dtype)
     context_classes: Callable[[Any, int], List[int]]   # graph context classes below the limit
+    kernel_set: Optional[str] = None                # ops/build.py: what a checkout without a built library compiles
 
 
 # --------------------------------------------------------------------------- DeepSeek-V4
@@ -138,7 +139,7 @@ FAMILIES = {
                                          _dsv4_load, _dsv4_draw, _dsv4_budget, _dsv4_pool, _dsv4_build, _dsv4_classes),
     BEDALORN: ModelFamily("bedalorn", BedalornConfig, BedalornConfig.from_dict, (torch.bfloat16, torch.float32), 1,
                           _bedalorn_load, _bedalorn_draw, _bedalorn_budget, _bedalorn_pool, _bedalorn_build,
-                          _bedalorn_classes),
+                          _bedalorn_classes, "layered"),
 }
 
 

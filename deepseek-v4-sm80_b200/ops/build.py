@@ -10,6 +10,9 @@ Two shared objects are produced next to this file:
   page-table builders and tensor checks.  It needs no CUDA at run time, so CPU-only
   tests can load it.
 
+A checkout that serves one model family without a prior build compiles only that family's kernel set
+(``KERNEL_SETS``) into ``libdsv4_b200_<set>.so``; the full library, where it exists, serves every family.
+
 The reference builds its native code lazily on first use through TVM-FFI
 (python/minisgl/kernel/utils.py:53-129); here the build is an explicit step so the
 objects travel with the source tree.
@@ -29,6 +32,17 @@ CSRC = HERE / "csrc"
 BUILD = HERE / "build"
 CUDA_LIB = HERE / "libdsv4_b200.so"
 HOST_LIB = HERE / "libdsv4_host.so"
+
+# sources (csrc/<name>.cu) a model family's forward pass and sampling need
+KERNEL_SETS = {
+    "layered": ("common", "comm", "elementwise", "sampling", "gemm_tcgen05", "gemm_prefill", "gemm_simt", "moe", "moe_bf16",
+                "residual", "latent_attn", "flash_attn", "wkv", "wkv_chunk"),
+}
+
+
+def cuda_lib_path(kernel_set=None) -> Path:
+    return CUDA_LIB if kernel_set is None else HERE / f"libdsv4_b200_{kernel_set}.so"
+
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -62,13 +76,14 @@ def _run(cmd, verbose):
         print(r.stdout, r.stderr, flush=True)
 
 
-def build_cuda(force: bool = False, verbose: bool = False, ptxas_v: bool = False) -> Path:
-    srcs = sorted(CSRC.glob("*.cu"))
+def build_cuda(force: bool = False, verbose: bool = False, ptxas_v: bool = False, kernel_set=None) -> Path:
+    srcs = sorted(CSRC.glob("*.cu")) if kernel_set is None else [CSRC / f"{n}.cu" for n in KERNEL_SETS[kernel_set]]
     hdrs = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
-    stamp = BUILD / "cuda.stamp"
+    lib = cuda_lib_path(kernel_set)
+    stamp = BUILD / f"cuda{'_' + kernel_set if kernel_set else ''}.stamp"
     dig = _digest(srcs + hdrs)
-    if not force and CUDA_LIB.exists() and stamp.exists() and stamp.read_text() == dig:
-        return CUDA_LIB
+    if not force and lib.exists() and stamp.exists() and stamp.read_text() == dig:
+        return lib
     BUILD.mkdir(exist_ok=True)
     nvcc = _nvcc()
     hdr_dig = _digest(hdrs)
@@ -87,9 +102,9 @@ def build_cuda(force: bool = False, verbose: bool = False, ptxas_v: bool = False
     with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 1)) as ex:
         objs = list(ex.map(one, srcs))
     _run([nvcc, "-gencode", "arch=compute_100a,code=sm_100a", "-shared", "-Xcompiler", "-fPIC", *objs,
-          "-o", CUDA_LIB, "-lcudart_static", "-lpthread", "-ldl", "-lrt"], verbose)
+          "-o", lib, "-lcudart_static", "-lpthread", "-ldl", "-lrt"], verbose)
     stamp.write_text(dig)
-    return CUDA_LIB
+    return lib
 
 
 def build_host(force: bool = False, verbose: bool = False) -> Path:

@@ -23,15 +23,26 @@ class NativeError(RuntimeError):
     pass
 
 
+_KERNEL_SET = None
+
+
+def prefer_kernel_set(name) -> None:
+    """Named before the library is first used: where no full library has been built, only this set's sources are."""
+    global _KERNEL_SET
+    _KERNEL_SET = name
+
+
 def cuda_lib() -> ctypes.CDLL:
     """Loads (building first if it is missing and nvcc exists) the sm_100a kernel library."""
     global _CUDA_LIB
     if _CUDA_LIB is None:
-        path = _HERE / "libdsv4_b200.so"
-        if not path.exists() or os.environ.get("MINISGL_REBUILD_KERNELS") == "1":
-            from . import build
+        from . import build
 
-            build.build_cuda(verbose=False)
+        rebuild = os.environ.get("MINISGL_REBUILD_KERNELS") == "1"
+        kernel_set = None if build.CUDA_LIB.exists() or rebuild else _KERNEL_SET
+        path = build.cuda_lib_path(kernel_set)
+        if not path.exists() or rebuild:
+            build.build_cuda(verbose=False, kernel_set=kernel_set)
         _CUDA_LIB = ctypes.CDLL(str(path))
         _CUDA_LIB.dsv4_abi_version.restype = ctypes.c_int
     return _CUDA_LIB
