@@ -13,6 +13,8 @@ import sys
 from dataclasses import dataclass
 from typing import List, Optional, Tuple
 
+import torch
+
 from ..dsv4_release import RECIPES
 from ..parallel.info import DistributedInfo
 from ..scheduler.config import SchedulerConfig
@@ -60,7 +62,7 @@ class ServerArgs(SchedulerConfig):
 
 
 def build_parser() -> argparse.ArgumentParser:
-    p = argparse.ArgumentParser(prog="minisgl", description="B200-native DeepSeek-V4 serving engine")
+    p = argparse.ArgumentParser(prog="minisgl", description="B200-native serving engine (DeepSeek-V4, Bedalorn)")
     p.add_argument("--model", "--model-path", dest="model_path", required=True)
     p.add_argument("--served-model-name", default=None)
     p.add_argument("--tp-size", "--tensor-parallel-size", dest="tp_size", type=int, default=1)
@@ -83,6 +85,8 @@ def build_parser() -> argparse.ArgumentParser:
     p.add_argument("--num-pages", dest="num_page_override", type=int, default=None)
     p.add_argument("--page-size", type=int, default=256)
     p.add_argument("--shell-mode", action="store_true")
+    p.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16",
+                   help="activation type of the layers (float32: families that run in 32-bit only)")
     p.add_argument("--device", choices=["cuda", "cpu"], default="cuda",
                    help="cpu runs the PyTorch oracle of every operator: for trying the serving stack without a GPU")
     return p
@@ -121,7 +125,7 @@ def parse_args(argv: Optional[List[str]] = None, run_shell: bool = False) -> Ser
         stats_log_interval=ns.stats_log_interval, disable_log_stats=ns.disable_log_stats,
         server_host=ns.server_host, server_port=ns.server_port, num_tokenizer=ns.num_tokenizer,
         served_model_name=ns.served_model_name, shell_mode=shell, explicit_fields=explicit, device=ns.device,
-        _unique_suffix=f".pid={os.getpid()}",
+        dtype=getattr(torch, ns.dtype), _unique_suffix=f".pid={os.getpid()}",
     )
     if shell:  # an interactive shell serves one request at a time and keeps the log quiet
         kw.update(max_running_req=1, cuda_graph_max_bs=1, silent_output=True)

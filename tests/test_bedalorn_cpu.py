@@ -200,3 +200,24 @@ def test_trace_rejects_bad_steps(mixed):
     for entry in ({"id": "a", "tokens": []}, {"id": "a", "tokens": [mixed.cfg["vocab"]]}, {"id": "a", "tokens": [0] * 65}):
         with pytest.raises(ValueError):
             t.step([entry])
+
+
+def test_command_line_serves_the_model(tmp_path):
+    """``python -m minisgl``: the backend processes serve the design like any other model; the shell's answer is the plain
+    model's greedy continuation."""
+    from test_server_e2e_cpu import _write_tokenizer
+
+    case = K.Case("single", tmp_path / "model", "cpu", torch.float32)
+    _write_tokenizer(case.folder, case.cfg["vocab"])
+    env = dict(os.environ, PYTHONPATH=ROOT + os.pathsep + os.environ.get("PYTHONPATH", ""), LOG_LEVEL="ERROR",
+               MINISGL_SHELL_MAX_TOKENS="5", MINISGL_SHELL_TEMPERATURE="0.0")
+    r = subprocess.run([sys.executable, "-m", "minisgl", "--model", case.folder, "--device", "cpu", "--dtype", "float32",
+                        "--shell-mode", "--page-size", "16", "--num-pages", "16", "--context-length", "128"],
+                       cwd=ROOT, env=env, input="w10 w11 w12\n/exit\n", capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0, r.stdout[-1000:] + r.stderr[-2000:]
+    ids = [10, 11, 12]
+    for _ in range(5):
+        case.plain.reset()
+        ids.append(int(case.plain.step(ids)[-1].argmax()))
+    names = {0: "<s>", 1: "</s>", 2: "<unk>", 3: "<think>", 4: "</think>"}
+    assert " ".join(names.get(i, f"w{i}") for i in ids[3:]) in " ".join(r.stdout.split()), (ids, r.stdout)
