@@ -7,7 +7,7 @@ cache manager, every step is one prepared batch (portions of prompts beside sing
 is a decode batch and replays the captured graph), and a request that ends gives its pages and its slot back.
 
 A step is one JSON object on a line:
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": ["a"]}
+    {"step": 4, "entries": [{"id": "x", "tokens": [11, 2], "want": [1]}, {"id": "y", "tokens": [40]}], "end": ["y"]}
 ``want``: places among the entry's tokens whose logits are written (in order) to OUT/<step>.f32 as little-endian fp32
 [wanted, vocab].  After every step the line "done <step>" is printed.
 """

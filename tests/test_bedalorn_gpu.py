@@ -34,10 +34,10 @@ def test_layers_one_by_one(case):
     case.want(toks)
     assert len(seen) == len(case.plain.residuals)
     for n, (got, want) in enumerate(zip(seen, case.plain.residuals)):
-        if case.dtype == torch.float32:
-            assert P.rel_err(got, want) < 3e-5, n
-        else:
-            case.compare(got, want, n)
+        case.compare(got, want, n)
+        if case.dtype == torch.float32:      # a few positions amplify rounding (a head's norm of a small output), most do not
+            d = (got.cpu().to(P.F) - want).pow(2).mean(-1).sqrt() / want.pow(2).mean(-1).sqrt()
+            assert float(d.median()) < 5e-6, (n, float(d.median()))
 
 
 def test_schedules(case):
