@@ -4,7 +4,9 @@ with the same weights."""
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Any, Dict, List, Optional, Tuple
+from typing import Any, Dict, Optional, Tuple
+
+from .layered_config import DenseSpec, LayeredConfig, LayerSpec, LoopSpec, parse_loop, serving_limits
 
 ARCHITECTURE = "Bedalorn"
 
@@ -25,11 +27,6 @@ class WKVSpec:
 
 
 @dataclass(frozen=True)
-class DenseSpec:
-    ff: int
-
-
-@dataclass(frozen=True)
 class ExpertsSpec:
     ff: int
     experts: int
@@ -37,28 +34,7 @@ class ExpertsSpec:
 
 
 @dataclass(frozen=True)
-class LayerSpec:
-    mixer: Any
-    ff: Any           # DenseSpec, ExpertsSpec or None
-
-
-@dataclass(frozen=True)
-class LoopSpec:
-    start: int
-    stop: int
-    times: int
-
-
-@dataclass(frozen=True)
-class LayerRun:
-    """One pass of one layer.  ``enters``: the number of the loop pass that begins right before it, or None."""
-
-    layer: int
-    enters: Optional[int] = None
-
-
-@dataclass(frozen=True)
-class BedalornConfig:
+class BedalornConfig(LayeredConfig):
     layers: Tuple[LayerSpec, ...]
     hidden_size: int
     vocab_size: int
@@ -72,28 +48,9 @@ class BedalornConfig:
     model_type: str = "bedalorn"
     window_size: int = 0
 
-    @property
-    def num_layers(self) -> int:
-        return len(self.layers)
-
-    @property
-    def runs(self) -> List[LayerRun]:
-        """The layer runs of one forward, in order."""
-        n, lp = len(self.layers), self.loop
-        if lp is None:
-            return [LayerRun(i) for i in range(n)]
-        out = [LayerRun(i) for i in range(lp.start)]
-        for t in range(lp.times):
-            out += [LayerRun(i, t if i == lp.start else None) for i in range(lp.start, lp.stop)]
-        return out + [LayerRun(i) for i in range(lp.stop, n)]
-
-    def run_stores(self) -> list:
-        """What every run keeps between forwards (kvcache/latent_pool.py)."""
-        out = []
-        for r in self.runs:
-            m = self.layers[r.layer].mixer
-            out.append(("latent", m.kv_rank) if isinstance(m, LatentAttentionSpec) else ("state", m.heads, m.dim))
-        return out
+    def mixer_store(self, mixer: Any) -> tuple:
+        latent = isinstance(mixer, LatentAttentionSpec)
+        return ("latent", mixer.kv_rank) if latent else ("state", mixer.heads, mixer.dim)
 
     # ------------------------------------------------------------------ config.json
     @staticmethod
@@ -101,17 +58,10 @@ class BedalornConfig:
         if raw.get("architecture") != ARCHITECTURE:
             raise ValueError(f"architecture {raw.get('architecture')!r} is not {ARCHITECTURE}")
         layers = tuple(_layer(i, e) for i, e in enumerate(raw["layers"]))
-        loop = raw.get("loop")
-        if loop:
-            loop = LoopSpec(int(loop["start"]), int(loop["stop"]), int(loop["times"]))
-            if not (0 <= loop.start < loop.stop <= len(layers) and loop.times >= 1):
-                raise ValueError(f"loop {loop} does not fit {len(layers)} layers")
         return BedalornConfig(
             layers=layers, hidden_size=int(raw["width"]), vocab_size=int(raw["vocab"]),
-            norm_eps=float(raw["norm"]["eps"]), logit_scale=float(raw["logit_scale"]), loop=loop or None,
-            max_position=int(raw.get("max_position_embeddings") or 1 << 20),
-            eos_token_id=int(raw["eos_token_id"]) if raw.get("eos_token_id") is not None else -1,
-            bos_token_id=int(raw["bos_token_id"]) if raw.get("bos_token_id") is not None else -1)
+            norm_eps=float(raw["norm"]["eps"]), logit_scale=float(raw["logit_scale"]),
+            loop=parse_loop(raw, len(layers)), **serving_limits(raw, 1 << 20))
 
     def to_dict(self) -> Dict[str, Any]:
         """The inverse of from_dict."""

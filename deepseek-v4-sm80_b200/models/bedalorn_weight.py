@@ -15,7 +15,7 @@ from typing import Callable, Dict
 import torch
 
 from .bedalorn_config import BedalornConfig, DenseSpec, LatentAttentionSpec
-from .weight import _index_checkpoint
+from .weight import tensor_reader
 
 MIXES = ("r", "k", "v", "g", "w")
 
@@ -114,20 +114,7 @@ def build_weights(cfg: BedalornConfig, get: Callable[[str], torch.Tensor], devic
 
 def load_checkpoint(folder: str, cfg: BedalornConfig, device) -> Dict[str, torch.Tensor]:
     """Streams a safetensors checkpoint into runtime tensors on ``device``."""
-    import safetensors
-
-    where = _index_checkpoint(folder)
-    handles: Dict[str, object] = {}
-
-    def fetch(name: str) -> torch.Tensor:
-        if name not in where:
-            raise KeyError(f"the checkpoint has no tensor {name!r}")
-        f = where[name]
-        if f not in handles:
-            handles[f] = safetensors.safe_open(f, framework="pt", device="cpu")
-        return handles[f].get_tensor(name)
-
-    return build_weights(cfg, fetch, device)
+    return build_weights(cfg, tensor_reader(folder), device)
 
 
 def random_weights(cfg: BedalornConfig, device, seed: int = 0, decay_rank: int = 64) -> Dict[str, torch.Tensor]:

@@ -1,8 +1,9 @@
-"""Layer mechanisms written against the operator facade, with their sizes and constants as parameters.  They read an fp32
-residual stream and add to it in place; activations between the projections have the serving type (bf16 or fp32)."""
+"""Layer mechanisms written against the operator facade, with their sizes and constants as parameters.  Those of the designs
+without a norm behind the sub-layer add to the fp32 residual stream in place, the others return their fp32 output;
+activations between the projections have the serving type (bf16 or fp32)."""
 from __future__ import annotations
 
-from typing import Dict
+from typing import Dict, Optional, Tuple
 
 import torch
 
@@ -75,3 +76,58 @@ class ExpertsFF:
     def __call__(self, h: torch.Tensor, x: torch.Tensor, fb: ForwardBatch) -> dict:
         idx, wts = O.route_topk(h, self.router, self.bias, self.top, fb.num_valid)
         return {"experts": (O.gated_experts(h, idx, wts, self.w13, self.w2), wts, idx)}
+
+
+class GroupedAttention:
+    """Causal attention over paged keys and values, several query heads to a key head.  Optional parts, by the weights there
+    are: projection biases (``qkv.b``), rotary positions on the leading dimensions (``freq``), a sink logit per head
+    (``sink``), a bias by distance (``rel``); and a query temperature (coef, every) that grows with the position."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, heads: int, kv_heads: int, dim: int, vdim: int, scale: float,
+                 softcap: float, q_temp: Optional[Tuple[float, int]] = None):
+        self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        self.scale, self.softcap, self.q_temp = scale, softcap, q_temp
+        self.qkv, self.o = w[prefix + "qkv"], w[prefix + "o"]
+        self.bias, self.freq, self.sink, self.rel = (w.get(prefix + n) for n in ("qkv.b", "freq", "sink", "rel"))
+
+    def __call__(self, h: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+        q = O.rotate_store(O.linear(h, self.qkv), self.bias, self.freq, self.q_temp, keys, values, fb, self.heads,
+                           self.kv_heads, self.dim, self.vdim)
+        v = O.grouped_attention(q, keys, values, fb, self.kv_heads, self.scale, self.softcap, self.sink, self.rel)
+        return O.linear(v, self.o, out_dtype=torch.float32)
+
+
+class ChannelDelta:
+    """Gated delta rule with one decay per head and key channel: short convolutions over q, k and v, unit query and key
+    vectors, the recurrence, per-head norm with a sigmoid gate."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, heads: int, kv_heads: int, dim: int, vdim: int, eps: float):
+        self.heads, self.kv_heads, self.dim, self.vdim, self.eps = heads, kv_heads, dim, vdim, eps
+        self.inp, self.a2, self.g2, self.o = (w[prefix + n] for n in ("in", "a2", "g2", "o"))
+        self.conv, self.a_log, self.dt_bias, self.gain = (w[prefix + n] for n in ("conv", "A_log", "dt_bias", "norm"))
+        up = lambda n: -(-n // 8) * 8          # every part of the merged projection starts at a multiple of eight
+        ra, rg = self.a2.shape[1], self.g2.shape[1]
+        qk = up(kv_heads * dim)
+        self.at_v, self.at_a = 2 * qk, 2 * qk + up(heads * vdim)
+        self.cols_a = slice(self.at_a, self.at_a + ra)
+        self.cols_g = slice(self.at_a + up(ra), self.at_a + up(ra) + rg)
+        self.at_b = self.at_a + up(ra) + up(rg)
+
+    def __call__(self, h: torch.Tensor, state: torch.Tensor, before: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+        p = O.linear(h, self.inp)
+        rate = O.linear(p[:, self.cols_a], self.a2, out_dtype=torch.float32)
+        gate = O.linear(p[:, self.cols_g], self.g2)
+        q, k, v = O.conv_unit(p, self.conv, before, fb, self.heads, self.kv_heads, self.dim, self.vdim)
+        y = O.delta_rule(q, k, v, rate, self.dt_bias, self.a_log, p, self.at_b, gate, self.gain, self.eps, state, before, fb,
+                         self.heads, self.kv_heads)
+        return O.linear(y, self.o, out_dtype=torch.float32)
+
+
+class GatedFF:
+    """down(act(gate h) * (up h)); gate and up are one projection whose epilogue pairs them."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, act: str):
+        self.gu, self.down, self.act = w[prefix + "gu"], w[prefix + "down"], act
+
+    def __call__(self, h: torch.Tensor) -> torch.Tensor:
+        return O.linear(O.gated_linear(h, self.gu, self.act), self.down, out_dtype=torch.float32)

@@ -11,6 +11,8 @@ from ..kvcache.paged import PoolSizes
 from ..utils.misc import div_ceil
 from .bedalorn_config import ARCHITECTURE as BEDALORN
 from .bedalorn_config import BedalornConfig
+from .buvalix_config import ARCHITECTURE as BUVALIX
+from .buvalix_config import BuvalixConfig
 from .config import ModelConfig
 
 
@@ -95,7 +97,27 @@ def _dsv4_classes(cfg, limit: int) -> List[int]:
     return [c for c in (4 * cfg.index_topk, DSV4_RELEASE.graph_short_context) if c < limit]
 
 
-# --------------------------------------------------------------------------- Bedalorn
+# --------------------------------------------------------------------------- layered designs
+def _layered_budget(cfg, c, dtype) -> KVBudget:
+    from ..kvcache import layered_pool as P
+
+    stores = cfg.run_stores()
+    # a model without attention layers still counts pages (they bound the sequence lengths)
+    return KVBudget(max(P.bytes_per_page(stores, c.page_size, dtype), 1),
+                    (c.max_running_req + 1) * P.bytes_per_req_slot(stores, cfg.hidden_size, dtype), 0, 1)
+
+
+def _layered_pool(cfg, sizes: PoolSizes, device, dtype):
+    from ..kvcache.layered_pool import LayeredPool
+
+    return LayeredPool(cfg.run_stores(), cfg.hidden_size, sizes, device, dtype)
+
+
+def _layered_classes(cfg, limit: int) -> List[int]:
+    # a class fixes how many ways the keys of a small decode batch are split
+    return [c for c in (2048, 32768) if c < limit]
+
+
 def _bedalorn_load(folder, cfg, device, rank, size, moe_mode):
     from .bedalorn_weight import load_checkpoint
 
@@ -108,38 +130,39 @@ def _bedalorn_draw(cfg, device, rank, size, moe_mode, seed, on_host):
     return random_weights(cfg, device, seed)
 
 
-def _bedalorn_budget(cfg, c, dtype) -> KVBudget:
-    from ..kvcache import latent_pool as P
-
-    stores = cfg.run_stores()
-    # a model without attention layers still counts pages (they bound the sequence lengths)
-    return KVBudget(max(P.bytes_per_page(stores, c.page_size, dtype), 1),
-                    (c.max_running_req + 1) * P.bytes_per_req_slot(stores, cfg.hidden_size), 0, 1)
-
-
-def _bedalorn_pool(cfg, sizes: PoolSizes, device, dtype):
-    from ..kvcache.latent_pool import LatentStatePool
-
-    return LatentStatePool(cfg.run_stores(), cfg.hidden_size, sizes, device, dtype)
-
-
 def _bedalorn_build(cfg, weights, pool, comm, moe_mode, dtype):
     from .bedalorn import BedalornModel
 
     return BedalornModel(cfg, weights, pool, comm, moe_mode, dtype)
 
 
-def _bedalorn_classes(cfg, limit: int) -> List[int]:
-    # a class fixes how many ways the keys of a small decode batch are split
-    return [c for c in (2048, 32768) if c < limit]
+def _buvalix_load(folder, cfg, device, rank, size, moe_mode):
+    from .buvalix_weight import load_checkpoint
+
+    return load_checkpoint(folder, cfg, device)
+
+
+def _buvalix_draw(cfg, device, rank, size, moe_mode, seed, on_host):
+    from .buvalix_weight import random_weights
+
+    return random_weights(cfg, device, seed)
+
+
+def _buvalix_build(cfg, weights, pool, comm, moe_mode, dtype):
+    from .buvalix import BuvalixModel
+
+    return BuvalixModel(cfg, weights, pool, comm, moe_mode, dtype)
 
 
 FAMILIES = {
     "DeepseekV4ForCausalLM": ModelFamily("deepseek_v4", ModelConfig, ModelConfig.from_hf, (torch.bfloat16,), 64,
                                          _dsv4_load, _dsv4_draw, _dsv4_budget, _dsv4_pool, _dsv4_build, _dsv4_classes),
     BEDALORN: ModelFamily("bedalorn", BedalornConfig, BedalornConfig.from_dict, (torch.bfloat16, torch.float32), 1,
-                          _bedalorn_load, _bedalorn_draw, _bedalorn_budget, _bedalorn_pool, _bedalorn_build,
-                          _bedalorn_classes, "layered"),
+                          _bedalorn_load, _bedalorn_draw, _layered_budget, _layered_pool, _bedalorn_build,
+                          _layered_classes, "layered"),
+    BUVALIX: ModelFamily("buvalix", BuvalixConfig, BuvalixConfig.from_dict, (torch.bfloat16, torch.float32), 1,
+                         _buvalix_load, _buvalix_draw, _layered_budget, _layered_pool, _buvalix_build,
+                         _layered_classes, "grouped"),
 }
 
 

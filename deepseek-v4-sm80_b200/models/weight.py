@@ -209,6 +209,24 @@ def _index_checkpoint(folder: str) -> Dict[str, str]:
     return out
 
 
+def tensor_reader(folder: str, device="cpu") -> Callable[[str], torch.Tensor]:
+    """name -> tensor of a safetensors checkpoint, files opened as they are needed."""
+    import safetensors
+
+    where = _index_checkpoint(folder)
+    handles: Dict[str, object] = {}
+
+    def fetch(name: str) -> torch.Tensor:
+        if name not in where:
+            raise KeyError(f"the checkpoint has no tensor {name!r}")
+        f = where[name]
+        if f not in handles:
+            handles[f] = safetensors.safe_open(f, framework="pt", device=str(device))
+        return handles[f].get_tensor(name)
+
+    return fetch
+
+
 def load_checkpoint(folder: str, cfg: ModelConfig, device, rank: int = 0, size: int = 1, moe_mode: str = "tp",
                     progress: Optional[Callable[[str], None]] = None) -> Dict[str, torch.Tensor]:
     """Streams a DeepSeek-V4 safetensors checkpoint into sharded runtime tensors on ``device``."""

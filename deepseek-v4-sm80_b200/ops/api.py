@@ -329,6 +329,61 @@ def wkv(p, a, w0, u, gain, state, prev, tail, fb, heads: int, eps: float):
     return _layers(p).wkv(p, a, w0, u, gain, state, prev, tail, fb, heads, eps)
 
 
+# --------------------------------------------------------------------------- layer norms, grouped attention, delta rule
+def _mixers(t):
+    from . import cuda_mixers, ref_mixers
+
+    return cuda_mixers if t.is_cuda else ref_mixers
+
+
+def residual_layer_norm(x, eps: float, dtype, norm=None, sub=None, add=None, rows=None, keep: bool = True):
+    """One step of the fp32 stream x [T, D] with layer norms around the sub-layers: x += N(y; w, b) for ``sub`` = (y fp32
+    [T, D], w, b), then x += ``add`` [T, D] (activations), then returns N(x; w, b) as activations for ``norm`` = (w, b), else
+    None.  ``rows``: only these rows are computed and returned.  keep=False (always with ``rows``): x itself may be left
+    as it was."""
+    return _mixers(x).residual_layer_norm(x, eps, dtype, norm, sub, add, rows, keep and rows is None)
+
+
+def gated_linear(h, w, act: str, block: int = 16):
+    """act(gate h) * (up h) for w [2F, D] in alternating blocks of ``block`` gate and up rows -> [T, F]."""
+    return _mixers(h).gated_linear(h, w, act, block)
+
+
+def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads: int, kv_heads: int, dim: int, vdim: int):
+    """Behind the projection q | k | v of grouped attention: adds ``bias`` (or None), turns neighbouring pairs of the first
+    2 * len(freq) dimensions of every q and k head by position * freq (or not), multiplies q by its temperature
+    1 + coef * ln(floor((position + 1) / every) + 1) for q_temp = (coef, every), writes keys and values to the rows
+    ``fb.out_loc`` of the caches and returns q [T, H, dim]."""
+    return _mixers(qkv).rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads, kv_heads, dim, vdim)
+
+
+def grouped_attention(q, keys, values, fb, kv_heads: int, scale: float, softcap: float = 0.0, sink=None, rel=None):
+    """Causal attention of q [T, H, dim] over the cached keys and values of every request, H / kv_heads query heads to a key
+    head.  score = softcap * tanh(q.k * scale / softcap) (0: not capped) + rel[h, min(distance, last)]; ``sink`` [H] adds
+    exp(sink) to the denominator.  Returns [T, H * vdim]."""
+    return _mixers(q).grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel)
+
+
+def conv_unit(p, taps, before, fb, heads: int, kv_heads: int, dim: int, vdim: int):
+    """Short causal convolution per channel and silu over the q, k and v columns of p (each part starts at a multiple of
+    eight columns), taps [n, channels], the inputs ahead of a portion from ``before`` [slots + 1, n - 1, channels]; then q and
+    k as unit vectors, q times dim^-1/2.  Returns (q fp32 [T, kv_heads * dim], k, v [T, H * vdim]).  :func:`delta_rule` of the
+    same layer must follow: it moves ``before`` on."""
+    return _mixers(p).conv_unit(p, taps, before, fb, heads, kv_heads, dim, vdim)
+
+
+def delta_rule(q, k, v, rate, dt_bias, a_log, p, at_b: int, gate, gain, eps: float, state, before, fb, heads: int,
+               kv_heads: int):
+    """Gated delta rule per head, S [dim, vdim] fp32 in ``state`` [slots + 1, H, dim, vdim]:
+
+        S <- diag(g) S,  u = beta (v - S^T k),  S <- S + k u^T,  o = S^T q
+        g = exp(-exp(a_log) softplus(rate + dt_bias)) per key channel,  beta = sigmoid(p[:, at_b + head])
+
+    and y = o / rms(o) * gain * sigmoid(gate) per head -> [T, H * vdim].  Also keeps the last inputs of the convolutions
+    (the q, k, v columns of p) in ``before``."""
+    return _mixers(p).delta_rule(q, k, v, rate, dt_bias, a_log, p, at_b, gate, gain, eps, state, before, fb, heads, kv_heads)
+
+
 # --------------------------------------------------------------------------- sampling
 def sample(logits, temperature, top_k, top_p, uniform, mask_ids=None):
     if logits.is_cuda:

@@ -37,6 +37,8 @@ HOST_LIB = HERE / "libdsv4_host.so"
 KERNEL_SETS = {
     "layered": ("common", "comm", "elementwise", "sampling", "gemm_tcgen05", "gemm_prefill", "gemm_simt", "moe", "moe_bf16",
                 "residual", "latent_attn", "flash_attn", "wkv", "wkv_chunk"),
+    "grouped": ("common", "comm", "elementwise", "sampling", "gemm_tcgen05", "gemm_prefill", "gemm_simt", "residual",
+                "grouped_attn", "flash_attn", "delta", "delta_chunk"),
 }
 
 

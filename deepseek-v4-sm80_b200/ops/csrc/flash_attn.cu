@@ -1,9 +1,11 @@
-// Causal multi-head attention of long prompt portions on tcgen05, keys and values expanded from the cached latents.
+// Causal multi-head attention of long prompt portions on tcgen05 over keys and values that lie side by side: gathered from
+// a paged cache (grouped_attn.cu: kv_gather, several query heads to a key head, optionally capped scores, a bias by distance
+// and a sink), or expanded from cached latents (latent_attn.cu).
 //
-// The absorbed form (latent_attn.cu) multiplies every (query, key) pair over the whole latent rank, twice.  For a portion
-// of many tokens it is cheaper to expand the request's latents once,  K = C W_uk^T  and  V^T = W_uv C^T  (two plain
-// projections; the second one comes out with the keys contiguous, which is the K-major operand of the PV product), and to
-// run ordinary attention over `dim` and `vdim` per head.
+// For latents, the absorbed form (latent_attn.cu) multiplies every (query, key) pair over the whole latent rank, twice.  For
+// a portion of many tokens it is cheaper to expand the request's latents once,  K = C W_uk^T  and  V^T = W_uv C^T  (two
+// plain projections; the second one comes out with the keys contiguous, which is the K-major operand of the PV product),
+// and to run ordinary attention over `dim` and `vdim` per head.
 //
 // One CTA: one head, 256 consecutive queries of one request as two 128-row tiles that share every key / value tile (128
 // keys).  The tensor core works on one tile while the softmax warps work on the other:
@@ -12,7 +14,7 @@
 //   warps 2-5   softmax of tile 0, warps 6-9 of tile 1: one thread per row; P_t overwrites S_t in place as bf16
 // Tensor memory: S0 | S1 | O0 | O1, 128 columns each.  O stays there; it is rescaled only when a row's maximum has grown by
 // more than 2^8 since the last time (the sums stay far from overflow, the quotient does not depend on it).
-#include "vec.cuh"
+#include "mma16.cuh"
 
 namespace {
 
@@ -23,8 +25,15 @@ constexpr int kColO = 256;
 
 struct FlashArgs {
   const int* items;     // [n_items][5]: first query row, queries, context position of the first, first key row, keys
-  int heads, dim, vdim, ldo;
+  int heads, group, dim, vdim, ldo;   // group: query heads that share a key head
   float scale2;         // scale * log2(e)
+  // capped scores (CAP): in powers of two, cap2 tanh(s c) for the raw product s
+  float c, cap2;
+  float small;          // |s| up to here: s (p0 + p1 s^2 + p2 s^4 + p3 s^6), an odd polynomial
+  float p0, p1, p2, p3;
+  const float* sink;    // [heads] or null
+  const float* rel;     // [heads][n_rel] (BIAS)
+  int n_rel;
 };
 
 struct FlashBars {
@@ -33,19 +42,19 @@ struct FlashBars {
   int abort_flag;
 };
 
+constexpr int kWin = 160;                    // distances between a warp's 32 queries and a tile's 128 keys (159)
+constexpr int kBiasBytes = 8 * kWin * 4;
+
 template <int NB>     // 64-wide blocks of dim
 struct FlashCfg {
   static constexpr int kQ = 2 * NB * kBlk, kK = NB * kBlk, kV = 2 * kBlk;
-  static constexpr int kSmem = kQ + 2 * (kK + kV) + 1024 + (int)sizeof(FlashBars);
+  static constexpr int kSmem = kQ + 2 * (kK + kV) + kBiasBytes + 1024 + (int)sizeof(FlashBars);
 };
 
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
+// What happens to a score between the product and the softmax.
+enum ScoreMode : int { kScaled = 0, kCapped = 1, kCappedBias = 2 };
 
-template <int NB>
+template <int NB, int MODE>
 __global__ void __launch_bounds__(kFThreads, 1)
 flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                   const __grid_constant__ CUtensorMap tmV, __nv_bfloat16* __restrict__ out, const FlashArgs a) {
@@ -55,10 +64,11 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   uint8_t* qs = smem;                       // [2 tiles][NB] blocks
   uint8_t* ks = qs + C::kQ;                 // [2 stages][NB] blocks
   uint8_t* vs = ks + 2 * C::kK;             // [2 stages][2] blocks of [vdim rows][64 keys]
-  FlashBars* b = reinterpret_cast<FlashBars*>(vs + 2 * C::kV);
+  float* wins = reinterpret_cast<float*>(vs + 2 * C::kV);   // [8 warps][kWin] bias by distance
+  FlashBars* b = reinterpret_cast<FlashBars*>(wins + 8 * kWin);
   volatile int* abort_flag = &b->abort_flag;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int head = blockIdx.x;
+  const int head = blockIdx.x, kv_head = head / a.group;
 
   if (threadIdx.x == 0) {
     mbar_init(&b->q_full, 1);
@@ -101,11 +111,11 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         if (i >= 2 && !mbar_wait<32>(&b->k_empty[s], ph, abort_flag, 81)) break;
         mbar_expect_tx(&b->k_full[s], C::kK);
         for (int j = 0; j < NB; ++j)
-          tma_load_3d(ks + s * C::kK + j * kBlk, &tmK, &b->k_full[s], j * 64, head, kv0 + i * kQT);
+          tma_load_3d(ks + s * C::kK + j * kBlk, &tmK, &b->k_full[s], j * 64, kv_head, kv0 + i * kQT);
         if (i >= 2 && !mbar_wait<32>(&b->v_empty[s], ph, abort_flag, 82)) break;
         mbar_expect_tx(&b->v_full[s], v_bytes);
         for (int j = 0; j < 2; ++j)
-          tma_load_3d(vs + s * C::kV + j * kBlk, &tmV, &b->v_full[s], kv0 + i * kQT + j * 64, 0, head);
+          tma_load_3d(vs + s * C::kV + j * kBlk, &tmV, &b->v_full[s], kv0 + i * kQT + j * 64, 0, kv_head);
       }
     }
   } else if (warp == 1) {
@@ -168,9 +178,22 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const uint32_t sp = tmem + t * 128 + lane_base, op = tmem + kColO + t * 128 + lane_base;
     const int last = row < nq ? pos0 + row : -1;              // last key the row sees
     const int first_masked = (pos0 + t * kQT + quarter * 32 + 1) / kQT;  // key tiles before it are seen whole by the warp
+    const float sc = MODE == kScaled ? a.scale2 : 1.f;        // the other modes leave scores in powers of two
+    float* win = wins + (warp - 2) * kWin;
+    const float* rel = MODE == kCappedBias ? a.rel + (size_t)head * a.n_rel : nullptr;
+    const float rel_far = MODE == kCappedBias ? rel[a.n_rel - 1] * kLog2e : 0.f;
     float m = -1e30f, l = 0.f;
     bool ok = true;
     for (int i = 0; i < n; ++i) {
+      const int base = pos0 + t * kQT + quarter * 32 - i * kQT;   // distance of the warp's first query and the tile's first key
+      const bool all_far = base - (kQT - 1) >= a.n_rel - 1;
+      if (MODE == kCappedBias && !all_far) {
+        __syncwarp();
+#pragma unroll
+        for (int x = 0; x < kWin; x += 32)
+          win[x + lane] = rel[max(min(base - (kQT - 1) + x + lane, a.n_rel - 1), 0)] * kLog2e;
+        __syncwarp();
+      }
       ok = mbar_wait<16>(&b->s_full[t], i & 1, abort_flag, 88);
       if (!ok) break;
       tc_fence_after();
@@ -183,6 +206,31 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 #pragma unroll
         for (int j = 0; j < 32; ++j) s[c * 32 + j] = __uint_as_float(r[j]);
       }
+      if (MODE != kScaled) {
+        float big = fabsf(s[0]);
+#pragma unroll
+        for (int j = 1; j < kQT; ++j) big = fmaxf(big, fabsf(s[j]));
+        if (__all_sync(0xffffffffu, big <= a.small)) {
+#pragma unroll
+          for (int j = 0; j < kQT; ++j) {
+            const float x = s[j] * s[j];
+            s[j] *= fmaf(fmaf(fmaf(a.p3, x, a.p2), x, a.p1), x, a.p0);
+          }
+        } else {
+          const float e = 2.f * kLog2e * a.c;
+#pragma unroll
+          for (int j = 0; j < kQT; ++j) s[j] = softcap_ex2(s[j], e, a.cap2);
+        }
+        if (MODE == kCappedBias) {
+          if (all_far) {
+#pragma unroll
+            for (int j = 0; j < kQT; ++j) s[j] += rel_far;
+          } else {
+#pragma unroll
+            for (int j = 0; j < kQT; ++j) s[j] += win[kQT - 1 + lane - j];
+          }
+        }
+      }
       if (i >= first_masked || row >= nq) {
         const int lim = last - i * kQT;
 #pragma unroll
@@ -192,7 +240,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       float mx = s[0];
 #pragma unroll
       for (int j = 1; j < kQT; ++j) mx = fmaxf(mx, s[j]);
-      mx *= a.scale2;
+      mx *= sc;
       const bool grow = mx > m + 8.f;
       if (__any_sync(0xffffffffu, grow)) {
         const float mn = grow ? mx : m, f = ex2(m - mn);
@@ -216,7 +264,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         uint32_t pk[16];
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
-          const float p0 = ex2(fmaf(s[c * 32 + 2 * j], a.scale2, -m)), p1 = ex2(fmaf(s[c * 32 + 2 * j + 1], a.scale2, -m));
+          const float p0 = ex2(fmaf(s[c * 32 + 2 * j], sc, -m)), p1 = ex2(fmaf(s[c * 32 + 2 * j + 1], sc, -m));
           sum0 += p0, sum1 += p1;
           const __nv_bfloat162 p = __floats2bfloat162_rn(p0, p1);
           pk[j] = *reinterpret_cast<const uint32_t*>(&p);
@@ -230,7 +278,13 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     }
     if (ok && mbar_wait<16>(&b->o_full[t], 0, abort_flag, 89)) {
       tc_fence_after();
-      const float inv = 1.f / l;
+      float f = 1.f;
+      if (a.sink) {            // one more term of the sum, without a key or a value
+        const float s2 = a.sink[head] * kLog2e, mm = fmaxf(m, s2);
+        f = ex2(m - mm);
+        l = l * f + ex2(s2 - mm);
+      }
+      const float inv = f / l;
       __nv_bfloat16* dst = out + (size_t)(q0 + row) * a.ldo + head * a.vdim;
 #pragma unroll 1
       for (int c = 0; c < vp; c += 16) {
@@ -258,63 +312,58 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   if (warp == 1) tmem_dealloc(tmem, 512);
 }
 
-// ctx[dst + j] = cache[page_table[slot][j]] for the keys j of every listed request, zeros in the padding behind them.
-// list: [segs][3] = slot, keys, first row of the copy; rows [dst, dst of the next request) belong to a request.
-__global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* __restrict__ cache, uint4* __restrict__ ctx,
-                                                            const int* __restrict__ list, int segs, int total,
-                                                            const int* __restrict__ page_table, int ld_pt, int r8) {
-  pdl_entry();
-  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (row >= total) return;
-  int lo = 0, hi = segs - 1;
-  while (lo < hi) {
-    const int mid = (lo + hi + 1) >> 1;
-    if (list[mid * 3 + 2] <= row) lo = mid; else hi = mid - 1;
-  }
-  const int j = row - list[lo * 3 + 2];
-  const bool in = j < list[lo * 3 + 1];
-  const size_t src = in ? (size_t)page_table[(size_t)list[lo * 3] * ld_pt + j] * r8 : 0;
-  for (int i = lane; i < r8; i += 32) ctx[(size_t)row * r8 + i] = in ? cache[src + i] : make_uint4(0, 0, 0, 0);
-}
-
-template <int NB>
+template <int NB, int MODE>
 int launch_flash(const CUtensorMap& q, const CUtensorMap& k, const CUtensorMap& v, void* out, const FlashArgs& a,
                  int n_items, cudaStream_t st) {
   using C = FlashCfg<NB>;
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(flash_attn_kernel<NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmem) != cudaSuccess)
+    if (cudaFuncSetAttribute(flash_attn_kernel<NB, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmem) !=
+        cudaSuccess)
       return 655;
     set = true;
   }
-  dsv4_launch(flash_attn_kernel<NB>, dim3(a.heads, n_items), kFThreads, C::kSmem, st, q, k, v, (__nv_bfloat16*)out, a);
+  dsv4_launch(flash_attn_kernel<NB, MODE>, dim3(a.heads, n_items), kFThreads, C::kSmem, st, q, k, v, (__nv_bfloat16*)out, a);
   return (int)cudaGetLastError();
+}
+template <int NB>
+int dispatch_flash(int mode, const CUtensorMap& q, const CUtensorMap& k, const CUtensorMap& v, void* out,
+                   const FlashArgs& a, int n_items, cudaStream_t st) {
+  if (mode == kScaled) return launch_flash<NB, kScaled>(q, k, v, out, a, n_items, st);
+  if (mode == kCapped) return launch_flash<NB, kCapped>(q, k, v, out, a, n_items, st);
+  return launch_flash<NB, kCappedBias>(q, k, v, out, a, n_items, st);
 }
 
 }  // namespace
 
-DSV4_API int dsv4_latent_gather(const void* cache, void* ctx, const int* list, int segs, int total,
-                                const int* page_table, int ld_pt, int rank, cudaStream_t st) {
-  if (total <= 0) return 0;
-  if (rank % 8 || segs < 1) return 650;
-  dsv4_launch(latent_gather_kernel, (total + 3) / 4, 128, 0, st, (const uint4*)cache, (uint4*)ctx, list, segs, total,
-              page_table, ld_pt, rank / 8);
-  return (int)cudaGetLastError();
-}
-
-// q: bf16 [rows, heads * dim] (row stride ldq), k: [kv_rows, heads * dim], vt: [heads * vdim, kv_rows] (row stride
-// kv_rows), out: [rows, heads * vdim].  items as in FlashArgs, at most 256 queries each; first key rows are multiples of 8.
+// q: bf16 [rows, heads * dim] (row stride ldq), k: [kv_rows, kv_heads * dim], vt: [kv_heads * vdim, kv_rows] (row stride
+// kv_rows), out: [rows, heads * vdim]; query head h reads key head h / (heads / kv_heads).  items as in FlashArgs, at most 256
+// queries each; first key rows are multiples of 8.  Scores: cap tanh(q.k scale / cap) (cap 0: q.k scale), plus rel[h,
+// min(distance, n_rel - 1)] if rel is given; sink [heads] or null adds e^sink to the sum of a row's weights.
 DSV4_API int dsv4_flash_attention(const void* q, int ldq, const void* k, const void* vt, void* out, const int* items,
-                                  int n_items, int rows, int kv_rows, int heads, int dim, int vdim, float scale,
+                                  int n_items, int rows, int kv_rows, int heads, int kv_heads, int dim, int vdim,
+                                  float scale, float cap, const float* sink, const float* rel, int n_rel,
                                   cudaStream_t st) {
   if (n_items <= 0) return 0;
   if (dim % 8 || vdim % 8 || ldq % 8 || kv_rows % 8 || dim < 8 || dim > 128 || vdim < 8 || vdim > 128 || n_items > 65535)
     return 651;
+  if (kv_heads < 1 || heads % kv_heads || (rel && n_rel < 1)) return 656;
   CUtensorMap tq, tk, tv;
   if (dsv4_make_tmap_3d(&tq, q, dim, heads, rows, (uint64_t)dim * 2, (uint64_t)ldq * 2, 64, 1, kQT)) return 652;
-  if (dsv4_make_tmap_3d(&tk, k, dim, heads, kv_rows, (uint64_t)dim * 2, (uint64_t)heads * dim * 2, 64, 1, kQT)) return 653;
+  if (dsv4_make_tmap_3d(&tk, k, dim, kv_heads, kv_rows, (uint64_t)dim * 2, (uint64_t)kv_heads * dim * 2, 64, 1, kQT)) return 653;
   const int vp = (vdim + 15) & ~15;
-  if (dsv4_make_tmap_3d(&tv, vt, kv_rows, vdim, heads, (uint64_t)kv_rows * 2, (uint64_t)vdim * kv_rows * 2, 64, vp)) return 654;
-  const FlashArgs a{items, heads, dim, vdim, heads * vdim, scale * 1.4426950408889634f};
-  return dim <= 64 ? launch_flash<1>(tq, tk, tv, out, a, n_items, st) : launch_flash<2>(tq, tk, tv, out, a, n_items, st);
+  if (dsv4_make_tmap_3d(&tv, vt, kv_rows, vdim, kv_heads, (uint64_t)kv_rows * 2, (uint64_t)vdim * kv_rows * 2, 64, vp)) return 654;
+  FlashArgs a{items, heads, heads / kv_heads, dim, vdim, heads * vdim, scale * kLog2e};
+  a.sink = sink, a.rel = rel, a.n_rel = rel ? n_rel : 0;
+  if (cap > 0.f) {
+    // tanh x = x - x^3 / 3 + 2 x^5 / 15 - 17 x^7 / 315 + ..., to 2e-6 relative for x up to 0.3
+    const float c = scale / cap, cap2 = cap * kLog2e, c2 = c * c;
+    a.c = c, a.cap2 = cap2, a.small = 0.3f / fabsf(c);
+    a.p0 = cap2 * c, a.p1 = -a.p0 * c2 / 3.f, a.p2 = a.p0 * c2 * c2 * (2.f / 15.f), a.p3 = a.p0 * c2 * c2 * c2 * (-17.f / 315.f);
+  } else {
+    a.small = INFINITY, a.p0 = a.scale2;      // only reached with a bias
+  }
+  const int mode = rel ? kCappedBias : cap > 0.f ? kCapped : kScaled;
+  return dim <= 64 ? dispatch_flash<1>(mode, tq, tk, tv, out, a, n_items, st)
+                   : dispatch_flash<2>(mode, tq, tk, tv, out, a, n_items, st);
 }

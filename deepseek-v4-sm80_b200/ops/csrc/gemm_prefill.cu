@@ -107,7 +107,8 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_kernel(const __grid_const
       tc_fence_after();
       const int row = m * kPM + q * 32 + lane;
       const uint32_t d0 = tmem + acc * kPN + ((uint32_t)(q * 32) << 16);
-      OutT* dst = out + (size_t)row * g.ldo + (size_t)b * g.N + n * kPN;
+      const bool gated = g.act == kActGeluGate;
+      OutT* dst = out + (size_t)row * g.ldo + (gated ? (size_t)n * (kPN / 2) : (size_t)b * g.N + n * kPN);
       const int cols = min(kPN, g.N - n * kPN);
       const bool vec = ((uintptr_t)dst & 15) == 0;
 #pragma unroll 1
@@ -119,6 +120,11 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_kernel(const __grid_const
         float v[32];
 #pragma unroll
         for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
+        if (gated) {
+          gate_block(v);
+          st_f16x(dst + c / 2, v);
+          continue;
+        }
         if (g.act) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] = gemm_act(v[j], g.act);
@@ -182,6 +188,7 @@ DSV4_API int dsv4_gemm_prefill(const void* x, const void* w, void* out, int M, i
                                int out_fp32, int accumulate, int act, int batches, int sms, cudaStream_t st) {
   if (M <= 0 || N <= 0) return 0;
   if (K % 8 || ldx % 8 || ldw % 8 || batches < 1 || sms < 1) return 660;
+  if (act == kActGeluGate && (N % 32 || ldo % 16 || batches != 1 || accumulate)) return 664;
   CUtensorMap ta, tb;
   if (dsv4_make_tmap_2d(&ta, x, 1, (uint64_t)K * batches, M, (uint64_t)ldx * 2, 64, kPM, 3)) return 661;
   if (dsv4_make_tmap_2d(&tb, w, 1, K, (uint64_t)N * batches, (uint64_t)ldw * 2, 64, kPN, 3)) return 662;

@@ -1,0 +1,654 @@
+// Causal attention with several query heads to a key head over paged keys and values (bf16 or fp32 caches): what happens
+// between the q | k | v projection and the output projection.
+//
+//   s_ij = cap tanh(q_i . k_j scale / cap) + rel[h, min(i - j, last)],    w_ij = e^{s_ij} / (e^{sink_h} + sum_j' e^{s_ij'})
+//
+// cap, rel and sink are optional.  Kernels:
+//   rotate_store     bias, rotation, query temperature; keys and values to their cache rows
+//   grouped_attn     tensor cores (mma.sync): the (token, query head) rows of a key head are consecutive, and all of them see
+//                    a prefix of the same keys, so a CTA takes 16 .. 64 rows of one request and key head and streams the keys
+//                    and values once for all of them.  grid.y splits the keys when the row tiles alone leave SMs idle;
+//                    grouped_merge adds the partial results in split order.  Decode, and short portions of prompts.
+//   grouped_row      one warp per row on the CUDA cores, fp32 throughout: models served in 32-bit floats, other sizes
+//   kv_gather        a request's keys and (transposed) values side by side, for the prompt kernel in flash_attn.cu
+#include "mma16.cuh"
+
+namespace {
+
+// ------------------------------------------------------------------ behind the projection
+struct RotateArgs {
+  int ld;                    // row stride of qkv
+  const float* bias;         // [(H + G) dim + G vdim] or null
+  const float* freq;         // [pairs] or null
+  int pairs;
+  float coef;                // query temperature 1 + coef ln((pos + 1) / every + 1); every 0: none
+  int every;
+  const int* pos;
+  const int* out_loc;
+  int heads, kv_heads, dim, vdim;
+};
+
+// One CTA per token; cos and sin of its angles in shared memory.  W consecutive values per thread (even, or 1).
+template <typename T, int W>
+__global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__ qkv, T* __restrict__ q,
+                                                           T* __restrict__ keys, T* __restrict__ values,
+                                                           const RotateArgs a) {
+  pdl_entry();
+  extern __shared__ float2 cs[];
+  const int t = blockIdx.x, pos = a.pos[t], loc = a.out_loc[t];
+  for (int i = threadIdx.x; i < a.pairs; i += 256) {
+    float s, c;
+    sincosf((float)pos * a.freq[i], &s, &c);
+    cs[i] = make_float2(c, s);
+  }
+  const float temp = a.every ? 1.f + a.coef * logf((float)((pos + 1) / a.every + 1)) : 1.f;
+  __syncthreads();
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
+  const T* src = qkv + (size_t)t * a.ld;
+  for (int i = threadIdx.x * W; i < nq + nk + nv; i += 256 * W) {
+    float v[W];
+    if constexpr (W == 1) {
+      v[0] = ld_f(src + i) + (a.bias ? a.bias[i] : 0.f);
+    } else {
+#pragma unroll
+      for (int j = 0; j < W; j += 4) {
+        float4 x = ld_f4(src + i + j);
+        if (a.bias) {
+          const float4 b = ld_f4(a.bias + i + j);
+          x.x += b.x, x.y += b.y, x.z += b.z, x.w += b.w;
+        }
+        v[j] = x.x, v[j + 1] = x.y, v[j + 2] = x.z, v[j + 3] = x.w;
+      }
+    }
+    if (i < nq + nk) {
+      const int e = i % a.dim;
+      if constexpr (W == 1) {
+        if (e < 2 * a.pairs) {
+          const int o = e & 1 ? i - 1 : i + 1;
+          const float2 r = cs[e >> 1];
+          const float other = ld_f(src + o) + (a.bias ? a.bias[o] : 0.f);
+          v[0] = e & 1 ? v[0] * r.x + other * r.y : v[0] * r.x - other * r.y;
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < W; j += 2)
+          if (e + j < 2 * a.pairs) {
+            const float2 r = cs[(e + j) >> 1];
+            const float x = v[j], y = v[j + 1];
+            v[j] = x * r.x - y * r.y, v[j + 1] = y * r.x + x * r.y;
+          }
+      }
+    }
+    T* dst;
+    if (i < nq) {
+#pragma unroll
+      for (int j = 0; j < W; ++j) v[j] *= temp;
+      dst = q + (size_t)t * nq + i;
+    } else {
+      if (loc < 0) continue;
+      dst = i < nq + nk ? keys + (size_t)loc * nk + (i - nq) : values + (size_t)loc * nv + (i - nq - nk);
+    }
+    if constexpr (W == 1) {
+      st_f(dst, v[0]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < W; j += 4) st_f4(dst + j, make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]));
+    }
+  }
+}
+
+// ------------------------------------------------------------------ few rows: tensor cores
+struct AttnArgs {
+  const int* slots;
+  const int* pos;
+  const int* page_table;
+  int ld_pt;
+  const int* tiles;      // [tiles][2]: row range of a tile (rows of a key head: token * group + query head), or null: tiles
+                         // of every token's own rows
+  int n_tiles;
+  const int* num_valid;  // tokens >= *num_valid are padding, or null
+  int rows;              // tokens
+  int kv_heads, group, dim, vdim;
+  float scale, cap;      // cap 0: scores are not capped
+  const float* sink;     // [H] or null
+  const float* rel;      // [H][n_rel] or null
+  int n_rel;
+  int nsplit;
+  float* part_acc;       // [T * H][nsplit][vdim]
+  float* part_ml;        // [T * H][nsplit][2]
+};
+
+constexpr int kKT = 64;       // keys per tile
+constexpr int kSP = kKT + 4;  // floats per score row
+
+template <int P, int MT>      // head sizes padded to P, MT x 16 rows
+struct AttnCfg {
+  static constexpr int M = MT * 16;
+  static constexpr int RG = MT == 4 ? 2 : 1;       // warp row groups of the S phase
+  static constexpr int WM = MT / RG;               // m16 tiles per warp
+  static constexpr int KG = 8 / RG;                // key groups
+  static constexpr int WN = kKT / KG / 8;          // n8 tiles per warp
+  static constexpr int DW = P / 8;                 // output columns per warp
+  static constexpr int NT = DW / 8;
+  static constexpr int SMEM = M * P * 2 + 4 * kKT * P * 2 + M * kSP * 4 + M * kKT * 2 + 4 * M * 4;
+};
+
+template <int P, int MT>
+__global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* __restrict__ q,
+                                                           const __nv_bfloat16* __restrict__ keys,
+                                                           const __nv_bfloat16* __restrict__ values,
+                                                           __nv_bfloat16* __restrict__ o, const AttnArgs a) {
+  pdl_entry();
+  using C = AttnCfg<P, MT>;
+  constexpr int M = C::M, WM = C::WM, WN = C::WN, NT = C::NT;
+  extern __shared__ __align__(128) uint8_t attn_smem[];
+  __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(attn_smem);  // [M][P] swizzled
+  __nv_bfloat16* ksm = qs + M * P;                                  // [2][kKT][P] swizzled
+  __nv_bfloat16* vsm = ksm + 2 * kKT * P;                           // [2][kKT][P] swizzled
+  float* ss = reinterpret_cast<float*>(vsm + 2 * kKT * P);          // [M][kSP]
+  __nv_bfloat16* pb = reinterpret_cast<__nv_bfloat16*>(ss + M * kSP);  // [M][kKT] swizzled
+  float* ms = reinterpret_cast<float*>(pb + M * kKT);
+  float* ls = ms + M;
+  float* alpha = ls + M;
+  int* see = reinterpret_cast<int*>(alpha + M);                     // keys the row sees
+
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = blockIdx.z, split = blockIdx.y, R = a.group, dch = a.dim / 8, vch = a.vdim / 8;
+  const int ldq = a.kv_heads * R * a.dim, ldk = a.kv_heads * a.dim, ldv = a.kv_heads * a.vdim;
+  int row0, row1;
+  if (a.tiles) {
+    row0 = a.tiles[blockIdx.x * 2], row1 = a.tiles[blockIdx.x * 2 + 1];
+  } else {
+    const int tpt = (R + M - 1) / M, t = blockIdx.x / tpt;
+    row0 = t * R + blockIdx.x % tpt * M;
+    row1 = min(row0 + M, (t + 1) * R);
+  }
+  if (a.num_valid && row0 / R >= *a.num_valid) return;
+  const int t_last = (row1 - 1) / R;
+  const int nkeys = a.pos[t_last] + 1;   // of the tile's last token, the one that sees most
+  const int* pt = a.page_table + (size_t)a.slots[t_last] * a.ld_pt;
+  // place of row r of the tile in q (elements) and in the lists of (token, head) rows
+  auto head_row = [&](int r) { return (size_t)((row0 + r) / R) * (a.kv_heads * R) + g * R + (row0 + r) % R; };
+
+  const int ktiles = (nkeys + kKT - 1) / kKT;
+  const int per = (ktiles + a.nsplit - 1) / a.nsplit;
+  const int kt0 = split * per, kt1 = min(kt0 + per, ktiles);
+  if (kt0 >= kt1) {  // nothing for this split: an empty partial
+    if (a.nsplit > 1)
+      for (int r = tid; r < row1 - row0; r += 256) {
+        float* ml = a.part_ml + (head_row(r) * a.nsplit + split) * 2;
+        ml[0] = -1e30f, ml[1] = 0.f;
+      }
+    return;
+  }
+
+  for (int i = tid; i < M * (P / 8); i += 256) {
+    const int r = i / (P / 8), c = i % (P / 8);
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (row0 + r < row1 && c < dch)
+      v = reinterpret_cast<const uint4*>(q + (size_t)((row0 + r) / R) * ldq + (g * R + (row0 + r) % R) * a.dim)[c];
+    reinterpret_cast<uint4*>(qs + r * P)[swz(r, c)] = v;
+  }
+  if (tid < M) {
+    ms[tid] = -1e30f, ls[tid] = 0.f;
+    see[tid] = row0 + tid < row1 ? a.pos[(row0 + tid) / R] + 1 : 0;
+  }
+
+  // four threads fetch the key and the value of one row
+  const int fk = tid >> 2, fp = tid & 3;
+  auto key_loc = [&](int kt) {
+    const int key = kt * kKT + fk;
+    return (kt < kt1 && key < nkeys) ? pt[key] : -1;
+  };
+  auto issue = [&](int loc, int buf) {
+    __nv_bfloat16 *kd = ksm + ((size_t)buf * kKT + fk) * P, *vd = vsm + ((size_t)buf * kKT + fk) * P;
+    const __nv_bfloat16 *kp = keys + (size_t)max(loc, 0) * ldk + g * a.dim, *vp = values + (size_t)max(loc, 0) * ldv + g * a.vdim;
+#pragma unroll
+    for (int c = fp; c < P / 8; c += 4) {
+      const bool in_k = loc >= 0 && c < dch, in_v = loc >= 0 && c < vch;
+      cpa16_zfill(kd + swz(fk, c) * 8, in_k ? kp + c * 8 : keys, in_k);
+      cpa16_zfill(vd + swz(fk, c) * 8, in_v ? vp + c * 8 : values, in_v);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+
+  float acc[MT][NT][4];
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < NT; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
+
+  issue(key_loc(kt0), kt0 & 1);
+  int loc_next = key_loc(kt0 + 1);
+  const float sc2 = a.scale * kLog2e, cap2 = a.cap * kLog2e;   // scores in powers of two
+  const float ce = a.cap > 0.f ? 2.f * kLog2e / cap2 : 0.f;
+  const int rg = warp / C::KG, kg = warp % C::KG;
+  const int kend = (a.dim + 31) / 32 * 2;                      // 16-wide steps of the score product, two at a time
+  for (int kt = kt0; kt < kt1; ++kt) {
+    const int buf = kt & 1;
+    if (kt + 1 < kt1) {
+      issue(loc_next, buf ^ 1);
+      loc_next = key_loc(kt + 2);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const __nv_bfloat16 *kb = ksm + (size_t)buf * kKT * P, *vb = vsm + (size_t)buf * kKT * P;
+    // ---- scores: rows [rg * WM * 16, +WM * 16) x keys [kg * WN * 8, +WN * 8)
+    {
+      float s[2][WM][WN][4] = {};
+#pragma unroll 2
+      for (int ks = 0; ks < kend; ks += 2) {
+        uint32_t bf[WN][4];
+#pragma unroll
+        for (int j = 0; j < WN; ++j) {
+          const int br = (kg * WN + j) * 8 + (lane & 7);
+          ldsm4(bf[j], kb + br * P + swz(br, ks * 2 + (lane >> 3)) * 8);
+        }
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int i = 0; i < WM; ++i) {
+            const int ar = (rg * WM + i) * 16 + (lane & 15);
+            uint32_t af[4];
+            ldsm4(af, qs + ar * P + swz(ar, (ks + h) * 2 + (lane >> 4)) * 8);
+#pragma unroll
+            for (int j = 0; j < WN; ++j) mma16816(s[h][i][j], af, bf[j][2 * h], bf[j][2 * h + 1]);
+          }
+      }
+#pragma unroll
+      for (int i = 0; i < WM; ++i)
+#pragma unroll
+        for (int j = 0; j < WN; ++j) {
+          const int r = (rg * WM + i) * 16 + (lane >> 2), c = (kg * WN + j) * 8 + (lane & 3) * 2;
+          *reinterpret_cast<float2*>(ss + r * kSP + c) =
+              make_float2((s[0][i][j][0] + s[1][i][j][0]) * sc2, (s[0][i][j][1] + s[1][i][j][1]) * sc2);
+          *reinterpret_cast<float2*>(ss + (r + 8) * kSP + c) =
+              make_float2((s[0][i][j][2] + s[1][i][j][2]) * sc2, (s[0][i][j][3] + s[1][i][j][3]) * sc2);
+        }
+    }
+    __syncthreads();
+    // ---- cap, bias, online softmax
+    {
+      constexpr int TPR = 256 / M, PER = kKT / TPR;  // threads per row, keys per thread (4, 8 or 16)
+      const int r = tid / TPR, seg = tid % TPR;
+      const int lim = see[r] - kt * kKT - seg * PER;
+      float v[PER];
+      float mx = -1e30f;
+#pragma unroll
+      for (int i = 0; i < PER; i += 4) {
+        const float4 f = *reinterpret_cast<const float4*>(ss + r * kSP + seg * PER + i);
+        v[i] = f.x, v[i + 1] = f.y, v[i + 2] = f.z, v[i + 3] = f.w;
+      }
+      if (a.cap > 0.f) {
+#pragma unroll
+        for (int i = 0; i < PER; ++i) v[i] = softcap_ex2(v[i], ce, cap2);
+      }
+      if (a.rel && lim > 0) {       // distance of key i: lim - 1 - i
+        const float* rel = a.rel + (size_t)(g * R + (row0 + r) % R) * a.n_rel;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) v[i] = fmaf(rel[max(min(lim - 1 - i, a.n_rel - 1), 0)], kLog2e, v[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        v[i] = i < lim ? v[i] : -INFINITY;
+        mx = fmaxf(mx, v[i]);
+      }
+#pragma unroll
+      for (int off = TPR / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+      const float m_old = ms[r], m_new = fmaxf(m_old, mx);
+      float sum = 0.f;
+      __align__(16) __nv_bfloat16 e[PER];
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        e[i] = f2bf(exp2f(v[i] - m_new));
+        sum += bf2f(e[i]);   // the weights as they enter the product add up to what they are divided by
+      }
+#pragma unroll
+      for (int off = TPR / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+      if constexpr (PER >= 8) {
+#pragma unroll
+        for (int i = 0; i < PER; i += 8)
+          reinterpret_cast<uint4*>(pb + r * kKT)[swz(r, (seg * PER + i) / 8)] = *reinterpret_cast<uint4*>(e + i);
+      } else {
+        *reinterpret_cast<uint2*>(pb + r * kKT + swz(r, seg / 2) * 8 + (seg & 1) * 4) = *reinterpret_cast<uint2*>(e);
+      }
+      __syncwarp();
+      if (seg == 0) {
+        const float al = exp2f(m_old - m_new);
+        alpha[r] = al;
+        ms[r] = m_new;
+        ls[r] = ls[r] * al + sum;
+      }
+    }
+    __syncthreads();
+    // ---- o += P V: all rows, output columns [warp * DW, +DW)
+    if (warp * C::DW < a.vdim) {
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        const float a0 = alpha[i * 16 + (lane >> 2)], a1 = alpha[i * 16 + (lane >> 2) + 8];
+#pragma unroll
+        for (int j = 0; j < NT; ++j) acc[i][j][0] *= a0, acc[i][j][1] *= a0, acc[i][j][2] *= a1, acc[i][j][3] *= a1;
+      }
+#pragma unroll
+      for (int kk = 0; kk < kKT / 16; ++kk) {
+        uint32_t pf[MT][4];
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+          const int pr = i * 16 + (lane & 15);
+          ldsm4(pf[i], pb + pr * kKT + swz(pr, kk * 2 + (lane >> 4)) * 8);
+        }
+        const int vr = kk * 16 + (lane & 15);
+        if constexpr (NT == 1) {
+          uint32_t v0, v1;
+          ldsm2_t(v0, v1, vb + vr * P + swz(vr, warp) * 8);
+#pragma unroll
+          for (int i = 0; i < MT; ++i) mma16816(acc[i][0], pf[i], v0, v1);
+        } else {
+#pragma unroll
+          for (int j = 0; j < NT; j += 2) {
+            uint32_t vf[4];
+            ldsm4_t(vf, vb + vr * P + swz(vr, warp * (C::DW / 8) + j + (lane >> 4)) * 8);
+#pragma unroll
+            for (int i = 0; i < MT; ++i) {
+              mma16816(acc[i][j], pf[i], vf[0], vf[1]);
+              mma16816(acc[i][j + 1], pf[i], vf[2], vf[3]);
+            }
+          }
+        }
+      }
+    }
+    __syncthreads();
+  }
+  // ---- result or partial
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int r = i * 16 + (lane >> 2) + half * 8;
+      if (row0 + r >= row1) continue;
+      const size_t row = head_row(r);
+      float inv = 1.f;
+      if (a.nsplit == 1) {
+        float l = ls[r], f = 1.f;
+        if (a.sink) {   // one more term of the sum, without a key or a value
+          const float s2 = a.sink[g * R + (row0 + r) % R] * kLog2e, mm = fmaxf(ms[r], s2);
+          f = exp2f(ms[r] - mm);
+          l = l * f + exp2f(s2 - mm);
+        }
+        inv = f / l;
+      }
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const int c = warp * C::DW + j * 8 + (lane & 3) * 2;
+        if (c >= a.vdim) continue;
+        const float x = acc[i][j][half * 2], y = acc[i][j][half * 2 + 1];
+        if (a.nsplit > 1)
+          *reinterpret_cast<float2*>(a.part_acc + (row * a.nsplit + split) * a.vdim + c) = make_float2(x, y);
+        else
+          *reinterpret_cast<__nv_bfloat162*>(o + row * a.vdim + c) = __floats2bfloat162_rn(x * inv, y * inv);
+      }
+    }
+  if (a.nsplit > 1 && tid < M && row0 + tid < row1) {
+    float* ml = a.part_ml + (head_row(tid) * a.nsplit + split) * 2;
+    ml[0] = ms[tid], ml[1] = ls[tid];
+  }
+}
+
+// o[row] = sum_s acc_s 2^(m_s - M) / (2^(sink - M) + sum_s l_s 2^(m_s - M)) for the rows of the tiles of M rows that
+// grouped_attn_kernel worked on; one warp per row.
+__global__ void __launch_bounds__(128) grouped_merge_kernel(__nv_bfloat16* __restrict__ o, const AttnArgs a, int M) {
+  pdl_entry();
+  const int R = a.group, n = a.nsplit, g = blockIdx.y, lane = threadIdx.x & 31;
+  int row0, row1;
+  if (a.tiles) {
+    row0 = a.tiles[blockIdx.x * 2], row1 = a.tiles[blockIdx.x * 2 + 1];
+  } else {
+    const int tpt = (R + M - 1) / M, t = blockIdx.x / tpt;
+    row0 = t * R + blockIdx.x % tpt * M;
+    row1 = min(row0 + M, (t + 1) * R);
+  }
+  if (a.num_valid && row0 / R >= *a.num_valid) return;
+  for (int r = row0 + (threadIdx.x >> 5); r < row1; r += 4) {
+    const int h = g * R + r % R;
+    const size_t row = (size_t)(r / R) * (a.kv_heads * R) + h;
+    const float* ml = a.part_ml + row * n * 2;
+    const float s2 = a.sink ? a.sink[h] * kLog2e : -1e30f;
+    // lane s holds split s (at most 32)
+    const float ms = lane < n ? ml[lane * 2] : -1e30f, ls = lane < n ? ml[lane * 2 + 1] : 0.f;
+    const float mx = fmaxf(warp_max(ms), s2);
+    const float f = ls > 0.f ? exp2f(ms - mx) : 0.f;
+    const float inv = 1.f / (warp_sum(ls * f) + (a.sink ? exp2f(s2 - mx) : 0.f));
+    for (int c0 = 0; c0 < a.vdim; c0 += 32) {
+      const int c = c0 + lane;
+      float v = 0.f;
+      for (int s = 0; s < n; ++s) {
+        const float fs = __shfl_sync(0xffffffffu, f, s);
+        if (fs > 0.f && c < a.vdim) v = fmaf(a.part_acc[(row * n + s) * a.vdim + c], fs, v);
+      }
+      if (c < a.vdim) o[row * a.vdim + c] = f2bf(v * inv);
+    }
+  }
+}
+
+// ------------------------------------------------------------------ one warp per row, fp32 arithmetic
+template <typename T, int NI>
+__global__ void __launch_bounds__(128) grouped_row_kernel(const T* __restrict__ q, const T* __restrict__ keys,
+                                                          const T* __restrict__ values, T* __restrict__ o,
+                                                          const AttnArgs a) {
+  pdl_entry();
+  constexpr int KB = 4;     // keys at a time
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int H = a.kv_heads * a.group;
+  if (row >= a.rows * H) return;
+  const int t = row / H, h = row % H, g = h / a.group;
+  if (a.num_valid && t >= *a.num_valid) return;
+  const int nkeys = a.pos[t] + 1;
+  const int* pt = a.page_table + (size_t)a.slots[t] * a.ld_pt;
+  const T *kb = keys + g * a.dim, *vb = values + g * a.vdim;
+  const size_t ldk = (size_t)a.kv_heads * a.dim, ldv = (size_t)a.kv_heads * a.vdim;
+  const float* rel = a.rel ? a.rel + (size_t)h * a.n_rel : nullptr;
+  float qv[NI], acc[NI];
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int c = i * 32 + lane;
+    qv[i] = c < a.dim ? ld_f(q + (size_t)row * a.dim + c) : 0.f;
+    acc[i] = 0.f;
+  }
+  float m = -1e30f, l = 0.f;
+  if (a.sink) m = a.sink[h], l = 1.f;
+  for (int k0 = 0; k0 < nkeys; k0 += 32) {
+    const int mine = pt[min(k0 + lane, nkeys - 1)];
+    const int n = min(32, nkeys - k0);
+    for (int k = 0; k < n; k += KB) {
+      size_t loc[KB];
+      float s[KB];
+#pragma unroll
+      for (int j = 0; j < KB; ++j) {
+        loc[j] = (size_t)__shfl_sync(0xffffffffu, mine, k + j);    // places past the last key repeat it
+        const T* kp = kb + loc[j] * ldk;
+        s[j] = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i)
+          if (i * 32 + lane < a.dim) s[j] = fmaf(qv[i], ld_f(kp + i * 32 + lane), s[j]);
+      }
+      float mn = m;
+#pragma unroll
+      for (int j = 0; j < KB; ++j) {
+        s[j] = warp_sum(s[j]) * a.scale;
+        if (a.cap > 0.f) s[j] = a.cap * tanhf(s[j] / a.cap);
+        if (rel) s[j] += rel[min(max(nkeys - 1 - (k0 + k + j), 0), a.n_rel - 1)];
+        if (k + j >= n) s[j] = -INFINITY;
+        mn = fmaxf(mn, s[j]);
+      }
+      const float al = expf(m - mn);
+      m = mn;
+      l *= al;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) acc[i] *= al;
+#pragma unroll
+      for (int j = 0; j < KB; ++j) {
+        const float p = expf(s[j] - mn);
+        const T* vp = vb + loc[j] * ldv;
+        l += p;
+#pragma unroll
+        for (int i = 0; i < NI; ++i)
+          if (i * 32 + lane < a.vdim) acc[i] = fmaf(p, ld_f(vp + i * 32 + lane), acc[i]);
+      }
+    }
+  }
+  const float inv = 1.f / l;
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int c = i * 32 + lane;
+    if (c < a.vdim) st_f(o + (size_t)row * a.vdim + c, acc[i] * inv);
+  }
+}
+
+// ------------------------------------------------------------------ keys and values of long portions, side by side
+// ctx_k[dst + j] = keys of key j of every listed request; ctx_vt[:, dst + j] = its values; zeros in the padding behind them.
+// list: [segs][3] = slot, keys, first row of the copy (a multiple of 64).  One CTA: 64 keys x 64 columns of k or v.
+__global__ void __launch_bounds__(256) kv_gather_kernel(const __nv_bfloat16* __restrict__ keys,
+                                                        const __nv_bfloat16* __restrict__ values,
+                                                        __nv_bfloat16* __restrict__ ctx_k, __nv_bfloat16* __restrict__ ctx_vt,
+                                                        const int* __restrict__ list, int segs, int total,
+                                                        const int* __restrict__ page_table, int ld_pt, int kw, int vw) {
+  pdl_entry();
+  __shared__ __nv_bfloat16 tile[64][66];
+  const int row0 = blockIdx.x * 64, kblocks = (kw + 63) / 64, tid = threadIdx.x;
+  int lo = 0, hi = segs - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (list[mid * 3 + 2] <= row0) lo = mid; else hi = mid - 1;
+  }
+  const int j0 = row0 - list[lo * 3 + 2], n = list[lo * 3 + 1];
+  const int* pt = page_table + (size_t)list[lo * 3] * ld_pt;
+  const bool is_k = (int)blockIdx.y < kblocks;
+  const int c0 = (is_k ? blockIdx.y : blockIdx.y - kblocks) * 64, w = is_k ? kw : vw;
+  const __nv_bfloat16* src = is_k ? keys : values;
+  for (int i = tid; i < 64 * 8; i += 256) {
+    const int r = i >> 3, c = (i & 7) * 8;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (j0 + r < n && c0 + c < w) v = *reinterpret_cast<const uint4*>(src + (size_t)pt[j0 + r] * w + c0 + c);
+    if (is_k) {
+      if (row0 + r < total && c0 + c < w) *reinterpret_cast<uint4*>(ctx_k + (size_t)(row0 + r) * w + c0 + c) = v;
+    } else {
+      uint32_t* d = reinterpret_cast<uint32_t*>(&tile[r][c]);
+      d[0] = v.x, d[1] = v.y, d[2] = v.z, d[3] = v.w;
+    }
+  }
+  if (is_k) return;
+  __syncthreads();
+  for (int i = tid; i < 64 * 8; i += 256) {
+    const int c = i >> 3, r = (i & 7) * 8;
+    if (c0 + c >= w) continue;
+    __align__(16) __nv_bfloat16 v[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = tile[r + e][c];
+    *reinterpret_cast<uint4*>(ctx_vt + (size_t)(c0 + c) * total + row0 + r) = *reinterpret_cast<uint4*>(v);
+  }
+}
+
+template <int P, int MT>
+int launch_attn(const void* q, const void* k, const void* v, void* o, const AttnArgs& a, cudaStream_t st) {
+  using C = AttnCfg<P, MT>;
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(grouped_attn_kernel<P, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM) !=
+        cudaSuccess)
+      return 671;
+    set = true;
+  }
+  dsv4_launch(grouped_attn_kernel<P, MT>, dim3(a.n_tiles, a.nsplit, a.kv_heads), 256, C::SMEM, st, (const __nv_bfloat16*)q,
+              (const __nv_bfloat16*)k, (const __nv_bfloat16*)v, (__nv_bfloat16*)o, a);
+  if (a.nsplit > 1)
+    dsv4_launch(grouped_merge_kernel, dim3(a.n_tiles, a.kv_heads), 128, 0, st, (__nv_bfloat16*)o, a, C::M);
+  return (int)cudaGetLastError();
+}
+template <int P>
+int dispatch_attn(int m, const void* q, const void* k, const void* v, void* o, const AttnArgs& a, cudaStream_t st) {
+  switch (m) {
+    case 16: return launch_attn<P, 1>(q, k, v, o, a, st);
+    case 32: return launch_attn<P, 2>(q, k, v, o, a, st);
+    case 64: return launch_attn<P, 4>(q, k, v, o, a, st);
+    default: return 672;
+  }
+}
+template <typename T>
+int launch_row(const void* q, const void* k, const void* v, void* o, const AttnArgs& a, cudaStream_t st) {
+  const int grid = (a.rows * a.kv_heads * a.group + 3) / 4, w = a.dim > a.vdim ? a.dim : a.vdim;
+  const T *tq = (const T*)q, *tk = (const T*)k, *tv = (const T*)v;
+  if (w <= 64)
+    dsv4_launch(grouped_row_kernel<T, 2>, grid, 128, 0, st, tq, tk, tv, (T*)o, a);
+  else if (w <= 128)
+    dsv4_launch(grouped_row_kernel<T, 4>, grid, 128, 0, st, tq, tk, tv, (T*)o, a);
+  else if (w <= 256)
+    dsv4_launch(grouped_row_kernel<T, 8>, grid, 128, 0, st, tq, tk, tv, (T*)o, a);
+  else if (w <= 512)
+    dsv4_launch(grouped_row_kernel<T, 16>, grid, 128, 0, st, tq, tk, tv, (T*)o, a);
+  else
+    return 673;
+  return (int)cudaGetLastError();
+}
+
+template <typename T, int W>
+void launch_rotate(const void* qkv, void* q, void* keys, void* values, const RotateArgs& a, int rows, cudaStream_t st) {
+  dsv4_launch(rotate_store_kernel<T, W>, rows, 256, a.pairs * sizeof(float2), st, (const T*)qkv, (T*)q, (T*)keys,
+              (T*)values, a);
+}
+
+}  // namespace
+
+// qkv [rows, ld]: q (heads x dim) | k (kv_heads x dim) | v (kv_heads x vdim); q_out [rows, heads * dim]; caches
+// [locations, kv_heads * dim] and [locations, kv_heads * vdim].  pairs: rotated pairs per head; every 0: no temperature.
+DSV4_API int dsv4_rotate_store(const void* qkv, int ld, const float* bias, const float* freq, int pairs, float coef, int every,
+                               const int* pos, const int* out_loc, void* q_out, void* keys, void* values, int rows,
+                               int heads, int kv_heads, int dim, int vdim, int fp32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (pairs < 0 || 2 * pairs > dim || pairs > 4096 || (pairs && !freq) || every < 0) return 674;
+  const RotateArgs a{ld, bias, freq, pairs, coef, every, pos, out_loc, heads, kv_heads, dim, vdim};
+  const bool wide = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0;
+  if (fp32)
+    wide ? launch_rotate<float, 4>(qkv, q_out, keys, values, a, rows, st)
+         : launch_rotate<float, 1>(qkv, q_out, keys, values, a, rows, st);
+  else
+    wide ? launch_rotate<__nv_bfloat16, 8>(qkv, q_out, keys, values, a, rows, st)
+         : launch_rotate<__nv_bfloat16, 1>(qkv, q_out, keys, values, a, rows, st);
+  return (int)cudaGetLastError();
+}
+
+// q [rows, heads * dim], o [rows, heads * vdim].  m: rows per CTA (16, 32 or 64; 0 = the one-warp-per-row kernel, which takes
+// every token).  tiles: [n_tiles][2] row ranges (see AttnArgs), or null: n_tiles covers every token's own rows.  nsplit > 1
+// (at most 32) needs part_acc [rows * heads, nsplit, vdim] and part_ml [rows * heads, nsplit, 2].
+DSV4_API int dsv4_grouped_attention(const void* q, const void* keys, const void* values, void* o, const int* slots,
+                                    const int* pos, const int* page_table, int ld_pt, const int* tiles, int n_tiles,
+                                    const int* num_valid, int rows, int kv_heads, int group, int dim, int vdim, float scale,
+                                    float cap, const float* sink, const float* rel, int n_rel, int m, int nsplit,
+                                    float* part_acc, float* part_ml, int fp32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (nsplit < 1 || nsplit > 32 || (nsplit > 1 && (!part_acc || !part_ml)) || (rel && n_rel < 1)) return 675;
+  if (kv_heads < 1 || kv_heads > 65535 || group < 1) return 676;
+  const AttnArgs a{slots, pos, page_table, ld_pt, tiles, n_tiles, num_valid, rows, kv_heads, group, dim, vdim, scale, cap,
+                   sink, rel, n_rel, nsplit, part_acc, part_ml};
+  if (m == 0)
+    return fp32 ? launch_row<float>(q, keys, values, o, a, st) : launch_row<__nv_bfloat16>(q, keys, values, o, a, st);
+  if (fp32 || dim % 8 || vdim % 8) return 677;
+  if (n_tiles <= 0) return 0;
+  const int w = dim > vdim ? dim : vdim;
+  if (w <= 64) return dispatch_attn<64>(m, q, keys, values, o, a, st);
+  if (w <= 128) return dispatch_attn<128>(m, q, keys, values, o, a, st);
+  if (w <= 256) return dispatch_attn<256>(m, q, keys, values, o, a, st);
+  return 678;
+}
+
+// ctx_k [total, kw], ctx_vt [vw, total]; total and the first rows of list are multiples of 64.
+DSV4_API int dsv4_kv_gather(const void* keys, const void* values, void* ctx_k, void* ctx_vt, const int* list, int segs,
+                            int total, const int* page_table, int ld_pt, int kw, int vw, cudaStream_t st) {
+  if (total <= 0) return 0;
+  if (kw % 8 || vw % 8 || total % 64 || segs < 1) return 679;
+  dsv4_launch(kv_gather_kernel, dim3(total / 64, (kw + 63) / 64 + (vw + 63) / 64), 256, 0, st, (const __nv_bfloat16*)keys,
+              (const __nv_bfloat16*)values, (__nv_bfloat16*)ctx_k, (__nv_bfloat16*)ctx_vt, list, segs, total, page_table,
+              ld_pt, kw, vw);
+  return (int)cudaGetLastError();
+}

@@ -13,7 +13,7 @@
 //
 // latent_attn_row_kernel computes the same with one warp per row on the CUDA cores, in fp32 throughout: models served in
 // 32-bit floats, and ranks the tensor-core kernel does not take.
-#include "vec.cuh"
+#include "mma16.cuh"
 
 namespace {
 
@@ -95,29 +95,6 @@ __device__ __forceinline__ bool find_tile(const LatArgs& a, int b, int& row0, in
 }
 
 // ------------------------------------------------------------------ tensor-core kernel
-__device__ __forceinline__ void cpa16_zfill(void* smem, const void* g, bool valid) {
-  const int sz = valid ? 16 : 0;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(smem)), "l"(g), "r"(sz) : "memory");
-}
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// 16-byte chunk c of row r sits at chunk (c ^ (r & 7)) within its group of eight
-__device__ __forceinline__ int swz(int r, int c) { return (c & ~7) | ((c ^ r) & 7); }
-
 constexpr int kKT = 64;   // keys per tile
 constexpr int kSP = kKT + 4;  // floats per score row
 
@@ -419,6 +396,25 @@ __global__ void __launch_bounds__(128) latent_attn_row_kernel(const T* __restric
   }
 }
 
+// ctx[dst + j] = cache[page_table[slot][j]] for the keys j of every listed request, zeros in the padding behind them.
+// list: [segs][3] = slot, keys, first row of the copy; rows [dst, dst of the next request) belong to a request.
+__global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* __restrict__ cache, uint4* __restrict__ ctx,
+                                                            const int* __restrict__ list, int segs, int total,
+                                                            const int* __restrict__ page_table, int ld_pt, int r8) {
+  pdl_entry();
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= total) return;
+  int lo = 0, hi = segs - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (list[mid * 3 + 2] <= row) lo = mid; else hi = mid - 1;
+  }
+  const int j = row - list[lo * 3 + 2];
+  const bool in = j < list[lo * 3 + 1];
+  const size_t src = in ? (size_t)page_table[(size_t)list[lo * 3] * ld_pt + j] * r8 : 0;
+  for (int i = lane; i < r8; i += 32) ctx[(size_t)row * r8 + i] = in ? cache[src + i] : make_uint4(0, 0, 0, 0);
+}
+
 template <int RP, int MT>
 int launch_lat(const void* q, const void* cache, void* o, const LatArgs& a, int tiles, cudaStream_t st) {
   using C = LatCfg<RP, MT>;
@@ -492,4 +488,13 @@ DSV4_API int dsv4_latent_attention(const void* q, const void* cache, void* o, co
   if (rank <= 384) return dispatch_lat<384>(m, q, cache, o, a, tiles, st);
   if (rank <= 512) return dispatch_lat<512>(m, q, cache, o, a, tiles, st);
   return 636;
+}
+
+DSV4_API int dsv4_latent_gather(const void* cache, void* ctx, const int* list, int segs, int total,
+                                const int* page_table, int ld_pt, int rank, cudaStream_t st) {
+  if (total <= 0) return 0;
+  if (rank % 8 || segs < 1) return 650;
+  dsv4_launch(latent_gather_kernel, (total + 3) / 4, 128, 0, st, (const uint4*)cache, (uint4*)ctx, list, segs, total,
+              page_table, ld_pt, rank / 8);
+  return (int)cudaGetLastError();
 }

@@ -139,6 +139,139 @@ __global__ void __launch_bounds__(256) silu_mul_kernel(const T* __restrict__ gu,
   st_f(out + i, g / (1.f + expf(-g)) * u);
 }
 
+// ------------------------------------------------------------------ layer norms around the sub-layers
+struct LayerNormArgs {
+  float* x;                   // [rows, d] stream, updated in place if keep
+  const long long* rows_idx;  // not null: output row r belongs to stream row rows_idx[r], and the stream is left alone
+  const float *sub, *sub_w, *sub_b;  // a sub-layer's output [rows, d], normed and added; or null
+  const void* add;            // activations [rows, d], added; or null
+  const float *w, *b;         // norm of the sum; null: no output
+  float eps;
+  int d, keep;
+};
+
+// Mean and 1 / standard deviation of a row of d values of which this thread holds NV x 4 (or walks every 256th); two passes:
+// the deviations are summed around the mean itself.
+template <int NV>
+__device__ __forceinline__ float2 row_stats(const float4 (&v)[NV], int d, float eps, float* sh) {
+  float s = 0.f;
+#pragma unroll
+  for (int n = 0; n < NV; ++n)
+    if ((n * 256 + (int)threadIdx.x) * 4 < d) s += (v[n].x + v[n].y) + (v[n].z + v[n].w);
+  const float mean = cta_sum(s, sh) / d;
+  float q = 0.f;
+#pragma unroll
+  for (int n = 0; n < NV; ++n)
+    if ((n * 256 + (int)threadIdx.x) * 4 < d) {
+      const float a = v[n].x - mean, b = v[n].y - mean, c = v[n].z - mean, e = v[n].w - mean;
+      q += (a * a + b * b) + (c * c + e * e);
+    }
+  return make_float2(mean, 1.f / sqrtf(cta_sum(q, sh) / d + eps));
+}
+__device__ __forceinline__ float4 norm4(const float4& v, const float2& st, const float4& w, const float4& b) {
+  return make_float4((v.x - st.x) * st.y * w.x + b.x, (v.y - st.x) * st.y * w.y + b.y, (v.z - st.x) * st.y * w.z + b.z,
+                     (v.w - st.x) * st.y * w.w + b.w);
+}
+
+// x += N(sub; sub_w, sub_b);  x += add;  out = N(x; w, b).  One CTA per row, the row stays in registers (NV x 4 values per
+// thread); NV = 0: any d, the sum passes through `out_row` in shared memory.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) residual_layer_norm_kernel(const LayerNormArgs a, T* __restrict__ out) {
+  pdl_entry();
+  __shared__ float sh[32];
+  extern __shared__ float rest[];
+  const int r = blockIdx.x, d = a.d;
+  const size_t src = (size_t)(a.rows_idx ? a.rows_idx[r] : r) * d;
+  const T* add = a.add ? static_cast<const T*>(a.add) + src : nullptr;
+  if constexpr (NV > 0) {
+    float4 x[NV], y[NV];
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int i = (n * 256 + threadIdx.x) * 4;
+      x[n] = y[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i >= d) continue;
+      x[n] = ld_f4(a.x + src + i);
+      if (a.sub) y[n] = ld_f4(a.sub + src + i);
+    }
+    if (a.sub) {
+      const float2 st = row_stats<NV>(y, d, a.eps, sh);
+#pragma unroll
+      for (int n = 0; n < NV; ++n) {
+        const int i = (n * 256 + threadIdx.x) * 4;
+        if (i >= d) continue;
+        const float4 v = norm4(y[n], st, ld_f4(a.sub_w + i), ld_f4(a.sub_b + i));
+        x[n].x += v.x, x[n].y += v.y, x[n].z += v.z, x[n].w += v.w;
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int i = (n * 256 + threadIdx.x) * 4;
+      if (i >= d) continue;
+      if (add) {
+        const float4 v = ld_f4(add + i);
+        x[n].x += v.x, x[n].y += v.y, x[n].z += v.z, x[n].w += v.w;
+      }
+      if (a.keep) st_f4(a.x + src + i, x[n]);
+    }
+    if (!a.w) return;
+    const float2 st = row_stats<NV>(x, d, a.eps, sh);
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int i = (n * 256 + threadIdx.x) * 4;
+      if (i < d) st_f4(out + (size_t)r * d + i, norm4(x[n], st, ld_f4(a.w + i), ld_f4(a.b + i)));
+    }
+  } else {
+    auto stats = [&](const float* v) {
+      float s = 0.f, q = 0.f;
+      for (int i = threadIdx.x; i < d; i += 256) s += v[i];
+      const float mean = cta_sum(s, sh) / d;
+      for (int i = threadIdx.x; i < d; i += 256) q += (v[i] - mean) * (v[i] - mean);
+      return make_float2(mean, 1.f / sqrtf(cta_sum(q, sh) / d + a.eps));
+    };
+    float2 st = make_float2(0.f, 0.f);
+    if (a.sub) st = stats(a.sub + src);
+    for (int i = threadIdx.x; i < d; i += 256) {   // every thread only reads back what it wrote itself
+      float v = a.x[src + i];
+      if (a.sub) v += (a.sub[src + i] - st.x) * st.y * a.sub_w[i] + a.sub_b[i];
+      if (add) v += ld_f(add + i);
+      if (a.keep) a.x[src + i] = v;
+      rest[i] = v;
+    }
+    if (!a.w) return;
+    st = stats(rest);
+    for (int i = threadIdx.x; i < d; i += 256) st_f(out + (size_t)r * d + i, (rest[i] - st.x) * st.y * a.w[i] + a.b[i]);
+  }
+}
+
+template <typename T>
+int launch_layer_norm(const LayerNormArgs& a, void* out, int rows, cudaStream_t st) {
+  auto go = [&](auto kern, size_t smem) { dsv4_launch(kern, rows, 256, smem, st, a, (T*)out); };
+  if (a.d % 4 || a.d > 8192) {
+    if (a.d > 11264) return 606;       // the row in 44 KB of shared memory
+    go(residual_layer_norm_kernel<T, 0>, (size_t)a.d * 4);
+  } else if (a.d <= 1024)
+    go(residual_layer_norm_kernel<T, 1>, 0);
+  else if (a.d <= 2048)
+    go(residual_layer_norm_kernel<T, 2>, 0);
+  else if (a.d <= 4096)
+    go(residual_layer_norm_kernel<T, 4>, 0);
+  else
+    go(residual_layer_norm_kernel<T, 8>, 0);
+  return (int)cudaGetLastError();
+}
+
+// gelu(gate) * up behind a projection without the gated epilogue: gu [rows, 2 f] in alternating blocks of 16 columns
+template <typename T>
+__global__ void __launch_bounds__(256) gelu_gate_kernel(const T* __restrict__ gu, T* __restrict__ out, long long total,
+                                                        int f) {
+  pdl_entry();
+  const long long i = blockIdx.x * 256ll + threadIdx.x;
+  if (i >= total) return;
+  const int c = (int)(i % f);
+  const T* g = gu + i / f * 2 * f + c / kGateBlock * 2 * kGateBlock + c % kGateBlock;
+  st_f(out + i, gelu_tanh(ld_f(g)) * ld_f(g + kGateBlock));
+}
+
 template <typename T>
 int launch_norm(const NormArgs& a, const void* erows, void* out, int rows, cudaStream_t st) {
   auto go = [&](auto kern) { dsv4_launch(kern, rows, 256, 0, st, a, (const T*)erows, (T*)out); };
@@ -194,5 +327,29 @@ DSV4_API int dsv4_silu_mul(const void* gu, void* out, int rows, int f, int fp32,
   else
     dsv4_launch(silu_mul_kernel<__nv_bfloat16>, grid, 256, 0, st, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, total,
                 f);
+  return (int)cudaGetLastError();
+}
+
+// x (+= N(sub; sub_w, sub_b)) (+= add);  out = N(x; w, b), N the layer norm of a row.  add and out: activations.  With
+// rows_idx the rows are gathered first and x is left alone.
+DSV4_API int dsv4_residual_layer_norm(float* x, const long long* rows_idx, const float* sub, const float* sub_w,
+                                      const float* sub_b, const void* add, const float* w, const float* b, float eps,
+                                      int keep, void* out, int rows, int d, int fp32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (rows_idx && keep) return 604;
+  if ((w && !out) || (sub && (!sub_w || !sub_b)) || (w && !b)) return 605;
+  const LayerNormArgs a{x, rows_idx, sub, sub_w, sub_b, add, w, b, eps, d, keep};
+  return fp32 ? launch_layer_norm<float>(a, out, rows, st) : launch_layer_norm<__nv_bfloat16>(a, out, rows, st);
+}
+
+DSV4_API int dsv4_gelu_gate(const void* gu, void* out, int rows, int f, int fp32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (f % kGateBlock) return 607;
+  const long long total = (long long)rows * f;
+  const unsigned grid = (unsigned)((total + 255) / 256);
+  if (fp32)
+    dsv4_launch(gelu_gate_kernel<float>, grid, 256, 0, st, (const float*)gu, (float*)out, total, f);
+  else
+    dsv4_launch(gelu_gate_kernel<__nv_bfloat16>, grid, 256, 0, st, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, total, f);
   return (int)cudaGetLastError();
 }

@@ -49,13 +49,41 @@ __device__ __forceinline__ float cta_sum(float v, float* sh) {
 }
 
 // Epilogue activations of the projections (the numbers are part of the host interface).
-enum GemmAct : int { kActNone = 0, kActRelu2 = 1, kActTanh = 2 };
+// kActGeluGate pairs columns: the weight rows come in blocks of 16 gate and 16 up rows, and the result is half as wide.
+enum GemmAct : int { kActNone = 0, kActRelu2 = 1, kActTanh = 2, kActGeluGate = 3 };
+constexpr int kGateBlock = 16;
 __device__ __forceinline__ float gemm_act(float v, int act) {
   if (act == kActRelu2) {
     v = fmaxf(v, 0.f);
     return v * v;
   }
   return act == kActTanh ? tanhf(v) : v;
+}
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+// 0.5 z (1 + tanh(w)) = z sigmoid(2 w),  w = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh(float z) {
+  return z * sigmoid_f(1.5957691216057308f * fmaf(0.044715f * z * z, z, z));
+}
+// v: a row's 32 consecutive columns (16 gate, 16 up) -> its 16 gated values in v[0..15]
+__device__ __forceinline__ void gate_block(float* v) {
+#pragma unroll
+  for (int j = 0; j < kGateBlock; ++j) v[j] = gelu_tanh(v[j]) * v[j + kGateBlock];
+}
+// 16 consecutive values, dst 16-byte aligned
+__device__ __forceinline__ void st_f16x(__nv_bfloat16* dst, const float* v) {
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    uint4 u;
+    __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) p[e] = __floats2bfloat162_rn(v[8 * i + 2 * e], v[8 * i + 2 * e + 1]);
+    reinterpret_cast<uint4*>(dst)[i] = u;
+  }
+}
+__device__ __forceinline__ void st_f16x(float* dst, const float* v) {
+#pragma unroll
+  for (int i = 0; i < 4; ++i) st_f4(dst + 4 * i, make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]));
 }
 
 // First and last row of a request's rows in the batch: rows of a request stand together at consecutive positions.

@@ -202,7 +202,7 @@ def expanded_attention(q, cache, fb, uk, uv, heads, scale):
     k, vt = linear(ctx, uk), linear(uv, ctx)
     out = torch.empty(t, heads * vdim, dtype=q.dtype, device=q.device)
     nv.call("flash_attention", nv.ptr(q), I(q.stride(0)), nv.ptr(k), nv.ptr(vt), nv.ptr(out), nv.ptr(items), I(n_items),
-            I(t), I(rows), I(heads), I(dim), I(vdim), F(scale))
+            I(t), I(rows), I(heads), I(heads), I(dim), I(vdim), F(scale), F(0.0), nv.ptr(None), nv.ptr(None), I(0))
     return out
 
 

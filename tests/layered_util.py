@@ -1,4 +1,4 @@
-"""Shared pieces of the Bedalorn tests: forwards over a shuffled page table, and traces through the engine."""
+"""Shared pieces of the tests of the layered designs: forwards over a shuffled page table, and traces through the engine."""
 import torch
 
 from minisgl.models.base import ForwardBatch

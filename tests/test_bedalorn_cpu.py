@@ -11,7 +11,7 @@ import torch
 
 import bedalorn_cases as K
 import plain_bedalorn as P
-from bedalorn_util import replay
+from layered_util import replay
 from minisgl.core import SamplingParams
 from minisgl.llm import LLM
 from minisgl.models import bedalorn_weight as W

@@ -23,7 +23,7 @@ def mixed(request, tmp_path):
 
 
 def test_layers_one_by_one(case):
-    from bedalorn_util import replay
+    from layered_util import replay
     import plain_bedalorn as P
 
     toks = K.tokens(case.cfg, 70, 5)
@@ -86,7 +86,7 @@ def test_poisoned_storage_changes_nothing(tmp_path):
     """Whatever pages and slots held before, a new request starts clean."""
     case = K.Case("state", tmp_path, "cuda", torch.bfloat16)
     reqs = {"a": K.tokens(case.cfg, 90, 3), "b": K.tokens(case.cfg, 1, 4)}
-    from bedalorn_util import replay
+    from layered_util import replay
 
     def run(poison):
         t = case.trace(192)

@@ -5,7 +5,7 @@ import pytest
 import torch
 
 import plain_bedalorn as P
-from bedalorn_util import make_fb
+from layered_util import make_fb
 from minisgl.ops import api as O
 from minisgl.ops import cuda_layers as C
 
