@@ -44,9 +44,9 @@ def parse():
     ap.add_argument("--moe-mode", default="ep", choices=["ep", "tp"])
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--no-fused-comm", action="store_true")
-    ap.add_argument("--design", default="", choices=["", "bedalorn"],
-                    help="instead of the headline: prefill / decode throughput of this design beside DeepSeek-V4 at equal "
-                         "size (one JSON line per model and workload, one GPU)")
+    ap.add_argument("--design", default="", choices=["", "bedalorn", "buvalix"],
+                    help="instead of the headline: prefill / decode throughput of this design beside the closest other "
+                         "model at equal size (one JSON line per model and workload, one GPU)")
     ap.add_argument("--sizes", default="small,large", help="with --design: model sizes to run")
     ap.add_argument("--profile", action="store_true", help="with --design: add per-launcher device times")
     args = ap.parse_args()
@@ -155,7 +155,7 @@ def main():
     if args.design:
         from minisgl.benchmark import designs
 
-        designs.main(args.sizes.split(","), args.profile)
+        designs.main(args.design, args.sizes.split(","), args.profile)
         return
     import torch
     import torch.distributed as dist

@@ -1,8 +1,10 @@
-"""Prefill and decode throughput of the Bedalorn design beside the closest other model (DeepSeek-V4) at equal size.
+"""Prefill and decode throughput of a layered design beside the closest other model at equal size: Bedalorn beside DeepSeek-V4,
+Buvalix beside Bedalorn.
 
-    python bench.py --design bedalorn [--sizes small,large] [--profile]
+    python bench.py --design bedalorn|buvalix [--sizes small,large] [--profile]
 
-Equal size: the same width, layer runs, attention heads, experts (number, chosen, intermediate size) and vocabulary, random
+Equal size: the same width, layer runs, attention heads, vocabulary and feed-forward weights (DeepSeek-V4: the same experts;
+Buvalix's gated feed-forwards have three matrices, so the Bedalorn model beside it has dense ones half as wide again), random
 weights, one GPU, through the offline API.  Per model and workload one JSON line: device time of the forwards (CUDA
 events), tokens per second, and with ``--profile`` the per-launcher share of one eager forward of each phase.
 Workloads: prefill forwards of 8 x 1 024 and 1 x 8 192 tokens; decode steps of 128 sequences at 1 024 tokens of context and
@@ -19,19 +21,50 @@ SIZES = {
     "small": (2048, 16, 32, 512, 8192, 32, 4, 1024, 8, 1, 32768),
     "large": (4096, 32, 64, 512, 16384, 32, 4, 2048, 4, 2, 65536),
 }
+DENSE_SIZES = {
+    # width, attention heads, key heads, delta heads, wkv heads, latent rank, gated ff, layers, loop passes, vocab
+    "small": (2048, 16, 4, 16, 32, 512, 5632, 8, 1, 32768),
+    "large": (4096, 32, 8, 32, 64, 512, 11264, 4, 2, 65536),
+}
 WORKLOADS = [("prefill", 8, 1024), ("prefill", 1, 8192), ("decode", 128, 1024), ("decode", 8, 8192)]
 
 
+def _loop(n: int, passes: int):
+    from minisgl.models.layered_config import LoopSpec
+
+    return LoopSpec(0, n, passes) if passes > 1 else None
+
+
 def bedalorn_config(size: str):
-    from minisgl.models.bedalorn_config import (BedalornConfig, DenseSpec, ExpertsSpec, LatentAttentionSpec, LayerSpec,
-                                                LoopSpec, WKVSpec)
+    from minisgl.models.bedalorn_config import BedalornConfig, DenseSpec, ExpertsSpec, LatentAttentionSpec, LayerSpec, WKVSpec
 
     d, h, hw, rank, ff, e, top, eff, n, passes, vocab = SIZES[size]
     attn = LatentAttentionSpec(h, 128, 128, rank, 128 ** -0.5)
     moe = ExpertsSpec(eff, e, top)
     layers = tuple(LayerSpec(WKVSpec(hw, 64), moe) if i % 4 == 2 else
                    LayerSpec(attn, DenseSpec(ff) if i % 4 == 0 else moe) for i in range(n))
-    return BedalornConfig(layers, d, vocab, 1e-6, 1.0, LoopSpec(0, n, passes) if passes > 1 else None, 1 << 17)
+    return BedalornConfig(layers, d, vocab, 1e-6, 1.0, _loop(n, passes), 1 << 17)
+
+
+def bedalorn_dense_config(size: str):
+    from minisgl.models.bedalorn_config import BedalornConfig, DenseSpec, LatentAttentionSpec, LayerSpec, WKVSpec
+
+    d, h, _, _, hw, rank, ff, n, passes, vocab = DENSE_SIZES[size]
+    attn = LatentAttentionSpec(h, 128, 128, rank, 128 ** -0.5)
+    layers = tuple(LayerSpec(WKVSpec(hw, 64) if i % 4 == 2 else attn, DenseSpec(ff * 3 // 2)) for i in range(n))
+    return BedalornConfig(layers, d, vocab, 1e-6, 1.0, _loop(n, passes), 1 << 17)
+
+
+def buvalix_config(size: str):
+    from minisgl.models.buvalix_config import (BuvalixConfig, ChannelDeltaSpec, DenseSpec, GroupedAttentionSpec, LayerSpec,
+                                               QueryTemperature, RotarySpec)
+
+    d, h, g, hd, _, _, ff, n, passes, vocab = DENSE_SIZES[size]
+    rotary = GroupedAttentionSpec(h, g, 128, 128, 128 ** -0.5, 30.0, rot=RotarySpec(64, 1e5), bias=True, sink=True)
+    bucket = GroupedAttentionSpec(h, g, 128, 128, 128 ** -0.5, 40.0, q_temp=QueryTemperature(0.1, 512), bias_max=2048)
+    delta = ChannelDeltaSpec(hd, hd, 128, 128, 4)
+    layers = tuple(LayerSpec((rotary, bucket, delta, rotary)[i % 4], DenseSpec(ff)) for i in range(n))
+    return BuvalixConfig(layers, d, vocab, 1e-6, _loop(n, passes), 1 << 17)
 
 
 def dsv4_config(size: str):
@@ -120,16 +153,21 @@ def run(cfg, phase: str, batch: int, context: int, profile: bool, steps: int = 3
     return out
 
 
-def main(sizes=("small", "large"), profile: bool = False, workloads=None, models=("bedalorn", "dsv4")) -> None:
+PAIRS = {
+    "bedalorn": {"bedalorn": bedalorn_config, "dsv4": dsv4_config},
+    "buvalix": {"buvalix": buvalix_config, "bedalorn": bedalorn_dense_config},
+}
+
+
+def main(design: str, sizes=("small", "large"), profile: bool = False, workloads=None) -> None:
     import gc
 
     import torch
 
-    makers = {"bedalorn": bedalorn_config, "dsv4": dsv4_config}
     for size in sizes:
-        for name in models:
+        for name, make in PAIRS[design].items():
             for phase, batch, context in workloads or WORKLOADS:
-                r = run(makers[name](size), phase, batch, context, profile)
+                r = run(make(size), phase, batch, context, profile)
                 print(json.dumps({"design": name, "size": size, **r}), flush=True)
                 gc.collect()
                 torch.cuda.empty_cache()

@@ -26,6 +26,9 @@ MODELS = {
     "wide": P.config([P.rotary_layer(2, 1, 160, 144, 64, 1e4, 0.1, 15.0, 40), P.delta_layer(2, 1, 136, 152, 4)], width=72, vocab=88),
 }
 LIMIT = {torch.float32: 1e-4, torch.bfloat16: 4e-2}
+# Unit vectors and head norms of small vectors amplify rounding: in bf16 a few positions are further off, with every backend
+# at the same places.
+STRAY, WORST = 0.03, 0.16
 
 
 class Case(layered_checks.Case):
@@ -33,4 +36,4 @@ class Case(layered_checks.Case):
         cfg = MODELS[name]
         tensors = P.tensors(cfg, seed=len(name))
         super().__init__(cfg, tensors, P.PlainBuvalix(cfg, tensors), P.write_model(cfg, tensors, folder), device, dtype,
-                         LIMIT[dtype])
+                         LIMIT[dtype], STRAY if dtype == torch.bfloat16 else 0.0, WORST)

@@ -52,22 +52,23 @@ def softcap(s, cap):
 
 def attend(q, k, v, group, scale, cap, sink, bias):
     """q [T, H, dim] at the last T places of k [n, G, dim], v [n, G, vdim]; query head h reads key head h // group.  sink
-    [H] or None; bias(distances) -> [keys, H] or None."""
+    [H] or None; bias(distances) -> [.., H] or None."""
     t, heads = q.shape[:2]
-    n0 = k.shape[0] - t
-    out = torch.empty(t, heads, v.shape[2], dtype=F)
-    for i in range(t):
-        see = n0 + i + 1
-        add = bias(see - 1 - torch.arange(see)) if bias is not None else None
-        for h in range(heads):
-            s = softcap((k[:see, h // group] @ q[i, h]) * scale, cap)
-            if add is not None:
-                s = s + add[:, h]
-            top = s.max() if sink is None else torch.maximum(s.max(), sink[h])
-            e = torch.exp(s - top)
-            total = e.sum() + (0.0 if sink is None else torch.exp(sink[h] - top))
-            out[i, h] = (e / total) @ v[:see, h // group]
-    return out
+    n = k.shape[0]
+    away = (n - t + torch.arange(t))[:, None] - torch.arange(n)[None, :]          # [T, n], negative: not seen
+    out = []
+    for h in range(heads):
+        s = softcap(q[:, h] @ k[:, h // group].T * scale, cap)
+        if bias is not None:
+            s = s + bias(away.clamp_min(0))[..., h]
+        s = torch.where(away >= 0, s, torch.full_like(s, -math.inf))
+        top = s.max(-1, keepdim=True).values
+        if sink is not None:
+            top = torch.maximum(top, sink[h])
+        e = torch.exp(s - top)
+        total = e.sum(-1, keepdim=True) + (0.0 if sink is None else torch.exp(sink[h] - top))
+        out.append((e / total) @ v[:, h // group])
+    return torch.stack(out, 1)
 
 
 def rotary_attention_mixer(h, p, m, past):
