@@ -11,6 +11,7 @@ with a dummy request); a third, small class covers contexts where top-k selectio
 from __future__ import annotations
 
 import bisect
+import gc
 from typing import Dict, List, Optional, Tuple
 
 import torch
@@ -84,6 +85,20 @@ class GraphRunner:
         b.slots.fill_(e.dummy_slot)
         b.out_loc.fill_(e.pool.dummy_page * e.page_size)
         b.num_valid.fill_(1)
+        # a collection in the middle of a capture may free another engine's graphs or buffers, which invalidates the capture
+        gc.collect()
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            self._capture_buckets()
+        finally:
+            if collecting:
+                gc.enable()
+        native.assert_device_ok()
+        logger.info_rank0("captured %d CUDA graphs (buckets %s, context classes %s)", len(self.graphs), self.buckets,
+                          self.classes)
+
+    def _capture_buckets(self) -> None:
         torch.cuda.synchronize()
         stream = torch.cuda.Stream()
         for bs in sorted(self.buckets, reverse=True):
@@ -102,9 +117,6 @@ class GraphRunner:
                 self.logits[(bs, ci)] = out[0]
                 self.capture_status["captured"] += 1
         torch.cuda.synchronize()
-        native.assert_device_ok()
-        logger.info_rank0("captured %d CUDA graphs (buckets %s, context classes %s)", len(self.graphs), self.buckets,
-                          self.classes)
 
     # ------------------------------------------------------------------ replay
     def padded_size(self, bs: int) -> int:

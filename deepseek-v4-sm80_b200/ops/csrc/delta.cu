@@ -20,7 +20,110 @@ struct ConvArgs {
   int rows, d, e, kv_heads, heads;
 };
 
-// One warp per (token, head of q, k or v).  Inputs ahead of the portion come from the slot.
+// A head of q, k or v.
+struct ConvUnit {
+  int part, head, width, ch0, col0;
+  __device__ __forceinline__ ConvUnit(const ConvArgs& a, int unit) {
+    part = unit < a.kv_heads ? 0 : unit < 2 * a.kv_heads ? 1 : 2;
+    head = unit - part * a.kv_heads, width = part == 2 ? a.e : a.d;
+    ch0 = part * a.cols.nqk + head * width;
+    col0 = a.cols.col(ch0);
+  }
+};
+
+// One warp per head and TB tokens, N taps: every input is read once, the taps and the last N - 1 inputs stay in registers.
+// NI x 4 x 32 channels at most, sizes multiples of 4.
+template <typename T, int NI, int N, int TB>
+__global__ void __launch_bounds__(256) conv_unit_tile_kernel(const T* __restrict__ p, const T* __restrict__ before,
+                                                             float* __restrict__ q, float* __restrict__ k,
+                                                             T* __restrict__ v, const ConvArgs a) {
+  pdl_entry();
+  const int t0 = (blockIdx.y * 8 + (threadIdx.x >> 5)) * TB, lane = threadIdx.x & 31;
+  if (t0 >= a.rows) return;
+  const ConvUnit un(a, blockIdx.x);
+  const int C = 2 * a.cols.nqk + a.cols.nv;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  int slot[TB], pos[TB];
+  float4 x[TB][NI], w[N][NI], old[N > 1 ? N - 1 : 1][NI];    // old[b]: b + 1 tokens back
+#pragma unroll
+  for (int i = 0; i < TB; ++i) {
+    const int t = min(t0 + i, a.rows - 1);
+    slot[i] = a.slots[t], pos[i] = a.pos[t];
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int c = (n * 32 + lane) * 4;
+      x[i][n] = c < un.width ? ld_f4(p + (size_t)t * a.cols.ld + un.col0 + c) : zero;
+    }
+  }
+#pragma unroll
+  for (int b = 0; b < N; ++b)
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int c = (n * 32 + lane) * 4;
+      w[b][n] = c < un.width ? ld_f4(a.taps + (size_t)(N - 1 - b) * C + un.ch0 + c) : zero;   // b tokens back
+    }
+#pragma unroll
+  for (int i = 0; i < TB; ++i) {
+    const int t = t0 + i;
+    if (t >= a.rows) return;
+    if (i == 0 || slot[i] != slot[i > 0 ? i - 1 : 0] || pos[i] != pos[i > 0 ? i - 1 : 0] + 1) {
+      int have = 1;               // rows of this portion that the convolution reads; older inputs come from the slot
+#pragma unroll
+      for (int b = 1; b < N; ++b)
+        if (have == b && t - b >= 0 && a.slots[t - b] == slot[i] && a.pos[t - b] == pos[i] - b) ++have;
+#pragma unroll
+      for (int b = 1; b < N; ++b)
+#pragma unroll
+        for (int n = 0; n < NI; ++n) {
+          const int c = (n * 32 + lane) * 4;
+          float4 o = zero;
+          if (c < un.width && pos[i] - b >= 0) {
+            if (b < have) {
+              o = ld_f4(p + (size_t)(t - b) * a.cols.ld + un.col0 + c);
+            } else {
+              const T* src = before + ((size_t)slot[i] * (N - 1) + N - 2 - (b - have)) * C + un.ch0 + c;
+              o = make_float4(ld_f(src), ld_f(src + 1), ld_f(src + 2), ld_f(src + 3));
+            }
+          }
+          old[b - 1][n] = o;
+        }
+    }
+    float4 y[NI];
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      float4 s = make_float4(x[i][n].x * w[0][n].x, x[i][n].y * w[0][n].y, x[i][n].z * w[0][n].z, x[i][n].w * w[0][n].w);
+#pragma unroll
+      for (int b = 1; b < N; ++b) {
+        const float4 o = old[b - 1][n], f = w[b][n];
+        s.x = fmaf(o.x, f.x, s.x), s.y = fmaf(o.y, f.y, s.y), s.z = fmaf(o.z, f.z, s.z), s.w = fmaf(o.w, f.w, s.w);
+      }
+      s.x *= sigmoid_for<T>(s.x), s.y *= sigmoid_for<T>(s.y), s.z *= sigmoid_for<T>(s.z), s.w *= sigmoid_for<T>(s.w);
+      ss += (s.x * s.x + s.y * s.y) + (s.z * s.z + s.w * s.w);
+      y[n] = s;
+#pragma unroll
+      for (int b = N - 2; b > 0; --b) old[b][n] = old[b - 1][n];
+      if (N > 1) old[0][n] = x[i][n];
+    }
+    float sc = 1.f;
+    if (un.part < 2) {
+      sc = 1.f / sqrtf(warp_sum(ss) + 1e-6f);
+      if (un.part == 0) sc *= 1.f / sqrtf((float)a.d);
+    }
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int c = (n * 32 + lane) * 4;
+      if (c >= un.width) continue;
+      const float4 s = make_float4(y[n].x * sc, y[n].y * sc, y[n].z * sc, y[n].w * sc);
+      if (un.part == 2)
+        st_f4(v + (size_t)t * a.cols.nv + un.head * un.width + c, s);
+      else
+        st_f4((un.part ? k : q) + (size_t)t * a.cols.nqk + un.head * un.width + c, s);
+    }
+  }
+}
+
+// Any number of taps, any sizes: one warp per (token, head of q, k or v).
 template <typename T, int W>     // W consecutive channels per lane and step (4, or 1 for sizes that are no multiple of 4)
 __global__ void __launch_bounds__(256) conv_unit_kernel(const T* __restrict__ p, const T* __restrict__ before,
                                                         float* __restrict__ q, float* __restrict__ k, T* __restrict__ v,
@@ -28,11 +131,9 @@ __global__ void __launch_bounds__(256) conv_unit_kernel(const T* __restrict__ p,
   pdl_entry();
   const int t = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (t >= a.rows) return;
-  const int unit = blockIdx.x, n = a.cols.taps, C = 2 * a.cols.nqk + a.cols.nv;
-  const int part = unit < a.kv_heads ? 0 : unit < 2 * a.kv_heads ? 1 : 2;
-  const int head = unit - part * a.kv_heads, width = part == 2 ? a.e : a.d;
-  const int ch0 = part * a.cols.nqk + head * width;
-  const int col0 = a.cols.col(ch0);
+  const int n = a.cols.taps, C = 2 * a.cols.nqk + a.cols.nv;
+  const ConvUnit un(a, blockIdx.x);
+  const int part = un.part, head = un.head, width = un.width, ch0 = un.ch0, col0 = un.col0;
   const int slot = a.slots[t], pos = a.pos[t];
   int have = 1;                   // rows of this portion up to and including this one that the convolution reads
   while (have < n && t - have >= 0 && a.slots[t - have] == slot && a.pos[t - have] == pos - have) ++have;
@@ -285,14 +386,14 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __rest
       const int c = (i * 32 + lane) * 4;
       if (c >= e) continue;
       const float4 gt = ld_f4(gate + r * e + c), gn = ld_f4(gain + c);
-      st_f4(y + r * e + c, make_float4(keep[i].x * inv * gn.x * sigmoid_f(gt.x), keep[i].y * inv * gn.y * sigmoid_f(gt.y),
-                                       keep[i].z * inv * gn.z * sigmoid_f(gt.z), keep[i].w * inv * gn.w * sigmoid_f(gt.w)));
+      st_f4(y + r * e + c, make_float4(keep[i].x * inv * gn.x * sigmoid_for<T>(gt.x), keep[i].y * inv * gn.y * sigmoid_for<T>(gt.y),
+                                       keep[i].z * inv * gn.z * sigmoid_for<T>(gt.z), keep[i].w * inv * gn.w * sigmoid_for<T>(gt.w)));
     }
     return;
   }
   for (int c = lane; c < e; c += 32) x += o[c] * o[c];
   const float inv = 1.f / sqrtf(warp_sum(x) / e + eps);
-  for (int c = lane; c < e; c += 32) st_f(y + r * e + c, o[c] * inv * gain[c] * sigmoid_f(ld_f(gate + r * e + c)));
+  for (int c = lane; c < e; c += 32) st_f(y + r * e + c, o[c] * inv * gain[c] * sigmoid_for<T>(ld_f(gate + r * e + c)));
 }
 
 template <typename T, int DP, int VB>
@@ -314,10 +415,32 @@ int dispatch_scan(const void* p, const void* v, const void* gate, void* before, 
   if (a.d <= 256 && vb == 64) return launch_scan<T, 256, 64>(p, v, gate, before, y, a, segs, st);
   return 680;
 }
+template <typename T, int NI, int N>
+void launch_conv_tile(const void* p, const void* before, float* q, float* k, void* v, const ConvArgs& a, cudaStream_t st) {
+  const int units = 2 * a.kv_heads + a.heads;
+  if (a.rows <= 1024)
+    dsv4_launch(conv_unit_tile_kernel<T, NI, N, 1>, dim3(units, (a.rows + 7) / 8), 256, 0, st, (const T*)p, (const T*)before,
+                q, k, (T*)v, a);
+  else
+    dsv4_launch(conv_unit_tile_kernel<T, NI, N, 4>, dim3(units, (a.rows + 31) / 32), 256, 0, st, (const T*)p,
+                (const T*)before, q, k, (T*)v, a);
+}
+template <typename T, int NI>
+bool dispatch_conv_tile(const void* p, const void* before, float* q, float* k, void* v, const ConvArgs& a, cudaStream_t st) {
+  switch (a.cols.taps) {
+    case 2: launch_conv_tile<T, NI, 2>(p, before, q, k, v, a, st); return true;
+    case 3: launch_conv_tile<T, NI, 3>(p, before, q, k, v, a, st); return true;
+    case 4: launch_conv_tile<T, NI, 4>(p, before, q, k, v, a, st); return true;
+    default: return false;
+  }
+}
 template <typename T>
 void launch_conv(const void* p, const void* before, float* q, float* k, void* v, const ConvArgs& a, bool wide,
                  cudaStream_t st) {
   const dim3 grid(2 * a.kv_heads + a.heads, (a.rows + 7) / 8);
+  if (wide && (a.d > 128 || a.e > 128 ? dispatch_conv_tile<T, 2>(p, before, q, k, v, a, st)
+                                      : dispatch_conv_tile<T, 1>(p, before, q, k, v, a, st)))
+    return;
   if (wide)
     dsv4_launch(conv_unit_kernel<T, 4>, grid, 256, 0, st, (const T*)p, (const T*)before, q, k, (T*)v, a);
   else

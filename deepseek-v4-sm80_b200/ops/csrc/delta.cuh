@@ -5,6 +5,11 @@
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 // logarithm of the decay of a key channel; ea = exp(A_log) of the head
 __device__ __forceinline__ float log_decay(float rate, float dt_bias, float ea) { return -ea * softplus_f(rate + dt_bias); }
+// The same in two special-function instructions.  The absolute error stays at a rounding of the sum of logarithms it goes into.
+__device__ __forceinline__ float log_decay_fast(float rate, float dt_bias, float ea) {
+  const float x = rate + dt_bias;
+  return -ea * (fmaxf(x, 0.f) + __logf(1.f + __expf(-fabsf(x))));
+}
 
 // Where the parts of the merged projection stand, and the inputs the short convolutions keep.
 struct ConvCols {

@@ -198,36 +198,43 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       if (!ok) break;
       tc_fence_after();
       float s[kQT];
+      float big = 0.f;
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < kQT; c += 32) {
         uint32_t r[32];
-        tmem_ld_32x32(sp + c * 32, r);
+        tmem_ld_32x32(sp + c, r);
         tmem_ld_wait();
 #pragma unroll
-        for (int j = 0; j < 32; ++j) s[c * 32 + j] = __uint_as_float(r[j]);
+        for (int j = 0; j < 32; ++j) s[c + j] = __uint_as_float(r[j]);
+        if (MODE != kScaled) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) big = fmaxf(big, fabsf(s[c + j]));
+        }
       }
       if (MODE != kScaled) {
-        float big = fabsf(s[0]);
+        const bool small = __all_sync(0xffffffffu, big <= a.small);
+        const float e = 2.f * kLog2e * a.c;
 #pragma unroll
-        for (int j = 1; j < kQT; ++j) big = fmaxf(big, fabsf(s[j]));
-        if (__all_sync(0xffffffffu, big <= a.small)) {
+        for (int c = 0; c < kQT; c += 32) {
+          float* x = s + c;
+          if (small) {
 #pragma unroll
-          for (int j = 0; j < kQT; ++j) {
-            const float x = s[j] * s[j];
-            s[j] *= fmaf(fmaf(fmaf(a.p3, x, a.p2), x, a.p1), x, a.p0);
-          }
-        } else {
-          const float e = 2.f * kLog2e * a.c;
-#pragma unroll
-          for (int j = 0; j < kQT; ++j) s[j] = softcap_ex2(s[j], e, a.cap2);
-        }
-        if (MODE == kCappedBias) {
-          if (all_far) {
-#pragma unroll
-            for (int j = 0; j < kQT; ++j) s[j] += rel_far;
+            for (int j = 0; j < 32; ++j) {
+              const float y = x[j] * x[j];
+              x[j] *= fmaf(fmaf(fmaf(a.p3, y, a.p2), y, a.p1), y, a.p0);
+            }
           } else {
 #pragma unroll
-            for (int j = 0; j < kQT; ++j) s[j] += win[kQT - 1 + lane - j];
+            for (int j = 0; j < 32; ++j) x[j] = softcap_ex2(x[j], e, a.cap2);
+          }
+          if (MODE == kCappedBias) {
+            if (all_far) {
+#pragma unroll
+              for (int j = 0; j < 32; ++j) x[j] += rel_far;
+            } else {
+#pragma unroll
+              for (int j = 0; j < 32; ++j) x[j] += win[kQT - 1 + lane - c - j];
+            }
           }
         }
       }

@@ -61,6 +61,11 @@ __device__ __forceinline__ float gemm_act(float v, int act) {
 }
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+// the same for results that are rounded to T: 1e-6 relative is enough for bf16
+template <typename T>
+__device__ __forceinline__ float sigmoid_for(float z) {
+  return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-z)) : sigmoid_f(z);
+}
 // 0.5 z (1 + tanh(w)) = z sigmoid(2 w),  w = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float gelu_tanh(float z) {
   return z * sigmoid_f(1.5957691216057308f * fmaf(0.044715f * z * z, z, z));

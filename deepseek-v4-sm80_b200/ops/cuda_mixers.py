@@ -199,11 +199,10 @@ def delta_rule(q, k, v, rate, dt_bias, a_log, p, at_b, gate, gain, eps, state, b
         raw = torch.empty(t, heads * vdim, **f32)
         w, kr, qd = (torch.empty(n, heads, 32, dim, **f32) for _ in range(3))
         u0, b, decay = (torch.empty(n, heads, *s, **f32) for s in ((32, vdim), (32, 32), (dim,)))
-        vb = 16 if n_segs * heads * -(-vdim // 32) < num_sms(q.device) else 32
         nv.call("delta_chunked", nv.ptr(p), I(p.stride(0)), I(at_k), I(at_v), I(at_b), I(taps), nv.ptr(q), nv.ptr(k),
                 nv.ptr(v), nv.ptr(rate), nv.ptr(dt_bias), nv.ptr(a_log), nv.ptr(state), nv.ptr(before), nv.ptr(raw),
                 nv.ptr(fb.positions), nv.ptr(fb.seg_off), nv.ptr(chunks), I(n), nv.ptr(segs), I(n_segs), nv.ptr(w),
-                nv.ptr(kr), nv.ptr(qd), nv.ptr(u0), nv.ptr(b), nv.ptr(decay), I(heads), I(kv_heads), I(dim), I(vdim), I(vb),
+                nv.ptr(kr), nv.ptr(qd), nv.ptr(u0), nv.ptr(b), nv.ptr(decay), I(heads), I(kv_heads), I(dim), I(vdim),
                 _f32(p.dtype))
         norm(raw)
         return y

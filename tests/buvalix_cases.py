@@ -28,7 +28,7 @@ MODELS = {
 LIMIT = {torch.float32: 1e-4, torch.bfloat16: 4e-2}
 # Unit vectors and head norms of small vectors amplify rounding: in bf16 a few positions are further off, with every backend
 # at the same places.
-STRAY, WORST = 0.03, 0.16
+STRAY, WORST = 0.045, 0.16
 
 
 class Case(layered_checks.Case):

@@ -361,9 +361,3 @@ def test_delta_chunks_with_slow_and_fast_decays(rate_mean, monkeypatch):
     monkeypatch.setattr(C, "DELTA_CHUNKED", True)
     check_delta([(1, 0, 300), (2, 50, 70)], 2, 1, 32, 48, 4, torch.float32, 2e-4, rate_mean)
 
-
-def test_walk_blocks_of_both_widths(monkeypatch):
-    monkeypatch.setattr(C, "DELTA_CHUNKED", True)
-    for sms in (1, 100000):
-        monkeypatch.setattr(C, "num_sms", lambda _: sms)
-        check_delta([(1, 0, 130), (2, 7, 40)], 3, 3, 64, 72, 4, torch.float32, 1e-4)
