@@ -13,7 +13,7 @@ Merged or re-laid for the kernels:
 from __future__ import annotations
 
 import math
-from typing import Callable, Dict, List, Tuple
+from typing import Callable, Dict
 
 import torch
 
@@ -22,6 +22,7 @@ from .weight import tensor_reader
 
 FREE = -1     # a size that only the tensors give
 GATE_BLOCK = 16
+DELTA_PARTS = ("q", "k", "v", "a1", "g1", "b")     # the merged input projection of a channel_delta layer, in order
 
 
 def raw_shapes(cfg: BuvalixConfig) -> Dict[str, tuple]:
@@ -90,12 +91,6 @@ def interleave_gate(gate: torch.Tensor, up: torch.Tensor, block: int = GATE_BLOC
     return torch.stack(parts, 1).reshape(-1, d).contiguous()
 
 
-def delta_parts(m: ChannelDeltaSpec, a_rank: int, g_rank: int) -> List[Tuple[str, int]]:
-    """(name, rows) of the merged input projection of a channel_delta layer."""
-    return [("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.heads * m.vdim), ("a1", a_rank), ("g1", g_rank),
-            ("b", m.heads)]
-
-
 def build_weights(cfg: BuvalixConfig, get: Callable[[str], torch.Tensor], device) -> Dict[str, torch.Tensor]:
     """``get(name)`` returns a raw tensor; shapes are checked against the configuration."""
     want = raw_shapes(cfg)
@@ -120,13 +115,13 @@ def build_weights(cfg: BuvalixConfig, get: Callable[[str], torch.Tensor], device
         norm(p + "norm1")
         norm(p + "norm1b")
         if isinstance(m, ChannelDeltaSpec):
-            parts = {n: mat(q + n) for n in ("q", "k", "v", "a1", "g1", "b")}
+            parts = {n: mat(q + n) for n in DELTA_PARTS}
             a2, g2 = mat(q + "a2"), mat(q + "g2")
             for n, second in (("a1", a2), ("g1", g2)):
                 if parts[n].shape[0] != second.shape[1]:
                     raise ValueError(f"{q}{n}: {parts[n].shape[0]} rows feed {second.shape[1]} columns")
             pad8 = lambda t: torch.nn.functional.pad(t, (0, 0, 0, -t.shape[0] % 8))
-            w[q + "in"] = torch.cat([pad8(parts[n]) for n, _ in delta_parts(m, 0, 0)], 0)
+            w[q + "in"] = torch.cat([pad8(parts[n]) for n in DELTA_PARTS], 0)
             w[q + "a2"], w[q + "g2"] = a2, g2
             taps = torch.cat([raw(q + n + ".conv").to(device).float() for n in "qkv"], 0)
             w[q + "conv"] = taps.t().contiguous()

@@ -25,7 +25,7 @@ MODELS = {
     # heads wider than the prompt kernel and the chunked recurrence take
     "wide": P.config([P.rotary_layer(2, 1, 160, 144, 64, 1e4, 0.1, 15.0, 40), P.delta_layer(2, 1, 136, 152, 4)], width=72, vocab=88),
 }
-LIMIT = {torch.float32: 1e-4, torch.bfloat16: 4e-2}
+LIMIT = {torch.float32: 1e-4, torch.bfloat16: 5e-2}
 # Unit vectors and head norms of small vectors amplify rounding: in bf16 a few positions are further off, with every backend
 # at the same places.
 STRAY, WORST = 0.045, 0.16
