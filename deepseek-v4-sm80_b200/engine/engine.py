@@ -179,8 +179,13 @@ class Engine:
         return self.family.load(download_hf_weight(self.config.model_path), cfg, self.device, tp.rank, tp.size,
                                 self.config.moe_mode)
 
-    def _context_classes(self) -> List[int]:
+    def _context_limit(self) -> int:
         limit = self.config.max_seq_len_override or self.model_config.max_position
+        learned = getattr(self.model_config, "position_rows", 0)      # learned position vectors end somewhere
+        return min(limit, learned) if learned else limit
+
+    def _context_classes(self) -> List[int]:
+        limit = self._context_limit()
         return self.family.context_classes(self.model_config, limit) + [limit]
 
     # ------------------------------------------------------------------ memory
@@ -203,7 +208,7 @@ class Engine:
     def _plan_kv(self) -> Dict[str, int]:
         cfg, c = self.model_config, self.config
         ps = self.page_size
-        limit = c.max_seq_len_override or cfg.max_position
+        limit = self._context_limit()
         kv = self.family.budget(cfg, c, c.dtype)
         swa_slots, per_page, fixed = kv.window_slots, kv.bytes_per_page, kv.fixed_bytes
         want_pages = min(c.max_running_req * div_ceil(limit, ps) + div_ceil(c.max_prefill_length, ps), 1 << 18)

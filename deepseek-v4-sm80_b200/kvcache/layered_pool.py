@@ -12,7 +12,11 @@ position 0 from zeros.
 * ("state", heads, d): ``state[run]`` [slots, heads, d, d] fp32 and ``shift[run]`` [slots, width] fp32 (the last token's
   input);
 * ("delta", heads, d, e, channels, taps): ``state[run]`` [slots, heads, d, e] fp32 and ``conv[run]`` [slots, taps - 1,
-  channels], the last inputs of the short convolutions, oldest first.
+  channels], the last inputs of the short convolutions, oldest first;
+* ("linear", heads, d, columns, tops, channels, taps): ``state[run]`` [slots, heads, d, columns] fp32, ``top[run]`` [slots, tops]
+  fp32, running maxima, and ``conv[run]`` as above; tops or channels may be 0: then there is none.
+
+A run may keep things of several kinds, ``(kind, kind, ..)``, as long as no two have the same storage.
 
 The recurrent state of a prefix is not kept with its pages, so a model with recurrent layers does not reuse prefixes.
 """
@@ -28,17 +32,26 @@ RunStore = Tuple      # what a run keeps, as listed above
 PAGED = ("latent", "kv")
 
 
+def kinds(stores: Sequence[RunStore]):
+    """(run, kind) of everything that is kept."""
+    for run, s in enumerate(stores):
+        for k in (s,) if isinstance(s[0], str) else s:
+            yield run, k
+
+
 def bytes_per_page(stores: Sequence[RunStore], page_size: int, dtype: torch.dtype) -> int:
-    return sum(sum(s[1:]) for s in stores if s[0] in PAGED) * page_size * dtype.itemsize
+    return sum(sum(s[1:]) for _, s in kinds(stores) if s[0] in PAGED) * page_size * dtype.itemsize
 
 
 def bytes_per_req_slot(stores: Sequence[RunStore], width: int, dtype: torch.dtype) -> int:
     total = 0
-    for s in stores:
+    for _, s in kinds(stores):
         if s[0] == "state":
             total += (s[1] * s[2] * s[2] + width) * 4
         elif s[0] == "delta":
             total += s[1] * s[2] * s[3] * 4 + (s[5] - 1) * s[4] * dtype.itemsize
+        elif s[0] == "linear":
+            total += (s[1] * s[2] * s[3] + s[4]) * 4 + (s[6] - 1) * s[5] * dtype.itemsize
     return total
 
 
@@ -46,7 +59,7 @@ class LayeredPool(PagedPool):
     def __init__(self, stores: Sequence[RunStore], width: int, sizes: PoolSizes, device, dtype=torch.bfloat16):
         super().__init__(sizes, device)
         self.stores = tuple(stores)
-        self.prefix_reusable = all(s[0] in PAGED for s in stores)
+        self.prefix_reusable = all(s[0] in PAGED for _, s in kinds(stores))
         rows, slots = (sizes.num_pages + 1) * sizes.page_size, sizes.num_req_slots + 1
         act, f32 = dict(dtype=dtype, device=self.device), dict(dtype=torch.float32, device=self.device)
         self.latent: Dict[int, torch.Tensor] = {}
@@ -55,7 +68,8 @@ class LayeredPool(PagedPool):
         self.state: Dict[int, torch.Tensor] = {}
         self.shift: Dict[int, torch.Tensor] = {}
         self.conv: Dict[int, torch.Tensor] = {}
-        for run, s in enumerate(stores):
+        self.top: Dict[int, torch.Tensor] = {}
+        for run, s in kinds(stores):
             if s[0] == "latent":
                 self.latent[run] = torch.zeros(rows, s[1], **act)
             elif s[0] == "kv":
@@ -66,14 +80,20 @@ class LayeredPool(PagedPool):
             elif s[0] == "delta":
                 self.state[run] = torch.zeros(slots, s[1], s[2], s[3], **f32)
                 self.conv[run] = torch.zeros(slots, s[5] - 1, s[4], **act)
+            elif s[0] == "linear":
+                self.state[run] = torch.zeros(slots, s[1], s[2], s[3], **f32)
+                if s[4]:
+                    self.top[run] = torch.zeros(slots, s[4], **f32)
+                if s[5]:
+                    self.conv[run] = torch.zeros(slots, s[6] - 1, s[5], **act)
             else:
                 raise ValueError(f"unknown kind of storage {s[0]!r}")
         # scratch of the token shift, shared by all runs: where a portion's last row waits until the slot may change
         self.shift_tail = torch.zeros(slots, width, **f32) if self.shift else None
 
     def storage(self) -> List[torch.Tensor]:
-        kinds = (self.latent, self.keys, self.values, self.state, self.shift, self.conv)
-        return [t for kind in kinds for t in kind.values()]
+        all_kinds = (self.latent, self.keys, self.values, self.state, self.shift, self.conv, self.top)
+        return [t for kind in all_kinds for t in kind.values()]
 
     def storage_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in self.storage())

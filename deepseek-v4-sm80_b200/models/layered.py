@@ -51,12 +51,13 @@ class LayeredModel:
         O.check_index(fb.out_loc, -1, locs, "out_loc")
         O.check_index(fb.page_table, 0, locs, "page_table")
 
-    def embed(self, fb: ForwardBatch, want_act: bool):
-        """(fp32 stream, the embedding output as activations if wanted), with the index audit around it."""
+    def embed(self, fb: ForwardBatch, want_act: bool, **kw):
+        """(fp32 stream, the embedding output as activations if wanted), with the index audit around it; kw: further arguments of
+        ``embed_residual``."""
         if self._debug_bounds and fb.token_feedback is None:
             self.audit_inputs(fb)
         x, x0 = O.embed_residual(fb.input_ids, self.w["embed.weight"], self.dtype, fb.token_feedback,
-                                 fb.slots if fb.token_feedback is not None else None, want_act)
+                                 fb.slots if fb.token_feedback is not None else None, want_act, **kw)
         if self._debug_bounds and fb.token_feedback is not None:
             self.audit_inputs(fb)
         return x, x0

@@ -81,20 +81,29 @@ class ExpertsFF:
 class GroupedAttention:
     """Causal attention over paged keys and values, several query heads to a key head.  Optional parts, by the weights there
     are: projection biases (``qkv.b``), rotary positions on the leading dimensions (``freq``), a sink logit per head
-    (``sink``), a bias by distance (``rel``); and a query temperature (coef, every) that grows with the position."""
+    (``sink``), a bias by distance (``rel``, a table, or ``slope`` per head), norms over all rows of q and of k (``qk.norm``).
+    By the arguments: a query temperature (coef, every) that grows with the position; keys seen only within the query's chunk of
+    positions; values divided by their root mean square per head (``unit_v``) and multiplied by ``v_mul``."""
 
     def __init__(self, w: Dict[str, torch.Tensor], prefix: str, heads: int, kv_heads: int, dim: int, vdim: int, scale: float,
-                 softcap: float, q_temp: Optional[Tuple[float, int]] = None):
+                 softcap: float = 0.0, q_temp: Optional[Tuple[float, int]] = None, chunk: int = 0, unit_v: bool = False,
+                 eps: float = 0.0, v_mul: float = 1.0):
         self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
         self.scale, self.softcap, self.q_temp = scale, softcap, q_temp
-        self.qkv, self.o = w[prefix + "qkv"], w[prefix + "o"]
+        self.chunk, self.unit_v, self.eps, self.v_mul = chunk, unit_v, eps, v_mul
+        self.qkv, self.o = w.get(prefix + "qkv"), w[prefix + "o"]
         self.bias, self.freq, self.sink, self.rel = (w.get(prefix + n) for n in ("qkv.b", "freq", "sink", "rel"))
+        self.gain, self.slope = w.get(prefix + "qk.norm"), w.get(prefix + "slope")
+
+    def attend(self, qkv: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+        """What stands between the projections: q | k | v [T, ..] -> the heads' results [T, H * vdim]."""
+        q = O.rotate_store(qkv, self.bias, self.freq, self.q_temp, keys, values, fb, self.heads, self.kv_heads, self.dim,
+                           self.vdim, self.gain, self.unit_v, self.eps, self.v_mul)
+        return O.grouped_attention(q, keys, values, fb, self.kv_heads, self.scale, self.softcap, self.sink, self.rel,
+                                   self.slope, self.chunk)
 
     def __call__(self, h: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
-        q = O.rotate_store(O.linear(h, self.qkv), self.bias, self.freq, self.q_temp, keys, values, fb, self.heads,
-                           self.kv_heads, self.dim, self.vdim)
-        v = O.grouped_attention(q, keys, values, fb, self.kv_heads, self.scale, self.softcap, self.sink, self.rel)
-        return O.linear(v, self.o, out_dtype=torch.float32)
+        return O.linear(self.attend(O.linear(h, self.qkv), keys, values, fb), self.o, out_dtype=torch.float32)
 
 
 class ChannelDelta:
@@ -131,3 +140,97 @@ class GatedFF:
 
     def __call__(self, h: torch.Tensor) -> torch.Tensor:
         return O.linear(O.gated_linear(h, self.gu, self.act), self.down, out_dtype=torch.float32)
+
+
+def padded8(sizes) -> list:
+    """Column ranges of parts that stand side by side, each beginning at a multiple of eight columns."""
+    at, out = 0, []
+    for n in sizes:
+        out.append(slice(at, at + n))
+        at += -(-n // 8) * 8
+    return out
+
+
+class MLSTM:
+    """Matrix memory with exponential input gates and a running maximum: the normaliser is one more column of the state."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, heads: int, dim: int, vdim: int, cap: float, eps: float):
+        self.heads, self.dim, self.vdim, self.cap, self.eps = heads, dim, vdim, cap, eps
+        self.inp, self.gates, self.bias, self.gain, self.o = (w[prefix + n] for n in ("in", "gates", "gates.b", "norm", "o"))
+        self.cols = padded8([heads * dim, heads * dim, heads * vdim, heads * vdim])
+
+    def __call__(self, h: torch.Tensor, state: torch.Tensor, top: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+        p = O.linear(h, self.inp)
+        q, k, v, g = (p[:, c] for c in self.cols)
+        log_g, fac, floor = O.mlstm_gates(O.linear(h, self.gates, out_dtype=torch.float32), self.bias, self.cap, top, fb)
+        o = O.gla("given", q, k, v, (log_g, fac), state, fb, self.heads, self.heads, self.dim ** -0.5)
+        y = O.norm_heads(o, self.vdim, self.gain, self.eps, h.dtype, gate=g, floor=floor)
+        return O.linear(y, self.o, out_dtype=torch.float32)
+
+
+class ForgetRecurrence:
+    """Linear attention in which the forget gate of a key channel also decides what is written; per-head norm."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, heads: int, dim: int, vdim: int, eps: float, mul: float = 1.0):
+        self.heads, self.dim, self.vdim, self.eps, self.mul = heads, dim, vdim, eps, mul
+        self.f, self.bias, self.low, self.gain, self.o = (w[prefix + n] for n in ("f", "f.b", "lower", "norm", "o"))
+
+    def mix(self, h: torch.Tensor, q: torch.Tensor, v: torch.Tensor, state: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+        """What stands between the projections of q and v and the output's, times ``mul``."""
+        z = O.linear(h, self.f, out_dtype=torch.float32)
+        o = O.gla("forget", q, None, v, (z, self.bias, self.low), state, fb, self.heads, self.heads)
+        return O.norm_heads(o, self.vdim, self.gain, self.eps, h.dtype, mul=self.mul)
+
+
+class ParallelMixer:
+    """Attention and a recurrence side by side on the same input; their projections of it are one product (``in``)."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, left: GroupedAttention, right: ForgetRecurrence):
+        self.inp, self.left, self.right = w[prefix + "in"], left, right
+        l, r = left, right
+        self.cols = padded8([l.heads * l.dim + l.kv_heads * (l.dim + l.vdim), r.heads * r.dim, r.heads * r.vdim])
+
+    def __call__(self, h: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, state: torch.Tensor,
+                 fb: ForwardBatch) -> torch.Tensor:
+        p = O.linear(h, self.inp)
+        qkv, q, v = (p[:, c] for c in self.cols)
+        y = O.linear(self.left.attend(qkv, keys, values, fb), self.left.o, out_dtype=torch.float32)
+        return O.linear(self.right.mix(h, q, v, state, fb), self.right.o, out=y, accumulate=True)
+
+
+class Mamba2:
+    """State-space recurrence with a step size per head: one projection z | x | B | C, a short convolution over x, B and C, the
+    recurrence, a skip, the gate z and norms over equal parts."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, heads: int, vdim: int, groups: int, state: int,
+                 norm_groups: int, eps: float):
+        self.heads, self.groups, self.norm_groups, self.eps = heads, groups, norm_groups, eps
+        self.inp, self.dt, self.dt_bias, self.a_log = (w[prefix + n] for n in ("in", "dt", "dt_bias", "A_log"))
+        self.conv, self.conv_b, self.skip, self.gain, self.o = (w[prefix + n] for n in ("conv", "conv.b", "D", "norm", "o"))
+        inner, gn = heads * vdim, groups * state
+        self.z, self.xbc = padded8([inner, inner + 2 * gn])
+        self.x, self.b, self.c = slice(0, inner), slice(inner, inner + gn), slice(inner + gn, inner + 2 * gn)
+
+    def __call__(self, h: torch.Tensor, state: torch.Tensor, before: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+        p = O.linear(h, self.inp)
+        dt = O.linear(h, self.dt, out_dtype=torch.float32)
+        u = O.causal_conv(p[:, self.xbc], self.conv, self.conv_b, before, fb)
+        x = u[:, self.x]
+        o = O.gla("step", u[:, self.c], u[:, self.b], x, (dt, self.dt_bias, self.a_log), state, fb, self.heads, self.groups)
+        y = O.norm_groups(o, self.skip, x, p[:, self.z], self.gain, self.norm_groups, self.eps)
+        return O.linear(y, self.o, out_dtype=torch.float32)
+
+
+class SharedExpertsFF:
+    """Mixture of silu-gated experts weighted with a softmax over all router outputs, some of which stand for the input itself,
+    beside an expert that every token uses.  The weighted sum is left to the kernel that touches the streams next."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, top: int, scale: float):
+        self.top, self.scale = top, scale
+        self.router, self.bias, self.w13, self.w2 = (w[prefix + n] for n in ("router", "correction", "w13", "w2"))
+        self.shared = GatedFF(w, prefix + "shared.", "silu")
+
+    def __call__(self, h: torch.Tensor, fb: ForwardBatch) -> dict:
+        idx, wts = O.route_topk(h, self.router, self.bias, self.top, fb.num_valid, "softmax", self.scale)
+        rows = O.gated_experts(h, idx, wts, self.w13, self.w2)
+        return {"sub": self.shared(h), "experts": (rows, wts, idx, self.w13.shape[0], h)}

@@ -14,6 +14,8 @@ from .bedalorn_config import BedalornConfig
 from .buvalix_config import ARCHITECTURE as BUVALIX
 from .buvalix_config import BuvalixConfig
 from .config import ModelConfig
+from .zazilix_config import ARCHITECTURE as ZAZILIX
+from .zazilix_config import ZazilixConfig
 
 
 @dataclass(frozen=True)
@@ -154,6 +156,24 @@ def _buvalix_build(cfg, weights, pool, comm, moe_mode, dtype):
     return BuvalixModel(cfg, weights, pool, comm, moe_mode, dtype)
 
 
+def _zazilix_load(folder, cfg, device, rank, size, moe_mode):
+    from .zazilix_weight import load_checkpoint
+
+    return load_checkpoint(folder, cfg, device)
+
+
+def _zazilix_draw(cfg, device, rank, size, moe_mode, seed, on_host):
+    from .zazilix_weight import random_weights
+
+    return random_weights(cfg, device, seed)
+
+
+def _zazilix_build(cfg, weights, pool, comm, moe_mode, dtype):
+    from .zazilix import ZazilixModel
+
+    return ZazilixModel(cfg, weights, pool, comm, moe_mode, dtype)
+
+
 FAMILIES = {
     "DeepseekV4ForCausalLM": ModelFamily("deepseek_v4", ModelConfig, ModelConfig.from_hf, (torch.bfloat16,), 64,
                                          _dsv4_load, _dsv4_draw, _dsv4_budget, _dsv4_pool, _dsv4_build, _dsv4_classes),
@@ -163,6 +183,9 @@ FAMILIES = {
     BUVALIX: ModelFamily("buvalix", BuvalixConfig, BuvalixConfig.from_dict, (torch.bfloat16, torch.float32), 1,
                          _buvalix_load, _buvalix_draw, _layered_budget, _layered_pool, _buvalix_build,
                          _layered_classes, "grouped"),
+    ZAZILIX: ModelFamily("zazilix", ZazilixConfig, ZazilixConfig.from_dict, (torch.bfloat16, torch.float32), 1,
+                         _zazilix_load, _zazilix_draw, _layered_budget, _layered_pool, _zazilix_build,
+                         _layered_classes, "streams"),
 }
 
 

@@ -267,9 +267,20 @@ def _layers(t):
     return cuda_layers if t.is_cuda else ref_layers
 
 
-def embed_residual(ids, weight, dtype, feedback=None, slots=None, want_act: bool = False):
-    """(x fp32 [T, D], the same rows as activations of ``dtype`` or None); feedback / slots as in :func:`embed`."""
-    return _layers(ids).embed_residual(ids, weight, dtype, feedback, slots, want_act)
+def embed_residual(ids, weight, dtype, feedback=None, slots=None, want_act: bool = False, mul: float = 1.0, table=None,
+                   positions=None, streams=None):
+    """(x = embedding * mul + table[position] fp32 [T, D], the same rows as activations of ``dtype`` or None); feedback / slots
+    as in :func:`embed`.  ``table``: learned position vectors or None.  ``streams``: x is that many copies [T, streams, D]."""
+    return _layers(ids).embed_residual(ids, weight, dtype, feedback, slots, want_act, mul, table, positions, streams)
+
+
+def stream_norm(x, eps: float, dtype, pre=None, post=None, sub=None, experts=None, rows=None, keep: bool = True):
+    """One step of fp32 residual streams x [T, S, D] with constant mixing weights.  With ``post`` = out [S] | mix [S, S] (from,
+    to), flat: x_t <- sum_s mix[s, t] x_s + out[t] y for y = ``sub`` [T, D] fp32 + the weighted rows of ``experts`` = (expert rows
+    [T*k, D], weights [T, k], ids [T, k], n, h [T, D]); ids from n on stand for h itself, negative ones for nothing.  With ``pre``
+    = in [S] | gain: returns u / rms(u) * gain as activations for u = sum_s in[s] x_s, else None.  ``rows``: only these are
+    computed and returned.  keep=False (always with ``rows``): x itself may be left as it was."""
+    return _layers(x).stream_norm(x, eps, dtype, pre, post, sub, experts, rows, keep and rows is None)
 
 
 def residual_norm(x, gain, eps: float, dtype, mul: float = 1.0, rows=None, add=None, add2=None, vec=None, experts=None,
@@ -281,10 +292,11 @@ def residual_norm(x, gain, eps: float, dtype, mul: float = 1.0, rows=None, add=N
     return _layers(x).residual_norm(x, gain, eps, dtype, mul, rows, add, add2, vec, experts, cast)
 
 
-def route_topk(h, weight, bias, top: int, num_valid=None):
-    """Router of a softmax-over-the-selected mixture: logits z = h W^T + b in fp32, the ``top`` largest (lower id on
-    ties) and the softmax over them.  Rows >= num_valid get id -1."""
-    return _layers(h).route_topk(h, weight, bias, top, num_valid)
+def route_topk(h, weight, bias, top: int, num_valid=None, kind: str = "selected", scale: float = 1.0):
+    """Router of a mixture, logits z = h W^T in fp32; the weights are times ``scale``.  kind "selected": the ``top`` largest
+    z + b (lower id on ties) and the softmax over them; "softmax": p = softmax(z) over all, the ``top`` largest p + b, weighted
+    with their p.  Rows >= num_valid get id -1."""
+    return _layers(h).route_topk(h, weight, bias, top, num_valid, kind, scale)
 
 
 def gated_experts(h, idx, wts, w13, w2):
@@ -345,23 +357,29 @@ def residual_layer_norm(x, eps: float, dtype, norm=None, sub=None, add=None, row
 
 
 def gated_linear(h, w, act: str, block: int = 16):
-    """act(gate h) * (up h) for w [2F, D] in alternating blocks of ``block`` gate and up rows -> [T, F]."""
+    """act(gate h) * (up h), act "gelu_tanh" or "silu", for w [2F, D] in alternating blocks of ``block`` gate and up rows -> [T, F]."""
     return _mixers(h).gated_linear(h, w, act, block)
 
 
-def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads: int, kv_heads: int, dim: int, vdim: int):
-    """Behind the projection q | k | v of grouped attention: adds ``bias`` (or None), turns neighbouring pairs of the first
+def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads: int, kv_heads: int, dim: int, vdim: int, gain=None,
+                 unit_v: bool = False, eps: float = 0.0, v_mul: float = 1.0):
+    """Behind the projection q | k | v of grouped attention: adds ``bias`` (or None); with ``gain`` divides q and k by the root
+    mean square of all their rows and multiplies by it; with ``unit_v`` divides every head's values by their root mean square;
+    multiplies the values by ``v_mul``; turns neighbouring pairs of the first
     2 * len(freq) dimensions of every q and k head by position * freq (or not), multiplies q by its temperature
     1 + coef * ln(floor((position + 1) / every) + 1) for q_temp = (coef, every), writes keys and values to the rows
     ``fb.out_loc`` of the caches and returns q [T, H, dim]."""
-    return _mixers(qkv).rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads, kv_heads, dim, vdim)
+    return _mixers(qkv).rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads, kv_heads, dim, vdim, gain, unit_v, eps,
+                                     v_mul)
 
 
-def grouped_attention(q, keys, values, fb, kv_heads: int, scale: float, softcap: float = 0.0, sink=None, rel=None):
+def grouped_attention(q, keys, values, fb, kv_heads: int, scale: float, softcap: float = 0.0, sink=None, rel=None, slope=None,
+                      chunk: int = 0):
     """Causal attention of q [T, H, dim] over the cached keys and values of every request, H / kv_heads query heads to a key
-    head.  score = softcap * tanh(q.k * scale / softcap) (0: not capped) + rel[h, min(distance, last)]; ``sink`` [H] adds
-    exp(sink) to the denominator.  Returns [T, H * vdim]."""
-    return _mixers(q).grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel)
+    head.  score = softcap * tanh(q.k * scale / softcap) (0: not capped) + rel[h, min(distance, last)] - slope[h] * distance;
+    ``sink`` [H] adds exp(sink) to the denominator; with ``chunk`` position i only sees keys from i // chunk * chunk on.
+    Returns [T, H * vdim]."""
+    return _mixers(q).grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, slope, chunk)
 
 
 def conv_unit(p, taps, before, fb, heads: int, kv_heads: int, dim: int, vdim: int):
@@ -382,6 +400,51 @@ def delta_rule(q, k, v, rate, dt_bias, a_log, p, at_b: int, gate, gain, eps: flo
     and y = o / rms(o) * gain * sigmoid(gate) per head -> [T, H * vdim].  Also keeps the last inputs of the convolutions
     (the q, k, v columns of p) in ``before``."""
     return _mixers(p).delta_rule(q, k, v, rate, dt_bias, a_log, p, at_b, gate, gain, eps, state, before, fb, heads, kv_heads)
+
+
+# --------------------------------------------------------------------------- gated linear attention
+def _gla(t):
+    from . import cuda_gla, ref_gla
+
+    return cuda_gla if t.is_cuda else ref_gla
+
+
+def mlstm_gates(z, bias, cap: float, top, fb):
+    """Exponential input gates with a running maximum: z fp32 [T, 2 H] (input gates, then forget gates), i = cap tanh((z + b) /
+    cap), f = log sigmoid(cap tanh((z + b) / cap)), m = max(f + m, i) with m in ``top`` [slots + 1, H] (0 at the start of a
+    sequence).  Returns (log of the decay f + m_before - m, factor of the keys e^(i - m), floor e^-m), each fp32 [T, H]."""
+    return _gla(z).mlstm_gates(z, bias, cap, top, fb)
+
+
+def causal_conv(p, taps, bias, before, fb):
+    """silu of a short causal convolution per channel: p [T, C] (may be a column slice), taps [n, C] (the last row is the current
+    token's), bias [C]; ``before`` [slots + 1, n - 1, C] holds the inputs ahead of a portion and is moved on.  Returns [T, C]."""
+    return _gla(p).causal_conv(p, taps, bias, before, fb)
+
+
+def gla(kind: str, q, k, v, gates, state, fb, heads: int, groups: int, q_mul: float = 1.0):
+    """Gated linear attention per head, S <- diag(g) S + k v^T, o = S^T q, with S [d, columns] fp32 in ``state`` [slots + 1, H, d,
+    columns]; v [T, H * e]; q, k [T, groups * d], shared by H / groups heads.  Gates by kind:
+
+        "given"   (log g [T, H], factor of k [T, H]); the values have a column of ones at e
+        "step"    (raw [T, H], bias [H], A_log [H]): dt = softplus(raw + bias), log g = -exp(A_log) dt, factor dt
+        "forget"  (raw [T, H * d], bias [H * d], low [H * d]): g = low + (1 - low) sigmoid(raw + bias), k = 1 - g (k is None),
+                  q goes through silu
+
+    q is multiplied by ``q_mul``.  Returns o fp32 [T, H, columns]; columns from e on (e + 1 for "given") mean nothing."""
+    return _gla(v).gla(kind, q, k, v, gates, state, fb, heads, groups, q_mul)
+
+
+def norm_heads(o, e: int, gain, eps: float, dtype, gate=None, floor=None, mul: float = 1.0):
+    """o [T, H, columns] -> o / rms(o) * gain * mul over the first e columns of every head (* sigmoid(gate)), as activations
+    [T, H * e].  gain [e] or [H * e].  ``floor`` [T, H]: o is divided by max(|o[e]|, floor) + 1e-6 first."""
+    return _gla(o).norm_heads(o, e, gain, eps, dtype, gate, floor, mul)
+
+
+def norm_groups(o, skip, x, z, gain, groups: int, eps: float):
+    """(o + skip x) silu(z) per head, then divided by the root mean square of each of ``groups`` equal parts, times gain.  o [T, H,
+    columns] fp32, x and z [T, H * e] (may be column slices) -> [T, H * e]."""
+    return _gla(o).norm_groups(o, skip, x, z, gain, groups, eps)
 
 
 # --------------------------------------------------------------------------- sampling

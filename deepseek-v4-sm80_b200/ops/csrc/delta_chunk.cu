@@ -23,6 +23,7 @@
 // contraction index is free as long as A and B agree: with its places t, t + 4 standing for 2t, 2t + 1, a lane's two B values
 // are neighbours in memory, and a C fragment is the A fragment of the next product as it is (c0, c2, c1, c3).
 #include "delta.cuh"
+#include "tf32.cuh"
 
 namespace {
 
@@ -32,35 +33,6 @@ constexpr float kSafe = 60.f;
 constexpr int kAL = kC + 4;       // row stride of beta A in shared memory
 constexpr int kTL = kC + 8;       // row stride of arrays read as B fragments (8 mod 32: conflict-free 8-byte reads)
 
-// ------------------------------------------------------------------ three-term TF32 products
-struct Split {
-  uint32_t hi, lo;
-};
-__device__ __forceinline__ Split split(float x) {
-  Split s;
-  s.hi = __float_as_uint(x) & 0xffffe000u;
-  s.lo = __float_as_uint(x - __uint_as_float(s.hi));
-  return s;
-}
-__device__ __forceinline__ void mma_tf32(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
-                                         uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-struct FragA {
-  Split v[4];
-};
-__device__ __forceinline__ FragA frag_a(float a0, float a1, float a2, float a3) {
-  return FragA{{split(a0), split(a1), split(a2), split(a3)}};
-}
-__device__ __forceinline__ void mma3(float (&c)[4], const FragA& a, const float2& b) {
-  const Split x = split(b.x), y = split(b.y);
-  mma_tf32(c, a.v[0].lo, a.v[1].lo, a.v[2].lo, a.v[3].lo, x.hi, y.hi);
-  mma_tf32(c, a.v[0].hi, a.v[1].hi, a.v[2].hi, a.v[3].hi, x.lo, y.lo);
-  mma_tf32(c, a.v[0].hi, a.v[1].hi, a.v[2].hi, a.v[3].hi, x.hi, y.hi);
-}
 __device__ __forceinline__ float2 ld_f2(const float* p) { return *reinterpret_cast<const float2*>(p); }
 
 // ------------------------------------------------------------------ everything that depends on a chunk alone

@@ -1,6 +1,6 @@
 // Causal multi-head attention of long prompt portions on tcgen05 over keys and values that lie side by side: gathered from
 // a paged cache (grouped_attn.cu: kv_gather, several query heads to a key head, optionally capped scores, a bias by distance
-// and a sink), or expanded from cached latents (latent_attn.cu).
+// (a table, or falling with the distance) and a sink), or expanded from cached latents (latent_attn.cu).
 //
 // For latents, the absorbed form (latent_attn.cu) multiplies every (query, key) pair over the whole latent rank, twice.  For
 // a portion of many tokens it is cheaper to expand the request's latents once,  K = C W_uk^T  and  V^T = W_uv C^T  (two
@@ -32,8 +32,9 @@ struct FlashArgs {
   float small;          // |s| up to here: s (p0 + p1 s^2 + p2 s^4 + p3 s^6), an odd polynomial
   float p0, p1, p2, p3;
   const float* sink;    // [heads] or null
-  const float* rel;     // [heads][n_rel] (BIAS)
+  const float* rel;     // [heads][n_rel] (kCappedBias)
   int n_rel;
+  const float* slope;   // [heads] (kSloped)
 };
 
 struct FlashBars {
@@ -52,7 +53,7 @@ struct FlashCfg {
 };
 
 // What happens to a score between the product and the softmax.
-enum ScoreMode : int { kScaled = 0, kCapped = 1, kCappedBias = 2 };
+enum ScoreMode : int { kScaled = 0, kCapped = 1, kCappedBias = 2, kSloped = 3 };
 
 template <int NB, int MODE>
 __global__ void __launch_bounds__(kFThreads, 1)
@@ -182,6 +183,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     float* win = wins + (warp - 2) * kWin;
     const float* rel = MODE == kCappedBias ? a.rel + (size_t)head * a.n_rel : nullptr;
     const float rel_far = MODE == kCappedBias ? rel[a.n_rel - 1] * kLog2e : 0.f;
+    const float slope2 = MODE == kSloped ? a.slope[head] * kLog2e : 0.f;
     float m = -1e30f, l = 0.f;
     bool ok = true;
     for (int i = 0; i < n; ++i) {
@@ -206,12 +208,17 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         tmem_ld_wait();
 #pragma unroll
         for (int j = 0; j < 32; ++j) s[c + j] = __uint_as_float(r[j]);
-        if (MODE != kScaled) {
+        if (MODE == kCapped || MODE == kCappedBias) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) big = fmaxf(big, fabsf(s[c + j]));
         }
       }
-      if (MODE != kScaled) {
+      if (MODE == kSloped) {
+        const float from = slope2 * (float)(i * kQT - pos0 - row);      // minus the distance of the tile's first key
+#pragma unroll
+        for (int j = 0; j < kQT; ++j) s[j] = fmaf(s[j], a.scale2, fmaf(slope2, (float)j, from));
+      }
+      if (MODE == kCapped || MODE == kCappedBias) {
         const bool small = __all_sync(0xffffffffu, big <= a.small);
         const float e = 2.f * kLog2e * a.c;
 #pragma unroll
@@ -338,6 +345,7 @@ int dispatch_flash(int mode, const CUtensorMap& q, const CUtensorMap& k, const C
                    const FlashArgs& a, int n_items, cudaStream_t st) {
   if (mode == kScaled) return launch_flash<NB, kScaled>(q, k, v, out, a, n_items, st);
   if (mode == kCapped) return launch_flash<NB, kCapped>(q, k, v, out, a, n_items, st);
+  if (mode == kSloped) return launch_flash<NB, kSloped>(q, k, v, out, a, n_items, st);
   return launch_flash<NB, kCappedBias>(q, k, v, out, a, n_items, st);
 }
 
@@ -346,22 +354,23 @@ int dispatch_flash(int mode, const CUtensorMap& q, const CUtensorMap& k, const C
 // q: bf16 [rows, heads * dim] (row stride ldq), k: [kv_rows, kv_heads * dim], vt: [kv_heads * vdim, kv_rows] (row stride
 // kv_rows), out: [rows, heads * vdim]; query head h reads key head h / (heads / kv_heads).  items as in FlashArgs, at most 256
 // queries each; first key rows are multiples of 8.  Scores: cap tanh(q.k scale / cap) (cap 0: q.k scale), plus rel[h,
-// min(distance, n_rel - 1)] if rel is given; sink [heads] or null adds e^sink to the sum of a row's weights.
+// min(distance, n_rel - 1)] if rel is given; or, without cap and rel, less slope[h] * distance.  sink [heads] or null adds e^sink
+// to the sum of a row's weights.
 DSV4_API int dsv4_flash_attention(const void* q, int ldq, const void* k, const void* vt, void* out, const int* items,
                                   int n_items, int rows, int kv_rows, int heads, int kv_heads, int dim, int vdim,
                                   float scale, float cap, const float* sink, const float* rel, int n_rel,
-                                  cudaStream_t st) {
+                                  const float* slope, cudaStream_t st) {
   if (n_items <= 0) return 0;
   if (dim % 8 || vdim % 8 || ldq % 8 || kv_rows % 8 || dim < 8 || dim > 128 || vdim < 8 || vdim > 128 || n_items > 65535)
     return 651;
-  if (kv_heads < 1 || heads % kv_heads || (rel && n_rel < 1)) return 656;
+  if (kv_heads < 1 || heads % kv_heads || (rel && n_rel < 1) || (slope && (rel || cap > 0.f))) return 656;
   CUtensorMap tq, tk, tv;
   if (dsv4_make_tmap_3d(&tq, q, dim, heads, rows, (uint64_t)dim * 2, (uint64_t)ldq * 2, 64, 1, kQT)) return 652;
   if (dsv4_make_tmap_3d(&tk, k, dim, kv_heads, kv_rows, (uint64_t)dim * 2, (uint64_t)kv_heads * dim * 2, 64, 1, kQT)) return 653;
   const int vp = (vdim + 15) & ~15;
   if (dsv4_make_tmap_3d(&tv, vt, kv_rows, vdim, kv_heads, (uint64_t)kv_rows * 2, (uint64_t)vdim * kv_rows * 2, 64, vp)) return 654;
   FlashArgs a{items, heads, heads / kv_heads, dim, vdim, heads * vdim, scale * kLog2e};
-  a.sink = sink, a.rel = rel, a.n_rel = rel ? n_rel : 0;
+  a.sink = sink, a.rel = rel, a.n_rel = rel ? n_rel : 0, a.slope = slope;
   if (cap > 0.f) {
     // tanh x = x - x^3 / 3 + 2 x^5 / 15 - 17 x^7 / 315 + ..., to 2e-6 relative for x up to 0.3
     const float c = scale / cap, cap2 = cap * kLog2e, c2 = c * c;
@@ -370,7 +379,7 @@ DSV4_API int dsv4_flash_attention(const void* q, int ldq, const void* k, const v
   } else {
     a.small = INFINITY, a.p0 = a.scale2;      // only reached with a bias
   }
-  const int mode = rel ? kCappedBias : cap > 0.f ? kCapped : kScaled;
+  const int mode = slope ? kSloped : rel ? kCappedBias : cap > 0.f ? kCapped : kScaled;
   return dim <= 64 ? dispatch_flash<1>(mode, tq, tk, tv, out, a, n_items, st)
                    : dispatch_flash<2>(mode, tq, tk, tv, out, a, n_items, st);
 }

@@ -107,7 +107,7 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_kernel(const __grid_const
       tc_fence_after();
       const int row = m * kPM + q * 32 + lane;
       const uint32_t d0 = tmem + acc * kPN + ((uint32_t)(q * 32) << 16);
-      const bool gated = g.act == kActGeluGate;
+      const bool gated = gated_act(g.act);
       OutT* dst = out + (size_t)row * g.ldo + (gated ? (size_t)n * (kPN / 2) : (size_t)b * g.N + n * kPN);
       const int cols = min(kPN, g.N - n * kPN);
       const bool vec = ((uintptr_t)dst & 15) == 0;
@@ -121,7 +121,7 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_kernel(const __grid_const
 #pragma unroll
         for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
         if (gated) {
-          gate_block(v);
+          gate_block(v, g.act);
           st_f16x(dst + c / 2, v);
           continue;
         }
@@ -188,7 +188,7 @@ DSV4_API int dsv4_gemm_prefill(const void* x, const void* w, void* out, int M, i
                                int out_fp32, int accumulate, int act, int batches, int sms, cudaStream_t st) {
   if (M <= 0 || N <= 0) return 0;
   if (K % 8 || ldx % 8 || ldw % 8 || batches < 1 || sms < 1) return 660;
-  if (act == kActGeluGate && (N % 32 || ldo % 16 || batches != 1 || accumulate)) return 664;
+  if (gated_act(act) && (N % 32 || ldo % 16 || batches != 1 || accumulate)) return 664;
   CUtensorMap ta, tb;
   if (dsv4_make_tmap_2d(&ta, x, 1, (uint64_t)K * batches, M, (uint64_t)ldx * 2, 64, kPM, 3)) return 661;
   if (dsv4_make_tmap_2d(&tb, w, 1, K, (uint64_t)N * batches, (uint64_t)ldw * 2, 64, kPN, 3)) return 662;

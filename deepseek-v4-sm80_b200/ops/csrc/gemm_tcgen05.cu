@@ -429,10 +429,10 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       }
       write_out = false;
     }
-    if (!FP8 && write_out && g.act == kActGeluGate) {
+    if (!FP8 && write_out && gated_act(g.act)) {
 #pragma unroll
       for (int c = 0; c < BN / 32; ++c) {
-        gate_block(&acc[c * 32]);
+        gate_block(&acc[c * 32], g.act);
         if (grow < M && n0 + c * 32 < N) st_f16x(part + (size_t)grow * ld_part + (n0 + c * 32) / 2, &acc[c * 32]);
       }
       write_out = false;
@@ -502,7 +502,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       for (int f = t; f < total_f4; f += 128) {
         const int row = (int)my_rank * rows_per + f / f4_per_row, c4 = f % f4_per_row;
         const uint32_t addr = red_base + (uint32_t)(row * (BN + 4) + c4 * 4) * 4u;
-        if (!FP8 && g.act == kActGeluGate) {   // gate columns fetch their up columns, 16 further on
+        if (!FP8 && gated_act(g.act)) {   // gate columns fetch their up columns, 16 further on
           if (c4 & 4) continue;
           float4 a = make_float4(0.f, 0.f, 0.f, 0.f), u = a;
           for (int sp = 0; sp < S2; ++sp) {
@@ -511,9 +511,10 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             u.x += w.x, u.y += w.y, u.z += w.z, u.w += w.w;
           }
           const int col = n0 + c4 * 4;
+          const bool silu = g.act == kActSiluGate;
           if (m0 + row < M && col < N)
             st_f4(outb + (size_t)(m0 + row) * g.ldo + (col / 32) * kGateBlock + col % 32,
-                  make_float4(gelu_tanh(a.x) * u.x, gelu_tanh(a.y) * u.y, gelu_tanh(a.z) * u.z, gelu_tanh(a.w) * u.w));
+                  make_float4(gate_mul(a.x, u.x, silu), gate_mul(a.y, u.y, silu), gate_mul(a.z, u.z, silu), gate_mul(a.w, u.w, silu)));
           continue;
         }
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -652,7 +653,7 @@ DSV4_API int dsv4_gemm_bf16(const void* x, const void* w, void* out, int M, int 
                             int act, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if ((K % 8) || (ldx % 8) || (ldw % 8)) return 110;
-  if (act == kActGeluGate && (N % 32 || ldo % 16 || batches > 1 || accumulate_out)) return 117;
+  if (gated_act(act) && (N % 32 || ldo % 16 || batches > 1 || accumulate_out)) return 117;
   LaunchOpts o;
   o.batches = batches < 1 ? 1 : batches;
   o.splits = splits < 1 ? 1 : splits;

@@ -1,10 +1,11 @@
 // Causal attention with several query heads to a key head over paged keys and values (bf16 or fp32 caches): what happens
 // between the q | k | v projection and the output projection.
 //
-//   s_ij = cap tanh(q_i . k_j scale / cap) + rel[h, min(i - j, last)],    w_ij = e^{s_ij} / (e^{sink_h} + sum_j' e^{s_ij'})
+//   s_ij = cap tanh(q_i . k_j scale / cap) + rel[h, min(i - j, last)] - slope_h (i - j)
+//   w_ij = e^{s_ij} / (e^{sink_h} + sum_j' e^{s_ij'})
 //
-// cap, rel and sink are optional.  Kernels:
-//   rotate_store     bias, rotation, query temperature; keys and values to their cache rows
+// cap, rel, slope and sink are optional.  With a chunk size, position i only sees keys from i / chunk * chunk on.  Kernels:
+//   rotate_store     bias, norms, rotation, query temperature; keys and values to their cache rows
 //   grouped_attn     tensor cores (mma.sync): the (token, query head) rows of a key head are consecutive, and all of them see
 //                    a prefix of the same keys, so a CTA takes 16 .. 64 rows of one request and key head and streams the keys
 //                    and values once for all of them.  grid.y splits the keys when the row tiles alone leave SMs idle;
@@ -23,18 +24,24 @@ struct RotateArgs {
   int pairs;
   float coef;                // query temperature 1 + coef ln((pos + 1) / every + 1); every 0: none
   int every;
+  const float* gain;         // [(H + G) dim]: q and k are divided by the root mean square of all their rows, times this; or null
+  int unit_v;                // every head's values are divided by their root mean square
+  float eps, v_mul;          // and the values multiplied by v_mul
   const int* pos;
   const int* out_loc;
   int heads, kv_heads, dim, vdim;
 };
 
-// One CTA per token; cos and sin of its angles in shared memory.  W consecutive values per thread (even, or 1).
+// One CTA per token; cos and sin of its angles and the norms' factors in shared memory.  W consecutive values per thread (even,
+// or 1).
 template <typename T, int W>
 __global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__ qkv, T* __restrict__ q,
                                                            T* __restrict__ keys, T* __restrict__ values,
                                                            const RotateArgs a) {
   pdl_entry();
   extern __shared__ float2 cs[];
+  __shared__ float sh[32];
+  float* inv = reinterpret_cast<float*>(cs + a.pairs);   // of q, of k, of every value head
   const int t = blockIdx.x, pos = a.pos[t], loc = a.out_loc[t];
   for (int i = threadIdx.x; i < a.pairs; i += 256) {
     float s, c;
@@ -42,13 +49,33 @@ __global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__
     cs[i] = make_float2(c, s);
   }
   const float temp = a.every ? 1.f + a.coef * logf((float)((pos + 1) / a.every + 1)) : 1.f;
-  __syncthreads();
   const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
   const T* src = qkv + (size_t)t * a.ld;
+  auto at = [&](int i) { return ld_f(src + i) + (a.bias ? a.bias[i] : 0.f); };
+  if (a.gain) {
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x; i < nq + nk; i += 256) {
+      const float x = at(i);
+      if (i < nq) sq += x * x; else sk += x * x;
+    }
+    sq = cta_sum(sq, sh), sk = cta_sum(sk, sh);
+    if (threadIdx.x == 0) inv[0] = 1.f / sqrtf(sq / nq + a.eps), inv[1] = 1.f / sqrtf(sk / nk + a.eps);
+  }
+  if (a.unit_v)
+    for (int g = threadIdx.x >> 5; g < a.kv_heads; g += 8) {
+      float s = 0.f;
+      for (int i = threadIdx.x & 31; i < a.vdim; i += 32) {
+        const float x = at(nq + nk + g * a.vdim + i);
+        s += x * x;
+      }
+      s = warp_sum(s);
+      if ((threadIdx.x & 31) == 0) inv[2 + g] = 1.f / sqrtf(s / a.vdim + a.eps);
+    }
+  __syncthreads();
   for (int i = threadIdx.x * W; i < nq + nk + nv; i += 256 * W) {
     float v[W];
     if constexpr (W == 1) {
-      v[0] = ld_f(src + i) + (a.bias ? a.bias[i] : 0.f);
+      v[0] = at(i);
     } else {
 #pragma unroll
       for (int j = 0; j < W; j += 4) {
@@ -61,12 +88,17 @@ __global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__
       }
     }
     if (i < nq + nk) {
+      const float sc = a.gain ? inv[i >= nq] : 1.f;
+      if (a.gain) {
+#pragma unroll
+        for (int j = 0; j < W; ++j) v[j] *= sc * a.gain[i + j];
+      }
       const int e = i % a.dim;
       if constexpr (W == 1) {
         if (e < 2 * a.pairs) {
           const int o = e & 1 ? i - 1 : i + 1;
           const float2 r = cs[e >> 1];
-          const float other = ld_f(src + o) + (a.bias ? a.bias[o] : 0.f);
+          const float other = at(o) * (a.gain ? sc * a.gain[o] : 1.f);
           v[0] = e & 1 ? v[0] * r.x + other * r.y : v[0] * r.x - other * r.y;
         }
       } else {
@@ -78,6 +110,10 @@ __global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__
             v[j] = x * r.x - y * r.y, v[j + 1] = y * r.x + x * r.y;
           }
       }
+    } else {
+      const float sc = a.unit_v ? inv[2 + (i - nq - nk) / a.vdim] * a.v_mul : a.v_mul;
+#pragma unroll
+      for (int j = 0; j < W; ++j) v[j] *= sc;
     }
     T* dst;
     if (i < nq) {
@@ -113,6 +149,9 @@ struct AttnArgs {
   const float* sink;     // [H] or null
   const float* rel;      // [H][n_rel] or null
   int n_rel;
+  const float* slope;    // [H]: taken off per position of distance; or null
+  int chunk;             // > 0: keys are seen from the start of the query's chunk of this many positions on; the tokens of a
+                         // tile then lie in one chunk
   int nsplit;
   float* part_acc;       // [T * H][nsplit][vdim]
   float* part_ml;        // [T * H][nsplit][2]
@@ -165,8 +204,9 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
   }
   if (a.num_valid && row0 / R >= *a.num_valid) return;
   const int t_last = (row1 - 1) / R;
-  const int nkeys = a.pos[t_last] + 1;   // of the tile's last token, the one that sees most
-  const int* pt = a.page_table + (size_t)a.slots[t_last] * a.ld_pt;
+  const int key0 = a.chunk ? a.pos[t_last] / a.chunk * a.chunk : 0;   // first key; keys are counted from there
+  const int nkeys = a.pos[t_last] + 1 - key0;   // of the tile's last token, the one that sees most
+  const int* pt = a.page_table + (size_t)a.slots[t_last] * a.ld_pt + key0;
   // place of row r of the tile in q (elements) and in the lists of (token, head) rows
   auto head_row = [&](int r) { return (size_t)((row0 + r) / R) * (a.kv_heads * R) + g * R + (row0 + r) % R; };
 
@@ -191,7 +231,7 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
   }
   if (tid < M) {
     ms[tid] = -1e30f, ls[tid] = 0.f;
-    see[tid] = row0 + tid < row1 ? a.pos[(row0 + tid) / R] + 1 : 0;
+    see[tid] = row0 + tid < row1 ? a.pos[(row0 + tid) / R] + 1 - key0 : 0;
   }
 
   // four threads fetch the key and the value of one row
@@ -289,6 +329,11 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
         const float* rel = a.rel + (size_t)(g * R + (row0 + r) % R) * a.n_rel;
 #pragma unroll
         for (int i = 0; i < PER; ++i) v[i] = fmaf(rel[max(min(lim - 1 - i, a.n_rel - 1), 0)], kLog2e, v[i]);
+      }
+      if (a.slope) {
+        const float slope = row0 + r < row1 ? a.slope[g * R + (row0 + r) % R] * kLog2e : 0.f;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) v[i] = fmaf(-slope, (float)(lim - 1 - i), v[i]);
       }
 #pragma unroll
       for (int i = 0; i < PER; ++i) {
@@ -444,8 +489,9 @@ __global__ void __launch_bounds__(128) grouped_row_kernel(const T* __restrict__ 
   if (row >= a.rows * H) return;
   const int t = row / H, h = row % H, g = h / a.group;
   if (a.num_valid && t >= *a.num_valid) return;
-  const int nkeys = a.pos[t] + 1;
-  const int* pt = a.page_table + (size_t)a.slots[t] * a.ld_pt;
+  const int key0 = a.chunk ? a.pos[t] / a.chunk * a.chunk : 0, nkeys = a.pos[t] + 1 - key0;
+  const int* pt = a.page_table + (size_t)a.slots[t] * a.ld_pt + key0;
+  const float slope = a.slope ? a.slope[h] : 0.f;
   const T *kb = keys + g * a.dim, *vb = values + g * a.vdim;
   const size_t ldk = (size_t)a.kv_heads * a.dim, ldv = (size_t)a.kv_heads * a.vdim;
   const float* rel = a.rel ? a.rel + (size_t)h * a.n_rel : nullptr;
@@ -479,6 +525,7 @@ __global__ void __launch_bounds__(128) grouped_row_kernel(const T* __restrict__ 
         s[j] = warp_sum(s[j]) * a.scale;
         if (a.cap > 0.f) s[j] = a.cap * tanhf(s[j] / a.cap);
         if (rel) s[j] += rel[min(max(nkeys - 1 - (k0 + k + j), 0), a.n_rel - 1)];
+        s[j] = fmaf(-slope, (float)(nkeys - 1 - (k0 + k + j)), s[j]);
         if (k + j >= n) s[j] = -INFINITY;
         mn = fmaxf(mn, s[j]);
       }
@@ -508,7 +555,7 @@ __global__ void __launch_bounds__(128) grouped_row_kernel(const T* __restrict__ 
 
 // ------------------------------------------------------------------ keys and values of long portions, side by side
 // ctx_k[dst + j] = keys of key j of every listed request; ctx_vt[:, dst + j] = its values; zeros in the padding behind them.
-// list: [segs][3] = slot, keys, first row of the copy (a multiple of 64).  One CTA: 64 keys x 64 columns of k or v.
+// list: [segs][4] = slot, keys, first row of the copy (a multiple of 64), first key.  One CTA: 64 keys x 64 columns of k or v.
 __global__ void __launch_bounds__(256) kv_gather_kernel(const __nv_bfloat16* __restrict__ keys,
                                                         const __nv_bfloat16* __restrict__ values,
                                                         __nv_bfloat16* __restrict__ ctx_k, __nv_bfloat16* __restrict__ ctx_vt,
@@ -520,10 +567,10 @@ __global__ void __launch_bounds__(256) kv_gather_kernel(const __nv_bfloat16* __r
   int lo = 0, hi = segs - 1;
   while (lo < hi) {
     const int mid = (lo + hi + 1) >> 1;
-    if (list[mid * 3 + 2] <= row0) lo = mid; else hi = mid - 1;
+    if (list[mid * 4 + 2] <= row0) lo = mid; else hi = mid - 1;
   }
-  const int j0 = row0 - list[lo * 3 + 2], n = list[lo * 3 + 1];
-  const int* pt = page_table + (size_t)list[lo * 3] * ld_pt;
+  const int j0 = row0 - list[lo * 4 + 2], n = list[lo * 4 + 1];
+  const int* pt = page_table + (size_t)list[lo * 4] * ld_pt + list[lo * 4 + 3];
   const bool is_k = (int)blockIdx.y < kblocks;
   const int c0 = (is_k ? blockIdx.y : blockIdx.y - kblocks) * 64, w = is_k ? kw : vw;
   const __nv_bfloat16* src = is_k ? keys : values;
@@ -594,20 +641,21 @@ int launch_row(const void* q, const void* k, const void* v, void* o, const AttnA
 
 template <typename T, int W>
 void launch_rotate(const void* qkv, void* q, void* keys, void* values, const RotateArgs& a, int rows, cudaStream_t st) {
-  dsv4_launch(rotate_store_kernel<T, W>, rows, 256, a.pairs * sizeof(float2), st, (const T*)qkv, (T*)q, (T*)keys,
-              (T*)values, a);
+  const size_t smem = a.pairs * sizeof(float2) + (a.gain || a.unit_v ? (2 + a.kv_heads) * sizeof(float) : 0);
+  dsv4_launch(rotate_store_kernel<T, W>, rows, 256, smem, st, (const T*)qkv, (T*)q, (T*)keys, (T*)values, a);
 }
 
 }  // namespace
 
 // qkv [rows, ld]: q (heads x dim) | k (kv_heads x dim) | v (kv_heads x vdim); q_out [rows, heads * dim]; caches
-// [locations, kv_heads * dim] and [locations, kv_heads * vdim].  pairs: rotated pairs per head; every 0: no temperature.
+// [locations, kv_heads * dim] and [locations, kv_heads * vdim].  pairs: rotated pairs per head; every 0: no temperature; gain,
+// unit_v: norms as in RotateArgs.
 DSV4_API int dsv4_rotate_store(const void* qkv, int ld, const float* bias, const float* freq, int pairs, float coef, int every,
-                               const int* pos, const int* out_loc, void* q_out, void* keys, void* values, int rows,
+                               const float* gain, int unit_v, float eps, float v_mul, const int* pos, const int* out_loc, void* q_out, void* keys, void* values, int rows,
                                int heads, int kv_heads, int dim, int vdim, int fp32, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (pairs < 0 || 2 * pairs > dim || pairs > 4096 || (pairs && !freq) || every < 0) return 674;
-  const RotateArgs a{ld, bias, freq, pairs, coef, every, pos, out_loc, heads, kv_heads, dim, vdim};
+  if (pairs < 0 || 2 * pairs > dim || pairs > 4096 || (pairs && !freq) || every < 0 || kv_heads > 1024) return 674;
+  const RotateArgs a{ld, bias, freq, pairs, coef, every, gain, unit_v, eps, v_mul, pos, out_loc, heads, kv_heads, dim, vdim};
   const bool wide = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0;
   if (fp32)
     wide ? launch_rotate<float, 4>(qkv, q_out, keys, values, a, rows, st)
@@ -624,13 +672,14 @@ DSV4_API int dsv4_rotate_store(const void* qkv, int ld, const float* bias, const
 DSV4_API int dsv4_grouped_attention(const void* q, const void* keys, const void* values, void* o, const int* slots,
                                     const int* pos, const int* page_table, int ld_pt, const int* tiles, int n_tiles,
                                     const int* num_valid, int rows, int kv_heads, int group, int dim, int vdim, float scale,
-                                    float cap, const float* sink, const float* rel, int n_rel, int m, int nsplit,
-                                    float* part_acc, float* part_ml, int fp32, cudaStream_t st) {
+                                    float cap, const float* sink, const float* rel, int n_rel, const float* slope,
+                                    int chunk, int m, int nsplit, float* part_acc, float* part_ml, int fp32,
+                                    cudaStream_t st) {
   if (rows <= 0) return 0;
   if (nsplit < 1 || nsplit > 32 || (nsplit > 1 && (!part_acc || !part_ml)) || (rel && n_rel < 1)) return 675;
-  if (kv_heads < 1 || kv_heads > 65535 || group < 1) return 676;
+  if (kv_heads < 1 || kv_heads > 65535 || group < 1 || chunk < 0) return 676;
   const AttnArgs a{slots, pos, page_table, ld_pt, tiles, n_tiles, num_valid, rows, kv_heads, group, dim, vdim, scale, cap,
-                   sink, rel, n_rel, nsplit, part_acc, part_ml};
+                   sink, rel, n_rel, slope, chunk, nsplit, part_acc, part_ml};
   if (m == 0)
     return fp32 ? launch_row<float>(q, keys, values, o, a, st) : launch_row<__nv_bfloat16>(q, keys, values, o, a, st);
   if (fp32 || dim % 8 || vdim % 8) return 677;

@@ -35,6 +35,7 @@ struct PlanHeader {
 // table row; w = p[idx] / (sum + 1e-8) * scaling.  Rows >= num_valid get (-1, 0).
 // scoring 3: the bias belongs to the logits, the k largest z = score + bias are selected and weighted with the softmax
 // over the selected logits only (p = e^(z - max z); the largest is always selected, so the sum is at least 1).
+// scoring 2: p is the softmax over all logits; scoring 4: the same, and the weights are p * scaling as they are.
 __global__ void moe_topk_kernel(const float* __restrict__ scores, const float* __restrict__ bias,
                                 const int* __restrict__ tid2eid, const int* __restrict__ token_ids,
                                 const int* __restrict__ num_valid, int* __restrict__ idx, float* __restrict__ wts,
@@ -105,7 +106,7 @@ __global__ void moe_topk_kernel(const float* __restrict__ scores, const float* _
       if (scoring == 3) sel[i] = s;
     }
   }
-  if (scoring == 2) {
+  if (scoring == 2 || scoring == 4) {
     ssum = warp_sum(ssum);
 #pragma unroll
     for (int i = 0; i < MAXPER; ++i) p[i] /= ssum;
@@ -154,7 +155,7 @@ __global__ void moe_topk_kernel(const float* __restrict__ scores, const float* _
   }
   if (lane < k) {
     idx[row * k + lane] = myi;
-    wts[row * k + lane] = myw / (wsum + 1e-8f) * scaling;
+    wts[row * k + lane] = scoring == 4 ? myw * scaling : myw / (wsum + 1e-8f) * scaling;
   }
 }
 

@@ -5,14 +5,21 @@
 
 namespace {
 
-// x[t] = embed[id], also as activations (x0, may be null).  feedback as in embed_kernel: the token of row t is
-// feedback[slots[t]] and is written to ids[t].
+// x[t] = embed[id] * mul (+ pos_w[pos[t]]), `copies` times side by side, also as activations (x0, may be null).  feedback as
+// in embed_kernel: the token of row t is feedback[slots[t]] and is written to ids[t].
+struct EmbedArgs {
+  float mul;
+  const __nv_bfloat16* pos_w;   // [n_pos][d] learned position vectors, or null
+  const int* pos;
+  int n_pos, copies, d;
+};
 template <typename T>
 __global__ void __launch_bounds__(256) embed_residual_kernel(int* __restrict__ ids, const int* __restrict__ feedback,
                                                              const int* __restrict__ slots,
                                                              const __nv_bfloat16* __restrict__ w,
-                                                             float* __restrict__ x, T* __restrict__ x0, int d) {
+                                                             float* __restrict__ x, T* __restrict__ x0, const EmbedArgs a) {
   pdl_entry();
+  const int d = a.d;
   const int t = blockIdx.x;
   int id;
   if (feedback) {
@@ -22,9 +29,28 @@ __global__ void __launch_bounds__(256) embed_residual_kernel(int* __restrict__ i
     id = ids[t];
   }
   const __nv_bfloat16* src = w + (size_t)id * d;
+  const __nv_bfloat16* at = nullptr;
+  if (a.pos_w) {
+    const int p = a.pos[t];
+    if (p >= a.n_pos && threadIdx.x == 0) dsv4_set_error(DSV4_ERR_BAD_INDEX, 60, p);
+    at = a.pos_w + (size_t)min(p, a.n_pos - 1) * d;
+  }
+  if (d % 4 == 0) {
+    for (int i = threadIdx.x * 4; i < d; i += blockDim.x * 4) {
+      float4 v = ld_f4(src + i);
+      v.x *= a.mul, v.y *= a.mul, v.z *= a.mul, v.w *= a.mul;
+      if (at) {
+        const float4 p = ld_f4(at + i);
+        v.x += p.x, v.y += p.y, v.z += p.z, v.w += p.w;
+      }
+      for (int c = 0; c < a.copies; ++c) st_f4(x + ((size_t)t * a.copies + c) * d + i, v);
+      if (x0) st_f4(x0 + (size_t)t * d + i, v);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
-    const float v = bf2f(src[i]);
-    x[(size_t)t * d + i] = v;
+    const float v = bf2f(src[i]) * a.mul + (at ? bf2f(at[i]) : 0.f);
+    for (int c = 0; c < a.copies; ++c) x[((size_t)t * a.copies + c) * d + i] = v;
     if (x0) st_f(x0 + (size_t)t * d + i, v);
   }
 }
@@ -260,16 +286,16 @@ int launch_layer_norm(const LayerNormArgs& a, void* out, int rows, cudaStream_t 
   return (int)cudaGetLastError();
 }
 
-// gelu(gate) * up behind a projection without the gated epilogue: gu [rows, 2 f] in alternating blocks of 16 columns
+// gate(z) * up behind a projection without the gated epilogue: gu [rows, 2 f] in alternating blocks of 16 columns
 template <typename T>
-__global__ void __launch_bounds__(256) gelu_gate_kernel(const T* __restrict__ gu, T* __restrict__ out, long long total,
-                                                        int f) {
+__global__ void __launch_bounds__(256) gate_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, long long total, int f,
+                                                       bool silu) {
   pdl_entry();
   const long long i = blockIdx.x * 256ll + threadIdx.x;
   if (i >= total) return;
   const int c = (int)(i % f);
   const T* g = gu + i / f * 2 * f + c / kGateBlock * 2 * kGateBlock + c % kGateBlock;
-  st_f(out + i, gelu_tanh(ld_f(g)) * ld_f(g + kGateBlock));
+  st_f(out + i, gate_mul(ld_f(g), ld_f(g + kGateBlock), silu));
 }
 
 template <typename T>
@@ -290,17 +316,19 @@ int launch_norm(const NormArgs& a, const void* erows, void* out, int rows, cudaS
 
 }  // namespace
 
-// fp32: the activation type (0 = bf16, 1 = fp32).
+// fp32: the activation type (0 = bf16, 1 = fp32).  x [t, copies, d].
 DSV4_API int dsv4_embed_residual(int* ids, const int* feedback, const int* slots, const void* w, float* x, void* x0,
-                                 int t, int d, int fp32, cudaStream_t st) {
+                                 float mul, const void* pos_w, const int* pos, int n_pos, int copies, int t, int d, int fp32,
+                                 cudaStream_t st) {
   if (t <= 0) return 0;
-  if (feedback && !slots) return 600;
+  if ((feedback && !slots) || (pos_w && (!pos || n_pos < 1)) || copies < 1) return 600;
+  const EmbedArgs a{mul, (const __nv_bfloat16*)pos_w, pos, n_pos, copies, d};
   if (fp32)
     dsv4_launch(embed_residual_kernel<float>, t, 256, 0, st, ids, feedback, slots, (const __nv_bfloat16*)w, x,
-                (float*)x0, d);
+                (float*)x0, a);
   else
     dsv4_launch(embed_residual_kernel<__nv_bfloat16>, t, 256, 0, st, ids, feedback, slots, (const __nv_bfloat16*)w, x,
-                (__nv_bfloat16*)x0, d);
+                (__nv_bfloat16*)x0, a);
   return (int)cudaGetLastError();
 }
 
@@ -342,14 +370,16 @@ DSV4_API int dsv4_residual_layer_norm(float* x, const long long* rows_idx, const
   return fp32 ? launch_layer_norm<float>(a, out, rows, st) : launch_layer_norm<__nv_bfloat16>(a, out, rows, st);
 }
 
-DSV4_API int dsv4_gelu_gate(const void* gu, void* out, int rows, int f, int fp32, cudaStream_t st) {
+DSV4_API int dsv4_gate_mul(const void* gu, void* out, int rows, int f, int act, int fp32, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (f % kGateBlock) return 607;
+  if (f % kGateBlock || !gated_act(act)) return 607;
+  const bool silu = act == kActSiluGate;
   const long long total = (long long)rows * f;
   const unsigned grid = (unsigned)((total + 255) / 256);
   if (fp32)
-    dsv4_launch(gelu_gate_kernel<float>, grid, 256, 0, st, (const float*)gu, (float*)out, total, f);
+    dsv4_launch(gate_mul_kernel<float>, grid, 256, 0, st, (const float*)gu, (float*)out, total, f, silu);
   else
-    dsv4_launch(gelu_gate_kernel<__nv_bfloat16>, grid, 256, 0, st, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, total, f);
+    dsv4_launch(gate_mul_kernel<__nv_bfloat16>, grid, 256, 0, st, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, total, f,
+                silu);
   return (int)cudaGetLastError();
 }

@@ -49,9 +49,10 @@ __device__ __forceinline__ float cta_sum(float v, float* sh) {
 }
 
 // Epilogue activations of the projections (the numbers are part of the host interface).
-// kActGeluGate pairs columns: the weight rows come in blocks of 16 gate and 16 up rows, and the result is half as wide.
-enum GemmAct : int { kActNone = 0, kActRelu2 = 1, kActTanh = 2, kActGeluGate = 3 };
+// The gates pair columns: the weight rows come in blocks of 16 gate and 16 up rows, and the result is half as wide.
+enum GemmAct : int { kActNone = 0, kActRelu2 = 1, kActTanh = 2, kActGeluGate = 3, kActSiluGate = 4 };
 constexpr int kGateBlock = 16;
+__host__ __device__ __forceinline__ bool gated_act(int act) { return act == kActGeluGate || act == kActSiluGate; }
 __device__ __forceinline__ float gemm_act(float v, int act) {
   if (act == kActRelu2) {
     v = fmaxf(v, 0.f);
@@ -66,14 +67,15 @@ template <typename T>
 __device__ __forceinline__ float sigmoid_for(float z) {
   return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-z)) : sigmoid_f(z);
 }
-// 0.5 z (1 + tanh(w)) = z sigmoid(2 w),  w = sqrt(2 / pi) (z + 0.044715 z^3)
-__device__ __forceinline__ float gelu_tanh(float z) {
-  return z * sigmoid_f(1.5957691216057308f * fmaf(0.044715f * z * z, z, z));
+// gate(z) * up.  silu: z sigmoid(z);  gelu: 0.5 z (1 + tanh(w)) = z sigmoid(2 w),  w = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gate_mul(float z, float up, bool silu) {
+  const float w = silu ? z : 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+  return z * sigmoid_f(w) * up;
 }
 // v: a row's 32 consecutive columns (16 gate, 16 up) -> its 16 gated values in v[0..15]
-__device__ __forceinline__ void gate_block(float* v) {
+__device__ __forceinline__ void gate_block(float* v, int act) {
 #pragma unroll
-  for (int j = 0; j < kGateBlock; ++j) v[j] = gelu_tanh(v[j]) * v[j + kGateBlock];
+  for (int j = 0; j < kGateBlock; ++j) v[j] = gate_mul(v[j], v[j + kGateBlock], act == kActSiluGate);
 }
 // 16 consecutive values, dst 16-byte aligned
 __device__ __forceinline__ void st_f16x(__nv_bfloat16* dst, const float* v) {

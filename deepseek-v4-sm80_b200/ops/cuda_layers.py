@@ -20,14 +20,35 @@ def _f32(dtype) -> I:
 
 
 # --------------------------------------------------------------------------- residual stream
-@tensors(ids="i32[T]", weight="bf16[_,_]", feedback="?i32[_]", slots="?i32[T]")
-def embed_residual(ids, weight, dtype, feedback=None, slots=None, want_act=False):
+@tensors(ids="i32[T]", weight="bf16[_,D]", feedback="?i32[_]", slots="?i32[T]", table="?bf16[_,D]", positions="?i32[T]")
+def embed_residual(ids, weight, dtype, feedback=None, slots=None, want_act=False, mul=1.0, table=None, positions=None,
+                   streams=None):
     t, d = ids.shape[0], weight.shape[1]
-    x = torch.empty(t, d, dtype=torch.float32, device=ids.device)
+    x = torch.empty(*((t, d) if streams is None else (t, streams, d)), dtype=torch.float32, device=ids.device)
     act = torch.empty(t, d, dtype=dtype, device=ids.device) if want_act else None
-    nv.call("embed_residual", nv.ptr(ids), nv.ptr(feedback), nv.ptr(slots), nv.ptr(weight), nv.ptr(x), nv.ptr(act),
-            I(t), I(d), _f32(dtype))
+    nv.call("embed_residual", nv.ptr(ids), nv.ptr(feedback), nv.ptr(slots), nv.ptr(weight), nv.ptr(x), nv.ptr(act), F(mul),
+            nv.ptr(table), nv.ptr(positions), I(0 if table is None else table.shape[0]), I(streams or 1), I(t), I(d),
+            _f32(dtype))
     return x, act
+
+
+@tensors(x="f32[T,S,D]", pre="?f32[_]", post="?f32[_]", sub="?f32[T,D]", rows="?i64[_]")
+def stream_norm(x, eps, dtype, pre, post, sub, experts, rows, keep):
+    t, s, d = x.shape
+    assert (pre is None or pre.shape[0] == s + 1) and (post is None or post.shape[0] == s * (s + 1))
+    erows = wts = idx = h = None
+    topk = n_experts = 0
+    if experts is not None:
+        erows, wts, idx, n_experts, h = experts
+        topk = idx.shape[1]
+        assert erows.dtype == h.dtype == dtype and erows.shape == (t * topk, d) and h.shape == (t, d)
+        assert erows.is_contiguous() and h.is_contiguous() and idx.shape == wts.shape == (t, topk)
+    n_out = t if rows is None else rows.shape[0]
+    out = torch.empty(n_out, d, dtype=dtype, device=x.device) if pre is not None else None
+    nv.call("stream_norm", nv.ptr(x), nv.ptr(rows), nv.ptr(post), nv.ptr(sub), nv.ptr(erows), nv.ptr(wts), nv.ptr(idx),
+            I(topk), I(n_experts), nv.ptr(h), nv.ptr(pre), F(eps), I(1 if keep and post is not None else 0), nv.ptr(out),
+            I(n_out), I(s), I(d), _f32(dtype))
+    return out
 
 
 @tensors(x="f32[_,D]", gain="?f32[D]", rows="?i64[_]", add="?f32[_,D]", add2="?f32[_,D]", vec="?f32[D]")
@@ -47,8 +68,11 @@ def residual_norm(x, gain, eps, dtype, mul=1.0, rows=None, add=None, add2=None, 
 
 
 # --------------------------------------------------------------------------- mixture of experts
+ROUTERS = {"selected": 3, "softmax": 4}      # csrc/moe.cu: moe_topk_kernel
+
+
 @tensors(h="bf16|f32[T,D]", weight="bf16[E,D]", bias="f32[E]", num_valid="?i32[1]")
-def route_topk(h, weight, bias, top, num_valid=None):
+def route_topk(h, weight, bias, top, num_valid=None, kind="selected", scale=1.0):
     t, e = h.shape[0], weight.shape[0]
     if _tma_ok(h, weight, h.shape[1]):
         scores = gemm_bf16_partials(h, weight)      # [S, T, E]; the selection kernel adds the splits
@@ -57,7 +81,7 @@ def route_topk(h, weight, bias, top, num_valid=None):
     idx = torch.empty(t, top, dtype=torch.int32, device=h.device)
     wts = torch.empty(t, top, dtype=torch.float32, device=h.device)
     nv.call("moe_topk", nv.ptr(scores), nv.ptr(bias), nv.ptr(None), nv.ptr(None), nv.ptr(num_valid), nv.ptr(idx),
-            nv.ptr(wts), I(t), I(e), I(top), F(1.0), I(3), I(scores.shape[0]), L(scores.stride(0)))
+            nv.ptr(wts), I(t), I(e), I(top), F(scale), I(ROUTERS[kind]), I(scores.shape[0]), L(scores.stride(0)))
     return idx, wts
 
 
@@ -202,7 +226,7 @@ def expanded_attention(q, cache, fb, uk, uv, heads, scale):
     k, vt = linear(ctx, uk), linear(uv, ctx)
     out = torch.empty(t, heads * vdim, dtype=q.dtype, device=q.device)
     nv.call("flash_attention", nv.ptr(q), I(q.stride(0)), nv.ptr(k), nv.ptr(vt), nv.ptr(out), nv.ptr(items), I(n_items),
-            I(t), I(rows), I(heads), I(heads), I(dim), I(vdim), F(scale), F(0.0), nv.ptr(None), nv.ptr(None), I(0))
+            I(t), I(rows), I(heads), I(heads), I(dim), I(vdim), F(scale), F(0.0), nv.ptr(None), nv.ptr(None), I(0), nv.ptr(None))
     return out
 
 
@@ -223,20 +247,21 @@ WKV_CHUNKED = None
 WKV_CHUNK_MIN, WKV_CHUNK = 64, 32
 
 
-def _chunk_plan(fb, device):
-    """(chunks [n, 2], segments [m, 4]) of a forward for the chunked recurrence; the same for all layers."""
-    plan = getattr(fb, "chunk_plan", None)
+def _chunk_plan(fb, device, size=WKV_CHUNK):
+    """(chunks [n, 2], segments [m, 4]) of a forward for a recurrence in chunks of ``size``; the same for all layers."""
+    plans = fb.__dict__.setdefault("chunk_plans", {})
+    plan = plans.get(size)
     if plan is None:
         chunks, segs, row = [], [], 0
         for n, slot in zip(fb.seg_lens, fb.seg_slots):
             c0 = len(chunks)
-            chunks += [(row + i, min(WKV_CHUNK, n - i)) for i in range(0, n, WKV_CHUNK)]
+            chunks += [(row + i, min(size, n - i)) for i in range(0, n, size)]
             segs.append((slot, c0, len(chunks) - c0, row))
             row += n
         host = torch.tensor([v for t in (*chunks, *segs) for v in t], dtype=torch.int32).pin_memory()
         dev = host.to(device, non_blocking=True)
         k = 2 * len(chunks)
-        plan = fb.chunk_plan = (dev[:k], dev[k:], len(chunks), len(segs))
+        plan = plans[size] = (dev[:k], dev[k:], len(chunks), len(segs))
     return plan
 
 

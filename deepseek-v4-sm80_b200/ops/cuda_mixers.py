@@ -10,7 +10,7 @@ import torch
 from . import native as nv
 from .cuda import num_sms
 from .cuda_layers import KV_ALIGN, SMEM_BYTES, _chunk_plan, _f32
-from .gemm import _tma_ok, linear
+from .gemm import ACTS, _tma_ok, linear
 from .native import F, I
 from .tensorcheck import tensors
 
@@ -35,29 +35,33 @@ def residual_layer_norm(x, eps, dtype, norm, sub, add, rows, keep):
 
 
 # --------------------------------------------------------------------------- gated feed-forward
+GATE_ACTS = {"gelu_tanh": "gelu_gate", "silu": "silu_gate"}
+
+
 def gated_linear(h, w, act, block):
-    if act != "gelu_tanh" or block != 16:
+    if act not in GATE_ACTS or block != 16:
         raise ValueError(f"no kernel for the gate {act!r} in blocks of {block}")
     if _tma_ok(h, w, h.shape[1]):
-        return linear(h, w, act="gelu_gate")
+        return linear(h, w, act=GATE_ACTS[act])
     gu = linear(h, w)
     t, f = h.shape[0], w.shape[0] // 2
     out = torch.empty(t, f, dtype=h.dtype, device=h.device)
-    nv.call("gelu_gate", nv.ptr(gu), nv.ptr(out), I(t), I(f), _f32(h.dtype))
+    nv.call("gate_mul", nv.ptr(gu), nv.ptr(out), I(t), I(f), I(ACTS[GATE_ACTS[act]]), _f32(h.dtype))
     return out
 
 
 # --------------------------------------------------------------------------- grouped attention
-@tensors(qkv="bf16|f32[T,_]", bias="?f32[_]", freq="?f32[_]", keys="bf16|f32[R,_]", values="bf16|f32[R,_]")
-def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads, kv_heads, dim, vdim):
+@tensors(qkv="bf16|f32[T,_]s", bias="?f32[_]", freq="?f32[_]", keys="bf16|f32[R,_]", values="bf16|f32[R,_]", gain="?f32[_]")
+def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads, kv_heads, dim, vdim, gain, unit_v, eps, v_mul):
     t = qkv.shape[0]
     assert qkv.dtype == keys.dtype == values.dtype and qkv.shape[1] == (heads + kv_heads) * dim + kv_heads * vdim
     assert keys.shape[1] == kv_heads * dim and values.shape[1] == kv_heads * vdim
+    assert gain is None or gain.shape[0] == (heads + kv_heads) * dim
     q = torch.empty(t, heads, dim, dtype=qkv.dtype, device=qkv.device)
     coef, every = q_temp if q_temp is not None else (0.0, 0)
     nv.call("rotate_store", nv.ptr(qkv), I(qkv.stride(0)), nv.ptr(bias), nv.ptr(freq), I(0 if freq is None else freq.shape[0]),
-            F(coef), I(every), nv.ptr(fb.positions), nv.ptr(fb.out_loc), nv.ptr(q), nv.ptr(keys), nv.ptr(values), I(t),
-            I(heads), I(kv_heads), I(dim), I(vdim), _f32(qkv.dtype))
+            F(coef), I(every), nv.ptr(gain), I(1 if unit_v else 0), F(eps), F(v_mul), nv.ptr(fb.positions), nv.ptr(fb.out_loc),
+            nv.ptr(q), nv.ptr(keys), nv.ptr(values), I(t), I(heads), I(kv_heads), I(dim), I(vdim), _f32(qkv.dtype))
     return q
 
 
@@ -80,22 +84,34 @@ def _split_keys(tiles: int, kv_heads: int, m: int, width: int, max_context: int,
     return max(1, min(ctas // max(tiles * kv_heads, 1), -(-max_context // 128), 32))
 
 
-def _prefill_plan(fb, device, group: int, flash_ok: bool):
+def _pieces(fb, chunk: int):
+    """The portions of a forward, cut where a chunk of keys ends: (queries, keys seen by the last one, slot, first key)."""
+    for n, s, slot in zip(fb.seg_lens, fb.seg_ends, fb.seg_slots):
+        at, size = s - n, chunk or s
+        while at < s:
+            key0 = at // size * size
+            end = min(key0 + size, s)
+            yield end - at, end - key0, slot, key0
+            at = end
+
+
+def _prefill_plan(fb, device, group: int, flash_ok: bool, chunk: int):
     """How the requests of a prefill forward are spread over the two kernels; the same for all layers with this many query
-    heads to a key head: (flash requests [n, 3], flash items [m, 5], n, m, gathered rows, row tiles [k, 2], k, rows per tile,
-    longest context among the row tiles)."""
+    heads to a key head and this chunk size: (flash requests [n, 4], flash items [m, 5], n, m, gathered rows, row tiles [k, 2],
+    k, rows per tile, longest context among the row tiles)."""
     plans = fb.__dict__.setdefault("grouped_plans", {})
-    key = (group, flash_ok, GROUPED_PREFILL, FLASH_MIN)
+    key = (group, flash_ok, GROUPED_PREFILL, FLASH_MIN, chunk)
     if key in plans:
         return plans[key]
     least = 1 if GROUPED_PREFILL == "flash" else FLASH_MIN
-    flash = [flash_ok and n >= least for n in fb.seg_lens]
-    few = [n for n, f in zip(fb.seg_lens, flash) if not f]
+    pieces = list(_pieces(fb, chunk))
+    flash = [flash_ok and n >= least for n, _, _, _ in pieces]
+    few = [p[0] for p, f in zip(pieces, flash) if not f]
     m = row_tile(max(few) * group) if few else 16
     reqs, items, tiles, at, row, longest = [], [], [], 0, 0, 1
-    for n, s, slot, f in zip(fb.seg_lens, fb.seg_ends, fb.seg_slots, flash):
+    for (n, s, slot, key0), f in zip(pieces, flash):
         if f:
-            reqs.append((slot, s, at))
+            reqs.append((slot, s, at, key0))
             for q in range(0, n, 256):
                 k = min(256, n - q)
                 items.append((row + q, k, s - n + q, at, s - n + q + k))
@@ -107,13 +123,13 @@ def _prefill_plan(fb, device, group: int, flash_ok: bool):
     items.sort(key=lambda i: -i[4])                   # the longest first
     host = torch.tensor([v for t in (*reqs, *items, *tiles) for v in t], dtype=torch.int32).pin_memory()
     dev = host.to(device, non_blocking=True)
-    a, b = 3 * len(reqs), 3 * len(reqs) + 5 * len(items)
+    a, b = 4 * len(reqs), 4 * len(reqs) + 5 * len(items)
     plans[key] = (dev[:a], dev[a:b], len(reqs), len(items), at, dev[b:], len(tiles), m, longest)
     return plans[key]
 
 
-@tensors(q="bf16|f32[T,H,D]", keys="bf16|f32[R,_]", values="bf16|f32[R,_]", sink="?f32[H]", rel="?f32[H,_]")
-def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel):
+@tensors(q="bf16|f32[T,H,D]", keys="bf16|f32[R,_]", values="bf16|f32[R,_]", sink="?f32[H]", rel="?f32[H,_]", slope="?f32[H]")
+def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, slope, chunk):
     t, heads, dim = q.shape
     group, kw, vw = heads // kv_heads, keys.shape[1], values.shape[1]
     vdim = vw // kv_heads
@@ -121,11 +137,12 @@ def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel):
     out = torch.empty(t, heads * vdim, dtype=q.dtype, device=q.device)
     pt, n_rel = fb.page_table, 0 if rel is None else rel.shape[1]
     even = q.dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0
-    tiles, n_tiles, m, longest = None, 0, 0, fb.max_context
+    tiles, n_tiles, m, longest = None, 0, 0, min(fb.max_context, chunk) if chunk else fb.max_context
     if even and fb.seg_lens is not None:
         ctx = sum(-(-s // KV_ALIGN) * KV_ALIGN for s in fb.seg_ends)
         flash_ok = max(dim, vdim) <= 128 and GROUPED_PREFILL != "rows" and 2 * ctx * (kw + vw) <= FLASH_BYTES
-        reqs, items, n_reqs, n_items, rows, tiles, n_tiles, m, longest = _prefill_plan(fb, q.device, group, flash_ok)
+        flash_ok = flash_ok and not (slope is not None and (softcap or rel is not None))
+        reqs, items, n_reqs, n_items, rows, tiles, n_tiles, m, longest = _prefill_plan(fb, q.device, group, flash_ok, chunk)
         if n_items:
             ck = torch.empty(rows, kw, dtype=q.dtype, device=q.device)
             cv = torch.empty(vw, rows, dtype=q.dtype, device=q.device)
@@ -133,7 +150,7 @@ def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel):
                     nv.ptr(pt), I(pt.stride(0)), I(kw), I(vw))
             nv.call("flash_attention", nv.ptr(q), I(heads * dim), nv.ptr(ck), nv.ptr(cv), nv.ptr(out), nv.ptr(items),
                     I(n_items), I(t), I(rows), I(heads), I(kv_heads), I(dim), I(vdim), F(scale), F(softcap), nv.ptr(sink),
-                    nv.ptr(rel), I(n_rel))
+                    nv.ptr(rel), I(n_rel), nv.ptr(slope))
         if n_tiles == 0:
             return out
     elif even:
@@ -151,8 +168,8 @@ def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel):
             ml = torch.empty(t * heads, nsplit, 2, dtype=torch.float32, device=q.device)
     nv.call("grouped_attention", nv.ptr(q), nv.ptr(keys), nv.ptr(values), nv.ptr(out), nv.ptr(fb.slots), nv.ptr(fb.positions),
             nv.ptr(pt), I(pt.stride(0)), nv.ptr(tiles), I(n_tiles), nv.ptr(fb.num_valid), I(t), I(kv_heads), I(group), I(dim),
-            I(vdim), F(scale), F(softcap), nv.ptr(sink), nv.ptr(rel), I(n_rel), I(m), I(nsplit), nv.ptr(acc), nv.ptr(ml),
-            _f32(q.dtype))
+            I(vdim), F(scale), F(softcap), nv.ptr(sink), nv.ptr(rel), I(n_rel), nv.ptr(slope), I(chunk), I(m), I(nsplit), nv.ptr(acc),
+            nv.ptr(ml), _f32(q.dtype))
     return out
 
 

@@ -110,7 +110,8 @@ def _ws(m, n, bn, batches, splits, device):
 
 
 # epilogue activations of the projections (csrc/vec.cuh: GemmAct), applied to the fp32 sum
-ACTS = {None: 0, "relu2": 1, "tanh": 2, "gelu_gate": 3}     # gelu_gate: half as many columns come out (TMA operands only)
+ACTS = {None: 0, "relu2": 1, "tanh": 2, "gelu_gate": 3, "silu_gate": 4}
+GATES = ("gelu_gate", "silu_gate")          # half as many columns come out (TMA operands only)
 
 
 def _act(y, act):
@@ -169,7 +170,7 @@ def grouped_linear(x, w, groups: int, out=None, out_dtype=None, accumulate=False
     t, k = x.shape[0], x.shape[1] // groups
     n = w.shape[0] // groups
     if out is None:
-        cols = n // 2 if act == "gelu_gate" else groups * n
+        cols = n // 2 if act in GATES else groups * n
         out = torch.empty(t, cols, dtype=out_dtype or x.dtype, device=x.device)
     if not x.is_cuda:
         y = torch.einsum("tgk,gnk->tgn", x.reshape(t, groups, k).float(), w.reshape(groups, n, k).float())
@@ -189,7 +190,7 @@ def grouped_linear(x, w, groups: int, out=None, out_dtype=None, accumulate=False
                 I(out.stride(0)), f32, I(1 if accumulate else 0), I(bn), I(groups), I(splits), nv.ptr(ws), nv.ptr(cnt),
                 I(ACTS[act]))
     else:
-        assert act != "gelu_gate"
+        assert act not in GATES
         nv.call("gemm_simt", nv.ptr(x), nv.ptr(w), nv.ptr(out), I(t), I(n), I(k), I(x.stride(0)), I(w.stride(0)),
                 I(out.stride(0)), I(1 if x.dtype == torch.float32 else 0), f32, I(1 if accumulate else 0),
                 I(ACTS[act]), I(groups))

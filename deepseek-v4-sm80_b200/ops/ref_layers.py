@@ -19,11 +19,34 @@ def segments(fb):
     return list(zip(off[:-1], off[1:]))
 
 
-def embed_residual(ids, weight, dtype, feedback, slots, want_act):
+def embed_residual(ids, weight, dtype, feedback, slots, want_act, mul, table, positions, streams):
     if feedback is not None:
         ids.copy_(feedback[slots.long()])
-    x = weight[ids.long()].float()
-    return x, (x.to(dtype, copy=True) if want_act else None)    # the stream changes in place
+    x = weight[ids.long()].float() * mul
+    if table is not None:
+        x = x + table[positions.long()].float()
+    act = x.to(dtype, copy=True) if want_act else None           # the stream changes in place
+    return (x if streams is None else x[:, None].repeat(1, streams, 1)), act
+
+
+def stream_norm(x, eps, dtype, pre, post, sub, experts, rows, keep):
+    t, s, d = x.shape
+    new = x
+    if post is not None:
+        y = torch.zeros(t, d) if sub is None else sub
+        if experts is not None:
+            erows, wts, idx, n, h = experts
+            real = (idx >= 0) & (idx < n)
+            w = torch.where(real, wts, torch.zeros_like(wts))
+            y = y + (torch.where(real[..., None], erows.float().view(*idx.shape, -1), 0.0) * w[..., None]).sum(1)
+            y = y + torch.where(idx >= n, wts, torch.zeros_like(wts)).sum(1, keepdim=True) * h.float()
+        new = torch.einsum("tad,ab->tbd", x, post[s:].view(s, s)) + post[:s, None] * y[:, None]
+        if keep:
+            x.copy_(new)
+    if pre is None:
+        return None
+    u = torch.einsum("tsd,s->td", new if rows is None else new[rows], pre[:s])
+    return (_rms(u, eps) * pre[s]).to(dtype)
 
 
 def residual_norm(x, gain, eps, dtype, mul, rows, add, add2, vec, experts, cast):
@@ -40,10 +63,15 @@ def residual_norm(x, gain, eps, dtype, mul, rows, add, add2, vec, experts, cast)
     return (_rms(y, eps) * gain * mul).to(dtype)
 
 
-def route_topk(h, weight, bias, top, num_valid):
-    z = h.float() @ weight.float().t() + bias
-    idx = torch.sort(z, dim=-1, descending=True, stable=True).indices[:, :top]
-    w = torch.softmax(torch.gather(z, 1, idx), -1)
+def route_topk(h, weight, bias, top, num_valid, kind, scale):
+    z = h.float() @ weight.float().t()
+    if kind == "selected":
+        idx = torch.sort(z + bias, dim=-1, descending=True, stable=True).indices[:, :top]
+        w = torch.softmax(torch.gather(z + bias, 1, idx), -1) * scale
+    else:
+        p = torch.softmax(z, -1)
+        idx = torch.sort(p + bias, dim=-1, descending=True, stable=True).indices[:, :top]
+        w = torch.gather(p, 1, idx) * scale
     idx = idx.to(torch.int32)
     if num_valid is not None:
         idx[int(num_valid):] = -1

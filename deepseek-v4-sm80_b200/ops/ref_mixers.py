@@ -6,7 +6,7 @@ import math
 
 import torch
 
-from .ref_layers import segments
+from .ref_layers import _rms, segments
 
 
 def _layer_norm(x, w, b, eps):
@@ -29,15 +29,23 @@ def residual_layer_norm(x, eps, dtype, norm, sub, add, rows, keep):
 def gated_linear(h, w, act, block):
     y = (h.float() @ w.float().t()).to(h.dtype).float().view(h.shape[0], -1, 2, block)
     g, u = y[:, :, 0], y[:, :, 1]
-    assert act == "gelu_tanh"
-    a = 0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g ** 3)))
+    if act == "silu":
+        a = g * torch.sigmoid(g)
+    else:
+        assert act == "gelu_tanh"
+        a = 0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g ** 3)))
     return (a * u).reshape(h.shape[0], -1).to(h.dtype)
 
 
-def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads, kv_heads, dim, vdim):
+def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads, kv_heads, dim, vdim, gain, unit_v, eps, v_mul):
     t = qkv.shape[0]
     x = qkv.float() if bias is None else qkv.float() + bias
     q, k, v = x.split([heads * dim, kv_heads * dim, kv_heads * vdim], 1)
+    if gain is not None:
+        q, k = _rms(q, eps) * gain[: heads * dim], _rms(k, eps) * gain[heads * dim:]
+    if unit_v:
+        v = _rms(v.reshape(t, kv_heads, vdim), eps).reshape(t, -1)
+    v = v * v_mul
     pos = fb.positions
 
     def turn(y):
@@ -61,7 +69,7 @@ def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads, kv_heads, dim
     return q.to(qkv.dtype)
 
 
-def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel):
+def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, slope, chunk):
     t, heads, dim = q.shape
     vdim, group = values.shape[1] // kv_heads, heads // kv_heads
     out = torch.empty(t, heads, vdim, dtype=q.dtype)
@@ -76,7 +84,12 @@ def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel):
         away = fb.positions[a:b].long()[:, None] - torch.arange(n)[None, :]
         if rel is not None:
             s = s + rel[:, away.clamp(0, rel.shape[1] - 1)]
-        s = s.masked_fill(away < 0, float("-inf"))
+        if slope is not None:
+            s = s - slope[:, None, None] * away
+        hidden = away < 0
+        if chunk:
+            hidden = hidden | (torch.arange(n)[None, :] < (fb.positions[a:b].long() // chunk * chunk)[:, None])
+        s = s.masked_fill(hidden, float("-inf"))
         if sink is not None:
             s = torch.cat([s, sink[:, None, None].expand(heads, b - a, 1)], -1)
         p = torch.softmax(s, -1)[..., :n]
