@@ -1,10 +1,12 @@
 """Prefill and decode throughput of a layered design beside the closest other model at equal size: Bedalorn beside DeepSeek-V4,
-Buvalix beside Bedalorn.
+Buvalix beside Bedalorn, Zazilix beside Bedalorn (whose experts are the like feed-forwards) and Buvalix (whose recurrence and
+attention are the like mixers).
 
-    python bench.py --design bedalorn|buvalix [--sizes small,large] [--profile]
+    python bench.py --design bedalorn|buvalix|zazilix [--sizes small,large] [--profile]
 
 Equal size: the same width, layer runs, attention heads, vocabulary and feed-forward weights (DeepSeek-V4: the same experts;
-Buvalix's gated feed-forwards have three matrices, so the Bedalorn model beside it has dense ones half as wide again), random
+Buvalix's gated feed-forwards have three matrices, so the Bedalorn model beside it has dense ones half as wide again; Zazilix has
+one expert less than the Bedalorn model with experts everywhere, and a shared one), random
 weights, one GPU, through the offline API.  Per model and workload one JSON line: device time of the forwards (CUDA
 events), tokens per second, and with ``--profile`` the per-launcher share of one eager forward of each phase.
 Workloads: prefill forwards of 8 x 1 024 and 1 x 8 192 tokens; decode steps of 128 sequences at 1 024 tokens of context and
@@ -65,6 +67,30 @@ def buvalix_config(size: str):
     delta = ChannelDeltaSpec(hd, hd, 128, 128, 4)
     layers = tuple(LayerSpec((rotary, bucket, delta, rotary)[i % 4], DenseSpec(ff)) for i in range(n))
     return BuvalixConfig(layers, d, vocab, 1e-6, _loop(n, passes), 1 << 17)
+
+
+def zazilix_config(size: str):
+    from minisgl.models.layered_config import LayerSpec
+    from minisgl.models.zazilix_config import (ChunkAttentionSpec, ForgetSpec, MambaSpec, MixtureSpec, MLSTMSpec, ParallelSpec,
+                                               ZazilixConfig)
+
+    d, h, _, _, _, e, top, eff, n, passes, vocab = SIZES[size]
+    g, half = DENSE_SIZES[size][2], h // 2
+    memory = MLSTMSpec(h, 128, 128, 15.0)
+    both = ParallelSpec(ChunkAttentionSpec(h, g, 128, 128, 128 ** -0.5, 2048), ForgetSpec(half, 128, 128), 0.7, 0.7)
+    mamba = MambaSpec(d // 32, 64, 8, 128, 4, 8)                      # twice the width inside
+    ff = MixtureSpec(eff, e - 1, top - 1, 8, 1.0, eff)
+    layers = tuple(LayerSpec((memory, both, mamba, both)[i % 4], ff) for i in range(n * passes))
+    return ZazilixConfig(layers, d, vocab, 1e-6, 4, 1.0, 1 << 14, max_position=1 << 14)
+
+
+def bedalorn_experts_config(size: str):
+    from minisgl.models.bedalorn_config import BedalornConfig, ExpertsSpec, LatentAttentionSpec, LayerSpec, WKVSpec
+
+    d, h, hw, rank, _, e, top, eff, n, passes, vocab = SIZES[size]
+    attn, moe = LatentAttentionSpec(h, 128, 128, rank, 128 ** -0.5), ExpertsSpec(eff, e, top)
+    layers = tuple(LayerSpec(WKVSpec(hw, 64) if i % 4 in (0, 2) else attn, moe) for i in range(n * passes))
+    return BedalornConfig(layers, d, vocab, 1e-6, 1.0, None, 1 << 17)
 
 
 def dsv4_config(size: str):
@@ -156,6 +182,7 @@ def run(cfg, phase: str, batch: int, context: int, profile: bool, steps: int = 3
 PAIRS = {
     "bedalorn": {"bedalorn": bedalorn_config, "dsv4": dsv4_config},
     "buvalix": {"buvalix": buvalix_config, "bedalorn": bedalorn_dense_config},
+    "zazilix": {"zazilix": zazilix_config, "bedalorn": bedalorn_experts_config, "buvalix": buvalix_config},
 }
 
 

@@ -150,8 +150,8 @@ def random_weights(cfg: ZazilixConfig, device, seed: int = 0) -> Dict[str, torch
 
     def draw(name):
         s = shapes[name]
-        r = lambda std: torch.randn(*s, generator=g, device=device, dtype=torch.float32) * std
-        u = lambda lo, hi: torch.rand(*s, generator=g, device=device) * (hi - lo) + lo
+        r = lambda std: torch.randn(s, generator=g, device=device, dtype=torch.float32) * std
+        u = lambda lo, hi: torch.rand(s, generator=g, device=device) * (hi - lo) + lo
         if name in ("embed", "pos"):
             t = r(1.0 if name == "embed" else 0.1)
         elif name.endswith((".in", ".out", ".mix")) and ".hc" in name:

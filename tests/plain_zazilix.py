@@ -259,8 +259,9 @@ def config(layers, width=96, vocab=136, streams=3, scale=1.5, eps=2e-5, position
             "embedding": {"scale": scale}, "norm": {"eps": eps}, "max_positions": positions}
 
 
-def tensors(cfg, seed=0):
-    """Random tensors of the configuration in the checkpoint's names (bfloat16)."""
+def tensors(cfg, seed=0, clear=False):
+    """Random tensors of the configuration in the checkpoint's names (bfloat16).  clear: the routers' corrections alone decide which
+    experts are chosen, so that rounding never does."""
     g = torch.Generator().manual_seed(seed)
     width, n, out = cfg["width"], cfg["streams"], {}
 
@@ -332,6 +333,8 @@ def tensors(cfg, seed=0):
             r, q = ff["router"], p + "mlp."
             lin(q + "router", r["experts"] + r["identity"], width, 2.0)
             vec(q + "correction", r["experts"] + r["identity"], 0.1)
+            if clear:
+                out[q + "correction"] = torch.randperm(r["experts"] + r["identity"], generator=g) * 1.5
             for name, size in [(f"e{e}", ff["expert"]["ff"]) for e in range(r["experts"])] + [("shared", ff["shared"]["ff"])]:
                 lin(f"{q}{name}.gate", size, width, 1.5)
                 lin(f"{q}{name}.up", size, width)

@@ -273,13 +273,13 @@ def test_gathered_keys_and_values():
     from minisgl.ops import native as nv
     from minisgl.ops.native import I
 
-    reqs = torch.tensor([1, 70, 0, 2, 210, 128], dtype=torch.int32, device=DEV)
+    reqs = torch.tensor([1, 70, 0, 0, 2, 170, 128, 40], dtype=torch.int32, device=DEV)   # slot, keys, row, first key
     total = 128 + 256
     ck, cv = torch.full((total, kw), 9.0, device=DEV).bfloat16(), torch.full((vw, total), 9.0, device=DEV).bfloat16()
     nv.call("kv_gather", nv.ptr(keys), nv.ptr(values), nv.ptr(ck), nv.ptr(cv), nv.ptr(reqs), I(2), I(total),
             nv.ptr(fb.page_table), I(fb.page_table.stride(0)), I(kw), I(vw))
-    for slot, n, at, end in ((1, 70, 0, 128), (2, 210, 128, 384)):
-        loc = fb.page_table[slot, :n].long()
+    for slot, n, at, end, key0 in ((1, 70, 0, 128, 0), (2, 170, 128, 384, 40)):
+        loc = fb.page_table[slot, key0:key0 + n].long()
         assert torch.equal(ck[at:at + n], keys[loc]) and torch.equal(cv[:, at:at + n], values[loc].t())
         assert float(ck[at + n:end].abs().max()) == 0 and float(cv[:, at + n:end].abs().max()) == 0
 

@@ -1,0 +1,41 @@
+"""Whole-model cases of the Zazilix design: small configurations, checked with ``layered_checks``."""
+import torch
+
+import layered_checks
+import plain_zazilix as P
+from layered_checks import *  # noqa: F401,F403
+
+MODELS = {
+    # every mixer, a layer without feed-forward, chunks that end inside pages
+    "mixed": P.config([P.mlstm_layer(ff=P.moe()), P.parallel_layer(ff=P.moe(32, 5, 2, 3, 2.2, 40)), P.mamba_layer(ff=P.moe()),
+                       P.parallel_layer(4, 1, 24, 16, 37, 0.2, 3, 16, 8, 1.4, 0.5)]),
+    # recurrences only: nothing is paged
+    "recurrent": P.config([P.mamba_layer(6, 16, 3, 40, 4, 2, P.moe(24, 4, 2, 1)), P.mlstm_layer(2, 32, 48, 5.0),
+                           P.mamba_layer(3, 40, 1, 24, 2, 1)], width=64, vocab=80, streams=2),
+    # sizes of one: a stream, a head, a tap, chunks of one position; every router output is chosen
+    "single": P.config([P.parallel_layer(1, 1, 16, 16, 1, 0.5, 1, 8, 8, 1.0, 1.0, P.moe(16, 2, 3, 1, 1.0, 24)),
+                        P.mlstm_layer(1, 8, 8, 20.0), P.mamba_layer(1, 8, 1, 8, 1, 1)], width=48, vocab=64, streams=1),
+    # attention on chunks that are whole pages, and longer than most sequences; no expert passes its input on
+    "attention": P.config([P.parallel_layer(20, 1, 16, 24, 64, 0.4, 2, 16, 16, 0.7, 0.2, P.moe(48, 8, 2, 0, 2.5, 32)),
+                           P.parallel_layer(34, 2, 8, 8, 100, 0.5, 1, 16, 16, 2.0, 0.3),
+                           P.parallel_layer(4, 4, 48, 40, 700, 0.2, 1, 8, 24, 1.1, 0.4)], width=128, vocab=96, streams=4),
+    # rows that do not start on 16 bytes, nothing a multiple of eight
+    "ragged": P.config([P.mlstm_layer(3, 9, 7, 6.0, P.moe(21, 3, 2, 2, 1.3, 15)), P.parallel_layer(6, 2, 10, 14, 23, 0.3, 3, 7, 5),
+                        P.mamba_layer(3, 7, 3, 11, 5, 3)], width=50, vocab=77, streams=5),
+    # heads wider than the prompt kernel and the chunks of a recurrence take
+    "wide": P.config([P.parallel_layer(2, 1, 160, 144, 90, 0.08, 1, 136, 152), P.mlstm_layer(1, 200, 264, 12.0),
+                      P.mamba_layer(2, 136, 1, 144, 3, 2)], width=72, vocab=88),
+}
+LIMIT = {torch.float32: 1e-4, torch.bfloat16: 5e-2}
+# Head norms of small vectors amplify rounding: in bf16 a few positions are further off, with every backend at the same places.
+STRAY, WORST = 0.045, 0.16
+
+
+class Case(layered_checks.Case):
+    def __init__(self, name, folder, device, dtype):
+        cfg = MODELS[name]
+        # in bf16 a close call of a router may fall the other way: there the choice is clear (32-bit cases and the tests of the
+        # router alone have calls of every kind)
+        tensors = P.tensors(cfg, seed=len(name), clear=dtype == torch.bfloat16)
+        super().__init__(cfg, tensors, P.PlainZazilix(cfg, tensors), P.write_model(cfg, tensors, folder), device, dtype,
+                         LIMIT[dtype], STRAY if dtype == torch.bfloat16 else 0.0, WORST)
