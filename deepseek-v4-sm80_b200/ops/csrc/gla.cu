@@ -244,66 +244,81 @@ struct HeadNormArgs {
   const float* gain;       // [e], or [heads * e] (per_head)
   int per_head, ldg, ldy;  // row strides of gate and y
   float eps, mul;
-  int heads, e, ew;
-  long long total;
+  int heads, e, ew, total;
 };
-// y = o / rms(o) * gain * mul (* sigmoid(gate)), one warp per (row, head)
-template <typename T, int W>
+// y = o / rms(o) * gain * mul (* sigmoid(gate)), one warp per R consecutive (row, head)s of up to NI x 128 values, e and the strides
+// multiples of 4
+template <typename T, int NI, int R>
 __global__ void __launch_bounds__(256) gla_norm_heads_kernel(const T* __restrict__ gate, T* __restrict__ y, const HeadNormArgs a) {
   pdl_entry();
-  const long long r = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  const int r0 = (blockIdx.x * 8 + (threadIdx.x >> 5)) * R;
   const int lane = threadIdx.x & 31;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 o[R][NI], g[R][NI];
+  float den[R], ss[R];
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int at = min(r0 + i, a.total - 1), head = at % a.heads;
+    const size_t r = at, row = at / a.heads;
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int c = (n * 32 + lane) * 4;
+      o[i][n] = c < a.e ? ld_f4(a.o + r * a.ew + c) : zero;
+      g[i][n] = gate && c < a.e ? ld_f4(gate + row * a.ldg + head * a.e + c) : zero;
+    }
+    den[i] = a.floor ? fmaxf(fabsf(a.o[r * a.ew + a.e]), a.floor[r]) + 1e-6f : 1.f;
+  }
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const float f = 1.f / den[i];
+    ss[i] = 0.f;
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      float4& x = o[i][n];
+      x.x *= f, x.y *= f, x.z *= f, x.w *= f;
+      ss[i] += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
+    }
+  }
+#pragma unroll
+  for (int off = 16; off > 0; off >>= 1)
+#pragma unroll
+    for (int i = 0; i < R; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], off);
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    if (r0 + i >= a.total) break;
+    const size_t row = (r0 + i) / a.heads;
+    const int head = (r0 + i) % a.heads;
+    const float inv = a.mul / sqrtf(ss[i] / a.e + a.eps);
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int c = (n * 32 + lane) * 4;
+      if (c >= a.e) continue;
+      const float4 gn = ld_f4(a.gain + (a.per_head ? head * a.e : 0) + c), x = o[i][n], z = g[i][n];
+      float4 w = make_float4(x.x * inv * gn.x, x.y * inv * gn.y, x.z * inv * gn.z, x.w * inv * gn.w);
+      if (gate) w.x *= sigmoid_for<T>(z.x), w.y *= sigmoid_for<T>(z.y), w.z *= sigmoid_for<T>(z.z), w.w *= sigmoid_for<T>(z.w);
+      st_f4(y + row * a.ldy + head * a.e + c, w);
+    }
+  }
+}
+// any sizes, one warp per (row, head)
+template <typename T>
+__global__ void __launch_bounds__(256) gla_norm_heads_any_kernel(const T* __restrict__ gate, T* __restrict__ y,
+                                                                 const HeadNormArgs a) {
+  pdl_entry();
+  const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (r >= a.total) return;
   const size_t row = r / a.heads;
-  const int head = (int)(r % a.heads);
-  const float* o = a.o + r * a.ew;
-  const float den = a.floor ? fmaxf(fabsf(o[a.e]), a.floor[r]) + 1e-6f : 1.f;
+  const int head = r % a.heads;
+  const float* o = a.o + (size_t)r * a.ew;
+  const float f = 1.f / (a.floor ? fmaxf(fabsf(o[a.e]), a.floor[r]) + 1e-6f : 1.f);
   const float* gain = a.gain + (a.per_head ? head * a.e : 0);
-  const T* gp = gate ? gate + row * a.ldg + head * a.e : nullptr;
-  T* dst = y + row * a.ldy + head * a.e;
-  constexpr int NI = W == 4 ? 2 : 8;        // up to 256 values in registers
-  auto value = [&](int c, float (&x)[W]) {
-    ld_w<W>(o + c, x);
-#pragma unroll
-    for (int j = 0; j < W; ++j) x[j] /= den;
-  };
-  float keep[NI][W];
   float ss = 0.f;
-#pragma unroll
-  for (int i = 0; i < NI; ++i) {
-    const int c = (i * 32 + lane) * W;
-#pragma unroll
-    for (int j = 0; j < W; ++j) keep[i][j] = 0.f;
-    if (c < a.e) value(c, keep[i]);
-#pragma unroll
-    for (int j = 0; j < W; ++j) ss += keep[i][j] * keep[i][j];
-  }
-  for (int c = (NI * 32 + lane) * W; c < a.e; c += 32 * W) {
-    float x[W];
-    value(c, x);
-#pragma unroll
-    for (int j = 0; j < W; ++j) ss += x[j] * x[j];
-  }
+  for (int c = lane; c < a.e; c += 32) ss += o[c] * f * (o[c] * f);
   const float inv = a.mul / sqrtf(warp_sum(ss) / a.e + a.eps);
-  auto put = [&](int c, float (&x)[W]) {
-    float gn[W];
-    ld_w<W>(gain + c, gn);
-#pragma unroll
-    for (int j = 0; j < W; ++j) {
-      x[j] *= inv * gn[j];
-      if (gp) x[j] *= sigmoid_for<T>(ld_f(gp + c + j));
-    }
-    st_w<W>(dst + c, x);
-  };
-#pragma unroll
-  for (int i = 0; i < NI; ++i) {
-    const int c = (i * 32 + lane) * W;
-    if (c < a.e) put(c, keep[i]);
-  }
-  for (int c = (NI * 32 + lane) * W; c < a.e; c += 32 * W) {
-    float x[W];
-    value(c, x);
-    put(c, x);
+  for (int c = lane; c < a.e; c += 32) {
+    float x = o[c] * f * inv * gain[c];
+    if (gate) x *= sigmoid_for<T>(ld_f(gate + row * a.ldg + head * a.e + c));
+    st_f(y + row * a.ldy + head * a.e + c, x);
   }
 }
 
@@ -412,6 +427,20 @@ int dispatch_causal(const void* p, void* before, void* out, const CausalConvArgs
   return (int)cudaGetLastError();
 }
 template <typename T>
+int launch_norm_heads(const void* gate, void* y, const HeadNormArgs& a, cudaStream_t st) {
+  auto go = [&](auto kern, int r) {
+    dsv4_launch(kern, (unsigned)((a.total + 8 * r - 1) / (8 * r)), 256, 0, st, (const T*)gate, (T*)y, a);
+  };
+  const bool wide = a.e % 4 == 0 && a.ldy % 4 == 0 && a.ldg % 4 == 0 && ((uintptr_t)gate & (4 * sizeof(T) - 1)) == 0;
+  if (!wide || a.e > 256)
+    go(gla_norm_heads_any_kernel<T>, 1);
+  else if (a.e > 128)
+    go(gla_norm_heads_kernel<T, 2, 2>, 2);
+  else
+    go(gla_norm_heads_kernel<T, 1, 4>, 4);
+  return (int)cudaGetLastError();
+}
+template <typename T>
 int launch_norm_groups(const void* x, const void* z, void* y, const GroupNormArgs& a, int rows, cudaStream_t st) {
   const int w = a.heads * a.e / a.groups;
   const dim3 grid(rows, a.groups);
@@ -480,18 +509,9 @@ DSV4_API int dsv4_gla_norm_heads(const float* o, const float* floor, const void*
                                  float eps, float mul, void* y, int ldy, int rows, int heads, int e, int ew, int fp32,
                                  cudaStream_t st) {
   if (rows <= 0) return 0;
-  const HeadNormArgs a{o, floor, gain, per_head, ldg, ldy, eps, mul, heads, e, ew, (long long)rows * heads};
-  const unsigned grid = (unsigned)((a.total + 7) / 8);
-  const bool wide = e % 4 == 0 && ldy % 4 == 0;
-  auto go = [&](auto kern, auto t) {
-    using T = decltype(t);
-    dsv4_launch(kern, grid, 256, 0, st, (const T*)gate, (T*)y, a);
-  };
-  if (fp32)
-    wide ? go(gla_norm_heads_kernel<float, 4>, 0.f) : go(gla_norm_heads_kernel<float, 1>, 0.f);
-  else
-    wide ? go(gla_norm_heads_kernel<__nv_bfloat16, 4>, __nv_bfloat16()) : go(gla_norm_heads_kernel<__nv_bfloat16, 1>, __nv_bfloat16());
-  return (int)cudaGetLastError();
+  if ((long long)rows * heads > 1 << 30) return 705;
+  const HeadNormArgs a{o, floor, gain, per_head, ldg, ldy, eps, mul, heads, e, ew, rows * heads};
+  return fp32 ? launch_norm_heads<float>(gate, y, a, st) : launch_norm_heads<__nv_bfloat16>(gate, y, a, st);
 }
 
 // See GroupNormArgs; x, z: row strides ldx, ldz; y [rows, heads * e].

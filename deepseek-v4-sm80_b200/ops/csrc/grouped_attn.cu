@@ -32,48 +32,21 @@ struct RotateArgs {
   int heads, kv_heads, dim, vdim;
 };
 
-// One CTA per token; cos and sin of its angles and the norms' factors in shared memory.  W consecutive values per thread (even,
-// or 1).
-template <typename T, int W>
+// One CTA per token; cos and sin of its angles and the norms' sums in shared memory.  W consecutive values per thread and chunk
+// (even, or 1); NC > 0: all chunks of the row in registers, which the norms want.
+template <typename T, int W, int NC>
 __global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__ qkv, T* __restrict__ q,
                                                            T* __restrict__ keys, T* __restrict__ values,
                                                            const RotateArgs a) {
   pdl_entry();
   extern __shared__ float2 cs[];
-  __shared__ float sh[32];
-  float* inv = reinterpret_cast<float*>(cs + a.pairs);   // of q, of k, of every value head
-  const int t = blockIdx.x, pos = a.pos[t], loc = a.out_loc[t];
-  for (int i = threadIdx.x; i < a.pairs; i += 256) {
-    float s, c;
-    sincosf((float)pos * a.freq[i], &s, &c);
-    cs[i] = make_float2(c, s);
-  }
-  const float temp = a.every ? 1.f + a.coef * logf((float)((pos + 1) / a.every + 1)) : 1.f;
+  __shared__ float sums[2][8];
+  float* part = reinterpret_cast<float*>(cs + a.pairs);   // NC > 0: sums of squares of the chunks of v; else of the heads
+  const int t = blockIdx.x, pos = a.pos[t], loc = a.out_loc[t], warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
   const T* src = qkv + (size_t)t * a.ld;
   auto at = [&](int i) { return ld_f(src + i) + (a.bias ? a.bias[i] : 0.f); };
-  if (a.gain) {
-    float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < nq + nk; i += 256) {
-      const float x = at(i);
-      if (i < nq) sq += x * x; else sk += x * x;
-    }
-    sq = cta_sum(sq, sh), sk = cta_sum(sk, sh);
-    if (threadIdx.x == 0) inv[0] = 1.f / sqrtf(sq / nq + a.eps), inv[1] = 1.f / sqrtf(sk / nk + a.eps);
-  }
-  if (a.unit_v)
-    for (int g = threadIdx.x >> 5; g < a.kv_heads; g += 8) {
-      float s = 0.f;
-      for (int i = threadIdx.x & 31; i < a.vdim; i += 32) {
-        const float x = at(nq + nk + g * a.vdim + i);
-        s += x * x;
-      }
-      s = warp_sum(s);
-      if ((threadIdx.x & 31) == 0) inv[2 + g] = 1.f / sqrtf(s / a.vdim + a.eps);
-    }
-  __syncthreads();
-  for (int i = threadIdx.x * W; i < nq + nk + nv; i += 256 * W) {
-    float v[W];
+  auto load = [&](int i, float (&v)[W]) {
     if constexpr (W == 1) {
       v[0] = at(i);
     } else {
@@ -87,11 +60,78 @@ __global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__
         v[j] = x.x, v[j + 1] = x.y, v[j + 2] = x.z, v[j + 3] = x.w;
       }
     }
-    if (i < nq + nk) {
-      const float sc = a.gain ? inv[i >= nq] : 1.f;
-      if (a.gain) {
+  };
+  float row[NC > 0 ? NC : 1][W];
+  float sq = 0.f, sk = 0.f;
+  if constexpr (NC > 0) {
 #pragma unroll
-        for (int j = 0; j < W; ++j) v[j] *= sc * a.gain[i + j];
+    for (int n = 0; n < NC; ++n) {
+      const int i = (n * 256 + (int)threadIdx.x) * W;
+      if (i < nq + nk + nv) load(i, row[n]);
+    }
+#pragma unroll
+    for (int n = 0; n < NC; ++n) {
+      const int i = (n * 256 + (int)threadIdx.x) * W;
+      if (i >= nq + nk + nv) continue;
+      float s = 0.f;
+#pragma unroll
+      for (int j = 0; j < W; ++j) s = fmaf(row[n][j], row[n][j], s);
+      if (i < nq) sq += s;
+      else if (i < nq + nk) sk += s;
+      else if (a.unit_v) part[(i - nq - nk) / W] = s;
+    }
+  } else {
+    for (int i = threadIdx.x; a.gain && i < nq + nk; i += 256) {
+      const float x = at(i);
+      if (i < nq) sq += x * x; else sk += x * x;
+    }
+    for (int g = warp; a.unit_v && g < a.kv_heads; g += 8) {
+      float s = 0.f;
+      for (int i = lane; i < a.vdim; i += 32) {
+        const float x = at(nq + nk + g * a.vdim + i);
+        s += x * x;
+      }
+      s = warp_sum(s);
+      if (lane == 0) part[g] = s;
+    }
+  }
+  if (a.gain) {
+    sq = warp_sum(sq), sk = warp_sum(sk);
+    if (lane == 0) sums[0][warp] = sq, sums[1][warp] = sk;
+  }
+  for (int i = threadIdx.x; i < a.pairs; i += 256) {
+    float s, c;
+    sincosf((float)pos * a.freq[i], &s, &c);
+    cs[i] = make_float2(c, s);
+  }
+  const float temp = a.every ? 1.f + a.coef * logf((float)((pos + 1) / a.every + 1)) : 1.f;
+  __syncthreads();
+  float inv[2] = {1.f, 1.f};       // of q and of k
+  if (a.gain) {
+#pragma unroll
+    for (int p = 0; p < 2; ++p) {
+      float s = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) s += sums[p][w];
+      inv[p] = 1.f / sqrtf(s / (p ? nk : nq) + a.eps);
+    }
+  }
+  auto place = [&](int i, float (&v)[W]) {
+    if (i < nq + nk) {
+      const float sc = i < nq ? inv[0] : inv[1];
+      if (a.gain) {
+        float gn[W];
+        if constexpr (W == 1) {
+          gn[0] = a.gain[i];
+        } else {
+#pragma unroll
+          for (int j = 0; j < W; j += 4) {
+            const float4 f = ld_f4(a.gain + i + j);
+            gn[j] = f.x, gn[j + 1] = f.y, gn[j + 2] = f.z, gn[j + 3] = f.w;
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < W; ++j) v[j] *= sc * gn[j];
       }
       const int e = i % a.dim;
       if constexpr (W == 1) {
@@ -111,7 +151,17 @@ __global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__
           }
       }
     } else {
-      const float sc = a.unit_v ? inv[2 + (i - nq - nk) / a.vdim] * a.v_mul : a.v_mul;
+      float sc = a.v_mul;
+      if (a.unit_v) {
+        const int head = (i - nq - nk) / a.vdim;
+        float s = 0.f;
+        if constexpr (NC > 0) {
+          for (int p = 0; p < a.vdim / W; ++p) s += part[head * (a.vdim / W) + p];
+        } else {
+          s = part[head];
+        }
+        sc /= sqrtf(s / a.vdim + a.eps);
+      }
 #pragma unroll
       for (int j = 0; j < W; ++j) v[j] *= sc;
     }
@@ -121,7 +171,7 @@ __global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__
       for (int j = 0; j < W; ++j) v[j] *= temp;
       dst = q + (size_t)t * nq + i;
     } else {
-      if (loc < 0) continue;
+      if (loc < 0) return;
       dst = i < nq + nk ? keys + (size_t)loc * nk + (i - nq) : values + (size_t)loc * nv + (i - nq - nk);
     }
     if constexpr (W == 1) {
@@ -129,6 +179,18 @@ __global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__
     } else {
 #pragma unroll
       for (int j = 0; j < W; j += 4) st_f4(dst + j, make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]));
+    }
+  };
+  if constexpr (NC > 0) {
+#pragma unroll
+    for (int n = 0; n < NC; ++n) {
+      const int i = (n * 256 + (int)threadIdx.x) * W;
+      if (i < nq + nk + nv) place(i, row[n]);
+    }
+  } else {
+    for (int i = threadIdx.x * W; i < nq + nk + nv; i += 256 * W) {
+      load(i, row[0]);
+      place(i, row[0]);
     }
   }
 }
@@ -641,8 +703,18 @@ int launch_row(const void* q, const void* k, const void* v, void* o, const AttnA
 
 template <typename T, int W>
 void launch_rotate(const void* qkv, void* q, void* keys, void* values, const RotateArgs& a, int rows, cudaStream_t st) {
-  const size_t smem = a.pairs * sizeof(float2) + (a.gain || a.unit_v ? (2 + a.kv_heads) * sizeof(float) : 0);
-  dsv4_launch(rotate_store_kernel<T, W>, rows, 256, smem, st, (const T*)qkv, (T*)q, (T*)keys, (T*)values, a);
+  const int nv = a.kv_heads * a.vdim, chunks = ((a.heads + a.kv_heads) * a.dim + nv + 256 * W - 1) / (256 * W);
+  const bool norms = a.gain || a.unit_v, in_regs = norms && W > 1 && chunks <= 4;
+  const size_t smem = a.pairs * sizeof(float2) + (a.unit_v ? (in_regs ? nv / W : a.kv_heads) * sizeof(float) : 0);
+  auto go = [&](auto kern) {
+    dsv4_launch(kern, rows, 256, smem, st, (const T*)qkv, (T*)q, (T*)keys, (T*)values, a);
+  };
+  if constexpr (W > 1) {
+    if (in_regs && chunks <= 1) return go(rotate_store_kernel<T, W, 1>);
+    if (in_regs && chunks <= 2) return go(rotate_store_kernel<T, W, 2>);
+    if (in_regs) return go(rotate_store_kernel<T, W, 4>);
+  }
+  go(rotate_store_kernel<T, W, 0>);
 }
 
 }  // namespace
@@ -656,7 +728,7 @@ DSV4_API int dsv4_rotate_store(const void* qkv, int ld, const float* bias, const
   if (rows <= 0) return 0;
   if (pairs < 0 || 2 * pairs > dim || pairs > 4096 || (pairs && !freq) || every < 0 || kv_heads > 1024) return 674;
   const RotateArgs a{ld, bias, freq, pairs, coef, every, gain, unit_v, eps, v_mul, pos, out_loc, heads, kv_heads, dim, vdim};
-  const bool wide = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0;
+  const bool wide = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && ((uintptr_t)qkv & 15) == 0;
   if (fp32)
     wide ? launch_rotate<float, 4>(qkv, q_out, keys, values, a, rows, st)
          : launch_rotate<float, 1>(qkv, q_out, keys, values, a, rows, st);

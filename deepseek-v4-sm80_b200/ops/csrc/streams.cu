@@ -68,10 +68,21 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamArgs a, co
         if (S || j < ns) s[j] = ld_f4(x + (size_t)j * d + i);
       if (a.post) {
         float4 y = a.sub ? ld_f4(a.sub + tok * d + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
-        for (int k = 0; k < a.topk; ++k)
-          if ((unsigned)ei[k] < (unsigned)a.n_experts) fma4(y, ew[k], ld_f4(er + (size_t)k * d + i));
-        if (w_id != 0.f) fma4(y, w_id, ld_f4(hr + i));
+        if (a.topk) {
+          const float4 id = w_id != 0.f ? ld_f4(hr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+          for (int k0 = 0; k0 < a.topk; k0 += 4) {         // four rows in flight
+            float4 e[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+              const bool runs = k0 + k < a.topk && (unsigned)ei[k0 + k] < (unsigned)a.n_experts;
+              e[k] = runs ? ld_f4(er + (size_t)(k0 + k) * d + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+              if (k0 + k < a.topk) fma4(y, ew[k0 + k], e[k]);
+          }
+          fma4(y, w_id, id);
+        }
         float4 t[SM];
 #pragma unroll
         for (int j = 0; j < SM; ++j) {

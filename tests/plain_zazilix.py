@@ -291,7 +291,8 @@ def tensors(cfg, seed=0, clear=False):
         if kind == "mlstm":
             h = m["heads"]
             lin(q + "q", h * m["dim"], width, 2.0)
-            lin(q + "k", h * m["dim"], width)
+            lin(q + "k", h * m["dim"], width, 0.6)
+            out[q + "k"] += 0.4 * out[q + "q"]       # a token answers its own query: a head's output is no small difference
             lin(q + "v", h * m["vdim"], width)
             lin(q + "g", h * m["vdim"], width, 2.0)
             lin(q + "o", width, h * m["vdim"])

@@ -27,15 +27,19 @@ MODELS = {
                       P.mamba_layer(2, 136, 1, 144, 3, 2)], width=72, vocab=88),
 }
 LIMIT = {torch.float32: 1e-4, torch.bfloat16: 5e-2}
-# Head norms of small vectors amplify rounding: in bf16 a few positions are further off, with every backend at the same places.
-STRAY, WORST = 0.045, 0.16
+# Rounding is amplified where a head's output is a small difference: in bf16 a few positions are further off, with every backend
+# at the same places.
+STRAY, WORST = 0.02, 0.16
+SEEDS = {"mixed": 9}
 
 
 class Case(layered_checks.Case):
     def __init__(self, name, folder, device, dtype):
         cfg = MODELS[name]
+        if dtype == torch.bfloat16:
+            cfg = {**cfg, "norm": {"eps": 0.05}}      # small vectors stay small
         # in bf16 a close call of a router may fall the other way: there the choice is clear (32-bit cases and the tests of the
         # router alone have calls of every kind)
-        tensors = P.tensors(cfg, seed=len(name), clear=dtype == torch.bfloat16)
+        tensors = P.tensors(cfg, seed=SEEDS.get(name, len(name)), clear=dtype == torch.bfloat16)
         super().__init__(cfg, tensors, P.PlainZazilix(cfg, tensors), P.write_model(cfg, tensors, folder), device, dtype,
                          LIMIT[dtype], STRAY if dtype == torch.bfloat16 else 0.0, WORST)
