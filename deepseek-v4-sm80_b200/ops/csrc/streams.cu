@@ -30,10 +30,10 @@ __device__ __forceinline__ void fma4(float4& a, float w, const float4& v) {
   a.x = fmaf(w, v.x, a.x), a.y = fmaf(w, v.y, a.y), a.z = fmaf(w, v.z, a.z), a.w = fmaf(w, v.w, a.w);
 }
 
-// S streams (0: any number up to kMaxStreams), NV x 4 coordinates per thread; NV = 0: any d, one coordinate at a time and u in
-// shared memory.
-template <typename T, int S, int NV>
-__global__ void __launch_bounds__(256) stream_norm_kernel(const StreamArgs a, const T* __restrict__ erows,
+// S streams (0: any number up to kMaxStreams), NT threads, NV x 4 coordinates per thread; NV = 0: any d, one coordinate at a time
+// and u in shared memory.
+template <typename T, int S, int NV, int NT>
+__global__ void __launch_bounds__(NT, S > 0 && NV == 1 ? 1024 / NT : 1) stream_norm_kernel(const StreamArgs a, const T* __restrict__ erows,
                                                           const T* __restrict__ h, T* __restrict__ out) {
   pdl_entry();
   constexpr int SM = S ? S : kMaxStreams;
@@ -42,8 +42,8 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamArgs a, co
   extern __shared__ float rest[];
   const int r = blockIdx.x, d = a.d, ns = S ? S : a.streams;
   const size_t tok = a.rows_idx ? (size_t)a.rows_idx[r] : r;
-  for (int i = threadIdx.x; a.post && i < ns * (ns + 1); i += 256) post[i] = a.post[i];
-  for (int i = threadIdx.x; a.pre && i <= ns; i += 256) pre[i] = a.pre[i];
+  for (int i = threadIdx.x; a.post && i < ns * (ns + 1); i += NT) post[i] = a.post[i];
+  for (int i = threadIdx.x; a.pre && i <= ns; i += NT) pre[i] = a.pre[i];
   if ((int)threadIdx.x < a.topk) {
     const int e = a.eidx[tok * a.topk + threadIdx.x];
     ei[threadIdx.x] = e, ew[threadIdx.x] = e < 0 ? 0.f : a.wts[tok * a.topk + threadIdx.x];
@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamArgs a, co
     float4 u[NV];
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
-      const int i = (n * 256 + (int)threadIdx.x) * 4;
+      const int i = (n * NT + (int)threadIdx.x) * 4;
       u[n] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (i >= d) continue;
       float4 s[SM];
@@ -83,40 +83,34 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamArgs a, co
           }
           fma4(y, w_id, id);
         }
-        float4 t[SM];
 #pragma unroll
         for (int j = 0; j < SM; ++j) {
           if (!S && j >= ns) continue;
           const float o = post[j];
-          t[j] = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
+          float4 t = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
 #pragma unroll
           for (int q = 0; q < SM; ++q)
-            if (S || q < ns) fma4(t[j], post[ns + q * ns + j], s[q]);
+            if (S || q < ns) fma4(t, post[ns + q * ns + j], s[q]);
+          if (a.keep) st_f4(x + (size_t)j * d + i, t);
+          if (a.pre) fma4(u[n], pre[j], t);
         }
-#pragma unroll
-        for (int j = 0; j < SM; ++j) {
-          if (!S && j >= ns) continue;
-          s[j] = t[j];
-          if (a.keep) st_f4(x + (size_t)j * d + i, s[j]);
-        }
-      }
-      if (a.pre) {
+      } else if (a.pre) {
 #pragma unroll
         for (int j = 0; j < SM; ++j)
           if (S || j < ns) fma4(u[n], pre[j], s[j]);
-        ss += (u[n].x * u[n].x + u[n].y * u[n].y) + (u[n].z * u[n].z + u[n].w * u[n].w);
       }
+      ss += (u[n].x * u[n].x + u[n].y * u[n].y) + (u[n].z * u[n].z + u[n].w * u[n].w);
     }
     if (!a.pre) return;
     const float sc = pre[ns] / sqrtf(cta_sum(ss, sh) / d + a.eps);
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
-      const int i = (n * 256 + (int)threadIdx.x) * 4;
+      const int i = (n * NT + (int)threadIdx.x) * 4;
       if (i < d) st_f4(out + (size_t)r * d + i, make_float4(u[n].x * sc, u[n].y * sc, u[n].z * sc, u[n].w * sc));
     }
   } else {
-    for (int i = threadIdx.x; i < d; i += 256) {
-      float s[SM];
+    for (int i = threadIdx.x; i < d; i += NT) {
+      float s[SM], u = 0.f;
 #pragma unroll
       for (int j = 0; j < SM; ++j)
         if (S || j < ns) s[j] = x[(size_t)j * d + i];
@@ -125,51 +119,44 @@ __global__ void __launch_bounds__(256) stream_norm_kernel(const StreamArgs a, co
         for (int k = 0; k < a.topk; ++k)
           if ((unsigned)ei[k] < (unsigned)a.n_experts) y = fmaf(ew[k], ld_f(er + (size_t)k * d + i), y);
         if (w_id != 0.f) y = fmaf(w_id, ld_f(hr + i), y);
-        float t[SM];
-#pragma unroll
-        for (int j = 0; j < SM; ++j) {
-          if (!S && j >= ns) continue;
-          t[j] = post[j] * y;
+        for (int j = 0; j < ns; ++j) {
+          float t = post[j] * y;
 #pragma unroll
           for (int q = 0; q < SM; ++q)
-            if (S || q < ns) t[j] = fmaf(post[ns + q * ns + j], s[q], t[j]);
+            if (S || q < ns) t = fmaf(post[ns + q * ns + j], s[q], t);
+          if (a.keep) x[(size_t)j * d + i] = t;
+          if (a.pre) u = fmaf(pre[j], t, u);
         }
-#pragma unroll
-        for (int j = 0; j < SM; ++j) {
-          if (!S && j >= ns) continue;
-          s[j] = t[j];
-          if (a.keep) x[(size_t)j * d + i] = s[j];
-        }
-      }
-      if (a.pre) {
-        float u = 0.f;
+      } else if (a.pre) {
 #pragma unroll
         for (int j = 0; j < SM; ++j)
           if (S || j < ns) u = fmaf(pre[j], s[j], u);
-        rest[i] = u;
-        ss += u * u;
       }
+      if (a.pre) rest[i] = u;
+      ss += u * u;
     }
     if (!a.pre) return;
     const float sc = pre[ns] / sqrtf(cta_sum(ss, sh) / d + a.eps);
-    for (int i = threadIdx.x; i < d; i += 256) st_f(out + (size_t)r * d + i, rest[i] * sc);   // what the thread wrote itself
+    for (int i = threadIdx.x; i < d; i += NT) st_f(out + (size_t)r * d + i, rest[i] * sc);   // what the thread wrote itself
   }
 }
 
 template <typename T, int S>
 int launch_streams(const StreamArgs& a, const void* erows, const void* h, void* out, int rows, cudaStream_t st) {
-  auto go = [&](auto kern, size_t smem) { dsv4_launch(kern, rows, 256, smem, st, a, (const T*)erows, (const T*)h, (T*)out); };
+  auto go = [&](auto kern, int threads, size_t smem) {
+    dsv4_launch(kern, rows, threads, smem, st, a, (const T*)erows, (const T*)h, (T*)out);
+  };
   if (a.d % 4 || a.d > 8192) {
     if (a.d > 8192 + 2048) return 611;       // u in 40 KB of shared memory
-    go(stream_norm_kernel<T, S, 0>, (size_t)a.d * 4);
+    go(stream_norm_kernel<T, S, 0, 256>, 256, (size_t)a.d * 4);
   } else if (a.d <= 1024)
-    go(stream_norm_kernel<T, S, 1>, 0);
+    go(stream_norm_kernel<T, S, 1, 256>, 256, 0);
   else if (a.d <= 2048)
-    go(stream_norm_kernel<T, S, 2>, 0);
+    go(stream_norm_kernel<T, S, 1, 512>, 512, 0);
   else if (a.d <= 4096)
-    go(stream_norm_kernel<T, S, 4>, 0);
+    go(stream_norm_kernel<T, S, 2, 512>, 512, 0);
   else
-    go(stream_norm_kernel<T, S, 8>, 0);
+    go(stream_norm_kernel<T, S, 4, 512>, 512, 0);
   return (int)cudaGetLastError();
 }
 template <typename T>

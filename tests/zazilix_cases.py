@@ -29,7 +29,7 @@ MODELS = {
 LIMIT = {torch.float32: 1e-4, torch.bfloat16: 5e-2}
 # Rounding is amplified where a head's output is a small difference: in bf16 a few positions are further off, with every backend
 # at the same places.
-STRAY, WORST = 0.02, 0.16
+STRAY, WORST = 0.045, 0.16
 SEEDS = {"mixed": 9}
 
 
