@@ -2,7 +2,8 @@
 // around it:
 //   mlstm_gates      exponential input and sigmoid forget gates with a running maximum -> log g, factor of k, floor
 //   causal_conv      short causal convolution per channel with bias and silu, and the inputs it keeps
-//   gla_scan         the recurrence, state in registers
+//   gla_scan         the recurrence over a portion, state in registers
+//   gla_step         one token per request: the state streams through once
 //   gla_norm_*       normaliser, skip, gate and norms behind the recurrence
 #include "gla.cuh"
 
@@ -237,6 +238,81 @@ __global__ void __launch_bounds__(512) gla_scan_kernel(const T* __restrict__ q, 
   }
 }
 
+// One CTA per (row, head), one token: a thread takes four columns of every KG-th key, so a row of the state is one contiguous
+// access; the KG partial sums of a column meet in shared memory.
+template <typename T, int MODE>
+__global__ void __launch_bounds__(256, 3) gla_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v,
+                                                       const int* __restrict__ num_valid, const GlaArgs a) {
+  pdl_entry();
+  constexpr int B = 8;             // keys in flight
+  __shared__ float qs[256], ks[256], gs[MODE == kForget ? 256 : 1];
+  __shared__ float4 part[256];
+  const int row = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, d = a.d, ew = a.ew;
+  if (num_valid && row >= *num_valid) return;
+  const int nq = ew / 4, KG = 256 / nq, kg = tid / nq, col = tid % nq * 4, at_k = head / a.group * d;
+  const bool fresh = a.pos[row] == 0, active = kg < KG;
+  float4* st = reinterpret_cast<float4*>(a.state + ((size_t)a.slots[row] * a.heads + head) * d * ew + col);
+  float4 s[B];
+  auto fetch = [&](int k0) {
+#pragma unroll
+    for (int i = 0; i < B; ++i) {
+      const int key = k0 + i * KG + kg;
+      s[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (active && !fresh && key < d) s[i] = st[(size_t)key * nq];
+    }
+  };
+  fetch(0);
+  float keep = 0.f, fac = 1.f;
+  if constexpr (MODE != kForget) {
+    const HeadGate f = head_gate<MODE>(a, row, head);
+    keep = expf(f.log_g), fac = f.fac;
+  }
+  for (int c = tid; c < d; c += 256) {
+    float qv = ld_f(q + (size_t)row * a.ldq + at_k + c);
+    if constexpr (MODE == kForget) {
+      const int ch = head * d + c;
+      const ChannelGate f = channel_gate(a.raw[(size_t)row * a.heads * d + ch] + a.bias[ch], a.par[ch]);
+      ks[c] = f.write, gs[c] = f.keep;
+      qv *= sigmoid_f(qv);
+    } else {
+      ks[c] = ld_f(k + (size_t)row * a.ldk + at_k + c);
+    }
+    qs[c] = qv * a.q_mul;
+  }
+  float vv[4] = {};
+  if (active)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int c = col + j;
+      if (c < a.e) vv[j] = fac * ld_f(v + (size_t)row * a.ldv + head * a.e + c);
+      else if (MODE == kGiven && c == a.e) vv[j] = fac;
+    }
+  __syncthreads();
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int k0 = 0; k0 < d; k0 += B * KG) {
+    if (k0 > 0) fetch(k0);
+#pragma unroll
+    for (int i = 0; i < B; ++i) {
+      const int key = k0 + i * KG + kg;
+      if (!active || key >= d) continue;
+      const float g = MODE == kForget ? gs[MODE == kForget ? key : 0] : keep, kk = ks[key], qq = qs[key];
+      float4 x = s[i];
+      x.x = fmaf(g, x.x, kk * vv[0]), x.y = fmaf(g, x.y, kk * vv[1]), x.z = fmaf(g, x.z, kk * vv[2]), x.w = fmaf(g, x.w, kk * vv[3]);
+      o.x = fmaf(qq, x.x, o.x), o.y = fmaf(qq, x.y, o.y), o.z = fmaf(qq, x.z, o.z), o.w = fmaf(qq, x.w, o.w);
+      st[(size_t)key * nq] = x;
+    }
+  }
+  part[tid] = o;
+  __syncthreads();
+  if (tid < nq) {
+    for (int i = 1; i < KG; ++i) {
+      const float4 x = part[i * nq + tid];
+      o.x += x.x, o.y += x.y, o.z += x.z, o.w += x.w;
+    }
+    reinterpret_cast<float4*>(a.out + ((size_t)row * a.heads + head) * ew)[tid] = o;
+  }
+}
+
 // ------------------------------------------------------------------ behind the recurrence
 struct HeadNormArgs {
   const float* o;          // [rows][heads][ew]
@@ -396,9 +472,19 @@ int dispatch_gla(const void* q, const void* k, const void* v, const GlaArgs& a, 
   if (a.d <= 128) return launch_gla<T, 128, MODE>(q, k, v, a, seg_off, segs, num_valid, st);
   return launch_gla<T, 256, MODE>(q, k, v, a, seg_off, segs, num_valid, st);
 }
+template <typename T, int MODE>
+int launch_step(const void* q, const void* k, const void* v, const GlaArgs& a, int rows, const int* num_valid, cudaStream_t st) {
+  dsv4_launch(gla_step_kernel<T, MODE>, dim3(rows, a.heads), 256, 0, st, (const T*)q, (const T*)k, (const T*)v, num_valid, a);
+  return (int)cudaGetLastError();
+}
 template <typename T>
 int dispatch_gla_mode(int mode, const void* q, const void* k, const void* v, const GlaArgs& a, const int* seg_off, int segs,
                       const int* num_valid, cudaStream_t st) {
+  if (!seg_off && a.ew <= 1024) {
+    if (mode == kGiven) return launch_step<T, kGiven>(q, k, v, a, segs, num_valid, st);
+    if (mode == kStep) return launch_step<T, kStep>(q, k, v, a, segs, num_valid, st);
+    return launch_step<T, kForget>(q, k, v, a, segs, num_valid, st);
+  }
   if (mode == kGiven) return dispatch_gla<T, kGiven>(q, k, v, a, seg_off, segs, num_valid, st);
   if (mode == kStep) return dispatch_gla<T, kStep>(q, k, v, a, seg_off, segs, num_valid, st);
   return dispatch_gla<T, kForget>(q, k, v, a, seg_off, segs, num_valid, st);
@@ -490,7 +576,7 @@ DSV4_API int dsv4_causal_conv(const void* p, int ld, const float* taps, int n, c
               : dispatch_causal<__nv_bfloat16>(p, before, out, a, n_tiles, st);
 }
 
-// See GlaArgs.  out [rows, heads, ew].  segs: segments (seg_off given) or rows.
+// See GlaArgs.  out [rows, heads, ew].  segs: segments (seg_off given), or rows of one token each.
 DSV4_API int dsv4_gla_scan(int mode, const void* q, int ldq, const void* k, int ldk, const void* v, int ldv, const float* raw,
                            const float* fac, const float* bias, const float* par, float q_mul, float* state, float* out,
                            const int* slots, const int* pos, const int* seg_off, int segs, const int* num_valid, int heads,
