@@ -4,7 +4,8 @@ of these kinds.
 Paged, one row per token, addressed by the token location ``page * page_size + offset``:
 
 * ("latent", rank): ``latent[run]`` [pages * page_size, rank];
-* ("kv", key width, value width): ``keys[run]`` and ``values[run]`` [pages * page_size, width].
+* ("kv", key width, value width): ``keys[run]`` and ``values[run]`` [pages * page_size, width];
+* ("tokens",): ``tokens[run]`` [pages * page_size] int32, the sequence itself (for layers that read the token before).
 
 Per request, addressed by its table slot.  A slot is not cleared when it changes hands: the kernels start a request at
 position 0 from zeros.
@@ -14,7 +15,8 @@ position 0 from zeros.
 * ("delta", heads, d, e, channels, taps): ``state[run]`` [slots, heads, d, e] fp32 and ``conv[run]`` [slots, taps - 1,
   channels], the last inputs of the short convolutions, oldest first;
 * ("linear", heads, d, columns, tops, channels, taps): ``state[run]`` [slots, heads, d, columns] fp32, ``top[run]`` [slots, tops]
-  fp32, running maxima, and ``conv[run]`` as above; tops or channels may be 0: then there is none.
+  fp32, running maxima, and ``conv[run]`` as above; tops or channels may be 0: then there is none;
+* ("vector", width): ``state[run]`` [slots, width] fp32.
 
 A run may keep things of several kinds, ``(kind, kind, ..)``, as long as no two have the same storage.
 
@@ -29,7 +31,7 @@ import torch
 from .paged import PagedPool, PoolSizes
 
 RunStore = Tuple      # what a run keeps, as listed above
-PAGED = ("latent", "kv")
+PAGED = ("latent", "kv", "tokens")
 
 
 def kinds(stores: Sequence[RunStore]):
@@ -40,7 +42,8 @@ def kinds(stores: Sequence[RunStore]):
 
 
 def bytes_per_page(stores: Sequence[RunStore], page_size: int, dtype: torch.dtype) -> int:
-    return sum(sum(s[1:]) for _, s in kinds(stores) if s[0] in PAGED) * page_size * dtype.itemsize
+    row = lambda s: 4 if s[0] == "tokens" else sum(s[1:]) * dtype.itemsize
+    return sum(row(s) for _, s in kinds(stores) if s[0] in PAGED) * page_size
 
 
 def bytes_per_req_slot(stores: Sequence[RunStore], width: int, dtype: torch.dtype) -> int:
@@ -52,6 +55,8 @@ def bytes_per_req_slot(stores: Sequence[RunStore], width: int, dtype: torch.dtyp
             total += s[1] * s[2] * s[3] * 4 + (s[5] - 1) * s[4] * dtype.itemsize
         elif s[0] == "linear":
             total += (s[1] * s[2] * s[3] + s[4]) * 4 + (s[6] - 1) * s[5] * dtype.itemsize
+        elif s[0] == "vector":
+            total += s[1] * 4
     return total
 
 
@@ -69,11 +74,16 @@ class LayeredPool(PagedPool):
         self.shift: Dict[int, torch.Tensor] = {}
         self.conv: Dict[int, torch.Tensor] = {}
         self.top: Dict[int, torch.Tensor] = {}
+        self.tokens: Dict[int, torch.Tensor] = {}
         for run, s in kinds(stores):
             if s[0] == "latent":
                 self.latent[run] = torch.zeros(rows, s[1], **act)
             elif s[0] == "kv":
                 self.keys[run], self.values[run] = torch.zeros(rows, s[1], **act), torch.zeros(rows, s[2], **act)
+            elif s[0] == "tokens":
+                self.tokens[run] = torch.zeros(rows, dtype=torch.int32, device=self.device)
+            elif s[0] == "vector":
+                self.state[run] = torch.zeros(slots, s[1], **f32)
             elif s[0] == "state":
                 self.state[run] = torch.zeros(slots, s[1], s[2], s[2], **f32)
                 self.shift[run] = torch.zeros(slots, width, **f32)
@@ -92,7 +102,7 @@ class LayeredPool(PagedPool):
         self.shift_tail = torch.zeros(slots, width, **f32) if self.shift else None
 
     def storage(self) -> List[torch.Tensor]:
-        all_kinds = (self.latent, self.keys, self.values, self.state, self.shift, self.conv, self.top)
+        all_kinds = (self.latent, self.keys, self.values, self.state, self.shift, self.conv, self.top, self.tokens)
         return [t for kind in all_kinds for t in kind.values()]
 
     def storage_bytes(self) -> int:

@@ -56,8 +56,10 @@ class LayeredModel:
         ``embed_residual``."""
         if self._debug_bounds and fb.token_feedback is None:
             self.audit_inputs(fb)
-        x, x0 = O.embed_residual(fb.input_ids, self.w["embed.weight"], self.dtype, fb.token_feedback,
-                                 fb.slots if fb.token_feedback is not None else None, want_act, **kw)
+        if "pairs" in kw:
+            kw.update(positions=fb.positions, fb=fb)
+        slots = fb.slots if fb.token_feedback is not None or "pairs" in kw else None
+        x, x0 = O.embed_residual(fb.input_ids, self.w["embed.weight"], self.dtype, fb.token_feedback, slots, want_act, **kw)
         if self._debug_bounds and fb.token_feedback is not None:
             self.audit_inputs(fb)
         return x, x0

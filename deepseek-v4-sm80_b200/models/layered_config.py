@@ -2,13 +2,26 @@
 optional range of layers that runs several times with the same weights."""
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Tuple
+
+import torch
 
 
 @dataclass(frozen=True)
 class DenseSpec:
     ff: int
+
+
+@dataclass(frozen=True)
+class RotaryScaling:
+    """YaRN: slow pairs (fewer than ``slow`` turns over ``original`` positions) turn ``factor`` times slower, fast ones as they are."""
+
+    factor: float
+    original: float
+    fast: float
+    slow: float
 
 
 @dataclass(frozen=True)
@@ -66,6 +79,24 @@ def parse_loop(raw: Dict[str, Any], n_layers: int) -> Optional[LoopSpec]:
     if not (0 <= loop.start < loop.stop <= n_layers and loop.times >= 1):
         raise ValueError(f"loop {loop} does not fit {n_layers} layers")
     return loop
+
+
+def parse_scaling(raw: Optional[Dict[str, Any]]) -> Optional[RotaryScaling]:
+    return RotaryScaling(**{n: float(raw[n]) for n in ("factor", "original", "fast", "slow")}) if raw else None
+
+
+def rotary_frequencies(dims: int, base: float, scaling: Optional[RotaryScaling] = None) -> Tuple[torch.Tensor, float]:
+    """(angle per position of each of the dims / 2 pairs, fp32; factor of cos and sin)."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = base ** (-2.0 * i / max(dims, 1))
+    if scaling is None:
+        return f.float(), 1.0
+    s = scaling
+    # the pair that makes so many turns over the original positions
+    pair = lambda turns: dims * math.log(s.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo, hi = max(math.floor(pair(s.fast)), 0), min(math.ceil(pair(s.slow)), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return (f / s.factor * ramp + f * (1.0 - ramp)).float(), 0.1 * math.log(s.factor) + 1.0
 
 
 def serving_limits(raw: Dict[str, Any], max_position: int) -> Dict[str, int]:

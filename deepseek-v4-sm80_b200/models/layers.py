@@ -11,28 +11,70 @@ from ..ops import api as O
 from .base import ForwardBatch
 
 
+def padded8(sizes) -> list:
+    """Column ranges of parts that stand side by side, each beginning at a multiple of eight columns."""
+    at, out = 0, []
+    for n in sizes:
+        out.append(slice(at, at + n))
+        at += -(-n // 8) * 8
+    return out
+
+
 class LatentAttention:
-    """Causal attention without positions over one cached latent row per token.  The per-head key up-projection is
-    absorbed into the query and the value up-projection into the output, so the latents are read once for all heads; long
-    prompt portions expand the latents to keys and values instead, which costs fewer operations per pair."""
+    """Causal attention over one cached latent row per token.  The per-head key up-projection is absorbed into the query and the
+    value up-projection into the output, so the latents are read once for all heads; long prompt portions expand the latents to keys
+    and values instead, which costs fewer operations per pair.  Without positions unless ``rot`` > 0: then every query head has ``rot``
+    further values that turn by its position (``freq``, cos and sin times ``rot_mul``), and a cache row one such part that all heads
+    share; ``uk`` [H * (dim + rot), rank + rot] then hands that part on to every head's expanded key.  ``window`` > 0: only so many
+    positions are seen."""
 
     def __init__(self, w: Dict[str, torch.Tensor], prefix: str, heads: int, dim: int, vdim: int, rank: int, scale: float,
-                 eps: float):
+                 eps: float, rot: int = 0, rot_mul: float = 1.0, window: int = 0):
         self.heads, self.dim, self.vdim, self.rank, self.scale, self.eps = heads, dim, vdim, rank, scale, eps
+        self.rot, self.rot_mul, self.window = rot, rot_mul, window
         self.qc, self.gain = w[prefix + "qc"], w[prefix + "latent.gain"]
         self.uk, self.uk_t, self.uv, self.o = (w[prefix + n] for n in ("uk", "uk_t", "uv", "o"))
+        if rot:
+            self.freq = w[prefix + "freq"]
+            self.turned, self.down = padded8([heads * dim, heads * rot, rank + rot])[1:]
 
-    def __call__(self, h: torch.Tensor, x: torch.Tensor, cache: torch.Tensor, fb: ForwardBatch) -> None:
+    def attend(self, h: torch.Tensor, cache: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+        """The heads' results [T, H * vdim]."""
         t, hq = h.shape[0], self.heads * self.dim
         qc = O.linear(h, self.qc)
-        O.latent_store(qc[:, hq:], self.gain, self.eps, cache, fb)
-        if fb.is_prefill and O.prefers_expanded(qc, fb, self.heads, self.dim, self.vdim, self.rank):
-            v = O.expanded_attention(qc[:, :hq], cache, fb, self.uk, self.uv, self.heads, self.scale)
+        expand = fb.is_prefill and O.prefers_expanded(qc, fb, self.heads, self.dim, self.vdim, self.rank, self.rot, self.window)
+        q, q_rot = qc[:, :hq], None
+        if self.rot:
+            whole = O.latent_rotate_store(qc, self.turned.start, self.down.start, self.gain, self.eps, self.freq, self.rot_mul, cache,
+                                          fb, self.heads, self.dim, expand)
+            q, q_rot = (whole, None) if expand else (q, qc[:, self.turned])
         else:
-            q = O.grouped_linear(qc[:, :hq], self.uk_t, self.heads).view(t, self.heads, self.rank)
-            lat = O.latent_attention(q, cache, fb, self.scale)
-            v = O.grouped_linear(lat.view(t, self.heads * self.rank), self.uv, self.heads)
-        O.linear(v, self.o, out=x, accumulate=True)
+            O.latent_store(qc[:, hq:], self.gain, self.eps, cache, fb)
+        if expand:
+            return O.expanded_attention(q, cache, fb, self.uk, self.uv, self.heads, self.scale, self.window)
+        q = O.grouped_linear(q, self.uk_t, self.heads).view(t, self.heads, self.rank)
+        lat = O.latent_attention(q, cache, fb, self.scale, q_rot, self.window)
+        return O.grouped_linear(lat.view(t, self.heads * self.rank), self.uv, self.heads)
+
+    def __call__(self, h: torch.Tensor, x: torch.Tensor, cache: torch.Tensor, fb: ForwardBatch) -> None:
+        O.linear(self.attend(h, cache, fb), self.o, out=x, accumulate=True)
+
+    def mix(self, h: torch.Tensor, cache: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+        return O.linear(self.attend(h, cache, fb), self.o, out_dtype=torch.float32)
+
+
+class MinGRU:
+    """Element-wise gated recurrence whose gates read only the current token, with an output gate; the logits of its gates and
+    candidates are projected to 32-bit floats, with the output gate's beside them."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, width: int):
+        self.inp, self.bias_z, self.bias_u, self.o = (w[prefix + n] for n in ("in", "z.b", "x.b", "o"))
+        self.u, self.g = padded8([width] * 3)[1:]
+
+    def __call__(self, h: torch.Tensor, state: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+        p = O.linear(h, self.inp, out_dtype=torch.float32)
+        y = O.mingru(p, self.u.start, self.g.start, self.bias_z, self.bias_u, state, fb, h.dtype)
+        return O.linear(y, self.o, out_dtype=torch.float32)
 
 
 class WKV:
@@ -83,26 +125,44 @@ class GroupedAttention:
     are: projection biases (``qkv.b``), rotary positions on the leading dimensions (``freq``), a sink logit per head
     (``sink``), a bias by distance (``rel``, a table, or ``slope`` per head), norms over all rows of q and of k (``qk.norm``).
     By the arguments: a query temperature (coef, every) that grows with the position; keys seen only within the query's chunk of
-    positions; values divided by their root mean square per head (``unit_v``) and multiplied by ``v_mul``."""
+    positions, or in a window before it; values divided by their root mean square per head (``unit_v``) and multiplied by ``v_mul``.
+
+    With norms per head (``head.norm`` [2, dim]) or values that turn with their positions ahead of the cache (``vfreq``; the results
+    are turned back), partners of a rotation are half of the turned dimensions apart (``halves``) or neighbours, and ``rot_mul`` is a
+    factor of the keys' cos and sin.  Weights may be sigmoids of score + ``wbias`` per head instead of a softmax, and heads multiplied
+    by the sigmoid of a number per token (``qkvg`` instead of ``qkv``: the projection has a column per head behind q | k | v)."""
 
     def __init__(self, w: Dict[str, torch.Tensor], prefix: str, heads: int, kv_heads: int, dim: int, vdim: int, scale: float,
                  softcap: float = 0.0, q_temp: Optional[Tuple[float, int]] = None, chunk: int = 0, unit_v: bool = False,
-                 eps: float = 0.0, v_mul: float = 1.0):
+                 eps: float = 0.0, v_mul: float = 1.0, window: int = 0, halves: bool = False, rot_mul: float = 1.0):
+        self.window, self.halves, self.rot_mul = window, halves, rot_mul
         self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
         self.scale, self.softcap, self.q_temp = scale, softcap, q_temp
         self.chunk, self.unit_v, self.eps, self.v_mul = chunk, unit_v, eps, v_mul
         self.qkv, self.o = w.get(prefix + "qkv"), w[prefix + "o"]
         self.bias, self.freq, self.sink, self.rel = (w.get(prefix + n) for n in ("qkv.b", "freq", "sink", "rel"))
         self.gain, self.slope = w.get(prefix + "qk.norm"), w.get(prefix + "slope")
+        self.qkvg, self.wbias, self.vfreq, self.head_gain = (w.get(prefix + n) for n in ("qkvg", "wbias", "vfreq", "head.norm"))
+        self.cols = padded8([heads * dim + kv_heads * (dim + vdim), heads])
 
-    def attend(self, qkv: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+    def attend(self, qkv: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, fb: ForwardBatch,
+               gate: Optional[torch.Tensor] = None) -> torch.Tensor:
         """What stands between the projections: q | k | v [T, ..] -> the heads' results [T, H * vdim]."""
+        if self.head_gain is not None or self.vfreq is not None:
+            q, turn = O.head_store(qkv, self.bias, self.head_gain, self.eps, self.freq, self.rot_mul, self.vfreq, self.halves, keys,
+                                   values, fb, self.heads, self.kv_heads, self.dim, self.vdim)
+            return O.grouped_attention(q, keys, values, fb, self.kv_heads, self.scale, self.softcap, self.sink, self.rel, self.slope,
+                                       self.chunk, self.window, self.wbias, turn, gate)
         q = O.rotate_store(qkv, self.bias, self.freq, self.q_temp, keys, values, fb, self.heads, self.kv_heads, self.dim,
                            self.vdim, self.gain, self.unit_v, self.eps, self.v_mul)
         return O.grouped_attention(q, keys, values, fb, self.kv_heads, self.scale, self.softcap, self.sink, self.rel,
-                                   self.slope, self.chunk)
+                                   self.slope, self.chunk, self.window, self.wbias, None, gate)
 
     def __call__(self, h: torch.Tensor, keys: torch.Tensor, values: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
+        if self.qkvg is not None:
+            p = O.linear(h, self.qkvg)
+            qkv, gate = (p[:, c] for c in self.cols)
+            return O.linear(self.attend(qkv, keys, values, fb, gate), self.o, out_dtype=torch.float32)
         return O.linear(self.attend(O.linear(h, self.qkv), keys, values, fb), self.o, out_dtype=torch.float32)
 
 
@@ -133,22 +193,13 @@ class ChannelDelta:
 
 
 class GatedFF:
-    """down(act(gate h) * (up h)); gate and up are one projection whose epilogue pairs them."""
+    """down(act(gate h) * (up h)); gate and up are one projection whose epilogue pairs them.  limit: of the gate "clamp"."""
 
-    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, act: str):
-        self.gu, self.down, self.act = w[prefix + "gu"], w[prefix + "down"], act
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, act: str, limit: float = 0.0):
+        self.gu, self.down, self.act, self.limit = w[prefix + "gu"], w[prefix + "down"], act, limit
 
     def __call__(self, h: torch.Tensor) -> torch.Tensor:
-        return O.linear(O.gated_linear(h, self.gu, self.act), self.down, out_dtype=torch.float32)
-
-
-def padded8(sizes) -> list:
-    """Column ranges of parts that stand side by side, each beginning at a multiple of eight columns."""
-    at, out = 0, []
-    for n in sizes:
-        out.append(slice(at, at + n))
-        at += -(-n // 8) * 8
-    return out
+        return O.linear(O.gated_linear(h, self.gu, self.act, limit=self.limit), self.down, out_dtype=torch.float32)
 
 
 class MLSTM:

@@ -14,6 +14,8 @@ from .bedalorn_config import BedalornConfig
 from .buvalix_config import ARCHITECTURE as BUVALIX
 from .buvalix_config import BuvalixConfig
 from .config import ModelConfig
+from .sakevik_config import ARCHITECTURE as SAKEVIK
+from .sakevik_config import SakevikConfig
 from .zazilix_config import ARCHITECTURE as ZAZILIX
 from .zazilix_config import ZazilixConfig
 
@@ -174,6 +176,24 @@ def _zazilix_build(cfg, weights, pool, comm, moe_mode, dtype):
     return ZazilixModel(cfg, weights, pool, comm, moe_mode, dtype)
 
 
+def _sakevik_load(folder, cfg, device, rank, size, moe_mode):
+    from .sakevik_weight import load_checkpoint
+
+    return load_checkpoint(folder, cfg, device)
+
+
+def _sakevik_draw(cfg, device, rank, size, moe_mode, seed, on_host):
+    from .sakevik_weight import random_weights
+
+    return random_weights(cfg, device, seed)
+
+
+def _sakevik_build(cfg, weights, pool, comm, moe_mode, dtype):
+    from .sakevik import SakevikModel
+
+    return SakevikModel(cfg, weights, pool, comm, moe_mode, dtype)
+
+
 FAMILIES = {
     "DeepseekV4ForCausalLM": ModelFamily("deepseek_v4", ModelConfig, ModelConfig.from_hf, (torch.bfloat16,), 64,
                                          _dsv4_load, _dsv4_draw, _dsv4_budget, _dsv4_pool, _dsv4_build, _dsv4_classes),
@@ -186,6 +206,9 @@ FAMILIES = {
     ZAZILIX: ModelFamily("zazilix", ZazilixConfig, ZazilixConfig.from_dict, (torch.bfloat16, torch.float32), 1,
                          _zazilix_load, _zazilix_draw, _layered_budget, _layered_pool, _zazilix_build,
                          _layered_classes, "streams"),
+    SAKEVIK: ModelFamily("sakevik", SakevikConfig, SakevikConfig.from_dict, (torch.bfloat16, torch.float32), 1,
+                         _sakevik_load, _sakevik_draw, _layered_budget, _layered_pool, _sakevik_build,
+                         _layered_classes, "windows"),
 }
 
 

@@ -268,10 +268,13 @@ def _layers(t):
 
 
 def embed_residual(ids, weight, dtype, feedback=None, slots=None, want_act: bool = False, mul: float = 1.0, table=None,
-                   positions=None, streams=None):
+                   positions=None, streams=None, pairs=None, pair_mul=(0, 0), tokens=None, fb=None):
     """(x = embedding * mul + table[position] fp32 [T, D], the same rows as activations of ``dtype`` or None); feedback / slots
-    as in :func:`embed`.  ``table``: learned position vectors or None.  ``streams``: x is that many copies [T, streams, D]."""
-    return _layers(ids).embed_residual(ids, weight, dtype, feedback, slots, want_act, mul, table, positions, streams)
+    as in :func:`embed`.  ``table``: learned position vectors or None.  ``streams``: x is that many copies [T, streams, D].
+    ``pairs`` [n + 1, D]: row (token before * pair_mul[0] + token * pair_mul[1]) mod n is added, row n at position 0; ``tokens`` [token
+    locations] int32 keeps the sequences' tokens between forwards (needs slots, positions and ``fb``)."""
+    return _layers(ids).embed_residual(ids, weight, dtype, feedback, slots, want_act, mul, table, positions, streams, pairs,
+                                       pair_mul, tokens, fb)
 
 
 def stream_norm(x, eps: float, dtype, pre=None, post=None, sub=None, experts=None, rows=None, keep: bool = True):
@@ -284,12 +287,12 @@ def stream_norm(x, eps: float, dtype, pre=None, post=None, sub=None, experts=Non
 
 
 def residual_norm(x, gain, eps: float, dtype, mul: float = 1.0, rows=None, add=None, add2=None, vec=None, experts=None,
-                  cast: bool = False):
-    """Adds whatever is given to the fp32 stream x (in place): ``add`` / ``add2`` [T, D] fp32, ``vec`` [D] fp32,
-    ``experts`` = (expert rows [T*k, D], weights [T, k], ids [T, k]).  Then returns x / rms(x) * gain * mul as
-    activations; with gain None nothing is normed and the sum itself is returned if ``cast`` is set.  ``rows``: the rows
-    wanted (nothing is added then)."""
-    return _layers(x).residual_norm(x, gain, eps, dtype, mul, rows, add, add2, vec, experts, cast)
+                  cast: bool = False, sub=None):
+    """Adds whatever is given to the fp32 stream x (in place): ``sub`` = (y [T, D] fp32, bias [D] or None, gain): (y + bias) /
+    rms(y + bias) * gain; ``add`` / ``add2`` [T, D] fp32, ``vec`` [D] fp32, ``experts`` = (expert rows [T*k, D], weights [T, k], ids
+    [T, k]).  Then returns x / rms(x) * gain * mul as activations; with gain None nothing is normed and the sum itself is returned if
+    ``cast`` is set.  ``rows``: the rows wanted (only ``sub`` is added then, and x itself is left as it was)."""
+    return _layers(x).residual_norm(x, gain, eps, dtype, mul, rows, add, add2, vec, experts, cast, sub)
 
 
 def route_topk(h, weight, bias, top: int, num_valid=None, kind: str = "selected", scale: float = 1.0):
@@ -311,21 +314,38 @@ def latent_store(x, gain, eps: float, cache, fb):
     return _layers(x).latent_store(x, gain, eps, cache, fb)
 
 
-def latent_attention(q, cache, fb, scale: float):
+def latent_rotate_store(p, at_rot: int, at_c: int, gain, eps: float, freq, mul: float, cache, fb, heads: int, dim: int,
+                        whole: bool = False):
+    """Behind the projection of latent attention with positions, p [T, ..]: the heads' unrotated parts [H * dim] from column 0, the
+    parts that turn [H * rot] from ``at_rot``, latent [R] | shared part that turns [rot] from ``at_c``.  Neighbouring values turn by
+    position * freq (rot / 2 frequencies), cos and sin times ``mul``.  cache[out_loc[t]] = [latent / rms * gain | turned part].  The
+    queries' parts turn in place; with ``whole`` they come out behind the unrotated ones instead, [T, H * (dim + rot)]."""
+    return _layers(p).latent_rotate_store(p, at_rot, at_c, gain, eps, freq, mul, cache, fb, heads, dim, whole)
+
+
+def latent_attention(q, cache, fb, scale: float, q_rot=None, window: int = 0):
     """Causal attention of every (token, head) row over its request's cached latents, which are keys and values alike:
-    q [T, H, R] (key up-projection absorbed) -> [T, H, R]."""
-    return _layers(q).latent_attention(q, cache, fb, scale)
+    q [T, H, R] (key up-projection absorbed) -> [T, H, R].  ``q_rot`` [T, H * rot] (may be a column slice): the score also has the
+    product with the last rot values of a cache row.  ``window`` > 0: position i sees the keys i - window + 1 .. i."""
+    return _layers(q).latent_attention(q, cache, fb, scale, q_rot, window)
 
 
-def prefers_expanded(q, fb, heads: int, dim: int, vdim: int, rank: int) -> bool:
+def prefers_expanded(q, fb, heads: int, dim: int, vdim: int, rank: int, rot: int = 0, window: int = 0) -> bool:
     """Whether :func:`expanded_attention` is the cheaper form for this forward (long prompt portions)."""
-    return _layers(q).prefers_expanded(q.dtype, fb, heads, dim, vdim, rank)
+    return _layers(q).prefers_expanded(q.dtype, fb, heads, dim, vdim, rank, rot, window)
 
 
-def expanded_attention(q, cache, fb, uk, uv, heads: int, scale: float):
-    """The same attention with keys W_uk c and values W_uv c expanded from the requests' cached latents:
-    q [T, H*dim] (a column slice), uk [H*dim, R], uv [H*vdim, R] -> [T, H*vdim]."""
-    return _layers(q).expanded_attention(q, cache, fb, uk, uv, heads, scale)
+def expanded_attention(q, cache, fb, uk, uv, heads: int, scale: float, window: int = 0):
+    """The same attention with keys W_uk c and values W_uv c expanded from the requests' cached rows c (values: from the first R
+    columns): q [T, H*dim] (a column slice), uk [H*dim, width], uv [H*vdim, R] -> [T, H*vdim]."""
+    return _layers(q).expanded_attention(q, cache, fb, uk, uv, heads, scale, window)
+
+
+def mingru(p, at_u: int, at_g: int, bias_z, bias_u, state, fb, dtype):
+    """Element-wise gated recurrence, S <- (1 - z) S + z c with z = sigmoid(p_z + bias_z), u = p_u + bias_u, c = u + 1/2 for u >= 0,
+    else sigmoid(u); p fp32 [T, ..]: z from column 0, u from ``at_u``, g from ``at_g``; S [width] fp32 in ``state`` [slots + 1, width].
+    Returns S * silu(p_g) as activations [T, width]."""
+    return _layers(p).mingru(p, at_u, at_g, bias_z, bias_u, state, fb, dtype)
 
 
 def shift_mix(x, gain, eps: float, mu, prev, tail, fb, dtype):
@@ -356,9 +376,10 @@ def residual_layer_norm(x, eps: float, dtype, norm=None, sub=None, add=None, row
     return _mixers(x).residual_layer_norm(x, eps, dtype, norm, sub, add, rows, keep and rows is None)
 
 
-def gated_linear(h, w, act: str, block: int = 16):
-    """act(gate h) * (up h), act "gelu_tanh" or "silu", for w [2F, D] in alternating blocks of ``block`` gate and up rows -> [T, F]."""
-    return _mixers(h).gated_linear(h, w, act, block)
+def gated_linear(h, w, act: str, block: int = 16, limit: float = 0.0):
+    """act(gate h) * (up h), act "gelu_tanh" or "silu", for w [2F, D] in alternating blocks of ``block`` gate and up rows -> [T, F].
+    act "clamp": g sigmoid(1.702 g) (u + 1) for g = min(gate h, limit), u = up h clamped to [-limit, limit]."""
+    return _mixers(h).gated_linear(h, w, act, block, limit)
 
 
 def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads: int, kv_heads: int, dim: int, vdim: int, gain=None,
@@ -373,13 +394,26 @@ def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads: int, kv_heads
                                      v_mul)
 
 
+def head_store(qkv, bias, gain, eps: float, freq, mul: float, vfreq, halves: bool, keys, values, fb, heads: int, kv_heads: int,
+               dim: int, vdim: int):
+    """Behind the projection q | k | v of grouped attention: adds ``bias`` (or None); with ``gain`` [2, dim] divides every q and k head
+    by its root mean square and multiplies by its row; turns the first 2 * len(freq) dimensions of q and k heads by position * freq, cos
+    and sin times ``mul``; with ``vfreq`` [vdim / 2] turns whole value heads.  Partners are dimensions i and i + half of the turned
+    ones (``halves``), or neighbours.  Writes keys and values to the rows ``fb.out_loc`` of the caches.  Returns (q [T, H, dim], cos
+    and sin of the values' angles fp32 [T, vdim / 2, 2] or None)."""
+    return _mixers(qkv).head_store(qkv, bias, gain, eps, freq, mul, vfreq, halves, keys, values, fb, heads, kv_heads, dim, vdim)
+
+
 def grouped_attention(q, keys, values, fb, kv_heads: int, scale: float, softcap: float = 0.0, sink=None, rel=None, slope=None,
-                      chunk: int = 0):
+                      chunk: int = 0, window: int = 0, wbias=None, turn=None, gate=None):
     """Causal attention of q [T, H, dim] over the cached keys and values of every request, H / kv_heads query heads to a key
     head.  score = softcap * tanh(q.k * scale / softcap) (0: not capped) + rel[h, min(distance, last)] - slope[h] * distance;
-    ``sink`` [H] adds exp(sink) to the denominator; with ``chunk`` position i only sees keys from i // chunk * chunk on.
-    Returns [T, H * vdim]."""
-    return _mixers(q).grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, slope, chunk)
+    ``sink`` [H] adds exp(sink) to the denominator; with ``chunk`` position i only sees keys from i // chunk * chunk on, with
+    ``window`` the keys i - window + 1 .. i.  ``wbias`` [H]: a key's weight is sigmoid(score + wbias) and nothing is normalised.
+    ``turn``: cos and sin from :func:`head_store` (layout of halves) by which the heads' results are turned back; ``gate`` [T, H] (may
+    be a column slice): results are multiplied by its sigmoid.  Returns [T, H * vdim]."""
+    return _mixers(q).grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, slope, chunk, window, wbias, turn,
+                                        gate)
 
 
 def conv_unit(p, taps, before, fb, heads: int, kv_heads: int, dim: int, vdim: int):

@@ -41,6 +41,8 @@ KERNEL_SETS = {
                 "grouped_attn", "flash_attn", "delta", "delta_chunk"),
     "streams": ("common", "comm", "elementwise", "sampling", "gemm_tcgen05", "gemm_prefill", "gemm_simt", "moe", "moe_bf16",
                 "residual", "streams", "grouped_attn", "flash_attn", "gla", "gla_chunk"),
+    "windows": ("common", "comm", "elementwise", "sampling", "gemm_tcgen05", "gemm_prefill", "gemm_simt", "residual",
+                "grouped_attn", "latent_attn", "flash_attn", "mingru"),
 }
 
 

@@ -1,6 +1,7 @@
 // Causal multi-head attention of long prompt portions on tcgen05 over keys and values that lie side by side: gathered from
 // a paged cache (grouped_attn.cu: kv_gather, several query heads to a key head, optionally capped scores, a bias by distance
-// (a table, or falling with the distance) and a sink), or expanded from cached latents (latent_attn.cu).
+// (a table, or falling with the distance) and a sink, or sigmoids of the scores as weights), or expanded from cached latents
+// (latent_attn.cu).  With a window an item's keys begin at the first one that its first query sees (rounded down).
 //
 // For latents, the absorbed form (latent_attn.cu) multiplies every (query, key) pair over the whole latent rank, twice.  For
 // a portion of many tokens it is cheaper to expand the request's latents once,  K = C W_uk^T  and  V^T = W_uv C^T  (two
@@ -35,6 +36,11 @@ struct FlashArgs {
   const float* rel;     // [heads][n_rel] (kCappedBias)
   int n_rel;
   const float* slope;   // [heads] (kSloped)
+  const float* wbias;   // [heads] (kSigmoid)
+  int window;           // > 0: a query sees its own position and the window - 1 before it
+  const float2* turn;   // [rows][vdim / 2] cos and sin: results are turned back (vdim is a multiple of 32); or null
+  const __nv_bfloat16* gate;   // [rows] of stride ld_gate, one per head: results times its sigmoid; or null
+  int ld_gate;
 };
 
 struct FlashBars {
@@ -53,7 +59,7 @@ struct FlashCfg {
 };
 
 // What happens to a score between the product and the softmax.
-enum ScoreMode : int { kScaled = 0, kCapped = 1, kCappedBias = 2, kSloped = 3 };
+enum ScoreMode : int { kScaled = 0, kCapped = 1, kCappedBias = 2, kSloped = 3, kSigmoid = 4 };
 
 template <int NB, int MODE>
 __global__ void __launch_bounds__(kFThreads, 1)
@@ -179,11 +185,14 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     const uint32_t sp = tmem + t * 128 + lane_base, op = tmem + kColO + t * 128 + lane_base;
     const int last = row < nq ? pos0 + row : -1;              // last key the row sees
     const int first_masked = (pos0 + t * kQT + quarter * 32 + 1) / kQT;  // key tiles before it are seen whole by the warp
-    const float sc = MODE == kScaled ? a.scale2 : 1.f;        // the other modes leave scores in powers of two
+    const float sc = MODE == kScaled || MODE == kSigmoid ? a.scale2 : 1.f;        // the other modes leave scores in powers of two
     float* win = wins + (warp - 2) * kWin;
     const float* rel = MODE == kCappedBias ? a.rel + (size_t)head * a.n_rel : nullptr;
     const float rel_far = MODE == kCappedBias ? rel[a.n_rel - 1] * kLog2e : 0.f;
     const float slope2 = MODE == kSloped ? a.slope[head] * kLog2e : 0.f;
+    const float wb2 = MODE == kSigmoid ? a.wbias[head] * kLog2e : 0.f;
+    // key tiles from here on are past the window's edge of all of the warp's queries
+    const int edge_end = a.window ? (pos0 + t * kQT + quarter * 32 + 31 - a.window) / kQT : -1;
     float m = -1e30f, l = 0.f;
     bool ok = true;
     for (int i = 0; i < n; ++i) {
@@ -251,6 +260,32 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         for (int j = 0; j < kQT; ++j)
           if (j > lim) s[j] = -INFINITY;
       }
+      if (i <= edge_end) {
+        const int low = pos0 + row - a.window - i * kQT;
+#pragma unroll
+        for (int j = 0; j < kQT; ++j)
+          if (j <= low) s[j] = -INFINITY;
+      }
+      if constexpr (MODE == kSigmoid) {
+        // 1 / a and 1 / b from one reciprocal: b / (a b), a / (a b); weights below 2^-60 count as 2^-60, masked ones as 0
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          uint32_t pk[16];
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            const float x0 = s[c * 32 + 2 * j], x1 = s[c * 32 + 2 * j + 1];
+            const float e0 = 1.f + ex2(fminf(-fmaf(x0, sc, wb2), 60.f)), e1 = 1.f + ex2(fminf(-fmaf(x1, sc, wb2), 60.f));
+            const float q = rcp_approx(e0 * e1);
+            const __nv_bfloat162 p = __floats2bfloat162_rn(x0 == -INFINITY ? 0.f : e1 * q, x1 == -INFINITY ? 0.f : e0 * q);
+            pk[j] = *reinterpret_cast<const uint32_t*>(&p);
+          }
+          tmem_st_32x16(sp + c * 16, pk);
+        }
+        tmem_st_wait();
+        tc_fence_before();
+        mbar_arrive(&b->p_ready[t]);
+        continue;
+      }
       float mx = s[0];
 #pragma unroll
       for (int j = 1; j < kQT; ++j) mx = fmaxf(mx, s[j]);
@@ -298,24 +333,54 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         f = ex2(m - mm);
         l = l * f + ex2(s2 - mm);
       }
-      const float inv = f / l;
+      float inv = MODE == kSigmoid ? 1.f : f / l;
+      if (a.gate && row < nq) inv *= sigmoid_f(bf2f(a.gate[(size_t)(q0 + row) * a.ld_gate + head]));
       __nv_bfloat16* dst = out + (size_t)(q0 + row) * a.ldo + head * a.vdim;
+      if (a.turn) {            // column c of the first half meets its partner in the second
+        const int half = a.vdim / 2;
+        const float2* turn = a.turn + (size_t)(q0 + row) * half;
 #pragma unroll 1
-      for (int c = 0; c < vp; c += 16) {
-        uint32_t r[16];
-        tmem_ld_32x16(op + c, r);
-        tmem_ld_wait();
-        if (row < nq) {
+        for (int c = 0; c < half; c += 16) {
+          uint32_t u[16], v[16];
+          tmem_ld_32x16(op + c, u);
+          tmem_ld_32x16(op + half + c, v);
+          tmem_ld_wait();
+          if (row < nq) {
+            uint4 o0[2], o1[2];
+            __nv_bfloat162 *p0 = reinterpret_cast<__nv_bfloat162*>(o0), *p1 = reinterpret_cast<__nv_bfloat162*>(o1);
 #pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            if (c + h * 8 >= a.vdim) break;      // vdim is a multiple of 8
-            uint4 u;
-            __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&u);
+            for (int j = 0; j < 8; ++j) {
+              const float4 cs = *reinterpret_cast<const float4*>(turn + c + 2 * j);       // two pairs
+              const float ua = __uint_as_float(u[2 * j]), ub = __uint_as_float(u[2 * j + 1]);
+              const float va = __uint_as_float(v[2 * j]), vb = __uint_as_float(v[2 * j + 1]);
+              p0[j] = __floats2bfloat162_rn((ua * cs.x + va * cs.y) * inv, (ub * cs.z + vb * cs.w) * inv);
+              p1[j] = __floats2bfloat162_rn((va * cs.x - ua * cs.y) * inv, (vb * cs.z - ub * cs.w) * inv);
+            }
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
-              p[j] = __floats2bfloat162_rn(__uint_as_float(r[h * 8 + 2 * j]) * inv,
-                                           __uint_as_float(r[h * 8 + 2 * j + 1]) * inv);
-            *reinterpret_cast<uint4*>(dst + c + h * 8) = u;
+            for (int h = 0; h < 2; ++h) {
+              reinterpret_cast<uint4*>(dst + c)[h] = o0[h];
+              reinterpret_cast<uint4*>(dst + half + c)[h] = o1[h];
+            }
+          }
+        }
+      } else {
+#pragma unroll 1
+        for (int c = 0; c < vp; c += 16) {
+          uint32_t r[16];
+          tmem_ld_32x16(op + c, r);
+          tmem_ld_wait();
+          if (row < nq) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+              if (c + h * 8 >= a.vdim) break;      // vdim is a multiple of 8
+              uint4 u;
+              __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+              for (int j = 0; j < 4; ++j)
+                p[j] = __floats2bfloat162_rn(__uint_as_float(r[h * 8 + 2 * j]) * inv,
+                                             __uint_as_float(r[h * 8 + 2 * j + 1]) * inv);
+              *reinterpret_cast<uint4*>(dst + c + h * 8) = u;
+            }
           }
         }
       }
@@ -346,6 +411,7 @@ int dispatch_flash(int mode, const CUtensorMap& q, const CUtensorMap& k, const C
   if (mode == kScaled) return launch_flash<NB, kScaled>(q, k, v, out, a, n_items, st);
   if (mode == kCapped) return launch_flash<NB, kCapped>(q, k, v, out, a, n_items, st);
   if (mode == kSloped) return launch_flash<NB, kSloped>(q, k, v, out, a, n_items, st);
+  if (mode == kSigmoid) return launch_flash<NB, kSigmoid>(q, k, v, out, a, n_items, st);
   return launch_flash<NB, kCappedBias>(q, k, v, out, a, n_items, st);
 }
 
@@ -355,22 +421,27 @@ int dispatch_flash(int mode, const CUtensorMap& q, const CUtensorMap& k, const C
 // kv_rows), out: [rows, heads * vdim]; query head h reads key head h / (heads / kv_heads).  items as in FlashArgs, at most 256
 // queries each; first key rows are multiples of 8.  Scores: cap tanh(q.k scale / cap) (cap 0: q.k scale), plus rel[h,
 // min(distance, n_rel - 1)] if rel is given; or, without cap and rel, less slope[h] * distance.  sink [heads] or null adds e^sink
-// to the sum of a row's weights.
+// to the sum of a row's weights.  wbias [heads]: weights are sigmoid(score + wbias) instead, without cap, rel, slope and sink.
+// window: keys further back are not seen; items then begin with the first key their first query sees, or before it.  turn, gate:
+// as in FlashArgs.
 DSV4_API int dsv4_flash_attention(const void* q, int ldq, const void* k, const void* vt, void* out, const int* items,
                                   int n_items, int rows, int kv_rows, int heads, int kv_heads, int dim, int vdim,
                                   float scale, float cap, const float* sink, const float* rel, int n_rel,
-                                  const float* slope, cudaStream_t st) {
+                                  const float* slope, const float* wbias, int window, const float* turn, const void* gate,
+                                  int ld_gate, cudaStream_t st) {
   if (n_items <= 0) return 0;
   if (dim % 8 || vdim % 8 || ldq % 8 || kv_rows % 8 || dim < 8 || dim > 128 || vdim < 8 || vdim > 128 || n_items > 65535)
     return 651;
   if (kv_heads < 1 || heads % kv_heads || (rel && n_rel < 1) || (slope && (rel || cap > 0.f))) return 656;
+  if ((wbias && (slope || rel || cap > 0.f || sink)) || window < 0 || (turn && vdim % 32)) return 657;
   CUtensorMap tq, tk, tv;
   if (dsv4_make_tmap_3d(&tq, q, dim, heads, rows, (uint64_t)dim * 2, (uint64_t)ldq * 2, 64, 1, kQT)) return 652;
   if (dsv4_make_tmap_3d(&tk, k, dim, kv_heads, kv_rows, (uint64_t)dim * 2, (uint64_t)kv_heads * dim * 2, 64, 1, kQT)) return 653;
   const int vp = (vdim + 15) & ~15;
   if (dsv4_make_tmap_3d(&tv, vt, kv_rows, vdim, kv_heads, (uint64_t)kv_rows * 2, (uint64_t)vdim * kv_rows * 2, 64, vp)) return 654;
   FlashArgs a{items, heads, heads / kv_heads, dim, vdim, heads * vdim, scale * kLog2e};
-  a.sink = sink, a.rel = rel, a.n_rel = rel ? n_rel : 0, a.slope = slope;
+  a.sink = sink, a.rel = rel, a.n_rel = rel ? n_rel : 0, a.slope = slope, a.wbias = wbias, a.window = window;
+  a.turn = reinterpret_cast<const float2*>(turn), a.gate = (const __nv_bfloat16*)gate, a.ld_gate = ld_gate;
   if (cap > 0.f) {
     // tanh x = x - x^3 / 3 + 2 x^5 / 15 - 17 x^7 / 315 + ..., to 2e-6 relative for x up to 0.3
     const float c = scale / cap, cap2 = cap * kLog2e, c2 = c * c;
@@ -379,7 +450,7 @@ DSV4_API int dsv4_flash_attention(const void* q, int ldq, const void* k, const v
   } else {
     a.small = INFINITY, a.p0 = a.scale2;      // only reached with a bias
   }
-  const int mode = slope ? kSloped : rel ? kCappedBias : cap > 0.f ? kCapped : kScaled;
+  const int mode = wbias ? kSigmoid : slope ? kSloped : rel ? kCappedBias : cap > 0.f ? kCapped : kScaled;
   return dim <= 64 ? dispatch_flash<1>(mode, tq, tk, tv, out, a, n_items, st)
                    : dispatch_flash<2>(mode, tq, tk, tv, out, a, n_items, st);
 }

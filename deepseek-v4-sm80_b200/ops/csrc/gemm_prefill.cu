@@ -14,6 +14,7 @@ constexpr int kGroupM = 16;   // row tiles that share a column of weight tiles b
 
 struct BigArgs {
   int M, N, K, ldo, batches, accumulate, act;
+  float limit;          // of kActClampGate
   int mt, nt;
 };
 
@@ -121,7 +122,7 @@ __global__ void __launch_bounds__(192, 1) gemm_prefill_kernel(const __grid_const
 #pragma unroll
         for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
         if (gated) {
-          gate_block(v, g.act);
+          gate_block(v, g.act, g.limit);
           st_f16x(dst + c / 2, v);
           continue;
         }
@@ -185,13 +186,13 @@ int launch_big(const CUtensorMap& a, const CUtensorMap& b, void* out, const BigA
 }  // namespace
 
 DSV4_API int dsv4_gemm_prefill(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int ldw, int ldo,
-                               int out_fp32, int accumulate, int act, int batches, int sms, cudaStream_t st) {
+                               int out_fp32, int accumulate, int act, float limit, int batches, int sms, cudaStream_t st) {
   if (M <= 0 || N <= 0) return 0;
   if (K % 8 || ldx % 8 || ldw % 8 || batches < 1 || sms < 1) return 660;
   if (gated_act(act) && (N % 32 || ldo % 16 || batches != 1 || accumulate)) return 664;
   CUtensorMap ta, tb;
   if (dsv4_make_tmap_2d(&ta, x, 1, (uint64_t)K * batches, M, (uint64_t)ldx * 2, 64, kPM, 3)) return 661;
   if (dsv4_make_tmap_2d(&tb, w, 1, K, (uint64_t)N * batches, (uint64_t)ldw * 2, 64, kPN, 3)) return 662;
-  const BigArgs g{M, N, K, ldo, batches, accumulate, act, (M + kPM - 1) / kPM, (N + kPN - 1) / kPN};
+  const BigArgs g{M, N, K, ldo, batches, accumulate, act, limit, (M + kPM - 1) / kPM, (N + kPN - 1) / kPN};
   return out_fp32 ? launch_big<float>(ta, tb, out, g, sms, st) : launch_big<__nv_bfloat16>(ta, tb, out, g, sms, st);
 }

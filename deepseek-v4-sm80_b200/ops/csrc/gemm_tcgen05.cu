@@ -73,6 +73,7 @@ struct GemmArgs {
   int* sp_counters;          // [row blocks], zero between launches (sp_mode 2)
   SpCtx sp;
   int act;                   // epilogue activation (GemmAct), applied to the complete sum before it is added or stored
+  float limit;               // of kActClampGate
 };
 
 __device__ __forceinline__ void store_row_chunk(__nv_bfloat16* dst, const float* v, int ncols_valid) {
@@ -432,7 +433,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
     if (!FP8 && write_out && gated_act(g.act)) {
 #pragma unroll
       for (int c = 0; c < BN / 32; ++c) {
-        gate_block(&acc[c * 32], g.act);
+        gate_block(&acc[c * 32], g.act, g.limit);
         if (grow < M && n0 + c * 32 < N) st_f16x(part + (size_t)grow * ld_part + (n0 + c * 32) / 2, &acc[c * 32]);
       }
       write_out = false;
@@ -511,10 +512,10 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             u.x += w.x, u.y += w.y, u.z += w.z, u.w += w.w;
           }
           const int col = n0 + c4 * 4;
-          const bool silu = g.act == kActSiluGate;
           if (m0 + row < M && col < N)
             st_f4(outb + (size_t)(m0 + row) * g.ldo + (col / 32) * kGateBlock + col % 32,
-                  make_float4(gate_mul(a.x, u.x, silu), gate_mul(a.y, u.y, silu), gate_mul(a.z, u.z, silu), gate_mul(a.w, u.w, silu)));
+                  make_float4(gate_mul(a.x, u.x, g.act, g.limit), gate_mul(a.y, u.y, g.act, g.limit),
+                              gate_mul(a.z, u.z, g.act, g.limit), gate_mul(a.w, u.w, g.act, g.limit)));
           continue;
         }
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -558,6 +559,7 @@ struct LaunchOpts {
   const SpCtx* sp = nullptr;
   int* sp_counters = nullptr;
   int act = 0;
+  float limit = 0.f;
 };
 
 int g_weight_prefetch = 0;  // set by dsv4_gemm_set_weight_prefetch
@@ -590,7 +592,7 @@ int launch_gemm(const void* x, const void* w, OutT* out, int M, int N, int K, in
   }
   GemmArgs g{M, N, K, ldo, sa, sb, o.sb_ld ? o.sb_ld : (K + 127) / 128, accumulate_out, o.a_col_pb, o.b_row_pb,
              o.out_col_pb, o.splits, o.ws, o.counters, o.deposit_only, g_weight_prefetch, o.cluster, o.partial_stride,
-             o.sp_mode, o.sp_counters, o.sp ? *o.sp : SpCtx{}, o.act};
+             o.sp_mode, o.sp_counters, o.sp ? *o.sp : SpCtx{}, o.act, o.limit};
   if (o.sp_mode && (!o.sp || o.sp->rows_per_rank % kBM || o.batches != 1)) return 106;
   if (o.sp_mode >= 2 && (o.splits != 1 || !o.sp_counters)) return 107;
   if (o.cluster) {
@@ -647,10 +649,10 @@ DSV4_API long long dsv4_gemm_splitk_ws_elems(int M, int N, int bn, int batches, 
 // out dtype: 0 = bf16, 1 = fp32.  ld* are row strides in elements.  bn = 0 picks the tile width.
 // batches > 1: batch b uses A columns [b*K, (b+1)*K) of x (ldx covers all batches), W rows [b*N, (b+1)*N) and output
 // columns [b*N, (b+1)*N).  splits > 1 needs ws (dsv4_gemm_splitk_ws_elems floats) and counters (>= tiles ints, zero).
-// act: epilogue activation (GemmAct in vec.cuh).
+// act: epilogue activation (GemmAct in vec.cuh), limit: its bound where it has one.
 DSV4_API int dsv4_gemm_bf16(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int ldw, int ldo,
                             int out_fp32, int accumulate_out, int bn, int batches, int splits, float* ws, int* counters,
-                            int act, cudaStream_t stream) {
+                            int act, float limit, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if ((K % 8) || (ldx % 8) || (ldw % 8)) return 110;
   if (gated_act(act) && (N % 32 || ldo % 16 || batches > 1 || accumulate_out)) return 117;
@@ -658,7 +660,7 @@ DSV4_API int dsv4_gemm_bf16(const void* x, const void* w, void* out, int M, int 
   o.batches = batches < 1 ? 1 : batches;
   o.splits = splits < 1 ? 1 : splits;
   o.ws = ws, o.counters = counters;
-  o.act = act;
+  o.act = act, o.limit = limit;
   if (o.batches > 1) o.a_col_pb = K, o.b_row_pb = N, o.out_col_pb = N, o.a_cols = K * o.batches, o.b_rows = N * o.batches;
   if (o.splits > 1 && bn == 0) return 116;
   if (o.splits > 1 && (!ws || !counters)) o.cluster = 1;  // no workspace given: reduce inside a thread-block cluster

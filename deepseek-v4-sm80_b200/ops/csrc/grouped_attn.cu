@@ -2,14 +2,18 @@
 // between the q | k | v projection and the output projection.
 //
 //   s_ij = cap tanh(q_i . k_j scale / cap) + rel[h, min(i - j, last)] - slope_h (i - j)
-//   w_ij = e^{s_ij} / (e^{sink_h} + sum_j' e^{s_ij'})
+//   w_ij = e^{s_ij} / (e^{sink_h} + sum_j' e^{s_ij'})       or, without any normalisation,  w_ij = sigmoid(s_ij + b_h)
 //
-// cap, rel, slope and sink are optional.  With a chunk size, position i only sees keys from i / chunk * chunk on.  Kernels:
+// cap, rel, slope and sink are optional.  With a chunk size, position i only sees keys from i / chunk * chunk on; with a window, the
+// last `window` positions up to itself.  Where the values were turned by their positions ahead of the cache, a head's result is
+// turned back by the query's; and it may be multiplied by a gate per token and head.  Kernels:
 //   rotate_store     bias, norms, rotation, query temperature; keys and values to their cache rows
+//   head_store       the same with a norm per head, either layout of the rotated pairs, and values that turn
 //   grouped_attn     tensor cores (mma.sync): the (token, query head) rows of a key head are consecutive, and all of them see
 //                    a prefix of the same keys, so a CTA takes 16 .. 64 rows of one request and key head and streams the keys
 //                    and values once for all of them.  grid.y splits the keys when the row tiles alone leave SMs idle;
-//                    grouped_merge adds the partial results in split order.  Decode, and short portions of prompts.
+//                    grouped_merge adds the partial results in split order, turns them back and gates them.  Decode, and short
+//                    portions of prompts.
 //   grouped_row      one warp per row on the CUDA cores, fp32 throughout: models served in 32-bit floats, other sizes
 //   kv_gather        a request's keys and (transposed) values side by side, for the prompt kernel in flash_attn.cu
 #include "mma16.cuh"
@@ -195,6 +199,105 @@ __global__ void __launch_bounds__(256) rotate_store_kernel(const T* __restrict__
   }
 }
 
+// ------------------------------------------------------------------ norms per head, values that turn
+struct HeadStoreArgs {
+  int ld;                    // row stride of qkv
+  const float* bias;         // [(H + G) dim + G vdim] or null
+  const float* gain;         // [2][dim]: every q and k head is divided by its root mean square, times its row; or null
+  float eps;
+  const float* freq;         // [pairs]: the first 2 * pairs dimensions of q and k heads turn; or null
+  int pairs, halves;         // partners: dimensions i and i + pairs (halves), or 2 i and 2 i + 1
+  float mul;                 // factor of their cos and sin
+  const float* vfreq;        // [vdim / 2]: whole value heads turn, in the same layout; or null
+  float2* turn;              // [rows][vdim / 2]: cos and sin of the values' angles, for what turns the results back
+  const int *pos, *out_loc;
+  int heads, kv_heads, dim, vdim;
+};
+
+// One CTA per token.  The row with its bias passes through shared memory, where a warp norms a head in place and partners meet.
+// W consecutive values per thread and access.
+template <typename T, int W>
+__global__ void __launch_bounds__(256) head_store_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict__ keys,
+                                                         T* __restrict__ values, const HeadStoreArgs a) {
+  pdl_entry();
+  extern __shared__ __align__(16) float hs_row[];
+  const int t = blockIdx.x, pos = a.pos[t], loc = a.out_loc[t], warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim, n = nq + nk + nv, vhalf = a.vdim / 2;
+  float* row = hs_row;
+  float2* cs = reinterpret_cast<float2*>(hs_row + (n + 3) / 4 * 4);
+  float2* vcs = cs + a.pairs;
+  const T* src = qkv + (size_t)t * a.ld;
+  for (int i = threadIdx.x * W; i < n; i += 256 * W) {
+    if constexpr (W == 1) {
+      row[i] = ld_f(src + i) + (a.bias ? a.bias[i] : 0.f);
+    } else {
+#pragma unroll
+      for (int j = 0; j < W; j += 4) {
+        float4 x = ld_f4(src + i + j);
+        if (a.bias) {
+          const float4 b = ld_f4(a.bias + i + j);
+          x.x += b.x, x.y += b.y, x.z += b.z, x.w += b.w;
+        }
+        *reinterpret_cast<float4*>(row + i + j) = x;
+      }
+    }
+  }
+  for (int i = threadIdx.x; i < a.pairs; i += 256) {
+    float s, c;
+    sincosf((float)pos * a.freq[i], &s, &c);
+    cs[i] = make_float2(c * a.mul, s * a.mul);
+  }
+  for (int i = threadIdx.x; a.vfreq && i < vhalf; i += 256) {
+    float s, c;
+    sincosf((float)pos * a.vfreq[i], &s, &c);
+    vcs[i] = make_float2(c, s);
+    a.turn[(size_t)t * vhalf + i] = make_float2(c, s);
+  }
+  __syncthreads();
+  if (a.gain) {
+    for (int h = warp; h < a.heads + a.kv_heads; h += 8) {
+      float* x = row + h * a.dim;
+      const float* g = a.gain + (h < a.heads ? 0 : a.dim);
+      float s = 0.f;
+      for (int i = lane; i < a.dim; i += 32) s = fmaf(x[i], x[i], s);
+      const float sc = 1.f / sqrtf(warp_sum(s) / a.dim + a.eps);
+      for (int i = lane; i < a.dim; i += 32) x[i] *= sc * g[i];
+    }
+    __syncthreads();
+  }
+  for (int i = threadIdx.x * W; i < n; i += 256 * W) {
+    const bool is_v = i >= nq + nk;
+    const int e = is_v ? (i - nq - nk) % a.vdim : i % a.dim;
+    const int m = is_v ? (a.vfreq ? vhalf : 0) : a.pairs;
+    const float2* tab = is_v ? vcs : cs;
+    float v[W];
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+      const int k = e + j;
+      v[j] = row[i + j];
+      if (k >= 2 * m) continue;
+      const bool second = a.halves ? k >= m : k & 1;
+      const int pair = a.halves ? (second ? k - m : k) : k >> 1, away = a.halves ? m : 1;
+      const float other = row[second ? i + j - away : i + j + away];
+      const float2 r = tab[pair];
+      v[j] = second ? v[j] * r.x + other * r.y : v[j] * r.x - other * r.y;
+    }
+    T* dst;
+    if (i < nq) {
+      dst = q + (size_t)t * nq + i;
+    } else {
+      if (loc < 0) continue;
+      dst = is_v ? values + (size_t)loc * nv + (i - nq - nk) : keys + (size_t)loc * nk + (i - nq);
+    }
+    if constexpr (W == 1) {
+      st_f(dst, v[0]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < W; j += 4) st_f4(dst + j, make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]));
+    }
+  }
+}
+
 // ------------------------------------------------------------------ few rows: tensor cores
 struct AttnArgs {
   const int* slots;
@@ -214,10 +317,24 @@ struct AttnArgs {
   const float* slope;    // [H]: taken off per position of distance; or null
   int chunk;             // > 0: keys are seen from the start of the query's chunk of this many positions on; the tokens of a
                          // tile then lie in one chunk
+  int window;            // > 0: position i sees the keys i - window + 1 .. i
+  const float* wbias;    // [H]: a key's weight is sigmoid(score + wbias), not normalised; or null: softmax
+  const float2* turn;    // [rows][vdim / 2] cos and sin: results are turned back by these angles (partners half of vdim apart); or
+                         // null
+  const void* gate;      // [rows] activations of stride ld_gate, one per head: results are multiplied by its sigmoid; or null
+  int ld_gate;
   int nsplit;
+  int partial;           // results go to part_acc and part_ml, for grouped_merge
   float* part_acc;       // [T * H][nsplit][vdim]
   float* part_ml;        // [T * H][nsplit][2]
 };
+__device__ __forceinline__ int first_key(const AttnArgs& a, int pos) {
+  return a.chunk ? pos / a.chunk * a.chunk : a.window ? max(0, pos - a.window + 1) : 0;
+}
+// column c of a result whose pair (c mod half, + half) holds u and v, turned back
+__device__ __forceinline__ float turned_back(float u, float v, const float2& cs, bool second) {
+  return second ? v * cs.x - u * cs.y : u * cs.x + v * cs.y;
+}
 
 constexpr int kKT = 64;       // keys per tile
 constexpr int kSP = kKT + 4;  // floats per score row
@@ -231,7 +348,7 @@ struct AttnCfg {
   static constexpr int WN = kKT / KG / 8;          // n8 tiles per warp
   static constexpr int DW = P / 8;                 // output columns per warp
   static constexpr int NT = DW / 8;
-  static constexpr int SMEM = M * P * 2 + 4 * kKT * P * 2 + M * kSP * 4 + M * kKT * 2 + 4 * M * 4;
+  static constexpr int SMEM = M * P * 2 + 4 * kKT * P * 2 + M * kSP * 4 + M * kKT * 2 + 5 * M * 4;
 };
 
 template <int P, int MT>
@@ -251,7 +368,8 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
   float* ms = reinterpret_cast<float*>(pb + M * kKT);
   float* ls = ms + M;
   float* alpha = ls + M;
-  int* see = reinterpret_cast<int*>(alpha + M);                     // keys the row sees
+  int* see = reinterpret_cast<int*>(alpha + M);                     // end of the keys the row sees
+  int* from = see + M;                                              // and their beginning
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = blockIdx.z, split = blockIdx.y, R = a.group, dch = a.dim / 8, vch = a.vdim / 8;
@@ -266,7 +384,7 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
   }
   if (a.num_valid && row0 / R >= *a.num_valid) return;
   const int t_last = (row1 - 1) / R;
-  const int key0 = a.chunk ? a.pos[t_last] / a.chunk * a.chunk : 0;   // first key; keys are counted from there
+  const int key0 = first_key(a, a.pos[row0 / R]);                     // first key; keys are counted from there
   const int nkeys = a.pos[t_last] + 1 - key0;   // of the tile's last token, the one that sees most
   const int* pt = a.page_table + (size_t)a.slots[t_last] * a.ld_pt + key0;
   // place of row r of the tile in q (elements) and in the lists of (token, head) rows
@@ -276,7 +394,7 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
   const int per = (ktiles + a.nsplit - 1) / a.nsplit;
   const int kt0 = split * per, kt1 = min(kt0 + per, ktiles);
   if (kt0 >= kt1) {  // nothing for this split: an empty partial
-    if (a.nsplit > 1)
+    if (a.partial)
       for (int r = tid; r < row1 - row0; r += 256) {
         float* ml = a.part_ml + (head_row(r) * a.nsplit + split) * 2;
         ml[0] = -1e30f, ml[1] = 0.f;
@@ -294,6 +412,7 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
   if (tid < M) {
     ms[tid] = -1e30f, ls[tid] = 0.f;
     see[tid] = row0 + tid < row1 ? a.pos[(row0 + tid) / R] + 1 - key0 : 0;
+    from[tid] = a.window ? max(0, see[tid] - a.window) : 0;
   }
 
   // four threads fetch the key and the value of one row
@@ -375,7 +494,7 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
     {
       constexpr int TPR = 256 / M, PER = kKT / TPR;  // threads per row, keys per thread (4, 8 or 16)
       const int r = tid / TPR, seg = tid % TPR;
-      const int lim = see[r] - kt * kKT - seg * PER;
+      const int lim = see[r] - kt * kKT - seg * PER, low = from[r] - kt * kKT - seg * PER;
       float v[PER];
       float mx = -1e30f;
 #pragma unroll
@@ -399,18 +518,24 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
       }
 #pragma unroll
       for (int i = 0; i < PER; ++i) {
-        v[i] = i < lim ? v[i] : -INFINITY;
+        v[i] = i < lim && i >= low ? v[i] : -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
 #pragma unroll
       for (int off = TPR / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-      const float m_old = ms[r], m_new = fmaxf(m_old, mx);
+      const float m_old = ms[r], m_new = a.wbias ? 0.f : fmaxf(m_old, mx);
       float sum = 0.f;
       __align__(16) __nv_bfloat16 e[PER];
+      if (a.wbias) {
+        const float wb = row0 + r < row1 ? a.wbias[g * R + (row0 + r) % R] * kLog2e : 0.f;
 #pragma unroll
-      for (int i = 0; i < PER; ++i) {
-        e[i] = f2bf(exp2f(v[i] - m_new));
-        sum += bf2f(e[i]);   // the weights as they enter the product add up to what they are divided by
+        for (int i = 0; i < PER; ++i) e[i] = f2bf(sigmoid_ex2(v[i] + wb));
+      } else {
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+          e[i] = f2bf(exp2f(v[i] - m_new));
+          sum += bf2f(e[i]);   // the weights as they enter the product add up to what they are divided by
+        }
       }
 #pragma unroll
       for (int off = TPR / 2; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
@@ -423,10 +548,10 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
       }
       __syncwarp();
       if (seg == 0) {
-        const float al = exp2f(m_old - m_new);
+        const float al = a.wbias ? 1.f : exp2f(m_old - m_new);
         alpha[r] = al;
         ms[r] = m_new;
-        ls[r] = ls[r] * al + sum;
+        ls[r] = a.wbias ? 1.f : ls[r] * al + sum;
       }
     }
     __syncthreads();
@@ -477,7 +602,7 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
       if (row0 + r >= row1) continue;
       const size_t row = head_row(r);
       float inv = 1.f;
-      if (a.nsplit == 1) {
+      if (!a.partial && !a.wbias) {
         float l = ls[r], f = 1.f;
         if (a.sink) {   // one more term of the sum, without a key or a value
           const float s2 = a.sink[g * R + (row0 + r) % R] * kLog2e, mm = fmaxf(ms[r], s2);
@@ -491,20 +616,20 @@ __global__ void __launch_bounds__(256) grouped_attn_kernel(const __nv_bfloat16* 
         const int c = warp * C::DW + j * 8 + (lane & 3) * 2;
         if (c >= a.vdim) continue;
         const float x = acc[i][j][half * 2], y = acc[i][j][half * 2 + 1];
-        if (a.nsplit > 1)
+        if (a.partial)
           *reinterpret_cast<float2*>(a.part_acc + (row * a.nsplit + split) * a.vdim + c) = make_float2(x, y);
         else
           *reinterpret_cast<__nv_bfloat162*>(o + row * a.vdim + c) = __floats2bfloat162_rn(x * inv, y * inv);
       }
     }
-  if (a.nsplit > 1 && tid < M && row0 + tid < row1) {
+  if (a.partial && tid < M && row0 + tid < row1) {
     float* ml = a.part_ml + (head_row(tid) * a.nsplit + split) * 2;
     ml[0] = ms[tid], ml[1] = ls[tid];
   }
 }
 
 // o[row] = sum_s acc_s 2^(m_s - M) / (2^(sink - M) + sum_s l_s 2^(m_s - M)) for the rows of the tiles of M rows that
-// grouped_attn_kernel worked on; one warp per row.
+// grouped_attn_kernel worked on (the plain sum where weights are not normalised), turned back and gated; one warp per row.
 __global__ void __launch_bounds__(128) grouped_merge_kernel(__nv_bfloat16* __restrict__ o, const AttnArgs a, int M) {
   pdl_entry();
   const int R = a.group, n = a.nsplit, g = blockIdx.y, lane = threadIdx.x & 31;
@@ -525,16 +650,37 @@ __global__ void __launch_bounds__(128) grouped_merge_kernel(__nv_bfloat16* __res
     // lane s holds split s (at most 32)
     const float ms = lane < n ? ml[lane * 2] : -1e30f, ls = lane < n ? ml[lane * 2 + 1] : 0.f;
     const float mx = fmaxf(warp_max(ms), s2);
-    const float f = ls > 0.f ? exp2f(ms - mx) : 0.f;
-    const float inv = 1.f / (warp_sum(ls * f) + (a.sink ? exp2f(s2 - mx) : 0.f));
+    const float f = ls > 0.f ? a.wbias ? 1.f : exp2f(ms - mx) : 0.f;
+    const float sum = warp_sum(ls * f) + (a.sink ? exp2f(s2 - mx) : 0.f);
+    float mul = a.wbias ? 1.f : 1.f / sum;
+    if (a.gate) mul *= sigmoid_f(bf2f(static_cast<const __nv_bfloat16*>(a.gate)[(size_t)(r / R) * a.ld_gate + h]));
+    const float* acc = a.part_acc + row * n * a.vdim;
+    if (a.turn) {
+      const int half = a.vdim / 2;
+      const float2* turn = a.turn + (size_t)(r / R) * half;
+      for (int c0 = 0; c0 < half; c0 += 32) {
+        const int c = c0 + lane;
+        float u = 0.f, v = 0.f;
+        for (int s = 0; s < n; ++s) {
+          const float fs = __shfl_sync(0xffffffffu, f, s);
+          if (fs > 0.f && c < half) u = fmaf(acc[s * a.vdim + c], fs, u), v = fmaf(acc[s * a.vdim + c + half], fs, v);
+        }
+        if (c < half) {
+          const float2 cs = turn[c];
+          o[row * a.vdim + c] = f2bf(turned_back(u, v, cs, false) * mul);
+          o[row * a.vdim + c + half] = f2bf(turned_back(u, v, cs, true) * mul);
+        }
+      }
+      continue;
+    }
     for (int c0 = 0; c0 < a.vdim; c0 += 32) {
       const int c = c0 + lane;
       float v = 0.f;
       for (int s = 0; s < n; ++s) {
         const float fs = __shfl_sync(0xffffffffu, f, s);
-        if (fs > 0.f && c < a.vdim) v = fmaf(a.part_acc[(row * n + s) * a.vdim + c], fs, v);
+        if (fs > 0.f && c < a.vdim) v = fmaf(acc[s * a.vdim + c], fs, v);
       }
-      if (c < a.vdim) o[row * a.vdim + c] = f2bf(v * inv);
+      if (c < a.vdim) o[row * a.vdim + c] = f2bf(v * mul);
     }
   }
 }
@@ -551,9 +697,9 @@ __global__ void __launch_bounds__(128) grouped_row_kernel(const T* __restrict__ 
   if (row >= a.rows * H) return;
   const int t = row / H, h = row % H, g = h / a.group;
   if (a.num_valid && t >= *a.num_valid) return;
-  const int key0 = a.chunk ? a.pos[t] / a.chunk * a.chunk : 0, nkeys = a.pos[t] + 1 - key0;
+  const int key0 = first_key(a, a.pos[t]), nkeys = a.pos[t] + 1 - key0;
   const int* pt = a.page_table + (size_t)a.slots[t] * a.ld_pt + key0;
-  const float slope = a.slope ? a.slope[h] : 0.f;
+  const float slope = a.slope ? a.slope[h] : 0.f, wb = a.wbias ? a.wbias[h] : 0.f;
   const T *kb = keys + g * a.dim, *vb = values + g * a.vdim;
   const size_t ldk = (size_t)a.kv_heads * a.dim, ldv = (size_t)a.kv_heads * a.vdim;
   const float* rel = a.rel ? a.rel + (size_t)h * a.n_rel : nullptr;
@@ -591,14 +737,16 @@ __global__ void __launch_bounds__(128) grouped_row_kernel(const T* __restrict__ 
         if (k + j >= n) s[j] = -INFINITY;
         mn = fmaxf(mn, s[j]);
       }
-      const float al = expf(m - mn);
-      m = mn;
-      l *= al;
+      if (!a.wbias) {
+        const float al = expf(m - mn);
+        m = mn;
+        l *= al;
 #pragma unroll
-      for (int i = 0; i < NI; ++i) acc[i] *= al;
+        for (int i = 0; i < NI; ++i) acc[i] *= al;
+      }
 #pragma unroll
       for (int j = 0; j < KB; ++j) {
-        const float p = expf(s[j] - mn);
+        const float p = a.wbias ? sigmoid_f(s[j] + wb) : expf(s[j] - mn);
         const T* vp = vb + loc[j] * ldv;
         l += p;
 #pragma unroll
@@ -607,11 +755,27 @@ __global__ void __launch_bounds__(128) grouped_row_kernel(const T* __restrict__ 
       }
     }
   }
-  const float inv = 1.f / l;
+  float mul = a.wbias ? 1.f : 1.f / l;
+  if (a.gate) mul *= sigmoid_f(ld_f(static_cast<const T*>(a.gate) + (size_t)t * a.ld_gate + h));
+  if (a.turn) {
+    __shared__ float whole[4][NI * 32];
+    float* w = whole[threadIdx.x >> 5];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) w[i * 32 + lane] = acc[i];
+    __syncwarp();
+    const int half = a.vdim / 2;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int c = i * 32 + lane;
+      if (c >= a.vdim) continue;
+      const int u = c < half ? c : c - half;
+      acc[i] = turned_back(w[u], w[u + half], a.turn[(size_t)t * half + u], c >= half);
+    }
+  }
 #pragma unroll
   for (int i = 0; i < NI; ++i) {
     const int c = i * 32 + lane;
-    if (c < a.vdim) st_f(o + (size_t)row * a.vdim + c, acc[i] * inv);
+    if (c < a.vdim) st_f(o + (size_t)row * a.vdim + c, acc[i] * mul);
   }
 }
 
@@ -671,7 +835,7 @@ int launch_attn(const void* q, const void* k, const void* v, void* o, const Attn
   }
   dsv4_launch(grouped_attn_kernel<P, MT>, dim3(a.n_tiles, a.nsplit, a.kv_heads), 256, C::SMEM, st, (const __nv_bfloat16*)q,
               (const __nv_bfloat16*)k, (const __nv_bfloat16*)v, (__nv_bfloat16*)o, a);
-  if (a.nsplit > 1)
+  if (a.partial)
     dsv4_launch(grouped_merge_kernel, dim3(a.n_tiles, a.kv_heads), 128, 0, st, (__nv_bfloat16*)o, a, C::M);
   return (int)cudaGetLastError();
 }
@@ -738,20 +902,49 @@ DSV4_API int dsv4_rotate_store(const void* qkv, int ld, const float* bias, const
   return (int)cudaGetLastError();
 }
 
+// Norms per head and rotation in either layout, values included (see HeadStoreArgs).  qkv, q_out and the caches as above; turn [rows,
+// vdim / 2, 2] receives the values' cos and sin if vfreq is given.
+DSV4_API int dsv4_head_store(const void* qkv, int ld, const float* bias, const float* gain, float eps, const float* freq,
+                             int pairs, int halves, float mul, const float* vfreq, float* turn, const int* pos,
+                             const int* out_loc, void* q_out, void* keys, void* values, int rows, int heads, int kv_heads,
+                             int dim, int vdim, int fp32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (pairs < 0 || 2 * pairs > dim || (pairs && !freq) || (vfreq && (vdim % 2 || !turn))) return 680;
+  const HeadStoreArgs a{ld, bias, gain, eps, freq, pairs, halves, mul, vfreq, reinterpret_cast<float2*>(turn), pos, out_loc,
+                        heads, kv_heads, dim, vdim};
+  const int n = (heads + kv_heads) * dim + kv_heads * vdim;
+  const size_t smem = (size_t)(n + 3) / 4 * 16 + (pairs + (vfreq ? vdim / 2 : 0)) * sizeof(float2);
+  if (smem > 200 * 1024) return 681;
+  const bool wide = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && ((uintptr_t)qkv & 15) == 0;
+  auto go = [&](auto kern, auto type) {
+    using T = decltype(type);
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+      return 682;
+    dsv4_launch(kern, rows, 256, smem, st, (const T*)qkv, (T*)q_out, (T*)keys, (T*)values, a);
+    return (int)cudaGetLastError();
+  };
+  if (fp32) return wide ? go(head_store_kernel<float, 4>, float()) : go(head_store_kernel<float, 1>, float());
+  return wide ? go(head_store_kernel<__nv_bfloat16, 8>, __nv_bfloat16()) : go(head_store_kernel<__nv_bfloat16, 1>, __nv_bfloat16());
+}
+
 // q [rows, heads * dim], o [rows, heads * vdim].  m: rows per CTA (16, 32 or 64; 0 = the one-warp-per-row kernel, which takes
 // every token).  tiles: [n_tiles][2] row ranges (see AttnArgs), or null: n_tiles covers every token's own rows.  nsplit > 1
-// (at most 32) needs part_acc [rows * heads, nsplit, vdim] and part_ml [rows * heads, nsplit, 2].
+// (at most 32) needs part_acc [rows * heads, nsplit, vdim] and part_ml [rows * heads, nsplit, 2], and so do turn and gate unless
+// m is 0.
 DSV4_API int dsv4_grouped_attention(const void* q, const void* keys, const void* values, void* o, const int* slots,
                                     const int* pos, const int* page_table, int ld_pt, const int* tiles, int n_tiles,
                                     const int* num_valid, int rows, int kv_heads, int group, int dim, int vdim, float scale,
                                     float cap, const float* sink, const float* rel, int n_rel, const float* slope,
-                                    int chunk, int m, int nsplit, float* part_acc, float* part_ml, int fp32,
-                                    cudaStream_t st) {
+                                    int chunk, int window, const float* wbias, const float* turn, const void* gate, int ld_gate,
+                                    int m, int nsplit, float* part_acc, float* part_ml, int fp32, cudaStream_t st) {
   if (rows <= 0) return 0;
-  if (nsplit < 1 || nsplit > 32 || (nsplit > 1 && (!part_acc || !part_ml)) || (rel && n_rel < 1)) return 675;
-  if (kv_heads < 1 || kv_heads > 65535 || group < 1 || chunk < 0) return 676;
+  const int partial = nsplit > 1 || (m && (turn || gate));
+  if (nsplit < 1 || nsplit > 32 || (partial && (!part_acc || !part_ml)) || (rel && n_rel < 1)) return 675;
+  if (kv_heads < 1 || kv_heads > 65535 || group < 1 || chunk < 0 || window < 0 || (chunk && window)) return 676;
+  if ((wbias && sink) || (turn && vdim % 2)) return 683;
   const AttnArgs a{slots, pos, page_table, ld_pt, tiles, n_tiles, num_valid, rows, kv_heads, group, dim, vdim, scale, cap,
-                   sink, rel, n_rel, slope, chunk, nsplit, part_acc, part_ml};
+                   sink, rel, n_rel, slope, chunk, window, wbias, reinterpret_cast<const float2*>(turn), gate, ld_gate, nsplit,
+                   partial, part_acc, part_ml};
   if (m == 0)
     return fp32 ? launch_row<float>(q, keys, values, o, a, st) : launch_row<__nv_bfloat16>(q, keys, values, o, a, st);
   if (fp32 || dim % 8 || vdim % 8) return 677;

@@ -1,10 +1,14 @@
-// Latent attention without positions over a paged cache of latents: all heads of a token read the same row c_j (K = V =
-// c_j, `rank` values), because the per-head up-projections of keys and values are absorbed into the query and into the
-// output:  score = (W_uk^T q) . c_j * scale,   o_lat = sum_j softmax_j c_j,   o = W_uv o_lat.
+// Latent attention over a paged cache of latents: all heads of a token read the same row c_j (K = V = c_j, `rank` values), because
+// the per-head up-projections of keys and values are absorbed into the query and into the output:
+// score = (W_uk^T q) . c_j * scale,   o_lat = sum_j softmax_j c_j,   o = W_uv o_lat.
+//
+// Positions, where a design has them, turn `rot` further values of every query head and one part r_j that all heads share: a cache
+// row is then [c_j | r_j], the score (W_uk^T q . c_j + q_r . r_j) * scale, and the values are still c_j.  With a window, position i
+// sees the keys i - window + 1 .. i only.
 //
 // q and o are [T][heads][rank].  The (token, head) rows of a request are consecutive, and all of them see a prefix of the
 // same keys, so a CTA takes M = 16 .. 64 consecutive rows of one request -- heads of one token in decode, several tokens
-// in prefill -- and streams the request's latents once for all of them.  Position i sees every j <= i.
+// in prefill -- and streams the request's latents once for all of them.  Position i sees every j <= i (of its window).
 //   S phase : 8 warps share the M x 64 score tile (mma.sync m16n8k16, bf16 in, fp32 accumulate)
 //   softmax : online (max, sum) per row in fp32, probabilities to shared memory as bf16
 //   PV phase: warp w owns rank / 8 output columns of all M rows in registers
@@ -27,6 +31,10 @@ struct LatArgs {
   const int* num_valid;  // rows (tokens) >= *num_valid are padding, or null
   int rows;              // tokens
   int heads, rank;
+  int rot;               // further values of a cache row and of a query head, which only the score reads
+  const void* q_rot;     // [T] rows of stride ld_rot: head h's at h * rot
+  int ld_rot;
+  int window;            // > 0: position i sees the keys i - window + 1 .. i
   float scale;
   int nsplit;
   float* part_acc;       // [T * heads][nsplit][rank]
@@ -53,6 +61,66 @@ __global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__
   const int loc = out_loc[t];
   if (loc < 0) return;
   for (int i = lane; i < rank; i += 32) st_f(cache + (size_t)loc * rank + i, ld_f(r + i) * sc * gain[i]);
+}
+
+// ------------------------------------------------------------------ norm, rotation, store
+struct LatStoreArgs {
+  int ld;                // row stride of p
+  int at_rot, at_c;      // columns: the heads' unrotated parts from 0, their parts that turn, then latent | shared part that turns
+  const float* gain;     // [rank]
+  float eps;
+  const float* freq;     // [rot / 2]: neighbouring values turn by position * freq
+  float mul;             // factor of cos and sin
+  const int *pos, *out_loc;
+  int heads, dim, rot, rank;
+};
+
+// One CTA per token.  cache row = [x / rms(x) * gain | turned part]; the queries' parts turn in place (`whole` null) or go, behind
+// the unrotated ones, to whole [T][heads][dim + rot].
+template <typename T>
+__global__ void __launch_bounds__(256) latent_rotate_store_kernel(T* p, T* __restrict__ cache, T* __restrict__ whole,
+                                                                  const LatStoreArgs a) {
+  pdl_entry();
+  extern __shared__ float2 lat_cs[];
+  __shared__ float sh[32];
+  const int t = blockIdx.x, loc = a.out_loc[t], half = a.rot / 2, wide = a.dim + a.rot;
+  T* row = p + (size_t)t * a.ld;
+  for (int i = threadIdx.x; i < half; i += 256) {
+    float s, c;
+    sincosf((float)a.pos[t] * a.freq[i], &s, &c);
+    lat_cs[i] = make_float2(c * a.mul, s * a.mul);
+  }
+  const T* x = row + a.at_c;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < a.rank; i += 256) {
+    const float v = ld_f(x + i);
+    ss += v * v;
+  }
+  const float sc = 1.f / sqrtf(cta_sum(ss, sh) / a.rank + a.eps);    // its barriers also publish lat_cs
+  if (loc >= 0) {
+    T* dst = cache + (size_t)loc * (a.rank + a.rot);
+    for (int i = threadIdx.x; i < a.rank; i += 256) st_f(dst + i, ld_f(x + i) * sc * a.gain[i]);
+    for (int i = threadIdx.x; i < half; i += 256) {
+      const float u = ld_f(x + a.rank + 2 * i), v = ld_f(x + a.rank + 2 * i + 1);
+      const float2 cs = lat_cs[i];
+      st_f(dst + a.rank + 2 * i, u * cs.x - v * cs.y);
+      st_f(dst + a.rank + 2 * i + 1, v * cs.x + u * cs.y);
+    }
+  }
+  T* q = row + a.at_rot;
+  for (int i = threadIdx.x; i < a.heads * half; i += 256) {
+    const int h = i / half, k = i - h * half;
+    const float u = ld_f(q + 2 * i), v = ld_f(q + 2 * i + 1);
+    const float2 cs = lat_cs[k];
+    T* dst = whole ? whole + ((size_t)t * a.heads + h) * wide + a.dim + 2 * k : q + 2 * i;
+    st_f(dst, u * cs.x - v * cs.y);
+    st_f(dst + 1, v * cs.x + u * cs.y);
+  }
+  if (whole)
+    for (int i = threadIdx.x; i < a.heads * a.dim; i += 256) {
+      const int h = i / a.dim;
+      whole[((size_t)t * a.heads + h) * wide + (i - h * a.dim)] = row[i];
+    }
 }
 
 // ------------------------------------------------------------------ row tiles
@@ -107,7 +175,7 @@ struct LatCfg {
   static constexpr int WN = kKT / KG / 8;          // n8 tiles per warp
   static constexpr int DW = RP / 8;                // output columns per warp
   static constexpr int NT = DW / 8;
-  static constexpr int SMEM = M * RP * 2 + 2 * kKT * RP * 2 + M * kSP * 4 + M * kKT * 2 + 4 * M * 4;
+  static constexpr int SMEM = M * RP * 2 + 2 * kKT * RP * 2 + M * kSP * 4 + M * kKT * 2 + 5 * M * 4;
 };
 
 template <int RP, int MT>
@@ -125,16 +193,18 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __nv_bfloat16* _
   float* ms = reinterpret_cast<float*>(pb + M * kKT);
   float* ls = ms + M;
   float* alpha = ls + M;
-  int* see = reinterpret_cast<int*>(alpha + M);                    // keys the row sees
+  int* see = reinterpret_cast<int*>(alpha + M);                    // end of the keys the row sees
+  int* from = see + M;                                             // and their beginning
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int split = blockIdx.y, R = a.rank, rch = R / 8;
+  const int split = blockIdx.y, R = a.rank, rch = R / 8, W = R + a.rot, wch = W / 8;
   int row0, row1;
   if (!find_tile<M>(a, blockIdx.x, row0, row1)) return;
   if (a.num_valid && row0 / a.heads >= *a.num_valid) return;
   const int t_last = (row1 - 1) / a.heads;
-  const int keys = a.pos[t_last] + 1;   // of the tile's last token, the one that sees most
-  const int* pt = a.page_table + (size_t)a.slots[t_last] * a.ld_pt;
+  const int key0 = a.window ? max(0, a.pos[row0 / a.heads] - a.window + 1) : 0;   // first key; keys are counted from there
+  const int keys = a.pos[t_last] + 1 - key0;   // up to the tile's last token
+  const int* pt = a.page_table + (size_t)a.slots[t_last] * a.ld_pt + key0;
 
   const int ktiles = (keys + kKT - 1) / kKT;
   const int per = (ktiles + a.nsplit - 1) / a.nsplit;
@@ -151,12 +221,16 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __nv_bfloat16* _
   for (int i = tid; i < M * (RP / 8); i += 256) {
     const int r = i / (RP / 8), c = i % (RP / 8);
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (row0 + r < row1 && c < rch) v = reinterpret_cast<const uint4*>(q + (size_t)(row0 + r) * R)[c];
+    if (row0 + r < row1 && c < wch)
+      v = c < rch ? reinterpret_cast<const uint4*>(q + (size_t)(row0 + r) * R)[c]
+                  : reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.q_rot) +
+                                                   (size_t)((row0 + r) / a.heads) * a.ld_rot + (row0 + r) % a.heads * a.rot)[c - rch];
     reinterpret_cast<uint4*>(qs + r * RP)[swz(r, c)] = v;
   }
   if (tid < M) {
     ms[tid] = -1e30f, ls[tid] = 0.f;
-    see[tid] = row0 + tid < row1 ? a.pos[(row0 + tid) / a.heads] + 1 : 0;
+    see[tid] = row0 + tid < row1 ? a.pos[(row0 + tid) / a.heads] + 1 - key0 : 0;
+    from[tid] = a.window ? max(0, see[tid] - a.window) : 0;
   }
 
   // four threads fetch one latent row
@@ -167,10 +241,10 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __nv_bfloat16* _
   };
   auto issue = [&](int loc, int buf) {
     __nv_bfloat16* dst = kv + ((size_t)buf * kKT + fk) * RP;
-    const __nv_bfloat16* src = cache + (size_t)max(loc, 0) * R;
+    const __nv_bfloat16* src = cache + (size_t)max(loc, 0) * W;
 #pragma unroll
     for (int c = fp; c < RP / 8; c += 4) {
-      const bool in = loc >= 0 && c < rch;
+      const bool in = loc >= 0 && c < wch;
       cpa16_zfill(dst + swz(fk, c) * 8, in ? src + c * 8 : cache, in);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -235,7 +309,7 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __nv_bfloat16* _
     {
       constexpr int TPR = 256 / M, PER = kKT / TPR;  // threads per row, keys per thread (4, 8 or 16)
       const int r = tid / TPR, seg = tid % TPR;
-      const int lim = see[r] - kt * kKT - seg * PER;
+      const int lim = see[r] - kt * kKT - seg * PER, low = from[r] - kt * kKT - seg * PER;
       float v[PER];
       float mx = -1e30f;
 #pragma unroll
@@ -245,7 +319,7 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __nv_bfloat16* _
       }
 #pragma unroll
       for (int i = 0; i < PER; ++i) {
-        v[i] = i < lim ? v[i] : -INFINITY;
+        v[i] = i < lim && i >= low ? v[i] : -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
 #pragma unroll
@@ -277,7 +351,7 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __nv_bfloat16* _
     }
     __syncthreads();
     // ---- o += P C: all rows, output columns [warp * DW, +DW)
-    {
+    if (warp * C::DW < R) {
 #pragma unroll
       for (int i = 0; i < MT; ++i) {
         const float a0 = alpha[i * 16 + (lane >> 2)], a1 = alpha[i * 16 + (lane >> 2) + 8];
@@ -359,13 +433,14 @@ __global__ void __launch_bounds__(128) latent_attn_row_kernel(const T* __restric
   if (row >= a.rows * a.heads) return;
   const int t = row / a.heads;
   if (a.num_valid && t >= *a.num_valid) return;
-  const int keys = a.pos[t] + 1;
-  const int* pt = a.page_table + (size_t)a.slots[t] * a.ld_pt;
+  const int W = R + a.rot, key0 = a.window ? max(0, a.pos[t] - a.window + 1) : 0, keys = a.pos[t] + 1 - key0;
+  const int* pt = a.page_table + (size_t)a.slots[t] * a.ld_pt + key0;
+  const T* qr = static_cast<const T*>(a.q_rot) + (a.rot ? (size_t)t * a.ld_rot + row % a.heads * a.rot : 0);
   float qv[NI], acc[NI];
 #pragma unroll
   for (int i = 0; i < NI; ++i) {
     const int c = i * 32 + lane;
-    qv[i] = c < R ? ld_f(q + (size_t)row * R + c) * a.scale : 0.f;
+    qv[i] = c < R ? ld_f(q + (size_t)row * R + c) * a.scale : c < W ? ld_f(qr + c - R) * a.scale : 0.f;
     acc[i] = 0.f;
   }
   float m = -1e30f, l = 0.f;
@@ -373,11 +448,11 @@ __global__ void __launch_bounds__(128) latent_attn_row_kernel(const T* __restric
     const int mine = k0 + lane < keys ? pt[k0 + lane] : 0;
     const int n = min(32, keys - k0);
     for (int k = 0; k < n; ++k) {
-      const T* c = cache + (size_t)__shfl_sync(0xffffffffu, mine, k) * R;
+      const T* c = cache + (size_t)__shfl_sync(0xffffffffu, mine, k) * W;
       float cv[NI], s = 0.f;
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
-        cv[i] = i * 32 + lane < R ? ld_f(c + i * 32 + lane) : 0.f;
+        cv[i] = i * 32 + lane < W ? ld_f(c + i * 32 + lane) : 0.f;
         s = fmaf(qv[i], cv[i], s);
       }
       s = warp_sum(s);
@@ -396,8 +471,8 @@ __global__ void __launch_bounds__(128) latent_attn_row_kernel(const T* __restric
   }
 }
 
-// ctx[dst + j] = cache[page_table[slot][j]] for the keys j of every listed request, zeros in the padding behind them.
-// list: [segs][3] = slot, keys, first row of the copy; rows [dst, dst of the next request) belong to a request.
+// ctx[dst + j] = cache[page_table[slot][first + j]] for the keys of every listed request, zeros in the padding behind them.
+// list: [segs][4] = slot, keys, first row of the copy, first key; rows [dst, dst of the next request) belong to a request.
 __global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* __restrict__ cache, uint4* __restrict__ ctx,
                                                             const int* __restrict__ list, int segs, int total,
                                                             const int* __restrict__ page_table, int ld_pt, int r8) {
@@ -407,11 +482,11 @@ __global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* __restr
   int lo = 0, hi = segs - 1;
   while (lo < hi) {
     const int mid = (lo + hi + 1) >> 1;
-    if (list[mid * 3 + 2] <= row) lo = mid; else hi = mid - 1;
+    if (list[mid * 4 + 2] <= row) lo = mid; else hi = mid - 1;
   }
-  const int j = row - list[lo * 3 + 2];
-  const bool in = j < list[lo * 3 + 1];
-  const size_t src = in ? (size_t)page_table[(size_t)list[lo * 3] * ld_pt + j] * r8 : 0;
+  const int j = row - list[lo * 4 + 2];
+  const bool in = j < list[lo * 4 + 1];
+  const size_t src = in ? (size_t)page_table[(size_t)list[lo * 4] * ld_pt + list[lo * 4 + 3] + j] * r8 : 0;
   for (int i = lane; i < r8; i += 32) ctx[(size_t)row * r8 + i] = in ? cache[src + i] : make_uint4(0, 0, 0, 0);
 }
 
@@ -436,7 +511,9 @@ int dispatch_lat(int m, const void* q, const void* cache, void* o, const LatArgs
   switch (m) {
     case 16: return launch_lat<RP, 1>(q, cache, o, a, tiles, st);
     case 32: return launch_lat<RP, 2>(q, cache, o, a, tiles, st);
-    case 64: return launch_lat<RP, 4>(q, cache, o, a, tiles, st);
+    case 64:
+      if constexpr (RP <= 512) return launch_lat<RP, 4>(q, cache, o, a, tiles, st);
+      return 632;
     default: return 632;
   }
 }
@@ -444,13 +521,14 @@ template <typename T>
 int launch_row(const void* q, const void* cache, void* o, const LatArgs& a, cudaStream_t st) {
   const int grid = (a.rows * a.heads + 3) / 4;
   const T *tq = (const T*)q, *tc = (const T*)cache;
-  if (a.rank <= 128)
+  const int w = a.rank + a.rot;
+  if (w <= 128)
     dsv4_launch(latent_attn_row_kernel<T, 4>, grid, 128, 0, st, tq, tc, (T*)o, a);
-  else if (a.rank <= 256)
+  else if (w <= 256)
     dsv4_launch(latent_attn_row_kernel<T, 8>, grid, 128, 0, st, tq, tc, (T*)o, a);
-  else if (a.rank <= 512)
+  else if (w <= 512)
     dsv4_launch(latent_attn_row_kernel<T, 16>, grid, 128, 0, st, tq, tc, (T*)o, a);
-  else if (a.rank <= 1024)
+  else if (w <= 1024)
     dsv4_launch(latent_attn_row_kernel<T, 32>, grid, 128, 0, st, tq, tc, (T*)o, a);
   else
     return 633;
@@ -472,21 +550,43 @@ DSV4_API int dsv4_latent_store(const void* x, int ldx, const float* gain, float 
   return (int)cudaGetLastError();
 }
 
+// p [rows, ld]: the heads' unrotated parts (heads x dim) from column 0, the parts that turn (heads x rot, even) at at_rot, latent |
+// shared part that turns (rank + rot) at at_c; cache [locations, rank + rot].  whole [rows, heads, dim + rot] or null: see above.
+DSV4_API int dsv4_latent_rotate_store(void* p, int ld, int at_rot, int at_c, const float* gain, float eps, const float* freq,
+                                      float mul, const int* pos, const int* out_loc, void* cache, void* whole, int rows,
+                                      int heads, int dim, int rot, int rank, int fp32, cudaStream_t st) {
+  if (rows <= 0) return 0;
+  if (rot < 2 || rot % 2 || rot > 8192 || !freq) return 637;
+  const LatStoreArgs a{ld, at_rot, at_c, gain, eps, freq, mul, pos, out_loc, heads, dim, rot, rank};
+  if (fp32)
+    dsv4_launch(latent_rotate_store_kernel<float>, rows, 256, rot * 4, st, (float*)p, (float*)cache, (float*)whole, a);
+  else
+    dsv4_launch(latent_rotate_store_kernel<__nv_bfloat16>, rows, 256, rot * 4, st, (__nv_bfloat16*)p, (__nv_bfloat16*)cache,
+                (__nv_bfloat16*)whole, a);
+  return (int)cudaGetLastError();
+}
+
+// q_rot [rows] of stride ld_rot, heads x rot: the part of the score that positions turn (rot 0: none); cache [locations, rank + rot].
 // m: rows per CTA (16, 32 or 64; 0 = the one-warp-per-row kernel), tiles: row tiles of that height over all requests.
 // nsplit > 1 needs part_acc [T * heads, nsplit, rank] and part_ml [T * heads, nsplit, 2].
 DSV4_API int dsv4_latent_attention(const void* q, const void* cache, void* o, const int* slots, const int* pos,
                                    const int* page_table, int ld_pt, const int* seg_off, int nseg,
-                                   const int* num_valid, int rows, int heads, int rank, float scale, int m, int tiles,
-                                   int nsplit, float* part_acc, float* part_ml, int fp32, cudaStream_t st) {
+                                   const int* num_valid, int rows, int heads, int rank, const void* q_rot, int ld_rot,
+                                   int rot, int window, float scale, int m, int tiles, int nsplit, float* part_acc,
+                                   float* part_ml, int fp32, cudaStream_t st) {
   if (rows <= 0) return 0;
   if (nsplit < 1 || nsplit > 65535 || (nsplit > 1 && (!part_acc || !part_ml))) return 634;
-  const LatArgs a{slots, pos, page_table, ld_pt, seg_off, nseg, num_valid, rows, heads, rank, scale, nsplit, part_acc, part_ml};
+  if (rot < 0 || (rot && !q_rot) || window < 0) return 638;
+  const LatArgs a{slots, pos, page_table, ld_pt, seg_off, nseg, num_valid, rows, heads, rank, rot, q_rot, ld_rot, window, scale,
+                  nsplit, part_acc, part_ml};
   if (m == 0) return fp32 ? launch_row<float>(q, cache, o, a, st) : launch_row<__nv_bfloat16>(q, cache, o, a, st);
-  if (fp32 || rank % 8) return 635;
-  if (rank <= 128) return dispatch_lat<128>(m, q, cache, o, a, tiles, st);
-  if (rank <= 256) return dispatch_lat<256>(m, q, cache, o, a, tiles, st);
-  if (rank <= 384) return dispatch_lat<384>(m, q, cache, o, a, tiles, st);
-  if (rank <= 512) return dispatch_lat<512>(m, q, cache, o, a, tiles, st);
+  if (fp32 || rank % 8 || rot % 8 || ld_rot % 8) return 635;
+  const int w = rank + rot;
+  if (w <= 128) return dispatch_lat<128>(m, q, cache, o, a, tiles, st);
+  if (w <= 256) return dispatch_lat<256>(m, q, cache, o, a, tiles, st);
+  if (w <= 384) return dispatch_lat<384>(m, q, cache, o, a, tiles, st);
+  if (w <= 512) return dispatch_lat<512>(m, q, cache, o, a, tiles, st);
+  if (w <= 640) return dispatch_lat<640>(m, q, cache, o, a, tiles, st);
   return 636;
 }
 

@@ -40,6 +40,8 @@ __device__ __forceinline__ float rcp_approx(float x) {
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// 1 / (1 + 2^-x)
+__device__ __forceinline__ float sigmoid_ex2(float x) { return rcp_approx(1.f + ex2(-x)); }
 // cap * tanh(x / cap) in the units of cap, e = 2 log2(e) / cap in the units of x:  1 - 2 / (1 + e^(2 x / cap)).
 // The result's absolute error is a few 1e-7 of cap.
 __device__ __forceinline__ float softcap_ex2(float x, float e, float cap) {

@@ -50,9 +50,9 @@ __device__ __forceinline__ float cta_sum(float v, float* sh) {
 
 // Epilogue activations of the projections (the numbers are part of the host interface).
 // The gates pair columns: the weight rows come in blocks of 16 gate and 16 up rows, and the result is half as wide.
-enum GemmAct : int { kActNone = 0, kActRelu2 = 1, kActTanh = 2, kActGeluGate = 3, kActSiluGate = 4 };
+enum GemmAct : int { kActNone = 0, kActRelu2 = 1, kActTanh = 2, kActGeluGate = 3, kActSiluGate = 4, kActClampGate = 5 };
 constexpr int kGateBlock = 16;
-__host__ __device__ __forceinline__ bool gated_act(int act) { return act == kActGeluGate || act == kActSiluGate; }
+__host__ __device__ __forceinline__ bool gated_act(int act) { return act >= kActGeluGate && act <= kActClampGate; }
 __device__ __forceinline__ float gemm_act(float v, int act) {
   if (act == kActRelu2) {
     v = fmaxf(v, 0.f);
@@ -67,15 +67,20 @@ template <typename T>
 __device__ __forceinline__ float sigmoid_for(float z) {
   return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-z)) : sigmoid_f(z);
 }
-// gate(z) * up.  silu: z sigmoid(z);  gelu: 0.5 z (1 + tanh(w)) = z sigmoid(2 w),  w = sqrt(2 / pi) (z + 0.044715 z^3)
-__device__ __forceinline__ float gate_mul(float z, float up, bool silu) {
-  const float w = silu ? z : 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+// gate(z) * up.  silu: z sigmoid(z);  gelu: 0.5 z (1 + tanh(w)) = z sigmoid(2 w),  w = sqrt(2 / pi) (z + 0.044715 z^3);
+// clamp: g sigmoid(1.702 g) (u + 1) for g = min(z, limit), u = min(max(up, -limit), limit)
+__device__ __forceinline__ float gate_mul(float z, float up, int act, float limit) {
+  if (act == kActClampGate) {
+    z = fminf(z, limit);
+    return z * sigmoid_f(1.702f * z) * (fminf(fmaxf(up, -limit), limit) + 1.f);
+  }
+  const float w = act == kActSiluGate ? z : 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
   return z * sigmoid_f(w) * up;
 }
 // v: a row's 32 consecutive columns (16 gate, 16 up) -> its 16 gated values in v[0..15]
-__device__ __forceinline__ void gate_block(float* v, int act) {
+__device__ __forceinline__ void gate_block(float* v, int act, float limit) {
 #pragma unroll
-  for (int j = 0; j < kGateBlock; ++j) v[j] = gate_mul(v[j], v[j + kGateBlock], act == kActSiluGate);
+  for (int j = 0; j < kGateBlock; ++j) v[j] = gate_mul(v[j], v[j + kGateBlock], act, limit);
 }
 // 16 consecutive values, dst 16-byte aligned
 __device__ __forceinline__ void st_f16x(__nv_bfloat16* dst, const float* v) {

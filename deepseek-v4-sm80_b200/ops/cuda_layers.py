@@ -1,4 +1,4 @@
-"""Python wrappers around the sm_100a kernels of the layered models (csrc/residual.cu, latent_attn.cu, wkv.cu,
+"""Python wrappers around the sm_100a kernels of the layered models (csrc/residual.cu, latent_attn.cu, mingru.cu, wkv.cu,
 moe_bf16.cu, gemm_simt.cu), one function per facade op in :mod:`minisgl.ops.api`.  Activations are bf16 or fp32."""
 from __future__ import annotations
 
@@ -20,15 +20,19 @@ def _f32(dtype) -> I:
 
 
 # --------------------------------------------------------------------------- residual stream
-@tensors(ids="i32[T]", weight="bf16[_,D]", feedback="?i32[_]", slots="?i32[T]", table="?bf16[_,D]", positions="?i32[T]")
+@tensors(ids="i32[T]", weight="bf16[_,D]", feedback="?i32[_]", slots="?i32[T]", table="?bf16[_,D]", positions="?i32[T]",
+         pairs="?bf16[_,D]", tokens="?i32[_]")
 def embed_residual(ids, weight, dtype, feedback=None, slots=None, want_act=False, mul=1.0, table=None, positions=None,
-                   streams=None):
+                   streams=None, pairs=None, pair_mul=(0, 0), tokens=None, fb=None):
     t, d = ids.shape[0], weight.shape[1]
     x = torch.empty(*((t, d) if streams is None else (t, streams, d)), dtype=torch.float32, device=ids.device)
     act = torch.empty(t, d, dtype=dtype, device=ids.device) if want_act else None
+    buckets = 1 if pairs is None else pairs.shape[0] - 1
     nv.call("embed_residual", nv.ptr(ids), nv.ptr(feedback), nv.ptr(slots), nv.ptr(weight), nv.ptr(x), nv.ptr(act), F(mul),
-            nv.ptr(table), nv.ptr(positions), I(0 if table is None else table.shape[0]), I(streams or 1), I(t), I(d),
-            _f32(dtype))
+            nv.ptr(table), nv.ptr(positions), I(0 if table is None else table.shape[0]), I(streams or 1), nv.ptr(pairs),
+            I(buckets), I(pair_mul[0] % buckets), I(pair_mul[1] % buckets), nv.ptr(tokens),
+            nv.ptr(None if fb is None else fb.out_loc), nv.ptr(None if fb is None else fb.page_table),
+            I(0 if fb is None else fb.page_table.stride(0)), I(t), I(d), _f32(dtype))
     return x, act
 
 
@@ -52,7 +56,7 @@ def stream_norm(x, eps, dtype, pre, post, sub, experts, rows, keep):
 
 
 @tensors(x="f32[_,D]", gain="?f32[D]", rows="?i64[_]", add="?f32[_,D]", add2="?f32[_,D]", vec="?f32[D]")
-def residual_norm(x, gain, eps, dtype, mul=1.0, rows=None, add=None, add2=None, vec=None, experts=None, cast=False):
+def residual_norm(x, gain, eps, dtype, mul=1.0, rows=None, add=None, add2=None, vec=None, experts=None, cast=False, sub=None):
     n, d = x.shape
     erows = wts = idx = None
     topk = 0
@@ -60,9 +64,14 @@ def residual_norm(x, gain, eps, dtype, mul=1.0, rows=None, add=None, add2=None, 
         erows, wts, idx = experts
         topk = idx.shape[1]
         assert erows.dtype == dtype and erows.shape == (n * topk, d) and erows.is_contiguous()
+    y = bias = sub_gain = None
+    if sub is not None:
+        y, bias, sub_gain = sub
+        assert y.shape == (n, d) and y.dtype == torch.float32 and y.is_contiguous()
+        assert all(v is None or (v.shape == (d,) and v.dtype == torch.float32) for v in (bias, sub_gain))
     n_out = n if rows is None else rows.shape[0]
     out = torch.empty(n_out, d, dtype=dtype, device=x.device) if gain is not None or cast else None
-    nv.call("residual_norm", nv.ptr(x), nv.ptr(rows), nv.ptr(add), nv.ptr(add2), nv.ptr(vec), nv.ptr(erows),
+    nv.call("residual_norm", nv.ptr(x), nv.ptr(rows), nv.ptr(y), nv.ptr(bias), nv.ptr(sub_gain), nv.ptr(add), nv.ptr(add2), nv.ptr(vec), nv.ptr(erows),
             nv.ptr(wts), nv.ptr(idx), I(topk), nv.ptr(gain), F(eps), F(mul), nv.ptr(out), I(n_out), I(d), _f32(dtype))
     return out
 
@@ -130,37 +139,50 @@ def latent_store(x, gain, eps, cache, fb):
             I(x.shape[0]), I(x.shape[1]), _f32(x.dtype))
 
 
+@tensors(p="bf16|f32[T,_]s", gain="f32[R]", freq="f32[_]", cache="bf16|f32[_,_]")
+def latent_rotate_store(p, at_rot, at_c, gain, eps, freq, mul, cache, fb, heads, dim, whole):
+    t, rank, rot = p.shape[0], gain.shape[0], 2 * freq.shape[0]
+    assert p.dtype == cache.dtype and cache.shape[1] == rank + rot and p.shape[1] >= at_c + rank + rot
+    q = torch.empty(t, heads * (dim + rot), dtype=p.dtype, device=p.device) if whole else None
+    nv.call("latent_rotate_store", nv.ptr(p), I(p.stride(0)), I(at_rot), I(at_c), nv.ptr(gain), F(eps), nv.ptr(freq), F(mul),
+            nv.ptr(fb.positions), nv.ptr(fb.out_loc), nv.ptr(cache), nv.ptr(q), I(t), I(heads), I(dim), I(rot), I(rank),
+            _f32(p.dtype))
+    return q
+
+
 def latent_tiling(seg_lens, rows: int, heads: int, rank: int, max_context: int, sms: int):
-    """(rows per CTA, row tiles, key splits) of the tensor-core kernel.  Splitting the keys pays while the row tiles
+    """(rows per CTA, row tiles, key splits) of the tensor-core kernel.  rank: values of a cache row.  Splitting the keys pays while the row tiles
     alone leave SMs idle and a tile has several key tiles."""
     lens = seg_lens if seg_lens is not None else [1] * rows
     per_seg = max(lens) * heads
-    m = 16 if per_seg <= 16 else 32 if per_seg <= 32 else 64
+    m = 16 if per_seg <= 16 else 32 if per_seg <= 32 or rank > 512 else 64
     tiles = sum(-(-n * heads // m) for n in lens)
     rp = -(-rank // 128) * 128
-    smem = m * rp * 2 + 2 * 64 * rp * 2 + m * 68 * 4 + m * 64 * 2 + 16 * m
+    smem = m * rp * 2 + 2 * 64 * rp * 2 + m * 68 * 4 + m * 64 * 2 + 20 * m
     ctas = sms * max(1, min(SMEM_BYTES // smem, 4))
     ktiles = -(-max_context // 64)
     return m, tiles, max(1, min(ctas // max(tiles, 1), -(-ktiles // 2), 32))
 
 
-@tensors(q="bf16|f32[T,H,R]", cache="bf16|f32[_,R]")
-def latent_attention(q, cache, fb, scale):
+@tensors(q="bf16|f32[T,H,R]", cache="bf16|f32[_,_]", q_rot="?bf16|f32[T,_]s")
+def latent_attention(q, cache, fb, scale, q_rot, window):
     t, h, r = q.shape
-    assert q.dtype == cache.dtype
+    width = cache.shape[1]
+    assert q.dtype == cache.dtype and width - r == (0 if q_rot is None else q_rot.shape[1] // h)
     o = torch.empty_like(q)
     m = tiles = 0
     nsplit, acc, ml = 1, None, None
-    if q.dtype == torch.bfloat16 and r % 8 == 0 and r <= 512:
-        m, tiles, nsplit = latent_tiling(fb.seg_lens, t, h, r, fb.max_context, num_sms(q.device))
+    even = r % 8 == 0 and width % 8 == 0 and width <= 640 and (q_rot is None or (q_rot.stride(0) % 8 == 0 and q_rot.data_ptr() % 16 == 0))
+    if q.dtype == torch.bfloat16 and even:
+        m, tiles, nsplit = latent_tiling(fb.seg_lens, t, h, width, window_span(fb, window), num_sms(q.device))
         if nsplit > 1:
             acc = torch.empty(t * h, nsplit, r, dtype=torch.float32, device=q.device)
             ml = torch.empty(t * h, nsplit, 2, dtype=torch.float32, device=q.device)
     pt = fb.page_table
     nv.call("latent_attention", nv.ptr(q), nv.ptr(cache), nv.ptr(o), nv.ptr(fb.slots), nv.ptr(fb.positions), nv.ptr(pt),
             I(pt.stride(0)), nv.ptr(fb.seg_off), I(0 if fb.seg_off is None else fb.seg_off.shape[0] - 1),
-            nv.ptr(fb.num_valid), I(t), I(h), I(r), F(scale), I(m), I(tiles), I(nsplit), nv.ptr(acc), nv.ptr(ml),
-            _f32(q.dtype))
+            nv.ptr(fb.num_valid), I(t), I(h), I(r), nv.ptr(q_rot), I(0 if q_rot is None else q_rot.stride(0)), I(width - r),
+            I(window), F(scale), I(m), I(tiles), I(nsplit), nv.ptr(acc), nv.ptr(ml), _f32(q.dtype))
     return o
 
 
@@ -170,64 +192,104 @@ EXPAND_BYTES = 4 << 30                        # bound of the expanded keys and v
 ABSORBED_TFLOPS, EXPANDED_TFLOPS, GEMM_TFLOPS, EXPAND_US = 200.0, 900.0, 600.0, 25.0    # measured rates
 
 
-def prefers_expanded(q_dtype, fb, heads: int, dim: int, vdim: int, rank: int) -> bool:
+def window_span(fb, window: int, tile_tokens: int = 1) -> int:
+    """The most keys that a tile of so many tokens reads."""
+    return min(fb.max_context, window + tile_tokens - 1) if window else fb.max_context
+
+
+def prefers_expanded(q_dtype, fb, heads: int, dim: int, vdim: int, rank: int, rot: int = 0, window: int = 0) -> bool:
     """Whether a prefill forward should expand its requests' latents to keys and values (csrc/flash_attn.cu) instead of
     attending over the latents: expanding costs every request's whole context once, and then a query pays dim + vdim per
     key instead of twice the rank."""
     if fb.seg_ends is None or q_dtype != torch.bfloat16 or LATENT_PREFILL == "absorbed":
         return False
-    if dim % 8 or vdim % 8 or rank % 8 or dim > 128 or vdim > 128:
+    wide = dim + rot                 # of a query and an expanded key
+    if wide % 8 or vdim % 8 or rank % 8 or rot % 8 or wide > 128 or vdim > 128:
         return False
-    ctx = sum(-(-s // KV_ALIGN) * KV_ALIGN for s in fb.seg_ends)
-    if 2 * ctx * (heads * (dim + vdim) + rank) > EXPAND_BYTES:
+    reach = window or max(fb.seg_ends)
+    need = [min(s, n + reach - 1) for n, s in zip(fb.seg_lens, fb.seg_ends)]         # keys that a portion sees
+    ctx = sum(-(-s // KV_ALIGN) * KV_ALIGN for s in need)
+    if 2 * ctx * (heads * (wide + vdim) + rank + rot) > EXPAND_BYTES:
         return False
     if LATENT_PREFILL == "expanded":
         return True
-    pairs = sum(n * (s - n / 2) for n, s in zip(fb.seg_lens, fb.seg_ends))
-    tiled = sum(-(-n // 256) * 256 * (s - n / 2 + 64) for n, s in zip(fb.seg_lens, fb.seg_ends))
-    absorbed = 4e-6 * heads * rank * pairs / ABSORBED_TFLOPS \
+    each = [min(s - n / 2, reach) for n, s in zip(fb.seg_lens, fb.seg_ends)]         # keys that a query sees, on average
+    pairs = sum(n * k for n, k in zip(fb.seg_lens, each))
+    tiled = sum(-(-n // 256) * 256 * (k + (192 if window else 64)) for n, k in zip(fb.seg_lens, each))
+    absorbed = 2e-6 * heads * (2 * rank + rot) * pairs / ABSORBED_TFLOPS \
         + 2e-6 * sum(fb.seg_lens) * heads * rank * (dim + vdim) / GEMM_TFLOPS
-    expanded = 2e-6 * heads * (dim + vdim) * (tiled / EXPANDED_TFLOPS + ctx * rank / GEMM_TFLOPS) + EXPAND_US
+    expanded = 2e-6 * heads * ((wide + vdim) * tiled / EXPANDED_TFLOPS
+                               + ctx * (wide * (rank + rot) + vdim * rank) / GEMM_TFLOPS) + EXPAND_US
     return expanded < absorbed
 
 
 KV_ALIGN = 64       # a request's expanded keys start at a multiple of this (16-byte TMA boundaries of V^T)
 
 
-def _expanded_plan(fb, device):
-    """(request list [n, 3], work items [m, 5], expanded rows), one per forward: the same for all layers.  Items are
+def prompt_items(row: int, n: int, s: int, at: int, window: int = 0):
+    """Work items of the prompt kernel for a portion of ``n`` queries from row ``row`` on, the last ones of ``s`` keys that stand from
+    row ``at`` on: (first query row, queries, place of the first among the item's keys, first key row, keys).  With a window an item's
+    keys begin where its first query's do, rounded down so that TMA can fetch them."""
+    for q in range(0, n, 256):
+        m, pos = min(256, n - q), s - n + q
+        skip = max(0, pos - window + 1) // KV_ALIGN * KV_ALIGN if window else 0
+        yield row + q, m, pos - skip, at + skip, pos - skip + m
+
+
+def _expanded_plan(fb, device, window: int):
+    """(request list [n, 4], work items [m, 5], expanded rows), one per forward: the same for all layers of a window.  Items are
     ordered by the number of keys they see, longest first."""
-    plan = getattr(fb, "expanded_plan", None)
+    plans = fb.__dict__.setdefault("expanded_plans", {})
+    plan = plans.get(window)
     if plan is None:
         reqs, items, at, row = [], [], 0, 0
         for n, s, slot in zip(fb.seg_lens, fb.seg_ends, fb.seg_slots):
-            reqs.append((slot, s, at))
-            for q in range(0, n, 256):
-                m = min(256, n - q)
-                items.append((row + q, m, s - n + q, at, s - n + q + m))
-            at += -(-s // KV_ALIGN) * KV_ALIGN
+            key0 = max(0, s - n - window + 1) if window else 0
+            reqs.append((slot, s - key0, at, key0))
+            items += prompt_items(row, n, s - key0, at, window)
+            at += -(-(s - key0) // KV_ALIGN) * KV_ALIGN
             row += n
         items.sort(key=lambda i: -i[4])
         host = torch.tensor([v for t in (*reqs, *items) for v in t], dtype=torch.int32).pin_memory()
         dev = host.to(device, non_blocking=True)
-        k = 3 * len(reqs)
-        plan = fb.expanded_plan = (dev[:k], dev[k:], len(reqs), len(items), at)
+        k = 4 * len(reqs)
+        plan = plans[window] = (dev[:k], dev[k:], len(reqs), len(items), at)
     return plan
 
 
-@tensors(q="bf16[_,_]s", cache="bf16[_,R]", uk="bf16[_,R]", uv="bf16[_,R]")
-def expanded_attention(q, cache, fb, uk, uv, heads, scale):
-    t, dim, vdim, rank = q.shape[0], uk.shape[0] // heads, uv.shape[0] // heads, cache.shape[1]
-    reqs, items, n_reqs, n_items, rows = _expanded_plan(fb, q.device)
-    ctx = torch.empty(rows, rank, dtype=q.dtype, device=q.device)
+@tensors(q="bf16[_,_]s", cache="bf16[_,W]", uk="bf16[_,W]", uv="bf16[_,_]")
+def expanded_attention(q, cache, fb, uk, uv, heads, scale, window):
+    t, dim, vdim, width, rank = q.shape[0], uk.shape[0] // heads, uv.shape[0] // heads, cache.shape[1], uv.shape[1]
+    reqs, items, n_reqs, n_items, rows = _expanded_plan(fb, q.device, window)
+    ctx = torch.empty(rows, width, dtype=q.dtype, device=q.device)
     pt = fb.page_table
     nv.call("latent_gather", nv.ptr(cache), nv.ptr(ctx), nv.ptr(reqs), I(n_reqs), I(rows), nv.ptr(pt), I(pt.stride(0)),
-            I(rank))
-    k, vt = linear(ctx, uk), linear(uv, ctx)
+            I(width))
+    k, vt = linear(ctx, uk), linear(uv, ctx[:, :rank])
     out = torch.empty(t, heads * vdim, dtype=q.dtype, device=q.device)
     nv.call("flash_attention", nv.ptr(q), I(q.stride(0)), nv.ptr(k), nv.ptr(vt), nv.ptr(out), nv.ptr(items), I(n_items),
-            I(t), I(rows), I(heads), I(heads), I(dim), I(vdim), F(scale), F(0.0), nv.ptr(None), nv.ptr(None), I(0), nv.ptr(None))
+            I(t), I(rows), I(heads), I(heads), I(dim), I(vdim), F(scale), F(0.0), nv.ptr(None), nv.ptr(None), I(0), nv.ptr(None), nv.ptr(None),
+            I(window), nv.ptr(None), nv.ptr(None), I(0))
     return out
+
+
+# --------------------------------------------------------------------------- element-wise recurrence
+GRU_TILES = (32, 16, 8)          # elements per CTA of the parallel form
+
+
+@tensors(p="f32[T,_]s", bias_z="f32[W]", bias_u="f32[W]", state="f32[_,W]")
+def mingru(p, at_u, at_g, bias_z, bias_u, state, fb, dtype):
+    t, width = p.shape[0], state.shape[1]
+    assert p.shape[1] >= at_g + width
+    y = torch.empty(t, width, dtype=dtype, device=p.device)
+    segs = t if fb.seg_off is None else fb.seg_off.shape[0] - 1
+    fill = num_sms(p.device) * 2 // 3
+    ct = next((c for c in GRU_TILES if -(-width // c) * segs >= fill), GRU_TILES[-1])
+    nv.call("mingru", nv.ptr(p), I(p.stride(0)), I(at_u), I(at_g), nv.ptr(bias_z), nv.ptr(bias_u), nv.ptr(state), nv.ptr(y),
+            nv.ptr(fb.slots), nv.ptr(fb.positions), nv.ptr(fb.seg_off), I(segs),
+            nv.ptr(fb.num_valid if fb.seg_off is None else None), I(max(fb.seg_lens) if fb.seg_lens is not None else 1), I(ct),
+            I(width), _f32(dtype))
+    return y
 
 
 # --------------------------------------------------------------------------- recurrent time mixing

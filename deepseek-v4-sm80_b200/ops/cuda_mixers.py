@@ -9,7 +9,7 @@ import torch
 
 from . import native as nv
 from .cuda import num_sms
-from .cuda_layers import KV_ALIGN, SMEM_BYTES, _chunk_plan, _f32
+from .cuda_layers import KV_ALIGN, SMEM_BYTES, _chunk_plan, _f32, prompt_items, window_span
 from .gemm import ACTS, _tma_ok, linear
 from .native import F, I
 from .tensorcheck import tensors
@@ -35,18 +35,18 @@ def residual_layer_norm(x, eps, dtype, norm, sub, add, rows, keep):
 
 
 # --------------------------------------------------------------------------- gated feed-forward
-GATE_ACTS = {"gelu_tanh": "gelu_gate", "silu": "silu_gate"}
+GATE_ACTS = {"gelu_tanh": "gelu_gate", "silu": "silu_gate", "clamp": "clamp_gate"}
 
 
-def gated_linear(h, w, act, block):
+def gated_linear(h, w, act, block, limit):
     if act not in GATE_ACTS or block != 16:
         raise ValueError(f"no kernel for the gate {act!r} in blocks of {block}")
     if _tma_ok(h, w, h.shape[1]):
-        return linear(h, w, act=GATE_ACTS[act])
+        return linear(h, w, act=GATE_ACTS[act], limit=limit)
     gu = linear(h, w)
     t, f = h.shape[0], w.shape[0] // 2
     out = torch.empty(t, f, dtype=h.dtype, device=h.device)
-    nv.call("gate_mul", nv.ptr(gu), nv.ptr(out), I(t), I(f), I(ACTS[GATE_ACTS[act]]), _f32(h.dtype))
+    nv.call("gate_mul", nv.ptr(gu), nv.ptr(out), I(t), I(f), I(ACTS[GATE_ACTS[act]]), F(limit), _f32(h.dtype))
     return out
 
 
@@ -65,6 +65,22 @@ def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads, kv_heads, dim
     return q
 
 
+@tensors(qkv="bf16|f32[T,_]s", bias="?f32[_]", gain="?f32[2,_]", freq="?f32[_]", vfreq="?f32[_]", keys="bf16|f32[R,_]",
+         values="bf16|f32[R,_]")
+def head_store(qkv, bias, gain, eps, freq, mul, vfreq, halves, keys, values, fb, heads, kv_heads, dim, vdim):
+    t = qkv.shape[0]
+    assert qkv.dtype == keys.dtype == values.dtype and qkv.shape[1] == (heads + kv_heads) * dim + kv_heads * vdim
+    assert keys.shape[1] == kv_heads * dim and values.shape[1] == kv_heads * vdim
+    assert (gain is None or gain.shape[1] == dim) and (vfreq is None or 2 * vfreq.shape[0] == vdim)
+    q = torch.empty(t, heads, dim, dtype=qkv.dtype, device=qkv.device)
+    turn = None if vfreq is None else torch.empty(t, vdim // 2, 2, dtype=torch.float32, device=qkv.device)
+    nv.call("head_store", nv.ptr(qkv), I(qkv.stride(0)), nv.ptr(bias), nv.ptr(gain), F(eps), nv.ptr(freq),
+            I(0 if freq is None else freq.shape[0]), I(1 if halves else 0), F(mul), nv.ptr(vfreq), nv.ptr(turn),
+            nv.ptr(fb.positions), nv.ptr(fb.out_loc), nv.ptr(q), nv.ptr(keys), nv.ptr(values), I(t), I(heads), I(kv_heads), I(dim),
+            I(vdim), _f32(qkv.dtype))
+    return q, turn
+
+
 # Portions of at least FLASH_MIN tokens run on the prompt kernel (csrc/flash_attn.cu), shorter ones and single tokens on
 # grouped_attn.cu.  MINISGL_GROUPED_PREFILL: auto, flash (every portion that the kernel takes) or rows (none).
 GROUPED_PREFILL = os.environ.get("MINISGL_GROUPED_PREFILL", "auto")
@@ -79,14 +95,19 @@ def row_tile(rows_per_request: int) -> int:
 def _split_keys(tiles: int, kv_heads: int, m: int, width: int, max_context: int, sms: int) -> int:
     """Ways to split the keys: pays while the row tiles alone leave SMs idle and a tile has several key tiles."""
     p = 64 if width <= 64 else 128 if width <= 128 else 256
-    smem = m * p * 2 + 4 * 64 * p * 2 + m * 68 * 4 + m * 64 * 2 + 16 * m
+    smem = m * p * 2 + 4 * 64 * p * 2 + m * 68 * 4 + m * 64 * 2 + 20 * m
     ctas = sms * max(1, min(SMEM_BYTES // smem, 4))
     return max(1, min(ctas // max(tiles * kv_heads, 1), -(-max_context // 128), 32))
 
 
-def _pieces(fb, chunk: int):
-    """The portions of a forward, cut where a chunk of keys ends: (queries, keys seen by the last one, slot, first key)."""
+def _pieces(fb, chunk: int, window: int):
+    """The portions of a forward, cut where a chunk of keys ends: (queries, keys up to the last one's own, slot, first key).  With a
+    window the first key is the first that any of them sees."""
     for n, s, slot in zip(fb.seg_lens, fb.seg_ends, fb.seg_slots):
+        if window:
+            key0 = max(0, s - n - window + 1)
+            yield n, s - key0, slot, key0
+            continue
         at, size = s - n, chunk or s
         while at < s:
             key0 = at // size * size
@@ -95,16 +116,16 @@ def _pieces(fb, chunk: int):
             at = end
 
 
-def _prefill_plan(fb, device, group: int, flash_ok: bool, chunk: int):
+def _prefill_plan(fb, device, group: int, flash_ok: bool, chunk: int, window: int):
     """How the requests of a prefill forward are spread over the two kernels; the same for all layers with this many query
-    heads to a key head and this chunk size: (flash requests [n, 4], flash items [m, 5], n, m, gathered rows, row tiles [k, 2],
+    heads to a key head and this chunk size or window: (flash requests [n, 4], flash items [m, 5], n, m, gathered rows, row tiles [k, 2],
     k, rows per tile, longest context among the row tiles)."""
     plans = fb.__dict__.setdefault("grouped_plans", {})
-    key = (group, flash_ok, GROUPED_PREFILL, FLASH_MIN, chunk)
+    key = (group, flash_ok, GROUPED_PREFILL, FLASH_MIN, chunk, window)
     if key in plans:
         return plans[key]
     least = 1 if GROUPED_PREFILL == "flash" else FLASH_MIN
-    pieces = list(_pieces(fb, chunk))
+    pieces = list(_pieces(fb, chunk, window))
     flash = [flash_ok and n >= least for n, _, _, _ in pieces]
     few = [p[0] for p, f in zip(pieces, flash) if not f]
     m = row_tile(max(few) * group) if few else 16
@@ -112,13 +133,11 @@ def _prefill_plan(fb, device, group: int, flash_ok: bool, chunk: int):
     for (n, s, slot, key0), f in zip(pieces, flash):
         if f:
             reqs.append((slot, s, at, key0))
-            for q in range(0, n, 256):
-                k = min(256, n - q)
-                items.append((row + q, k, s - n + q, at, s - n + q + k))
+            items += prompt_items(row, n, s, at, window)
             at += -(-s // KV_ALIGN) * KV_ALIGN
         else:
             tiles += [(r, min(r + m, (row + n) * group)) for r in range(row * group, (row + n) * group, m)]
-            longest = max(longest, s)
+            longest = max(longest, min(s, window + m // group) if window else s)
         row += n
     items.sort(key=lambda i: -i[4])                   # the longest first
     host = torch.tensor([v for t in (*reqs, *items, *tiles) for v in t], dtype=torch.int32).pin_memory()
@@ -128,21 +147,26 @@ def _prefill_plan(fb, device, group: int, flash_ok: bool, chunk: int):
     return plans[key]
 
 
-@tensors(q="bf16|f32[T,H,D]", keys="bf16|f32[R,_]", values="bf16|f32[R,_]", sink="?f32[H]", rel="?f32[H,_]", slope="?f32[H]")
-def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, slope, chunk):
+@tensors(q="bf16|f32[T,H,D]", keys="bf16|f32[R,_]", values="bf16|f32[R,_]", sink="?f32[H]", rel="?f32[H,_]", slope="?f32[H]",
+         wbias="?f32[H]", turn="?f32[T,_,2]", gate="?bf16|f32[T,H]s")
+def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, slope, chunk, window, wbias, turn, gate):
     t, heads, dim = q.shape
     group, kw, vw = heads // kv_heads, keys.shape[1], values.shape[1]
     vdim = vw // kv_heads
-    assert q.dtype == keys.dtype == values.dtype and kw == kv_heads * dim
+    assert q.dtype == keys.dtype == values.dtype and kw == kv_heads * dim and (gate is None or gate.dtype == q.dtype)
+    assert turn is None or 2 * turn.shape[1] == vdim
+    ends = (nv.ptr(wbias), nv.ptr(turn), nv.ptr(gate), I(0 if gate is None else gate.stride(0)))
     out = torch.empty(t, heads * vdim, dtype=q.dtype, device=q.device)
     pt, n_rel = fb.page_table, 0 if rel is None else rel.shape[1]
     even = q.dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0
-    tiles, n_tiles, m, longest = None, 0, 0, min(fb.max_context, chunk) if chunk else fb.max_context
+    tiles, n_tiles, m, longest = None, 0, 0, min(fb.max_context, chunk) if chunk else window_span(fb, window)
     if even and fb.seg_lens is not None:
         ctx = sum(-(-s // KV_ALIGN) * KV_ALIGN for s in fb.seg_ends)
         flash_ok = max(dim, vdim) <= 128 and GROUPED_PREFILL != "rows" and 2 * ctx * (kw + vw) <= FLASH_BYTES
-        flash_ok = flash_ok and not (slope is not None and (softcap or rel is not None))
-        reqs, items, n_reqs, n_items, rows, tiles, n_tiles, m, longest = _prefill_plan(fb, q.device, group, flash_ok, chunk)
+        flash_ok = flash_ok and not (slope is not None and (softcap or rel is not None)) and (turn is None or vdim % 32 == 0)
+        flash_ok = flash_ok and not (wbias is not None and (softcap or rel is not None or slope is not None))
+        reqs, items, n_reqs, n_items, rows, tiles, n_tiles, m, longest = _prefill_plan(fb, q.device, group, flash_ok, chunk,
+                                                                                                  window)
         if n_items:
             ck = torch.empty(rows, kw, dtype=q.dtype, device=q.device)
             cv = torch.empty(vw, rows, dtype=q.dtype, device=q.device)
@@ -150,7 +174,7 @@ def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, 
                     nv.ptr(pt), I(pt.stride(0)), I(kw), I(vw))
             nv.call("flash_attention", nv.ptr(q), I(heads * dim), nv.ptr(ck), nv.ptr(cv), nv.ptr(out), nv.ptr(items),
                     I(n_items), I(t), I(rows), I(heads), I(kv_heads), I(dim), I(vdim), F(scale), F(softcap), nv.ptr(sink),
-                    nv.ptr(rel), I(n_rel), nv.ptr(slope))
+                    nv.ptr(rel), I(n_rel), nv.ptr(slope), ends[0], I(window), *ends[1:])
         if n_tiles == 0:
             return out
     elif even:
@@ -163,13 +187,13 @@ def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, 
     nsplit, acc, ml = 1, None, None
     if m:
         nsplit = _split_keys(n_tiles, kv_heads, m, max(dim, vdim), longest, num_sms(q.device))
-        if nsplit > 1:
+        if nsplit > 1 or turn is not None or gate is not None:
             acc = torch.empty(t * heads, nsplit, vdim, dtype=torch.float32, device=q.device)
             ml = torch.empty(t * heads, nsplit, 2, dtype=torch.float32, device=q.device)
     nv.call("grouped_attention", nv.ptr(q), nv.ptr(keys), nv.ptr(values), nv.ptr(out), nv.ptr(fb.slots), nv.ptr(fb.positions),
             nv.ptr(pt), I(pt.stride(0)), nv.ptr(tiles), I(n_tiles), nv.ptr(fb.num_valid), I(t), I(kv_heads), I(group), I(dim),
-            I(vdim), F(scale), F(softcap), nv.ptr(sink), nv.ptr(rel), I(n_rel), nv.ptr(slope), I(chunk), I(m), I(nsplit), nv.ptr(acc),
-            nv.ptr(ml), _f32(q.dtype))
+            I(vdim), F(scale), F(softcap), nv.ptr(sink), nv.ptr(rel), I(n_rel), nv.ptr(slope), I(chunk), I(window), *ends, I(m),
+            I(nsplit), nv.ptr(acc), nv.ptr(ml), _f32(q.dtype))
     return out
 
 

@@ -15,7 +15,7 @@ import ctypes
 import torch
 
 from . import native as nv
-from .native import I, L
+from .native import F, I, L
 
 _COUNTERS = {}
 NUM_SMS_HINT = 148
@@ -110,8 +110,8 @@ def _ws(m, n, bn, batches, splits, device):
 
 
 # epilogue activations of the projections (csrc/vec.cuh: GemmAct), applied to the fp32 sum
-ACTS = {None: 0, "relu2": 1, "tanh": 2, "gelu_gate": 3, "silu_gate": 4}
-GATES = ("gelu_gate", "silu_gate")          # half as many columns come out (TMA operands only)
+ACTS = {None: 0, "relu2": 1, "tanh": 2, "gelu_gate": 3, "silu_gate": 4, "clamp_gate": 5}
+GATES = ("gelu_gate", "silu_gate", "clamp_gate")          # half as many columns come out (TMA operands only)
 
 
 def _act(y, act):
@@ -141,7 +141,7 @@ def gemm_bf16(x, w, out=None, out_dtype=torch.bfloat16, accumulate=False, bn=0, 
     ws, cnt = _ws(m, n, bn, 1, splits, x.device)
     nv.call("gemm_bf16", nv.ptr(x2), nv.ptr(w), nv.ptr(o2), I(m), I(n), I(k), I(x2.stride(0)), I(w.stride(0)),
             I(o2.stride(0)), I(1 if out.dtype == torch.float32 else 0), I(1 if accumulate else 0), I(bn), I(1),
-            I(splits), nv.ptr(ws), nv.ptr(cnt), I(ACTS[act]))
+            I(splits), nv.ptr(ws), nv.ptr(cnt), I(ACTS[act]), F(0.0))
     return out
 
 
@@ -158,13 +158,14 @@ def prefill_tiles(m: int, n: int, groups: int) -> int:
     return -(-m // 128) * -(-n // 256) * groups if m > 128 else 0
 
 
-def linear(x, w, out=None, out_dtype=None, accumulate=False, act=None):
+def linear(x, w, out=None, out_dtype=None, accumulate=False, act=None, limit=0.0):
     """``x [T, K] @ w [N, K]^T`` for bf16 weights and bf16 or fp32 activations (rows may be strided).  bf16 runs on the
-    tensor cores; fp32 activations, and bf16 rows that TMA cannot fetch, on the fp32 kernel (csrc/gemm_simt.cu)."""
-    return grouped_linear(x, w, 1, out, out_dtype, accumulate, act)
+    tensor cores; fp32 activations, and bf16 rows that TMA cannot fetch, on the fp32 kernel (csrc/gemm_simt.cu).  limit: of the
+    activation "clamp_gate"."""
+    return grouped_linear(x, w, 1, out, out_dtype, accumulate, act, limit)
 
 
-def grouped_linear(x, w, groups: int, out=None, out_dtype=None, accumulate=False, act=None):
+def grouped_linear(x, w, groups: int, out=None, out_dtype=None, accumulate=False, act=None, limit=0.0):
     """``groups`` projections side by side in one launch: x [T, G*K] (rows may be strided), w [G*N, K] -> [T, G*N],
     group g reading its own K columns."""
     t, k = x.shape[0], x.shape[1] // groups
@@ -182,13 +183,13 @@ def grouped_linear(x, w, groups: int, out=None, out_dtype=None, accumulate=False
     if _tma_ok(x, w, k):
         if prefill_tiles(t, n, groups) >= PREFILL_MIN_TILES:
             nv.call("gemm_prefill", nv.ptr(x), nv.ptr(w), nv.ptr(out), I(t), I(n), I(k), I(x.stride(0)), I(w.stride(0)),
-                    I(out.stride(0)), f32, I(1 if accumulate else 0), I(ACTS[act]), I(groups), I(NUM_SMS_HINT))
+                    I(out.stride(0)), f32, I(1 if accumulate else 0), I(ACTS[act]), F(limit), I(groups), I(NUM_SMS_HINT))
             return out
         bn, splits = pick_tiling(t, n, (k + 63) // 64, groups, False, 0, 0)
         ws, cnt = _ws(t, n, bn, groups, splits, x.device)
         nv.call("gemm_bf16", nv.ptr(x), nv.ptr(w), nv.ptr(out), I(t), I(n), I(k), I(x.stride(0)), I(w.stride(0)),
                 I(out.stride(0)), f32, I(1 if accumulate else 0), I(bn), I(groups), I(splits), nv.ptr(ws), nv.ptr(cnt),
-                I(ACTS[act]))
+                I(ACTS[act]), F(limit))
     else:
         assert act not in GATES
         nv.call("gemm_simt", nv.ptr(x), nv.ptr(w), nv.ptr(out), I(t), I(n), I(k), I(x.stride(0)), I(w.stride(0)),
@@ -255,7 +256,7 @@ def gemm_bf16_grouped(x, w, groups: int, out=None):
     bn, splits = pick_tiling(t, n, (k + 63) // 64, groups, False, 0, 0)
     ws, cnt = _ws(t, n, bn, groups, splits, x.device)
     nv.call("gemm_bf16", nv.ptr(x), nv.ptr(w), nv.ptr(out), I(t), I(n), I(k), I(x.stride(0)), I(w.stride(0)),
-            I(out.stride(0)), I(0), I(0), I(bn), I(groups), I(splits), nv.ptr(ws), nv.ptr(cnt), I(0))
+            I(out.stride(0)), I(0), I(0), I(bn), I(groups), I(splits), nv.ptr(ws), nv.ptr(cnt), I(0), F(0.0))
     return out
 
 

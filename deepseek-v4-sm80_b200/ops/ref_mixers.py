@@ -6,7 +6,7 @@ import math
 
 import torch
 
-from .ref_layers import _rms, segments
+from .ref_layers import _hidden, _rms, segments
 
 
 def _layer_norm(x, w, b, eps):
@@ -26,10 +26,13 @@ def residual_layer_norm(x, eps, dtype, norm, sub, add, rows, keep):
     return None if norm is None else _layer_norm(y, norm[0], norm[1], eps).to(dtype)
 
 
-def gated_linear(h, w, act, block):
+def gated_linear(h, w, act, block, limit):
     y = (h.float() @ w.float().t()).to(h.dtype).float().view(h.shape[0], -1, 2, block)
     g, u = y[:, :, 0], y[:, :, 1]
-    if act == "silu":
+    if act == "clamp":
+        g = g.clamp(max=limit)
+        a, u = g * torch.sigmoid(1.702 * g), u.clamp(-limit, limit) + 1.0
+    elif act == "silu":
         a = g * torch.sigmoid(g)
     else:
         assert act == "gelu_tanh"
@@ -69,7 +72,33 @@ def rotate_store(qkv, bias, freq, q_temp, keys, values, fb, heads, kv_heads, dim
     return q.to(qkv.dtype)
 
 
-def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, slope, chunk):
+def head_store(qkv, bias, gain, eps, freq, mul, vfreq, halves, keys, values, fb, heads, kv_heads, dim, vdim):
+    t, pos = qkv.shape[0], fb.positions.float()
+    x = qkv.float() if bias is None else qkv.float() + bias
+    q, k, v = (y.reshape(t, -1, n) for y, n in zip(x.split([heads * dim, kv_heads * dim, kv_heads * vdim], 1), (dim, dim, vdim)))
+    if gain is not None:
+        q, k = _rms(q, eps) * gain[0], _rms(k, eps) * gain[1]
+
+    def turn(y, f, m):
+        if f is None:
+            return y
+        n, a = f.shape[0], pos[:, None, None] * f
+        c, s = torch.cos(a) * m, torch.sin(a) * m
+        if halves:
+            u, w = y[..., :n], y[..., n:2 * n]
+            return torch.cat([u * c - w * s, w * c + u * s, y[..., 2 * n:]], -1)
+        u, w = y[..., 0:2 * n:2], y[..., 1:2 * n:2]
+        return torch.cat([torch.stack([u * c - w * s, w * c + u * s], -1).flatten(2), y[..., 2 * n:]], -1)
+
+    q, k, v = turn(q, freq, mul), turn(k, freq, mul), turn(v, vfreq, 1.0)
+    ok = fb.out_loc >= 0
+    at = fb.out_loc[ok].long()
+    keys[at], values[at] = k[ok].flatten(1).to(keys.dtype), v[ok].flatten(1).to(values.dtype)
+    angles = None if vfreq is None else pos[:, None] * vfreq
+    return q.to(qkv.dtype), None if vfreq is None else torch.stack([torch.cos(angles), torch.sin(angles)], -1)
+
+
+def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, slope, chunk, window, wbias, turn, gate):
     t, heads, dim = q.shape
     vdim, group = values.shape[1] // kv_heads, heads // kv_heads
     out = torch.empty(t, heads, vdim, dtype=q.dtype)
@@ -86,15 +115,28 @@ def grouped_attention(q, keys, values, fb, kv_heads, scale, softcap, sink, rel, 
             s = s + rel[:, away.clamp(0, rel.shape[1] - 1)]
         if slope is not None:
             s = s - slope[:, None, None] * away
-        hidden = away < 0
+        hidden = _hidden(fb, a, b, n, window)
         if chunk:
             hidden = hidden | (torch.arange(n)[None, :] < (fb.positions[a:b].long() // chunk * chunk)[:, None])
         s = s.masked_fill(hidden, float("-inf"))
+        if wbias is not None:
+            p = torch.sigmoid(s + wbias[:, None, None])
+            out[a:b] = _finish(torch.einsum("htj,jhe->the", p, v), a, b, turn, gate).to(q.dtype)
+            continue
         if sink is not None:
             s = torch.cat([s, sink[:, None, None].expand(heads, b - a, 1)], -1)
         p = torch.softmax(s, -1)[..., :n]
-        out[a:b] = torch.einsum("htj,jhe->the", p, v).to(q.dtype)
+        out[a:b] = _finish(torch.einsum("htj,jhe->the", p, v), a, b, turn, gate).to(q.dtype)
     return out.view(t, heads * vdim)
+
+
+def _finish(o, a, b, turn, gate):
+    """Results [b - a, H, e] of the rows a .. b - 1, turned back and gated."""
+    if turn is not None:
+        u, v = o.chunk(2, -1)
+        c, s = turn[a:b, None, :, 0], turn[a:b, None, :, 1]
+        o = torch.cat([u * c + v * s, v * c - u * s], -1)
+    return o if gate is None else o * torch.sigmoid(gate[a:b].float())[..., None]
 
 
 def conv_unit(p, taps, before, fb, heads, kv_heads, dim, vdim):
