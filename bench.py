@@ -44,7 +44,7 @@ def parse():
     ap.add_argument("--moe-mode", default="ep", choices=["ep", "tp"])
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--no-fused-comm", action="store_true")
-    ap.add_argument("--design", default="", choices=["", "bedalorn", "buvalix", "zazilix"],
+    ap.add_argument("--design", default="", choices=["", "bedalorn", "buvalix", "zazilix", "sakevik"],
                     help="instead of the headline: prefill / decode throughput of this design beside the closest other "
                          "model at equal size (one JSON line per model and workload, one GPU)")
     ap.add_argument("--sizes", default="small,large", help="with --design: model sizes to run")

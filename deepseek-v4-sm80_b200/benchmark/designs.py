@@ -1,13 +1,14 @@
 """Prefill and decode throughput of a layered design beside the closest other model at equal size: Bedalorn beside DeepSeek-V4,
 Buvalix beside Bedalorn, Zazilix beside Bedalorn (whose experts are the like feed-forwards) and Buvalix (whose recurrence and
-attention are the like mixers).
+attention are the like mixers), Sakevik beside Buvalix (the like feed-forwards, attention and norms) and Bedalorn (the like latent
+attention).
 
-    python bench.py --design bedalorn|buvalix|zazilix [--sizes small,large] [--profile]
+    python bench.py --design bedalorn|buvalix|zazilix|sakevik [--sizes small,large] [--profile]
 
 Equal size: the same width, layer runs, attention heads, vocabulary and feed-forward weights (DeepSeek-V4: the same experts;
 Buvalix's gated feed-forwards have three matrices, so the Bedalorn model beside it has dense ones half as wide again; Zazilix has
-one expert less than the Bedalorn model with experts everywhere, and a shared one), random
-weights, one GPU, through the offline API.  Per model and workload one JSON line: device time of the forwards (CUDA
+one expert less than the Bedalorn model with experts everywhere, and a shared one; Sakevik's windows of 1 024 and 2 048 positions
+hold all of a short prompt), random weights, one GPU, through the offline API.  Per model and workload one JSON line: device time of the forwards (CUDA
 events), tokens per second, and with ``--profile`` the per-launcher share of one eager forward of each phase.
 Workloads: prefill forwards of 8 x 1 024 and 1 x 8 192 tokens; decode steps of 128 sequences at 1 024 tokens of context and
 of 8 sequences at 8 192.
@@ -82,6 +83,18 @@ def zazilix_config(size: str):
     ff = MixtureSpec(eff, e - 1, top - 1, 8, 1.0, eff)
     layers = tuple(LayerSpec((memory, both, mamba, both)[i % 4], ff) for i in range(n * passes))
     return ZazilixConfig(layers, d, vocab, 1e-6, 4, 1.0, 1 << 14, max_position=1 << 14)
+
+
+def sakevik_config(size: str):
+    from minisgl.models.layered_config import LayerSpec, RotaryScaling
+    from minisgl.models.sakevik_config import (ClampedSpec, MinGRUSpec, PairEmbeddingSpec, RotarySpec, SakevikConfig,
+                                               SigmoidAttentionSpec, WindowLatentSpec)
+
+    d, h, g, _, _, rank, ff, n, passes, vocab = DENSE_SIZES[size]
+    sigmoid = SigmoidAttentionSpec(h, g, 128, 128, 128 ** -0.5, 1024, RotarySpec(128, 1e5))
+    latent = WindowLatentSpec(h, 96, 32, 128, rank, 128 ** -0.5, 2048, RotarySpec(32, 1e5, RotaryScaling(8.0, 4096, 32.0, 1.0)))
+    layers = tuple(LayerSpec((sigmoid, latent, MinGRUSpec(d), sigmoid)[i % 4], ClampedSpec(ff, 7.0)) for i in range(n * passes))
+    return SakevikConfig(layers, d, vocab, 1e-6, 1.0, PairEmbeddingSpec(4 * vocab, 31, 17), 1.0, max_position=1 << 17)
 
 
 def bedalorn_experts_config(size: str):
@@ -183,6 +196,7 @@ PAIRS = {
     "bedalorn": {"bedalorn": bedalorn_config, "dsv4": dsv4_config},
     "buvalix": {"buvalix": buvalix_config, "bedalorn": bedalorn_dense_config},
     "zazilix": {"zazilix": zazilix_config, "bedalorn": bedalorn_experts_config, "buvalix": buvalix_config},
+    "sakevik": {"sakevik": sakevik_config, "buvalix": buvalix_config, "bedalorn": bedalorn_dense_config},
 }
 
 

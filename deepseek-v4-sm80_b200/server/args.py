@@ -62,7 +62,7 @@ class ServerArgs(SchedulerConfig):
 
 
 def build_parser() -> argparse.ArgumentParser:
-    p = argparse.ArgumentParser(prog="minisgl", description="B200-native serving engine (DeepSeek-V4, Bedalorn, Buvalix, Zazilix)")
+    p = argparse.ArgumentParser(prog="minisgl", description="B200-native serving engine (DeepSeek-V4, Bedalorn, Buvalix, Zazilix, Sakevik)")
     p.add_argument("--model", "--model-path", dest="model_path", required=True)
     p.add_argument("--served-model-name", default=None)
     p.add_argument("--tp-size", "--tensor-parallel-size", dest="tp_size", type=int, default=1)

@@ -13,7 +13,7 @@ MODELS = {
     "recurrent": P.config([P.mingru_layer(120, P.dense(24)), P.mingru_layer(36), P.mingru_layer(64)], width=64, vocab=80, buckets=7),
     # attention only: pages can be shared between requests; windows of whole pages, longer than most sequences, and of one position
     "attention": P.config([P.latent_layer(2, 32, 8, 16, 24, 64, ff=P.dense(32, 0.5)), P.attention_layer(20, 2, 16, 32, 64, 8),
-                           P.attention_layer(3, 3, 24, 8, 1, 24), P.latent_layer(5, 8, 24, 24, 64, 700, scaling=(2.0, 300, 4.0, 2.0)),
+                           P.attention_layer(3, 3, 24, 8, 1, 24), P.latent_layer(5, 8, 24, 24, 64, 700, scale=0.1, scaling=(2.0, 300, 4.0, 2.0)),
                            P.attention_layer(34, 1, 8, 16, 500, 4, 100.0, 0.5)], width=128, vocab=96),
     # sizes of one
     "single": P.config([P.attention_layer(1, 1, 2, 2, 2, 2), P.mingru_layer(1), P.latent_layer(1, 1, 2, 1, 1, 3)], width=48, vocab=64,
@@ -23,11 +23,13 @@ MODELS = {
                         P.mingru_layer(19, P.dense(13)), P.attention_layer(2, 2, 7, 6, 40, 4)], width=50, vocab=77, buckets=1009,
                        mul_prev=2654435761, mul_cur=40503),
     # heads wider than the prompt kernel takes, latents wider than a 64-row tile
-    "wide": P.config([P.attention_layer(2, 1, 160, 144, 90, 64), P.latent_layer(2, 64, 64, 48, 512, 80), P.mingru_layer(300),
-                      P.latent_layer(2, 96, 48, 136, 200, 50), P.attention_layer(2, 2, 96, 320, 30, 96)], width=72, vocab=88),
+    "wide": P.config([P.attention_layer(2, 1, 160, 144, 90, 64, scale=0.1), P.latent_layer(2, 64, 64, 48, 512, 80, scale=0.04), P.mingru_layer(300),
+                      P.latent_layer(2, 96, 48, 136, 200, 50, scale=0.04), P.attention_layer(2, 2, 96, 320, 30, 96, scale=0.1)], width=72, vocab=88),
 }
 LIMIT = {torch.float32: 1e-4, torch.bfloat16: 5e-2}
-STRAY, WORST = 0.02, 0.12
+# The stream enters the sub-layers unnormed and a norm stands behind them: where an output is a small difference its rounding is
+# amplified, with every backend at the same places.
+STRAY, WORST = 0.02, 0.2
 
 
 class Case(layered_checks.Case):
