@@ -214,8 +214,115 @@ struct HeadStoreArgs {
   int heads, kv_heads, dim, vdim;
 };
 
-// One CTA per token.  The row with its bias passes through shared memory, where a warp norms a head in place and partners meet.
-// W consecutive values per thread and access.
+// One CTA per token, the row in registers: a thread's unit is eight values of a head, two groups of four that hold each other's
+// partners.  Heads of q and k are a power of two of units wide, so that the lanes of a head sum up its squares.  Few tokens take a
+// thread per unit (NU = 1), many take CTAs of kUnitThreads.
+constexpr int kUnitThreads = 128;
+template <typename T, int NU>
+__global__ void __launch_bounds__(NU == 1 ? 1024 : kUnitThreads) head_store_units_kernel(const T* __restrict__ qkv, T* __restrict__ q,
+                                                                        T* __restrict__ keys, T* __restrict__ values,
+                                                                        const HeadStoreArgs a) {
+  pdl_entry();
+  extern __shared__ __align__(16) float hs_row[];
+  const int t = blockIdx.x, pos = a.pos[t], loc = a.out_loc[t], tid = threadIdx.x, nt = blockDim.x;
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim, n = nq + nk + nv, vhalf = a.vdim / 2;
+  float2* cs = reinterpret_cast<float2*>(hs_row);
+  float2* vcs = cs + a.pairs;
+  const T* src = qkv + (size_t)t * a.ld;
+  // first columns (in the row) of the two groups of unit u; m: turned pairs of its head, k: the unit's first pair (< m) or none
+  auto place = [&](int u, int& c0, int& c1, int& m, int& k) {
+    const bool is_v = u * 8 >= nq + nk;
+    const int w = is_v ? a.vdim : a.dim, base = is_v ? nq + nk : 0;
+    const int h = (u * 8 - base) / w, e = u - (base + h * w) / 8;      // unit of its head
+    m = is_v ? (a.vfreq ? vhalf : 0) : a.pairs;
+    k = e * 4;
+    c0 = base + h * w;
+    if (a.halves && k < m)
+      c1 = c0 + m + k, c0 += k;
+    else
+      c0 += e * 8, c1 = c0 + 4;
+  };
+  float4 x[NU][2];
+#pragma unroll
+  for (int i = 0; i < NU; ++i) {
+    const int u = i * nt + tid;
+    if (u * 8 >= n) continue;
+    int c0, c1, m, k;
+    place(u, c0, c1, m, k);
+    x[i][0] = ld_f4(src + c0), x[i][1] = ld_f4(src + c1);
+  }
+  for (int i = tid; i < a.pairs; i += nt) {
+    float s, c;
+    sincosf((float)pos * a.freq[i], &s, &c);
+    cs[i] = make_float2(c * a.mul, s * a.mul);
+  }
+  for (int i = tid; a.vfreq && i < vhalf; i += nt) {
+    float s, c;
+    sincosf((float)pos * a.vfreq[i], &s, &c);
+    vcs[i] = make_float2(c, s);
+    a.turn[(size_t)t * vhalf + i] = make_float2(c, s);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < NU; ++i) {
+    const int u = i * nt + tid;
+    const bool in = u * 8 < n;
+    int c0 = 0, c1 = 4, m = 0, k = 0;
+    float v[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = 0.f;
+    if (in) {
+      place(u, c0, c1, m, k);
+      float4 b0 = make_float4(0.f, 0.f, 0.f, 0.f), b1 = b0;
+      if (a.bias) b0 = ld_f4(a.bias + c0), b1 = ld_f4(a.bias + c1);
+      v[0] = x[i][0].x + b0.x, v[1] = x[i][0].y + b0.y, v[2] = x[i][0].z + b0.z, v[3] = x[i][0].w + b0.w;
+      v[4] = x[i][1].x + b1.x, v[5] = x[i][1].y + b1.y, v[6] = x[i][1].z + b1.z, v[7] = x[i][1].w + b1.w;
+    }
+    if (a.gain) {
+      float s = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) s = fmaf(v[j], v[j], s);
+      for (int off = a.dim / 16; off > 0; off >>= 1) s += __shfl_xor_sync(0xffffffffu, s, off);
+      if (in && c0 < nq + nk) {
+        const float sc = 1.f / sqrtf(s / a.dim + a.eps);
+        const float* g = a.gain + (c0 < nq ? 0 : a.dim);
+        const float4 g0 = ld_f4(g + c0 % a.dim), g1 = ld_f4(g + c1 % a.dim);
+        v[0] *= sc * g0.x, v[1] *= sc * g0.y, v[2] *= sc * g0.z, v[3] *= sc * g0.w;
+        v[4] *= sc * g1.x, v[5] *= sc * g1.y, v[6] *= sc * g1.z, v[7] *= sc * g1.w;
+      }
+    }
+    if (!in) continue;
+    if (k < m) {
+      const float4* tab = reinterpret_cast<const float4*>((c0 < nq + nk ? cs : vcs) + k);      // two pairs each
+      const float4 r0 = tab[0], r1 = tab[1];
+      const float co[4] = {r0.x, r0.z, r1.x, r1.z}, si[4] = {r0.y, r0.w, r1.y, r1.w};
+      if (a.halves) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float y = v[j] * co[j] - v[4 + j] * si[j];
+          v[4 + j] = v[4 + j] * co[j] + v[j] * si[j], v[j] = y;
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float y = v[2 * j] * co[j] - v[2 * j + 1] * si[j];
+          v[2 * j + 1] = v[2 * j + 1] * co[j] + v[2 * j] * si[j], v[2 * j] = y;
+        }
+      }
+    }
+    T *d0 = q + (size_t)t * nq + c0, *d1 = q + (size_t)t * nq + c1;
+    if (c0 >= nq) {
+      if (loc < 0) continue;
+      T* base = c0 < nq + nk ? keys + (size_t)loc * nk - nq : values + (size_t)loc * nv - (nq + nk);
+      d0 = base + c0, d1 = base + c1;
+    }
+    st_f4(d0, make_float4(v[0], v[1], v[2], v[3]));
+    st_f4(d1, make_float4(v[4], v[5], v[6], v[7]));
+  }
+}
+
+// Other sizes: the row with its bias passes through shared memory, where a warp norms a head in place and partners meet.  W
+// consecutive values per thread and access.
 template <typename T, int W>
 __global__ void __launch_bounds__(256) head_store_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict__ keys,
                                                          T* __restrict__ values, const HeadStoreArgs a) {
@@ -916,6 +1023,25 @@ DSV4_API int dsv4_head_store(const void* qkv, int ld, const float* bias, const f
   const size_t smem = (size_t)(n + 3) / 4 * 16 + (pairs + (vfreq ? vdim / 2 : 0)) * sizeof(float2);
   if (smem > 200 * 1024) return 681;
   const bool wide = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && ((uintptr_t)qkv & 15) == 0;
+  const int units = (n / 8 + kUnitThreads - 1) / kUnitThreads, lanes = dim / 8;
+  if (wide && pairs % 4 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0 && units <= 8) {
+    const int threads = rows <= 512 && n <= 8192 ? (n / 8 + 31) / 32 * 32 : kUnitThreads;
+    const size_t small = (pairs + (vfreq ? vdim / 2 : 0)) * sizeof(float2);
+    auto go = [&](auto kern, auto type) {
+      using T = decltype(type);
+      dsv4_launch(kern, rows, threads, small, st, (const T*)qkv, (T*)q_out, (T*)keys, (T*)values, a);
+    };
+    auto pick = [&](auto type) {
+      using T = decltype(type);
+      if (units <= 1 || threads != kUnitThreads) go(head_store_units_kernel<T, 1>, type);
+      else if (units <= 3) go(head_store_units_kernel<T, 3>, type);
+      else if (units <= 5) go(head_store_units_kernel<T, 5>, type);
+      else go(head_store_units_kernel<T, 8>, type);
+    };
+    if (fp32) pick(float());
+    else pick(__nv_bfloat16());
+    return (int)cudaGetLastError();
+  }
   auto go = [&](auto kern, auto type) {
     using T = decltype(type);
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)

@@ -76,12 +76,63 @@ struct LatStoreArgs {
 };
 
 // One CTA per token.  cache row = [x / rms(x) * gain | turned part]; the queries' parts turn in place (`whole` null) or go, behind
-// the unrotated ones, to whole [T][heads][dim + rot].
+// the unrotated ones, to whole [T][heads][dim + rot].  Four values at a time where every size is a multiple of four: the latent and a
+// first share of the queries' turned parts then wait in registers while angles and squares are summed up.
+__device__ __forceinline__ float4 turn4(const float4& v, const float2* cs) {
+  const float4 r = *reinterpret_cast<const float4*>(cs);      // two pairs
+  return make_float4(v.x * r.x - v.y * r.y, v.y * r.x + v.x * r.y, v.z * r.z - v.w * r.w, v.w * r.z + v.z * r.w);
+}
+constexpr int kLatThreads = 128;
+template <typename T>
+__global__ void __launch_bounds__(kLatThreads) latent_rotate_store4_kernel(T* p, T* __restrict__ cache, T* __restrict__ whole,
+                                                                           const LatStoreArgs a) {
+  pdl_entry();
+  extern __shared__ __align__(16) float2 lat_cs[];
+  __shared__ float sh[32];
+  const int t = blockIdx.x, tid = threadIdx.x, loc = a.out_loc[t], wide = a.dim + a.rot, r4 = a.rot / 4, c4 = a.rank / 4;
+  T* row = p + (size_t)t * a.ld;
+  const T* x = row + a.at_c;
+  T* q = row + a.at_rot;
+  const int nq = a.heads * r4;
+  float4 lat = make_float4(0.f, 0.f, 0.f, 0.f), mine = lat;
+  if (tid < c4) lat = ld_f4(x + tid * 4);
+  if (tid < nq) mine = ld_f4(q + tid * 4);
+  for (int i = tid; i < a.rot / 2; i += kLatThreads) {
+    float s, c;
+    sincosf((float)a.pos[t] * a.freq[i], &s, &c);
+    lat_cs[i] = make_float2(c * a.mul, s * a.mul);
+  }
+  float ss = lat.x * lat.x + lat.y * lat.y + lat.z * lat.z + lat.w * lat.w;
+  for (int i = tid + kLatThreads; i < c4; i += kLatThreads) {
+    const float4 v = ld_f4(x + i * 4);
+    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+  if (whole)                                       // the unrotated parts, next to their heads' turned ones
+    for (int i = tid; i < a.heads * (a.dim / 4); i += kLatThreads) {
+      const int h = i / (a.dim / 4);
+      st_f4(whole + ((size_t)t * a.heads + h) * wide + (i - h * (a.dim / 4)) * 4, ld_f4(row + i * 4));
+    }
+  const float sc = 1.f / sqrtf(cta_sum(ss, sh) / a.rank + a.eps);    // its barriers also publish lat_cs
+  if (loc >= 0) {
+    T* dst = cache + (size_t)loc * (a.rank + a.rot);
+    for (int i = tid; i < c4; i += kLatThreads) {
+      const float4 v = i == tid ? lat : ld_f4(x + i * 4), g = ld_f4(a.gain + i * 4);
+      st_f4(dst + i * 4, make_float4(v.x * sc * g.x, v.y * sc * g.y, v.z * sc * g.z, v.w * sc * g.w));
+    }
+    for (int i = tid; i < r4; i += kLatThreads) st_f4(dst + a.rank + i * 4, turn4(ld_f4(x + a.rank + i * 4), lat_cs + 2 * i));
+  }
+  for (int i = tid; i < nq; i += kLatThreads) {
+    const int h = i / r4, k = i - h * r4;
+    st_f4(whole ? whole + ((size_t)t * a.heads + h) * wide + a.dim + 4 * k : q + 4 * i,
+          turn4(i == tid ? mine : ld_f4(q + 4 * i), lat_cs + 2 * k));
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) latent_rotate_store_kernel(T* p, T* __restrict__ cache, T* __restrict__ whole,
                                                                   const LatStoreArgs a) {
   pdl_entry();
-  extern __shared__ float2 lat_cs[];
+  extern __shared__ __align__(16) float2 lat_cs[];
   __shared__ float sh[32];
   const int t = blockIdx.x, loc = a.out_loc[t], half = a.rot / 2, wide = a.dim + a.rot;
   T* row = p + (size_t)t * a.ld;
@@ -558,11 +609,17 @@ DSV4_API int dsv4_latent_rotate_store(void* p, int ld, int at_rot, int at_c, con
   if (rows <= 0) return 0;
   if (rot < 2 || rot % 2 || rot > 8192 || !freq) return 637;
   const LatStoreArgs a{ld, at_rot, at_c, gain, eps, freq, mul, pos, out_loc, heads, dim, rot, rank};
+  const bool fours = ld % 4 == 0 && at_rot % 4 == 0 && at_c % 4 == 0 && dim % 4 == 0 && rot % 4 == 0 && rank % 4 == 0 &&
+                     ((uintptr_t)p & 15) == 0;
+  auto go = [&](auto kern, int threads, auto type) {
+    using T = decltype(type);
+    dsv4_launch(kern, rows, threads, rot * 4, st, (T*)p, (T*)cache, (T*)whole, a);
+  };
+  using B = __nv_bfloat16;
   if (fp32)
-    dsv4_launch(latent_rotate_store_kernel<float>, rows, 256, rot * 4, st, (float*)p, (float*)cache, (float*)whole, a);
+    fours ? go(latent_rotate_store4_kernel<float>, kLatThreads, float()) : go(latent_rotate_store_kernel<float>, 256, float());
   else
-    dsv4_launch(latent_rotate_store_kernel<__nv_bfloat16>, rows, 256, rot * 4, st, (__nv_bfloat16*)p, (__nv_bfloat16*)cache,
-                (__nv_bfloat16*)whole, a);
+    fours ? go(latent_rotate_store4_kernel<B>, kLatThreads, B()) : go(latent_rotate_store_kernel<B>, 256, B());
   return (int)cudaGetLastError();
 }
 

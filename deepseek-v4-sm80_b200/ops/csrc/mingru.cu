@@ -7,7 +7,7 @@
 // S -> a S + b, which compose to (a1 a2, a2 b1 + b2): products of the decays themselves, so portions of any length run in parallel
 // without logarithms.
 //   mingru_step   one thread per request and W elements, token by token: decode and short portions
-//   mingru_scan   a CTA takes `CT` neighbouring elements of one request and all its tokens: 512 threads hold 8 tokens each, the
+//   mingru_scan   a CTA takes `CT` neighbouring elements of one request and all its tokens: 256 threads hold 8 tokens each, the
 //                 maps are combined over lanes and warps, the state is carried from tile to tile.  The next tile's inputs are
 //                 fetched before the current tile is combined.
 #include "vec.cuh"
@@ -23,12 +23,21 @@ struct MinGruArgs {
   int width;
 };
 
-// z and u with their biases -> the step's map (a, b)
+// z and u with their biases -> the step's map (a, b).  1 - sigmoid(z) = e^-z sigmoid(z), without cancellation.  Where bf16 comes out,
+// both reciprocals are one: 1 / p = q / (p q).
 template <typename T>
 __device__ __forceinline__ void gru_map(float z, float u, float& a, float& b) {
-  const float s = sigmoid_for<T>(z);
-  a = sigmoid_for<T>(-z);                                  // 1 - z without cancellation
-  b = s * (u >= 0.f ? u + 0.5f : sigmoid_for<T>(u));
+  if constexpr (sizeof(T) == 2) {
+    const float ez = __expf(fminf(-z, 40.f)), eu = __expf(fminf(-u, 40.f));
+    const float p = 1.f + ez, q = 1.f + eu, r = __fdividef(1.f, p * q);
+    const float s = q * r;
+    a = ez * s;
+    b = s * (u >= 0.f ? u + 0.5f : p * r);
+  } else {
+    const float ez = expf(fminf(-z, 80.f)), s = 1.f / (1.f + ez);
+    a = ez * s;
+    b = s * (u >= 0.f ? u + 0.5f : sigmoid_f(u));
+  }
 }
 
 template <typename T, int W>
@@ -63,10 +72,10 @@ __global__ void __launch_bounds__(128) mingru_step_kernel(T* __restrict__ y, con
   st_w<W>(st, s);
 }
 
-constexpr int kGruThreads = 512, kGruTokens = 8, kGruWarps = kGruThreads / 32;
+constexpr int kGruThreads = 256, kGruTokens = 8, kGruWarps = kGruThreads / 32;
 
 template <typename T, int CT>
-__global__ void __launch_bounds__(kGruThreads, 1) mingru_scan_kernel(T* __restrict__ y, const MinGruArgs a) {
+__global__ void __launch_bounds__(kGruThreads, 2) mingru_scan_kernel(T* __restrict__ y, const MinGruArgs a) {
   pdl_entry();
   constexpr int L = kGruTokens, SUB = 32 / CT, TT = kGruThreads / CT * L;   // token groups per warp, tokens per tile
   __shared__ float2 maps[2][kGruWarps][CT];

@@ -112,6 +112,13 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const NormArgs a, co
   if constexpr (NV > 0) {
     float4 keep[NV];
     float4 y[NV];
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {          // everything in flight before the first sum
+      const int i = (n * 256 + threadIdx.x) * 4;
+      if (i >= d) continue;
+      keep[n] = ld_f4(a.x + src + i);
+      if (a.sub) y[n] = ld_f4(a.sub + src + i);
+    }
     float sub_sc = 0.f;
     if (a.sub) {
       float s2 = 0.f;
@@ -119,7 +126,6 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const NormArgs a, co
       for (int n = 0; n < NV; ++n) {
         const int i = (n * 256 + threadIdx.x) * 4;
         if (i >= d) continue;
-        y[n] = ld_f4(a.sub + src + i);
         if (a.sub_bias) {
           const float4 u = ld_f4(a.sub_bias + i);
           y[n].x += u.x, y[n].y += u.y, y[n].z += u.z, y[n].w += u.w;
@@ -132,7 +138,7 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const NormArgs a, co
     for (int n = 0; n < NV; ++n) {
       const int i = (n * 256 + threadIdx.x) * 4;
       if (i >= d) continue;
-      float4 v = *reinterpret_cast<const float4*>(a.x + src + i);
+      float4 v = keep[n];
       if (adds) {
         if (a.sub) {
           const float4 g = ld_f4(a.sub_gain + i);

@@ -283,7 +283,7 @@ def mingru(p, at_u, at_g, bias_z, bias_u, state, fb, dtype):
     assert p.shape[1] >= at_g + width
     y = torch.empty(t, width, dtype=dtype, device=p.device)
     segs = t if fb.seg_off is None else fb.seg_off.shape[0] - 1
-    fill = num_sms(p.device) * 2 // 3
+    fill = num_sms(p.device) * 4 // 3
     ct = next((c for c in GRU_TILES if -(-width // c) * segs >= fill), GRU_TILES[-1])
     nv.call("mingru", nv.ptr(p), I(p.stride(0)), I(at_u), I(at_g), nv.ptr(bias_z), nv.ptr(bias_u), nv.ptr(state), nv.ptr(y),
             nv.ptr(fb.slots), nv.ptr(fb.positions), nv.ptr(fb.seg_off), I(segs),

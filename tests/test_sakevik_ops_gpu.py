@@ -135,7 +135,7 @@ def test_recurrence(width, dtype):
 def test_parallel_recurrence_at_its_edges(ct, dtype, monkeypatch):
     """Lengths around the tiles of every form; gates that forget within a token and ones that remember all of it."""
     monkeypatch.setattr(CL, "GRU_TILES", (ct,))
-    tile = 512 // ct * 8
+    tile = 256 // ct * 8
     for n in (17, tile - 1, tile, tile + 1, 2 * tile + 9):
         gru_case(45, [(2, 7, n), (4, 0, n + 3)], dtype, decay=3.0)
     gru_case(45, [(2, 7, 2 * tile + 9)], dtype, decay=12.0)
@@ -163,10 +163,12 @@ def test_recurrence_in_portions_carries_its_state(dtype):
 @BOTH
 @pytest.mark.parametrize("halves", [True, False])
 @pytest.mark.parametrize("heads,kv,dim,vdim,dims", [(6, 3, 32, 24, 24), (4, 1, 16, 64, 16), (3, 3, 7, 6, 4), (16, 4, 128, 128, 64),
-                                                    (2, 2, 24, 40, 0), (1, 1, 2, 2, 2), (5, 1, 12, 320, 10), (64, 8, 128, 128, 128)])
-def test_norm_and_rotation_per_head(heads, kv, dim, vdim, dims, halves, dtype):
-    fb, rows = make_fb([(1, 0, 5), (2, 22, 4), (0, 900, 2)], DEV)
-    t, n, eps, base, mul = 11, (heads + kv) * dim + kv * vdim, 1e-2, 700.0, 1.3
+                                                    (2, 2, 24, 40, 0), (1, 1, 2, 2, 2), (5, 1, 12, 320, 10), (64, 8, 128, 128, 128),
+                                                    (28, 4, 128, 64, 120), (96, 8, 128, 128, 64)])
+@pytest.mark.parametrize("long", [0, 520])       # few tokens and many run with other blocks
+def test_norm_and_rotation_per_head(heads, kv, dim, vdim, dims, long, halves, dtype):
+    fb, rows = make_fb([(1, 0, 5), (2, 22, 4), (0, 900, 2)] + [(3, 30, long)] * (long > 0), DEV)
+    t, n, eps, base, mul = 11 + long, (heads + kv) * dim + kv * vdim, 1e-2, 700.0, 1.3
     wide = rand(t, n + 8, std=0.3).to(dtype)          # a column slice of a wider projection
     bias, gain = rand(n, seed=1), rand(2, dim, seed=2, mean=1.0)
     freq, vfreq = rotary_frequencies(dims, base)[0] if dims else None, rotary_frequencies(vdim, base)[0]
